@@ -265,9 +265,50 @@ typedef struct {
   int32_t cross_len;       /* Whisper: encoder positions the cross attention reads (1500) */
   int32_t reserved;
 } lmb200_model_config;
-enum { LMB200_ARCH_LLAMA = 0, LMB200_ARCH_WHISPER_DECODER = 1 };
+enum { LMB200_ARCH_LLAMA = 0, LMB200_ARCH_WHISPER_DECODER = 1, LMB200_ARCH_LAYERED = 2 };
 
 int32_t lmb200_model_create(lmb200_ctx ctx, const lmb200_model_config* cfg, lmb200_model* model);
+
+/* A decoder whose layers are described one by one (LMB200_ARCH_LAYERED): every layer has its own mixer, sizes and
+ * constants.  Layer i is x <- x + (mixer(h) + ff(h)) with h the RMSNorm of x; the head follows a final RMSNorm and may be
+ * bounded by softcap * tanh(. / softcap).  Not in the reference, whose models repeat one kind of layer (src/NN.jl:417-507).
+ *  - LMB200_MIXER_LATENT_ATTENTION: causal attention whose keys and values are linear in one cached latent per token
+ *    (kv_rank wide) plus one rotated key part shared by the heads (rot_dim wide); queries come from a latent of q_rank;
+ *    every head's output is multiplied by a sigmoid gate.  kv_from >= 0: the layer has no latent of its own and reads the
+ *    cache of that earlier layer.
+ *  - LMB200_MIXER_RETENTION: linear attention with a fixed decay per head over a float32 state [dim, vdim] per head; the
+ *    output of a head is divided by its root mean square and gated with silu.
+ * Tensor names: "embed", "final.norm", "head"; per layer i "l<i>.norm1", "l<i>.mlp.up", "l<i>.mlp.down", and under
+ * "l<i>.mix.": latent attention dq, dq.norm, uq, dkv, dkv.norm, uk, uv, g, o; retention q, k, v, g, o. */
+enum { LMB200_MIXER_LATENT_ATTENTION = 0, LMB200_MIXER_RETENTION = 1 };
+enum { LMB200_ROT_HALF = 0, LMB200_ROT_INTERLEAVED = 1 };   /* pairs (i, i + rot_dims/2), or (2i, 2i + 1) */
+typedef struct {
+  int32_t mixer;
+  int32_t heads;
+  int32_t dim;             /* query / key width per head (latent attention: the part without positions) */
+  int32_t vdim;            /* value width per head */
+  int32_t q_rank;          /* latent attention */
+  int32_t kv_rank;         /* latent attention */
+  int32_t rot_dim;         /* latent attention: width of the part with positions */
+  int32_t kv_from;         /* latent attention: -1, or the layer whose latent cache is read */
+  int32_t rot_dims;        /* features that are rotated, from the first on (0: none; latent attention: rot_dim) */
+  int32_t rot_layout;      /* LMB200_ROT_* */
+  int32_t ff;              /* width of the feed-forward down(relu(up h)^2); 0: none */
+  float scale;             /* latent attention: factor of the scores */
+  double rot_base;         /* frequency i is rot_base^(-2 i / rot_dims) */
+  const double* decay;     /* retention: [heads], each in (0, 1]; copied */
+} lmb200_layer_config;
+typedef struct {
+  int32_t n_layers;
+  int32_t width;
+  int32_t vocab;
+  int32_t dtype;           /* LMB200_F32, or LMB200_BF16: weights, latent cache and GEMM inputs bf16; residual, norms, scores,
+                              states and accumulation float32 */
+  float eps;               /* of every RMSNorm */
+  float softcap;           /* 0: the logits are not bounded */
+} lmb200_layered_config;
+int32_t lmb200_model_create_layered(lmb200_ctx ctx, const lmb200_layered_config* cfg, const lmb200_layer_config* layers,
+                                    lmb200_model* model);
 /* Host-only view of the weight re-layout and tensor-parallel sharding (no GPU needed): the extent
  * of this rank's fused matrix `matrix` (0 qkv, 1 o_proj, 2 gate/up, 3 down_proj, 4 lm_head) and, for
  * one of its elements, which logical tensor (slot: q/k/v = 0/1/2, gate/up = 0/1, else 0) and which
@@ -308,7 +349,9 @@ int32_t lmb200_session_destroy(lmb200_session session);
 int32_t lmb200_session_reset(lmb200_session session);
 int32_t lmb200_session_position(lmb200_session session, int32_t* pos);
 /* Rewind (or move) the position of every sequence; cache contents at and beyond it are overwritten by
- * later steps.  lmb200_session_position reports the furthest position of any sequence. */
+ * later steps.  lmb200_session_position reports the furthest position of any sequence.  A sequence put to position 0 is
+ * free for a new request.  Layers with a recurrent state (LMB200_MIXER_RETENTION) allow position 0 (the state is emptied)
+ * and the present position only; anything else is LMB200_ESTATE. */
 int32_t lmb200_session_set_position(lmb200_session session, int32_t pos);
 /* One position per sequence (pos[batch] / pos_out[batch]).  The reference's [batch, seq] token tensor
  * gives every sequence the same length (src/NN.jl:448-455); a batch of real prompts has one length
@@ -342,6 +385,13 @@ int32_t lmb200_prefill(lmb200_session session, const int32_t* tokens, int32_t n,
  * do for equal lengths. */
 int32_t lmb200_prefill_ragged(lmb200_session session, const int32_t* tokens, const int32_t* lengths,
                               int32_t n_max, float* logits_out);
+/* The next lengths[b] >= 0 tokens of every sequence, appended at that sequence's position: `tokens` holds the ids of
+ * sequence 0, then those of sequence 1, and so on.  want[n_want] (ascending places in that packed order) chooses the
+ * positions whose logits come back, [n_want, vocab] in logits_out.  Prompts, portions of prompts and single tokens can be
+ * mixed in one call; the result at a position does not depend on how its tokens were cut into calls, beyond rounding.
+ * Replaces running the model over [batch, seq] tokens and slicing its logits (src/NN.jl:448-455). */
+int32_t lmb200_extend(lmb200_session session, const int32_t* tokens, const int32_t* lengths, int32_t n_want,
+                      const int32_t* want, float* logits_out);
 /* One token per sequence in, greedy next token out; host buffers, copies inside the call.
  * Replaces one iteration of the generation loop (src/Decoding.jl:91-130, examples/llama.jl:73-99). */
 int32_t lmb200_decode_step(lmb200_session session, const int32_t* tokens_in,

@@ -33,6 +33,17 @@ class ModelConfig(C.Structure):
                 ("reserved", C.c_int32)]
 
 
+class LayerConfig(C.Structure):
+    _fields_ = [(n, C.c_int32) for n in ("mixer", "heads", "dim", "vdim", "q_rank", "kv_rank", "rot_dim", "kv_from", "rot_dims",
+                                         "rot_layout", "ff")] + \
+               [("scale", C.c_float), ("rot_base", C.c_double), ("decay", C.POINTER(C.c_double))]
+
+
+class LayeredConfig(C.Structure):
+    _fields_ = [("n_layers", C.c_int32), ("width", C.c_int32), ("vocab", C.c_int32), ("dtype", C.c_int32), ("eps", C.c_float),
+                ("softcap", C.c_float)]
+
+
 _i32, _i64, _u64, _f32, _vp = C.c_int32, C.c_int64, C.c_uint64, C.c_float, C.c_void_p
 _pi64 = C.POINTER(C.c_int64)
 _pi32 = C.POINTER(C.c_int32)
@@ -87,6 +98,8 @@ SIGNATURES = {
     "lmb200_whisper_encoder_run": [_u64, _vp, _i32, _i32, _vp],
     "lmb200_whisper_encoder_cross_kv": [_u64, _u64],
     "lmb200_model_create": [_u64, C.POINTER(ModelConfig), C.POINTER(_u64)],
+    "lmb200_model_create_layered": [_u64, C.POINTER(LayeredConfig), C.POINTER(LayerConfig), C.POINTER(_u64)],
+    "lmb200_extend": [_u64, _vp, _vp, _i32, _vp, _vp],
     "lmb200_shard_extent": [C.POINTER(ModelConfig), _i32, _pi32, _pi32],
     "lmb200_shard_map": [C.POINTER(ModelConfig), _i32, _i32, _i32, _pi32, _pi32, _pi32],
     "lmb200_model_destroy": [_u64],

@@ -541,9 +541,28 @@ __device__ __forceinline__ void row_epilogue(const GemvParams& p, float (&v)[NV]
   }
   if (p.epi == EPI_STORE_F32) {
     if (row < p.rows) {
+      if (p.softcap > 0.f) {
+#pragma unroll
+        for (int b = 0; b < N; ++b) v[b] = p.softcap * tanhf(v[b] / p.softcap);
+      }
 #pragma unroll
       for (int b = 0; b < N; ++b)
         if (b0 + b < p.B) p.out[(int64_t)(b0 + b) * p.out_pitch + row] = v[b];
+    }
+    return;
+  }
+  if (p.epi == EPI_STORE_RELU2) {
+    if (row < p.act_row0) {
+#pragma unroll
+      for (int b = 0; b < N; ++b)
+        if (b0 + b < p.B) p.out[(int64_t)(b0 + b) * p.out_pitch + row] = v[b];
+    } else if (row - p.act_row0 < p.n_act) {
+      __nv_bfloat16* act = reinterpret_cast<__nv_bfloat16*>(p.act);
+#pragma unroll
+      for (int b = 0; b < N; ++b) {
+        const float u = fmaxf(v[b], 0.f);
+        if (b0 + b < p.B) act[LY::x_offset(b0 + b, p.act_col0 + row - p.act_row0, BP)] = __float2bfloat16_rn(u * u);
+      }
     }
     return;
   }

@@ -11,6 +11,7 @@ enum GemvEpilogue {
   EPI_SILU_GATE = 1,   // act[b, i] = silu(gate_i) * up_i         (rows interleaved 8 gate / 8 up)
   EPI_QKV_ROPE = 2,    // RoPE on q and k (if `rope`), q -> q_out, k/v appended to the cache at *pos
   EPI_GELU_ACT = 3,    // act[b, row] = gelu(acc)                  (Whisper fc1)
+  EPI_STORE_RELU2 = 5, // rows < act_row0: out[b, row] = acc; rows from act_row0: act[b, act_col0 + row - act_row0] = relu(acc)^2
   EPI_RESID_NORM = 4   // row-parallel projection + all-reduce + residual add + RMSNorm preparation (ResidNorm below)
 };
 
@@ -91,6 +92,8 @@ struct GemvParams {
   // EPI_STORE_F32
   float* out = nullptr;
   int out_pitch = 0;
+  float softcap = 0.f;       // > 0: out = softcap * tanh(acc / softcap)
+  int act_row0 = 0, act_col0 = 0;   // EPI_STORE_RELU2
   // EPI_SILU_GATE: act is a GEMV activation buffer of the same batch padding as x
   void* act = nullptr;
   int n_act = 0;

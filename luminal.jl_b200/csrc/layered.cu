@@ -1,0 +1,967 @@
+// Decoders described layer by layer (LMB200_ARCH_LAYERED): the layers' specifications, their weights, the per-layer caches and
+// states of a session, and the two ways a step runs.
+//   fused step   bf16 decoding, one token per sequence, captured in a CUDA graph: GEMVs whose epilogues carry the norm's scale,
+//                the feed-forward's activation, the residual sum and the next norm's preparation.  A layer's projections are
+//                one matrix, and so are its two output projections: retention takes three launches, latent attention seven.
+//   rows step    any number of tokens of any sequences, packed: prompts, portions of prompts, mixed calls; and every
+//                float32 step.
+#include <math.h>
+#include <stdio.h>
+#include <string.h>
+
+#include <algorithm>
+
+#include "latent.cuh"
+#include "model.cuh"
+#include "pdl.cuh"
+#include "retention.cuh"
+
+namespace lmb {
+
+// device buffers of a rows step over up to `cap_T` tokens
+struct RowsBuf {
+  int64_t cap_T = 0;
+  void* base = nullptr;
+  int64_t bytes = 0;
+  float *x = nullptr, *delta = nullptr, *proj = nullptr, *olat = nullptr;
+  void *xn = nullptr, *xq = nullptr, *q = nullptr, *qa = nullptr, *cat = nullptr;
+  int* meta = nullptr;          // tokens | seq | pos | last (sequence whose last token this is, or -1), cap_T each; then start | len | pos0, B each; want
+};
+
+struct LayeredScratch {
+  // fused step
+  float *proj = nullptr, *qf = nullptr, *olat = nullptr;
+  void *xq = nullptr, *qa = nullptr;
+  std::vector<GemvPlan> p_in, p_out, p_uq;
+  int *iota = nullptr, *ones = nullptr;          // [B]
+  LatentAttnPlan attn;
+  float* attn_part = nullptr;
+  unsigned* attn_counters = nullptr;
+  RowsBuf step, prompt;                          // float32 decode step; everything longer
+  float* want_logits = nullptr;
+  void* want_xn = nullptr;
+  int64_t want_cap = 0;
+  float* prompt_part = nullptr;                  // split partials of the absorbed attention in a rows step
+  unsigned* prompt_counters = nullptr;
+  int64_t prompt_part_floats = 0, prompt_counter_cap = 0;
+};
+
+namespace {
+
+constexpr int kBlockTokens = 2048;      // tokens per round of the absorbed attention in a rows step (bounds its scratch)
+constexpr uint64_t kIdLayered = 0x200000, kIdLayeredState = 0x300000;
+enum LatentSlot { L_DQ = 0, L_DKV = 1, L_G = 2, L_UP = 3 };
+enum RetentionSlot { R_Q = 0, R_K = 1, R_V = 2, R_G = 3, R_UP = 4 };
+
+bool is_latent(const LayerSpec& s) { return s.c.mixer == LMB200_MIXER_LATENT_ATTENTION; }
+int out_width(const LayerSpec& s) { return s.c.heads * s.c.vdim; }
+int q_width(const LayerSpec& s) { return s.c.heads * (s.c.dim + s.c.rot_dim); }
+int state_ld(const LayerSpec& s) { return (int)round_up(s.c.vdim, 4); }
+int row_ld(int n) { return (int)round_up(n, 8); }
+const LayerSpec& cache_spec(const Model* M, int l) { return M->specs[M->specs[l].c.kv_from >= 0 ? M->specs[l].c.kv_from : l]; }
+int cache_layer(const Model* M, int l) { return M->specs[l].c.kv_from >= 0 ? M->specs[l].c.kv_from : l; }
+
+int32_t check_layer(const lmb200_layer_config& c, const std::vector<LayerSpec>& before, int i) {
+  LMB_REQUIRE(c.mixer == LMB200_MIXER_LATENT_ATTENTION || c.mixer == LMB200_MIXER_RETENTION, "layer %d: mixer %d", i, c.mixer);
+  LMB_REQUIRE(c.heads >= 1 && c.dim >= 1 && c.vdim >= 1 && c.ff >= 0, "layer %d: non-positive size", i);
+  LMB_REQUIRE(c.rot_layout == LMB200_ROT_HALF || c.rot_layout == LMB200_ROT_INTERLEAVED, "layer %d: rot_layout %d", i, c.rot_layout);
+  LMB_REQUIRE(c.rot_dims >= 0 && c.rot_dims % 2 == 0 && (c.rot_dims == 0 || c.rot_base > 0), "layer %d: rotation of %d features, base %g", i,
+              c.rot_dims, c.rot_base);
+  if (c.mixer == LMB200_MIXER_LATENT_ATTENTION) {
+    LMB_REQUIRE(c.q_rank >= 1 && c.kv_rank >= 1 && c.rot_dim >= 0 && c.rot_dims <= c.rot_dim, "layer %d: ranks %d, %d, rotated %d of %d", i,
+                c.q_rank, c.kv_rank, c.rot_dims, c.rot_dim);
+    LMB_REQUIRE(c.dim <= 1024 && c.kv_rank <= 1024, "layer %d: head width %d, latent width %d (at most 1024)", i, c.dim, c.kv_rank);
+    LMB_REQUIRE(c.kv_from < i, "layer %d: kv_from %d is not an earlier layer", i, c.kv_from);
+    if (c.kv_from >= 0) {
+      const lmb200_layer_config& f = before[c.kv_from].c;
+      LMB_REQUIRE(f.mixer == c.mixer && f.kv_from < 0 && f.kv_rank == c.kv_rank && f.rot_dim == c.rot_dim && f.rot_dims == c.rot_dims &&
+                      f.rot_base == c.rot_base && f.rot_layout == c.rot_layout,
+                  "layer %d: layer %d has no latent cache of its own with the same widths and rotation", i, c.kv_from);
+    }
+  } else {
+    LMB_REQUIRE(c.decay, "layer %d: no decay", i);
+    LMB_REQUIRE(c.rot_dims <= c.dim && c.dim <= 2048 && c.vdim <= 4096, "layer %d: heads of %d x %d, %d features rotated", i, c.dim, c.vdim, c.rot_dims);
+    for (int h = 0; h < c.heads; ++h)
+      LMB_REQUIRE(c.decay[h] > 0.0 && c.decay[h] <= 1.0, "layer %d: decay %g of head %d", i, c.decay[h], h);
+  }
+  return LMB200_OK;
+}
+
+void stack(WMap& m, int slot, int row0, int rows, int col0, int cols) {
+  m.row_off[slot] = row0; m.src_rows[slot] = rows; m.col_off[slot] = col0; m.src_cols[slot] = cols;
+  if (m.n_src <= slot) m.n_src = slot + 1;
+}
+
+void derive_layer(LayerSpec& s, int width) {
+  const lmb200_layer_config& c = s.c;
+  s.m_in.kind = s.m_out.kind = s.m_uq.kind = s.m_ukv.kind = MAP_STACK;
+  int at = 0;
+  auto part = [&](int slot, int rows) {
+    s.row0[slot] = at;
+    stack(s.m_in, slot, at, rows, 0, width);
+    at += (int)round_up(rows, 32);
+  };
+  if (is_latent(s)) {
+    part(L_DQ, c.q_rank);
+    if (c.kv_from < 0) part(L_DKV, c.kv_rank + c.rot_dim);
+    part(L_G, c.heads);
+    s.n_store = at;
+    if (c.ff) part(L_UP, c.ff);
+    stack(s.m_uq, 0, 0, q_width(s), 0, c.q_rank);
+    s.m_uq.rows = q_width(s); s.m_uq.K = c.q_rank;
+    const int uv0 = (int)round_up(c.heads * c.dim, 32);
+    stack(s.m_ukv, 0, 0, c.heads * c.dim, 0, c.kv_rank);
+    stack(s.m_ukv, 1, uv0, out_width(s), 0, c.kv_rank);
+    s.m_ukv.rows = uv0 + out_width(s); s.m_ukv.K = c.kv_rank;
+    finish_map(s.m_uq);
+    finish_map(s.m_ukv);
+    s.lat_rot = (int)round_up(c.kv_rank, 8);
+    s.lat_ld = (int)round_up(s.lat_rot + c.rot_dim, 8);
+  } else {
+    part(R_Q, c.heads * c.dim);
+    part(R_K, c.heads * c.dim);
+    part(R_V, out_width(s));
+    part(R_G, out_width(s));
+    s.n_store = at;
+    if (c.ff) part(R_UP, c.ff);
+  }
+  s.m_in.rows = at; s.m_in.K = width;
+  s.cat0 = (int)round_up(out_width(s), 32);
+  stack(s.m_out, 0, 0, width, 0, out_width(s));
+  if (c.ff) stack(s.m_out, 1, 0, width, s.cat0, c.ff);
+  s.m_out.rows = width; s.m_out.K = c.ff ? s.cat0 + c.ff : out_width(s);
+  finish_map(s.m_in);
+  finish_map(s.m_out);
+}
+
+// where a tensor lives: a slot of a stacked matrix, a float32 vector, the embedding, and / or a row-major copy
+struct Target {
+  void* tiled = nullptr;
+  const WMap* map = nullptr;
+  int slot = 0;
+  void* plain = nullptr;         // row-major copy in the model dtype (float32 for vectors)
+  bool vec = false;
+  int64_t rows = 0, cols = 0;
+};
+
+bool find_target(Model* M, const std::string& n, Target* t) {
+  const lmb200_model_config& c = M->cfg;
+  auto vec = [&](float* d, int64_t len) { t->plain = d; t->vec = true; t->rows = 1; t->cols = len; return true; };
+  auto mat = [&](void* d, const WMap& m, int slot) {
+    t->tiled = d; t->map = &m; t->slot = slot; t->rows = m.src_rows[slot]; t->cols = m.src_cols[slot];
+    return true;
+  };
+  if (n == "embed") { t->plain = M->embed; t->rows = c.vocab; t->cols = c.hidden; return true; }
+  if (n == "final.norm") return vec(M->final_norm, c.hidden);
+  if (n == "head") return mat(M->lm_head, M->m_head, 0);
+  int layer = -1, used = 0;
+  if (sscanf(n.c_str(), "l%d.%n", &layer, &used) < 1 || used == 0 || layer < 0 || layer >= c.n_layers) return false;
+  const std::string tail = n.substr(used);
+  LayerSpec& s = M->specs[layer];
+  LayeredWeights& w = M->lw[layer];
+  if (tail == "norm1") return vec(w.norm, c.hidden);
+  const bool latent = is_latent(s);
+  if (s.c.ff && tail == "mlp.up") return mat(w.w_in, s.m_in, latent ? (int)L_UP : (int)R_UP);
+  if (s.c.ff && tail == "mlp.down") return mat(w.w_out, s.m_out, 1);
+  if (tail == "mix.o") return mat(w.w_out, s.m_out, 0);
+  if (latent) {
+    if (tail == "mix.dq") return mat(w.w_in, s.m_in, L_DQ);
+    if (tail == "mix.dq.norm") return vec(w.q_norm, s.c.q_rank);
+    if (tail == "mix.uq") return mat(w.w_uq, s.m_uq, 0);
+    if (tail == "mix.g") return mat(w.w_in, s.m_in, L_G);
+    if (s.c.kv_from < 0 && tail == "mix.dkv") return mat(w.w_in, s.m_in, L_DKV);
+    if (s.c.kv_from < 0 && tail == "mix.dkv.norm") return vec(w.kv_norm, s.c.kv_rank);
+    if (tail == "mix.uk") { mat(w.w_ukv, s.m_ukv, 0); t->plain = w.w_uk; return true; }
+    if (tail == "mix.uv") { mat(w.w_ukv, s.m_ukv, 1); t->plain = w.w_uv; return true; }
+    return false;
+  }
+  if (tail == "mix.q") return mat(w.w_in, s.m_in, R_Q);
+  if (tail == "mix.k") return mat(w.w_in, s.m_in, R_K);
+  if (tail == "mix.v") return mat(w.w_in, s.m_in, R_V);
+  if (tail == "mix.g") return mat(w.w_in, s.m_in, R_G);
+  return false;
+}
+
+// fills a tensor from `src` (device float32) or, src == NULL, from the generator
+int32_t fill_target(Model* M, const Target& t, uint64_t key, const float* src, int layout, float scale) {
+  if (t.vec) return fill_plain_dt(M, LMB200_F32, t.plain, t.rows, t.cols, key, src, 0, scale, src ? 0.f : 1.f);
+  if (t.plain) LMB_TRY(fill_plain_dt(M, M->cfg.dtype, t.plain, t.rows, t.cols, key, src, layout, scale, 0.f));
+  if (!t.tiled) return LMB200_OK;
+  FillSrc f{};
+  f.only_slot = t.slot; f.colmajor = layout; f.scale = scale;
+  f.key[t.slot] = key; f.src[t.slot] = src;
+  return fill_tiled_dt(M, t.tiled, *t.map, f);
+}
+
+}  // namespace
+
+void layered_free_model(Model* M) {
+  for (LayeredWeights& w : M->lw) {
+    cudaFree(w.w_in); cudaFree(w.w_out); cudaFree(w.w_uq); cudaFree(w.w_ukv); cudaFree(w.w_uk); cudaFree(w.w_uv);
+    cudaFree(w.norm); cudaFree(w.q_norm); cudaFree(w.kv_norm); cudaFree(w.inv_freq); cudaFree(w.decay);
+  }
+  M->lw.clear();
+}
+
+bool layered_has_state(const Model* M) {
+  for (const LayerSpec& s : M->specs)
+    if (!is_latent(s)) return true;
+  return false;
+}
+
+std::vector<std::string> layered_weight_names(const Model* M) {
+  std::vector<std::string> v = {"embed", "final.norm", "head"};
+  for (int l = 0; l < M->cfg.n_layers; ++l) {
+    const LayerSpec& s = M->specs[l];
+    const std::string p = "l" + std::to_string(l) + ".";
+    v.push_back(p + "norm1");
+    std::vector<const char*> mix = {"q", "k", "v", "g", "o"};
+    if (is_latent(s)) {
+      mix = {"dq", "dq.norm", "uq", "uk", "uv", "g", "o"};
+      if (s.c.kv_from < 0) { mix.push_back("dkv"); mix.push_back("dkv.norm"); }
+    }
+    for (const char* t : mix) v.push_back(p + "mix." + t);
+    if (s.c.ff) { v.push_back(p + "mlp.up"); v.push_back(p + "mlp.down"); }
+  }
+  return v;
+}
+
+int32_t layered_set_weight(Model* M, const char* name, const float* host, int32_t rank, const int64_t* dims, int32_t layout) {
+  Ctx* ctx = M->ctx;
+  Target t;
+  if (!find_target(M, name, &t)) return fail(LMB200_ENOTFOUND, "set_weight: unknown tensor '%s'", name);
+  LMB_TRY(check_weight_shape(name, rank, dims, t.rows, t.cols));
+  float* stage = nullptr;
+  LMB_TRY(dmalloc((void**)&stage, t.rows * t.cols * 4, false, ctx->stream));
+  int32_t rc = LMB200_OK;
+  if (cudaMemcpyAsync(stage, host, (size_t)(t.rows * t.cols) * 4, cudaMemcpyHostToDevice, ctx->stream) != cudaSuccess)
+    rc = fail(LMB200_ECUDA, "set_weight: upload failed");
+  if (rc == LMB200_OK) rc = fill_target(M, t, 0, stage, layout, 0.f);
+  cudaStreamSynchronize(ctx->stream);
+  cudaFree(stage);
+  if (rc == LMB200_OK) M->weights_set.insert(name);
+  return rc;
+}
+
+int32_t layered_init_random(Model* M, uint64_t seed, float sigma) {
+  Ctx* ctx = M->ctx;
+  LMB_CUDA(cudaSetDevice(ctx->device));
+  uint64_t id = kIdLayered;
+  for (const std::string& n : layered_weight_names(M)) {
+    Target t;
+    if (!find_target(M, n, &t)) return fail(LMB200_EINVAL, "init_random: '%s'", n.c_str());
+    LMB_TRY(fill_target(M, t, stream_key(seed, id++), nullptr, LMB200_ROWMAJOR, sigma / 131072.0f));
+  }
+  LMB_CUDA(cudaStreamSynchronize(ctx->stream));
+  M->all_weights_set = true;
+  return LMB200_OK;
+}
+
+// ---------------------------------------------------------------------------------------------
+// session
+// ---------------------------------------------------------------------------------------------
+namespace {
+
+template <typename F>
+int64_t max_over(const Model* M, F f) {
+  int64_t m = 0;
+  for (const LayerSpec& s : M->specs) m = std::max<int64_t>(m, f(s));
+  return m;
+}
+
+void free_rows(RowsBuf& r) {
+  cudaFree(r.base);
+  r = RowsBuf();
+}
+
+// the buffers for T tokens, carved out of one allocation (a larger request replaces it)
+int32_t ensure_rows(Session* S, RowsBuf& r, int64_t T, int64_t n_want) {
+  const Model* M = S->m;
+  const int64_t e = M->esz, W = M->cfg.hidden;
+  const int64_t need_meta = 4 * T + 3 * S->B + n_want;
+  if (T <= r.cap_T && need_meta <= 4 * r.cap_T + 3 * S->B + r.cap_T) return LMB200_OK;
+  T = std::max<int64_t>(T, r.cap_T);
+  free_rows(r);
+  const int64_t blk = std::min<int64_t>(T, kBlockTokens);
+  struct Piece { void** p; int64_t bytes; };
+  const Piece pieces[] = {
+      {(void**)&r.x, T * W * 4},
+      {(void**)&r.delta, T * W * 4},
+      {&r.xn, T * row_ld((int)W) * e},
+      {(void**)&r.proj, T * max_over(M, [&](const LayerSpec& s) { return is_latent(s) ? (int64_t)s.n_store * 4 : (int64_t)s.n_store * e; })},
+      {&r.xq, T * row_ld((int)max_over(M, [](const LayerSpec& s) { return s.c.q_rank; })) * e},
+      {&r.q, T * max_over(M, [](const LayerSpec& s) { return is_latent(s) ? q_width(s) : 0; }) * e},
+      {&r.qa, blk * max_over(M, [](const LayerSpec& s) { return is_latent(s) ? (int64_t)s.c.heads * s.lat_ld : 0; }) * e},
+      {(void**)&r.olat, blk * max_over(M, [](const LayerSpec& s) { return is_latent(s) ? (int64_t)s.c.heads * s.c.kv_rank : 0; }) * 4},
+      {&r.cat, T * max_over(M, [](const LayerSpec& s) { return row_ld(s.m_out.K); }) * e},
+      {(void**)&r.meta, (5 * T + 3 * S->B) * 4},
+  };
+  int64_t total = 0;
+  for (const Piece& p : pieces) total += round_up(p.bytes, 256);
+  LMB_TRY(dmalloc(&r.base, total, true, M->ctx->stream));
+  char* at = reinterpret_cast<char*>(r.base);
+  for (const Piece& p : pieces) { *p.p = at; at += round_up(p.bytes, 256); }
+  r.bytes = total;
+  r.cap_T = T;
+  return LMB200_OK;
+}
+
+// x[t] <- embedding row (tokens given) or x[t] + delta[t]; xn[t] = RMSNorm(x[t]) w in the model dtype.  Rows in order, or the rows
+// `pick` chooses (then x itself is left alone).  capture [.., n]: the new row of every sequence's last token.
+template <typename WT>
+__global__ void __launch_bounds__(256) rows_norm_kernel(float* __restrict__ x, const float* __restrict__ delta, const int* __restrict__ tokens,
+                                                        const WT* __restrict__ embed, int vocab, const int* __restrict__ pick,
+                                                        const float* __restrict__ w, WT* __restrict__ xn, int ldn, int n, float eps,
+                                                        float* __restrict__ capture, const int* __restrict__ last) {
+  extern __shared__ float row[];
+  __shared__ float red[8];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int i0 = blockIdx.x, tid = threadIdx.x;
+  const int64_t t = pick ? pick[i0] : i0;
+  const int tok = tokens ? tokens[t] : 0;
+  const bool ok = tok >= 0 && tok < vocab;
+  const int cap = capture && !pick ? last[t] : -1;
+  float ss = 0.f;
+  for (int i = tid; i < n; i += 256) {
+    float v;
+    if (tokens) v = ok ? to_f32(embed[(int64_t)tok * n + i]) : 0.f;
+    else v = x[t * n + i] + (delta ? delta[t * n + i] : 0.f);
+    if (!pick) x[t * n + i] = v;
+    if (cap >= 0) capture[(int64_t)cap * n + i] = v;
+    row[i] = v;
+    ss += v * v;
+  }
+#pragma unroll
+  for (int off = 16; off > 0; off >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, off);
+  if ((tid & 31) == 0) red[tid >> 5] = ss;
+  __syncthreads();
+  float tot = 0.f;
+#pragma unroll
+  for (int i = 0; i < 8; ++i) tot += red[i];
+  const float inv = 1.0f / sqrtf(tot / (float)n + eps);
+  if (xn)
+    for (int i = tid; i < n; i += 256) xn[(int64_t)i0 * ldn + i] = from_f32<WT>(row[i] * inv * w[i]);
+}
+
+// float32 GEMM over many tokens on the CUDA cores: 64 rows x 64 tokens per CTA, W in the 16 x 32 tiles of the float32 layout
+__global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__ W, const float* __restrict__ X, int ldx, int T, int rows, int K,
+                                                       const RowSegs segs) {
+  __shared__ float ws[32][68], xs[32][68];              // [k][row], [k][token]
+  pdl_launch_dependents();
+  pdl_wait();
+  const int row0 = blockIdx.x * 64, t0 = blockIdx.y * 64, tid = threadIdx.x;
+  const int KC = (K + 31) >> 5, RB = (rows + 15) >> 4;
+  const int tr = (tid & 15) * 4, tt = (tid >> 4) * 4;
+  float acc[4][4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
+  for (int kc = 0; kc < KC; ++kc) {
+    for (int i = tid; i < 64 * 32; i += 256) {
+      const int r = i >> 5, k = i & 31;
+      ws[k][r] = ((row0 + r) >> 4) < RB ? W[wtile_offset(row0 + r, kc * 32 + k, KC)] : 0.f;
+      xs[k][r] = t0 + r < T && kc * 32 + k < K ? X[(int64_t)(t0 + r) * ldx + kc * 32 + k] : 0.f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < 32; ++k) {
+      const float4 a = *reinterpret_cast<const float4*>(&ws[k][tr]), b = *reinterpret_cast<const float4*>(&xs[k][tt]);
+      const float av[4] = {a.x, a.y, a.z, a.w}, bv[4] = {b.x, b.y, b.z, b.w};
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(av[i], bv[j], acc[i][j]);
+    }
+    __syncthreads();
+  }
+  for (int i = 0; i < 4; ++i) {
+    const int row = row0 + tr + i;
+    for (int s = 0; s < segs.n; ++s) {
+      const RowSeg sg = segs.s[s];
+      const int r = row - sg.row0;
+      if (r < 0 || r >= sg.rows) continue;
+      for (int j = 0; j < 4; ++j) {
+        if (t0 + tt + j >= T) continue;
+        float y = acc[i][j];
+        if (sg.kind == SEG_RELU2) { y = fmaxf(y, 0.f); y = y * y; }
+        else if (sg.kind == SEG_SILU) y = y / (1.0f + expf(-y));
+        else if (sg.kind == SEG_SOFTCAP && segs.softcap > 0.f) y = segs.softcap * tanhf(y / segs.softcap);
+        reinterpret_cast<float*>(sg.dst)[(int64_t)(t0 + tt + j) * sg.pitch + r] = y;
+      }
+    }
+  }
+}
+
+int32_t rows_gemm(const Model* M, const void* W, const WMap& m, const void* X, int ldx, int T, const RowSegs& segs, cudaStream_t st) {
+  Ctx* ctx = M->ctx;
+  if (M->cfg.dtype == LMB200_BF16) return gemm_segments_bf16(ctx, W, X, ldx, T, m.rows, m.K, segs, st);
+  LMB_REQUIRE(ceil_div(T, 64) <= 65535, "layered: %d tokens in one call", T);
+  LMB_CUDA(launch_k(gemm_f32_kernel, dim3((unsigned)ceil_div(m.rows, 64), (unsigned)ceil_div(T, 64)), dim3(256), 0, st, (const float*)W,
+                    (const float*)X, ldx, T, m.rows, m.K, segs));
+  ctx->launches++;
+  return LMB200_OK;
+}
+
+LatentView latent_view(const Session* S, int l) {
+  const Model* M = S->m;
+  const LayerSpec& s = M->specs[l];
+  LatentView v;
+  v.H = s.c.heads; v.dim = s.c.dim; v.vdim = s.c.vdim; v.q_rank = s.c.q_rank; v.kv_rank = s.c.kv_rank;
+  v.rot_dim = s.c.rot_dim; v.rot_dims = s.c.rot_dims; v.rot_interleaved = s.c.rot_layout == LMB200_ROT_INTERLEAVED;
+  v.rot = s.lat_rot; v.ld = s.lat_ld;
+  v.seq_stride = (int64_t)S->cap * s.lat_ld;
+  v.inv_freq = M->lw[l].inv_freq;
+  v.scale = s.c.scale; v.eps = M->cfg.rms_eps;
+  return v;
+}
+
+RetentionView retention_view(const Session* S, int l) {
+  const Model* M = S->m;
+  const LayerSpec& s = M->specs[l];
+  RetentionView v;
+  v.B = S->B;
+  v.H = s.c.heads; v.dim = s.c.dim; v.vdim = s.c.vdim; v.rot_dims = s.c.rot_dims;
+  v.rot_interleaved = s.c.rot_layout == LMB200_ROT_INTERLEAVED;
+  v.inv_freq = M->lw[l].inv_freq; v.decay = M->lw[l].decay; v.decay_pitch = kDecayPow;
+  v.eps = M->cfg.rms_eps;
+  v.state = S->state[l];
+  return v;
+}
+
+// What a rows step runs over: packed tokens and, on the host, how they divide into sequences (empty: one token per sequence)
+struct RowsRun {
+  int T = 0;
+  const int *tokens = nullptr, *seq = nullptr, *pos = nullptr, *last = nullptr, *start = nullptr, *len = nullptr, *pos0 = nullptr;
+  int max_len = 1;
+  int ctx_len = 0;                       // no token looks at more positions than this
+  std::vector<int> h_start, h_len, h_pos0;
+};
+
+template <typename WT>
+int32_t norm_rows(Session* S, RowsBuf& r, const RowsRun& run, int n_rows, const float* delta, bool embed, const int* pick, const float* w, void* xn,
+                  float* capture, cudaStream_t st) {
+  const Model* M = S->m;
+  const int W = M->cfg.hidden;
+  LMB_CUDA(launch_k(rows_norm_kernel<WT>, dim3((unsigned)n_rows), dim3(256), (size_t)W * 4, st, r.x, delta, embed ? run.tokens : (const int*)nullptr,
+                    (const WT*)M->embed, M->cfg.vocab, pick, w, (WT*)xn, row_ld(W), W, M->cfg.rms_eps, capture, run.last));
+  M->ctx->launches++;
+  return LMB200_OK;
+}
+
+int32_t latent_rows(Session* S, RowsBuf& r, const RowsRun& run, int l, bool graph, cudaStream_t st) {
+  Model* M = S->m;
+  Ctx* ctx = M->ctx;
+  const LayerSpec& s = M->specs[l];
+  LayeredWeights& w = M->lw[l];
+  LayeredScratch& Z = *S->lay;
+  const int dt = M->cfg.dtype, T = run.T, e = M->esz, ldc = row_ld(s.m_out.K), ldq = row_ld(s.c.q_rank);
+  const bool own = s.c.kv_from < 0;
+  RowSegs in;
+  in.add(s.row0[L_DQ], s.c.q_rank, SEG_F32, r.proj + s.row0[L_DQ], s.n_store);
+  if (own) in.add(s.row0[L_DKV], s.c.kv_rank + s.c.rot_dim, SEG_F32, r.proj + s.row0[L_DKV], s.n_store);
+  in.add(s.row0[L_G], s.c.heads, SEG_F32, r.proj + s.row0[L_G], s.n_store);
+  if (s.c.ff) in.add(s.row0[L_UP], s.c.ff, SEG_RELU2, (char*)r.cat + (int64_t)s.cat0 * e, ldc);
+  LMB_TRY(rows_gemm(M, w.w_in, s.m_in, r.xn, row_ld(M->cfg.hidden), T, in, st));
+  LatentView v = latent_view(S, l);
+  v.T = T; v.seq = run.seq; v.pos = run.pos;
+  void* cache = S->latent[cache_layer(M, l)];
+  LMB_TRY(latent_prep(ctx, dt, v, r.proj, s.n_store, s.row0[L_DQ], own ? s.row0[L_DKV] : 0, w.q_norm, w.kv_norm, r.xq, ldq, 0,
+                      own ? cache : nullptr, st));
+  RowSegs qs;
+  qs.add(0, q_width(s), SEG_ACT, r.q, q_width(s));
+  LMB_TRY(rows_gemm(M, w.w_uq, s.m_uq, r.xq, ldq, T, qs, st));
+  for (int t0 = 0; t0 < T; t0 += kBlockTokens) {
+    LatentView b = v;
+    b.T = std::min(kBlockTokens, T - t0); b.seq = run.seq + t0; b.pos = run.pos + t0;
+    LMB_TRY(latent_absorb(ctx, dt, b, (const char*)r.q + (int64_t)t0 * q_width(s) * e, 0, w.w_uk, r.qa, st));
+    LatentAttnPlan plan = graph ? Z.attn : latent_attn_plan(ctx, dt, b.T, b.H, b.kv_rank, run.ctx_len);
+    float* part = graph ? Z.attn_part : Z.prompt_part;
+    unsigned* counters = graph ? Z.attn_counters : Z.prompt_counters;
+    LMB_REQUIRE(graph || (plan.part_floats <= Z.prompt_part_floats && plan.counters <= Z.prompt_counter_cap), "layered: attention scratch");
+    LMB_TRY(latent_attend(ctx, dt, b, r.qa, cache, plan, part, counters, r.olat, st));
+    LMB_TRY(latent_expand(ctx, dt, b, r.olat, w.w_uv, r.proj + (int64_t)t0 * s.n_store + s.row0[L_G], s.n_store,
+                          (char*)r.cat + (int64_t)t0 * ldc * e, ldc, 0, st));
+  }
+  return LMB200_OK;
+}
+
+int32_t retention_rows(Session* S, RowsBuf& r, const RowsRun& run, int l, cudaStream_t st) {
+  Model* M = S->m;
+  Ctx* ctx = M->ctx;
+  const LayerSpec& s = M->specs[l];
+  LayeredWeights& w = M->lw[l];
+  const int dt = M->cfg.dtype, T = run.T, e = M->esz, ldc = row_ld(s.m_out.K);
+  char* proj = reinterpret_cast<char*>(r.proj);
+  auto at = [&](int slot) { return (void*)(proj + (int64_t)s.row0[slot] * e); };
+  RowSegs in;
+  in.add(s.row0[R_Q], s.c.heads * s.c.dim, SEG_ACT, at(R_Q), s.n_store);
+  in.add(s.row0[R_K], s.c.heads * s.c.dim, SEG_ACT, at(R_K), s.n_store);
+  in.add(s.row0[R_V], out_width(s), SEG_ACT, at(R_V), s.n_store);
+  in.add(s.row0[R_G], out_width(s), SEG_SILU, at(R_G), s.n_store);
+  if (s.c.ff) in.add(s.row0[R_UP], s.c.ff, SEG_RELU2, (char*)r.cat + (int64_t)s.cat0 * e, ldc);
+  LMB_TRY(rows_gemm(M, w.w_in, s.m_in, r.xn, row_ld(M->cfg.hidden), T, in, st));
+  RetentionView v = retention_view(S, l);
+  v.start = run.start; v.len = run.len; v.pos0 = run.pos0; v.max_len = run.max_len;
+  v.q = at(R_Q); v.k = at(R_K); v.v = at(R_V); v.g = at(R_G);
+  v.q_pitch = v.k_pitch = v.v_pitch = v.g_pitch = s.n_store;
+  v.in_f32 = dt != LMB200_BF16; v.raw_gate = 0;
+  v.out = r.cat; v.ldo = ldc; v.bp = 0;
+  return retention_steps(ctx, dt, v, st);
+}
+
+// one pass over packed tokens; the residual rows of the last layer are left in x + delta (in x where outputs are captured)
+int32_t rows_step(Session* S, RowsBuf& r, const RowsRun& run, bool graph, cudaStream_t st) {
+  Model* M = S->m;
+  const int W = M->cfg.hidden, L = M->cfg.n_layers, bf = M->cfg.dtype == LMB200_BF16;
+  for (int l = 0; l < L; ++l) {
+    float* cap = S->capture_on && l > 0 ? S->capture + (int64_t)(l - 1) * S->B * W : nullptr;
+    const float* delta = l ? r.delta : nullptr;
+    LMB_TRY(bf ? norm_rows<__nv_bfloat16>(S, r, run, run.T, delta, l == 0, nullptr, M->lw[l].norm, r.xn, cap, st)
+               : norm_rows<float>(S, r, run, run.T, delta, l == 0, nullptr, M->lw[l].norm, r.xn, cap, st));
+    const LayerSpec& s = M->specs[l];
+    LMB_TRY(is_latent(s) ? latent_rows(S, r, run, l, graph, st) : retention_rows(S, r, run, l, st));
+    RowSegs out;
+    out.add(0, W, SEG_F32, r.delta, W);
+    LMB_TRY(rows_gemm(M, M->lw[l].w_out, s.m_out, r.cat, row_ld(s.m_out.K), run.T, out, st));
+  }
+  if (S->capture_on) {
+    float* cap = S->capture + (int64_t)(L - 1) * S->B * W;
+    LMB_TRY(norm_rows<float>(S, r, run, run.T, r.delta, false, nullptr, nullptr, nullptr, cap, st));
+  }
+  return LMB200_OK;
+}
+
+// final norm and head on the rows `pick` chooses: logits [n, pitch]
+int32_t rows_head(Session* S, RowsBuf& r, const RowsRun& run, const int* pick, int n, void* xn, float* logits, int pitch, cudaStream_t st) {
+  Model* M = S->m;
+  const int W = M->cfg.hidden;
+  const float* delta = S->capture_on ? nullptr : r.delta;
+  LMB_TRY(M->cfg.dtype == LMB200_BF16 ? norm_rows<__nv_bfloat16>(S, r, run, n, delta, false, pick, M->final_norm, xn, nullptr, st)
+                                      : norm_rows<float>(S, r, run, n, delta, false, pick, M->final_norm, xn, nullptr, st));
+  RowSegs h;
+  h.add(0, M->cfg.vocab, SEG_SOFTCAP, logits, pitch);
+  h.softcap = M->softcap;
+  return rows_gemm(M, M->lm_head, M->m_head, xn, row_ld(W), n, h, st);
+}
+
+// bf16, one token per sequence
+int32_t fused_step(Session* S, cudaStream_t st, bool with_head) {
+  Model* M = S->m;
+  Ctx* ctx = M->ctx;
+  LayeredScratch& Z = *S->lay;
+  const int B = S->B, hid = M->cfg.hidden, L = M->cfg.n_layers, dt = LMB200_BF16;
+  LMB_TRY(embed_prep_launch(S, M->lw[0].norm, st));
+  int tiles = (int)ceil_div(hid, S->embed_rows_per_cta);
+  auto inv_scale = [&]() { InvScale iv; iv.ssq = S->ssq; iv.tiles = tiles; iv.n = hid; iv.eps = M->cfg.rms_eps; return iv; };
+  for (int l = 0; l < L; ++l) {
+    const LayerSpec& s = M->specs[l];
+    LayeredWeights& w = M->lw[l];
+    {
+      GemvParams p = gemv_params(S, w.w_in, s.m_in, Z.p_in[l], S->xn);
+      p.epi = EPI_STORE_RELU2; p.inv = inv_scale();
+      p.out = Z.proj; p.out_pitch = s.n_store; p.act_row0 = s.n_store; p.act = S->act; p.act_col0 = s.cat0; p.n_act = s.c.ff;
+      if (is_latent(s)) gemv_prefetch_next(p, ctx, dt, w.w_uq, s.m_uq.rows, s.m_uq.K, Z.p_uq[l]);
+      else gemv_prefetch_next(p, ctx, dt, w.w_out, s.m_out.rows, s.m_out.K, Z.p_out[l]);
+      LMB_TRY(gemv_launch(ctx, dt, p, st));
+    }
+    if (is_latent(s)) {
+      const bool own = s.c.kv_from < 0;
+      LatentView v = latent_view(S, l);
+      v.T = B; v.seq = Z.iota; v.pos = S->pos;
+      void* cache = S->latent[cache_layer(M, l)];
+      LMB_TRY(latent_prep(ctx, dt, v, Z.proj, s.n_store, s.row0[L_DQ], own ? s.row0[L_DKV] : 0, w.q_norm, w.kv_norm, Z.xq, 0, S->Bp,
+                          own ? cache : nullptr, st));
+      GemvParams p = gemv_params(S, w.w_uq, s.m_uq, Z.p_uq[l], Z.xq);
+      p.epi = EPI_STORE_F32; p.out = Z.qf; p.out_pitch = q_width(s);
+      gemv_prefetch_next(p, ctx, dt, w.w_out, s.m_out.rows, s.m_out.K, Z.p_out[l]);
+      LMB_TRY(gemv_launch(ctx, dt, p, st));
+      LMB_TRY(latent_absorb(ctx, dt, v, Z.qf, 1, w.w_uk, Z.qa, st));
+      LMB_TRY(latent_attend(ctx, dt, v, Z.qa, cache, Z.attn, Z.attn_part, Z.attn_counters, Z.olat, st));
+      LMB_TRY(latent_expand(ctx, dt, v, Z.olat, w.w_uv, Z.proj + s.row0[L_G], s.n_store, S->act, 0, S->Bp, st));
+    } else {
+      RetentionView v = retention_view(S, l);
+      v.start = Z.iota; v.len = Z.ones; v.pos0 = S->pos;
+      v.q = Z.proj + s.row0[R_Q]; v.k = Z.proj + s.row0[R_K]; v.v = Z.proj + s.row0[R_V]; v.g = Z.proj + s.row0[R_G];
+      v.q_pitch = v.k_pitch = v.v_pitch = v.g_pitch = s.n_store;
+      v.in_f32 = 1; v.raw_gate = 1;
+      v.out = S->act; v.bp = S->Bp;
+      LMB_TRY(retention_steps(ctx, dt, v, st));
+    }
+    {
+      GemvParams p = gemv_params(S, w.w_out, s.m_out, Z.p_out[l], S->act);
+      p.epi = EPI_RESID_NORM;
+      p.rn.x = S->xT; p.rn.gain = l + 1 < L ? M->lw[l + 1].norm : M->final_norm; p.rn.xg = S->xn; p.rn.ssq = S->ssq;
+      p.rn.capture = S->capture_on ? S->capture + (int64_t)l * B * hid : nullptr;
+      if (l + 1 < L) gemv_prefetch_next(p, ctx, dt, M->lw[l + 1].w_in, M->specs[l + 1].m_in.rows, M->specs[l + 1].m_in.K, Z.p_in[l + 1]);
+      else if (with_head) gemv_prefetch_next(p, ctx, dt, M->lm_head, M->m_head.rows, M->m_head.K, S->p_head);
+      LMB_TRY(gemv_launch(ctx, dt, p, st));
+      tiles = gemv_plan_ctas(Z.p_out[l], s.m_out.rows);
+    }
+  }
+  if (with_head) {
+    GemvParams p = gemv_params(S, M->lm_head, M->m_head, S->p_head, S->xn);
+    p.epi = EPI_STORE_F32; p.inv = inv_scale(); p.out = S->logits; p.out_pitch = S->logits_pitch; p.softcap = M->softcap;
+    LMB_TRY(gemv_launch(ctx, dt, p, st));
+  }
+  return LMB200_OK;
+}
+
+RowsRun decode_run(const Session* S) {
+  const LayeredScratch& Z = *S->lay;
+  RowsRun run;
+  run.T = S->B;
+  run.tokens = S->tokens; run.seq = Z.iota; run.pos = S->pos; run.last = Z.iota;
+  run.start = Z.iota; run.len = Z.ones; run.pos0 = S->pos;
+  run.ctx_len = S->cap;
+  return run;
+}
+
+int32_t ensure_want(Session* S, int64_t n) {
+  LayeredScratch& Z = *S->lay;
+  if (n <= Z.want_cap) return LMB200_OK;
+  cudaFree(Z.want_logits); cudaFree(Z.want_xn);
+  Z.want_logits = nullptr; Z.want_xn = nullptr; Z.want_cap = 0;
+  LMB_TRY(dmalloc((void**)&Z.want_logits, n * S->m->cfg.vocab * 4, false, S->m->ctx->stream));
+  LMB_TRY(dmalloc(&Z.want_xn, n * row_ld(S->m->cfg.hidden) * S->m->esz, true, S->m->ctx->stream));
+  Z.want_cap = n;
+  return LMB200_OK;
+}
+
+}  // namespace
+
+int32_t layered_enqueue_step(Session* S, cudaStream_t st, bool with_head) {
+  if (S->m->cfg.dtype == LMB200_BF16) {
+    LMB_TRY(fused_step(S, st, with_head));
+  } else {
+    LayeredScratch& Z = *S->lay;
+    const RowsRun run = decode_run(S);
+    LMB_TRY(rows_step(S, Z.step, run, true, st));
+    if (with_head) LMB_TRY(rows_head(S, Z.step, run, Z.iota, S->B, Z.step.xn, S->logits, S->logits_pitch, st));
+  }
+  if (with_head) LMB_TRY(argmax_launch(S, st));
+  return advance_launch(S, st);
+}
+
+int32_t layered_session_create(Model* M, int batch, int max_ctx, lmb200_session* out) {
+  Ctx* ctx = M->ctx;
+  LMB_CUDA(cudaSetDevice(ctx->device));
+  const lmb200_model_config& c = M->cfg;
+  const bool bf = c.dtype == LMB200_BF16;
+  Session* S = new Session();
+  S->m = M; S->B = batch; S->max_ctx = max_ctx;
+  S->cap = (int)round_up(max_ctx, 64);
+  S->Bp = bf ? Layout<__nv_bfloat16>::batch_pad(batch) : Layout<float>::batch_pad(batch);
+  S->logits_pitch = (int)round_up(c.vocab, 16);
+  S->lay = new LayeredScratch();
+  LayeredScratch& Z = *S->lay;
+  int32_t rc = LMB200_OK;
+  auto alloc = [&](void** p, int64_t bytes) { if (rc == LMB200_OK) rc = dmalloc(p, bytes, true, ctx->stream); };
+  S->latent.assign(c.n_layers, nullptr);
+  S->state.assign(c.n_layers, nullptr);
+  int64_t lat_parts = 0, lat_counters = 0, prompt_parts = 0, prompt_counters = 0;
+  for (int l = 0; l < c.n_layers; ++l) {
+    const LayerSpec& s = M->specs[l];
+    if (!is_latent(s)) { alloc((void**)&S->state[l], (int64_t)batch * s.c.heads * s.c.dim * state_ld(s) * 4); continue; }
+    if (s.c.kv_from < 0) alloc(&S->latent[l], (int64_t)batch * S->cap * s.lat_ld * M->esz);
+  }
+  // one plan serves every latent layer: sized for the widest of them
+  const int heads = (int)max_over(M, [](const LayerSpec& s) { return is_latent(s) ? s.c.heads : 0; });
+  const int kvr = (int)max_over(M, [](const LayerSpec& s) { return is_latent(s) ? s.c.kv_rank : 0; });
+  if (heads) {
+    Z.attn = latent_attn_plan(ctx, c.dtype, batch, heads, kvr, S->cap);
+    lat_parts = Z.attn.part_floats; lat_counters = Z.attn.counters;
+    for (int T = 1; T <= kBlockTokens; T *= 2) {
+      const LatentAttnPlan p = latent_attn_plan(ctx, c.dtype, T, heads, kvr, S->cap);
+      prompt_parts = std::max(prompt_parts, 2 * p.part_floats); prompt_counters = std::max(prompt_counters, 2 * p.counters);
+    }
+    Z.prompt_part_floats = prompt_parts; Z.prompt_counter_cap = prompt_counters;
+  }
+  if (bf) {
+    int64_t max_part = 0;
+    int max_cnt = 0;
+    auto take = [&](const GemvPlan& g) { max_part = std::max(max_part, g.partial_floats); max_cnt = std::max(max_cnt, g.n_counters); return g; };
+    for (const LayerSpec& s : M->specs) {
+      Z.p_in.push_back(take(gemv_plan(ctx, c.dtype, batch, s.m_in.rows, s.m_in.K)));
+      Z.p_uq.push_back(is_latent(s) ? take(gemv_plan(ctx, c.dtype, batch, s.m_uq.rows, s.m_uq.K)) : GemvPlan());
+      Z.p_out.push_back(take(gemv_plan_resid(ctx, batch, s.m_out.rows, s.m_out.K)));
+      if (Z.p_out.back().cluster < 1 && rc == LMB200_OK) rc = fail(LMB200_EINVAL, "session_create: width %d has more than one wave of row groups", c.hidden);
+    }
+    S->p_head = take(gemv_plan(ctx, c.dtype, batch, M->m_head.rows, M->m_head.K));
+    S->embed_rows_per_cta = 32 * (int)ceil_div(c.hidden, 32 * 256);
+    auto x_bytes = [&](int64_t K) { return Layout<__nv_bfloat16>::x_elems((int)K, S->Bp) * 2; };
+    alloc(&S->xn, x_bytes(c.hidden));
+    alloc(&S->act, x_bytes(max_over(M, [](const LayerSpec& s) { return s.m_out.K; })));
+    alloc((void**)&S->xT, (int64_t)round_up(c.hidden, 128) * S->Bp * 4);
+    alloc((void**)&S->ssq, (int64_t)256 * 32 * 4);
+    alloc((void**)&S->gemv_partials, max_part * 4);
+    alloc((void**)&S->gemv_counters, (int64_t)max_cnt * 4);
+    alloc((void**)&Z.proj, batch * max_over(M, [](const LayerSpec& s) { return s.n_store; }) * 4);
+    alloc((void**)&Z.qf, batch * max_over(M, [](const LayerSpec& s) { return is_latent(s) ? q_width(s) : 0; }) * 4);
+    alloc(&Z.xq, x_bytes(std::max<int64_t>(1, max_over(M, [](const LayerSpec& s) { return s.c.q_rank; }))));
+    alloc(&Z.qa, batch * max_over(M, [](const LayerSpec& s) { return is_latent(s) ? (int64_t)s.c.heads * s.lat_ld : 0; }) * 2);
+    alloc((void**)&Z.olat, batch * max_over(M, [](const LayerSpec& s) { return is_latent(s) ? (int64_t)s.c.heads * s.c.kv_rank : 0; }) * 4);
+    S->fused = true;
+  } else if (rc == LMB200_OK) {
+    rc = ensure_rows(S, Z.step, batch, 0);
+  }
+  alloc((void**)&Z.attn_part, lat_parts * 4);
+  alloc((void**)&Z.attn_counters, lat_counters * 4);
+  alloc((void**)&Z.prompt_part, prompt_parts * 4);
+  alloc((void**)&Z.prompt_counters, prompt_counters * 4);
+  alloc((void**)&S->logits, (int64_t)batch * S->logits_pitch * 4);
+  alloc((void**)&S->tokens, (int64_t)batch * 4);
+  alloc((void**)&S->pos, (int64_t)batch * 4);
+  alloc((void**)&S->limit, (int64_t)batch * 4);
+  alloc((void**)&S->step_ctr, 4);
+  alloc((void**)&S->stop, (int64_t)(2 + batch) * 4);
+  alloc((void**)&S->tok_hist, (int64_t)(S->cap + 1) * batch * 4);
+  alloc((void**)&Z.iota, (int64_t)batch * 4);
+  alloc((void**)&Z.ones, (int64_t)batch * 4);
+  S->host_pos_v.assign(batch, 0);
+  if (rc == LMB200_OK) {
+    std::vector<int> iota(batch), ones(batch, 1), limit(batch, 0x7fffffff);
+    for (int b = 0; b < batch; ++b) iota[b] = b;
+    const int no_eot = -1;
+    const bool ok = cudaMemcpyAsync(Z.iota, iota.data(), batch * 4, cudaMemcpyHostToDevice, ctx->stream) == cudaSuccess &&
+                    cudaMemcpyAsync(Z.ones, ones.data(), batch * 4, cudaMemcpyHostToDevice, ctx->stream) == cudaSuccess &&
+                    cudaMemcpyAsync(S->limit, limit.data(), batch * 4, cudaMemcpyHostToDevice, ctx->stream) == cudaSuccess &&
+                    cudaMemcpyAsync(S->stop, &no_eot, 4, cudaMemcpyHostToDevice, ctx->stream) == cudaSuccess &&
+                    cudaStreamSynchronize(ctx->stream) == cudaSuccess;
+    if (!ok) rc = fail(LMB200_ECUDA, "session_create: upload failed");
+  }
+  if (rc != LMB200_OK) { lmb200_session_destroy(reinterpret_cast<lmb200_session>(S)); return rc; }
+  *out = reinterpret_cast<lmb200_session>(S);
+  return LMB200_OK;
+}
+
+void layered_session_free(Session* S) {
+  for (void* p : S->latent) cudaFree(p);
+  for (float* p : S->state) cudaFree(p);
+  S->latent.clear();
+  S->state.clear();
+  if (!S->lay) return;
+  LayeredScratch& Z = *S->lay;
+  cudaFree(Z.proj); cudaFree(Z.qf); cudaFree(Z.olat); cudaFree(Z.xq); cudaFree(Z.qa); cudaFree(Z.iota); cudaFree(Z.ones);
+  cudaFree(Z.attn_part); cudaFree(Z.attn_counters); cudaFree(Z.prompt_part); cudaFree(Z.prompt_counters);
+  cudaFree(Z.want_logits); cudaFree(Z.want_xn);
+  free_rows(Z.step);
+  free_rows(Z.prompt);
+  delete S->lay;
+  S->lay = nullptr;
+}
+
+int32_t layered_check_positions(const Session* S, const int32_t* pos) {
+  if (!layered_has_state(S->m)) return LMB200_OK;
+  for (int b = 0; b < S->B; ++b)
+    if (pos[b] != 0 && pos[b] != S->host_pos_v[b])
+      return fail(LMB200_ESTATE, "set_position: sequence %d is at %d; its recurrent state cannot be moved to position %d (0 empties it)", b,
+                  S->host_pos_v[b], pos[b]);
+  return LMB200_OK;
+}
+
+int32_t layered_clear_state(Session* S, const int32_t* new_pos) {
+  const Model* M = S->m;
+  for (int l = 0; l < M->cfg.n_layers; ++l) {
+    if (!S->state[l]) continue;
+    const LayerSpec& s = M->specs[l];
+    const int64_t per = (int64_t)s.c.heads * s.c.dim * state_ld(s);
+    for (int b = 0; b < S->B; ++b)
+      if (new_pos[b] == 0) LMB_CUDA(cudaMemsetAsync(S->state[l] + b * per, 0, (size_t)per * 4, M->ctx->stream));
+  }
+  return LMB200_OK;
+}
+
+int32_t layered_fill_random(Session* S, int32_t n_pos, uint64_t seed) {
+  Model* M = S->m;
+  const float scale = 1.0f / 131072.0f;
+  for (int l = 0; l < M->cfg.n_layers; ++l) {
+    const LayerSpec& s = M->specs[l];
+    const uint64_t key = stream_key(seed, kIdLayeredState + l);
+    if (S->latent[l]) {
+      if (n_pos == 0) continue;
+      for (int b = 0; b < S->B; ++b) {
+        char* base = reinterpret_cast<char*>(S->latent[l]) + (int64_t)b * S->cap * s.lat_ld * M->esz;
+        LMB_TRY(fill_plain_dt(M, M->cfg.dtype, base, n_pos, s.lat_ld, key + b, nullptr, 0, scale, 0.f));
+      }
+    } else if (S->state[l]) {
+      const int64_t rows = (int64_t)S->B * s.c.heads * s.c.dim;
+      if (n_pos == 0) LMB_CUDA(cudaMemsetAsync(S->state[l], 0, (size_t)(rows * state_ld(s)) * 4, M->ctx->stream));
+      else LMB_TRY(fill_plain_dt(M, LMB200_F32, S->state[l], rows, state_ld(s), key, nullptr, 0, scale, 0.f));
+    }
+  }
+  return LMB200_OK;
+}
+
+int32_t layered_extend(Session* S, const int32_t* tokens, const int32_t* lengths, int32_t n_want, const int32_t* want, float* logits_out,
+                       bool greedy) {
+  Model* M = S->m;
+  Ctx* ctx = M->ctx;
+  LayeredScratch& Z = *S->lay;
+  const int B = S->B, V = M->cfg.vocab;
+  LMB_CUDA(cudaSetDevice(ctx->device));
+  int T = 0, max_len = 0, ctx_len = 0;
+  bool single = true;
+  for (int b = 0; b < B; ++b) {
+    T += lengths[b];
+    max_len = std::max(max_len, lengths[b]);
+    ctx_len = std::max(ctx_len, S->host_pos_v[b] + lengths[b]);
+    single = single && lengths[b] == 1;
+  }
+  LMB_CUDA(cudaMemsetAsync(S->step_ctr, 0, 4, ctx->stream));
+  if (single) {                                   // the decode step
+    LMB_CUDA(cudaMemcpyAsync(S->tokens, tokens, (size_t)B * 4, cudaMemcpyHostToDevice, ctx->stream));
+    LMB_TRY(run_step(S, n_want > 0, logits_out != nullptr));
+    for (int i = 0; i < n_want && logits_out; ++i)
+      LMB_CUDA(cudaMemcpyAsync(logits_out + (int64_t)i * V, S->logits + (int64_t)want[i] * S->logits_pitch, (size_t)V * 4, cudaMemcpyDeviceToHost,
+                               ctx->stream));
+    LMB_CUDA(cudaStreamSynchronize(ctx->stream));
+    return check_device_error(ctx);
+  }
+  LMB_TRY(ensure_rows(S, Z.prompt, T, n_want));
+  RowsBuf& r = Z.prompt;
+  std::vector<int> meta((size_t)4 * T + 3 * B + n_want);
+  RowsRun run;
+  run.T = T; run.max_len = max_len; run.ctx_len = ctx_len;
+  int at = 0;
+  for (int b = 0; b < B; ++b) {
+    run.h_start.push_back(at); run.h_len.push_back(lengths[b]); run.h_pos0.push_back(S->host_pos_v[b]);
+    meta[(size_t)4 * T + b] = at; meta[(size_t)4 * T + B + b] = lengths[b]; meta[(size_t)4 * T + 2 * B + b] = S->host_pos_v[b];
+    for (int i = 0; i < lengths[b]; ++i, ++at) {
+      meta[at] = tokens[at];
+      meta[(size_t)T + at] = b;
+      meta[(size_t)2 * T + at] = S->host_pos_v[b] + i;
+      meta[(size_t)3 * T + at] = i == lengths[b] - 1 ? b : -1;
+    }
+  }
+  for (int i = 0; i < n_want; ++i) meta[(size_t)4 * T + 3 * B + i] = want[i];
+  LMB_CUDA(cudaMemcpyAsync(r.meta, meta.data(), meta.size() * 4, cudaMemcpyHostToDevice, ctx->stream));
+  run.tokens = r.meta; run.seq = r.meta + T; run.pos = r.meta + 2 * (int64_t)T; run.last = r.meta + 3 * (int64_t)T;
+  run.start = r.meta + 4 * (int64_t)T; run.len = run.start + B; run.pos0 = run.len + B;
+  const int* want_dev = run.pos0 + B;
+  int32_t rc = rows_step(S, r, run, false, ctx->stream);
+  if (rc == LMB200_OK && n_want > 0) {
+    const bool to_session = greedy && n_want == B;
+    rc = ensure_want(S, n_want);
+    float* logits = to_session ? S->logits : Z.want_logits;
+    const int pitch = to_session ? S->logits_pitch : V;
+    if (rc == LMB200_OK) rc = rows_head(S, r, run, want_dev, n_want, Z.want_xn, logits, pitch, ctx->stream);
+    if (rc == LMB200_OK && to_session) rc = argmax_launch(S, ctx->stream);
+    if (rc == LMB200_OK && logits_out &&
+        cudaMemcpy2DAsync(logits_out, (size_t)V * 4, logits, (size_t)pitch * 4, (size_t)V * 4, (size_t)n_want, cudaMemcpyDeviceToHost, ctx->stream) !=
+            cudaSuccess)
+      rc = fail(LMB200_ECUDA, "extend: logits copy failed");
+  }
+  const cudaError_t e = cudaStreamSynchronize(ctx->stream);       // also: `meta` is host memory of this call
+  LMB_TRY(rc);
+  if (e != cudaSuccess) return fail(LMB200_ECUDA, "extend: %s", cudaGetErrorString(e));
+  for (int b = 0; b < B; ++b) S->host_pos_v[b] += lengths[b];
+  LMB_TRY(push_positions(S));
+  return check_device_error(ctx);
+}
+
+// bytes a decode step has to move: every weight once, latent rows of T positions per sequence (once for all heads, again for
+// each layer that borrows them), recurrent states read and written
+int64_t layered_step_bytes(const Session* S, int32_t T) {
+  const Model* M = S->m;
+  const int64_t e = M->esz, W = M->cfg.hidden, B = S->B;
+  int64_t n = (int64_t)M->cfg.vocab * W * e + W * 4 + B * W * e;
+  for (int l = 0; l < M->cfg.n_layers; ++l) {
+    const LayerSpec& s = M->specs[l];
+    auto mat = [&](const WMap& m) { int64_t k = 0; for (int i = 0; i < m.n_src; ++i) k += (int64_t)m.src_rows[i] * m.src_cols[i]; return k * e; };
+    n += mat(s.m_in) + mat(s.m_out) + W * 4;
+    if (is_latent(s)) n += mat(s.m_uq) + mat(s.m_ukv) + B * (int64_t)(T + (s.c.kv_from < 0 ? 1 : 0)) * (s.c.kv_rank + s.c.rot_dim) * e;
+    else n += 2 * B * (int64_t)s.c.heads * s.c.dim * s.c.vdim * 4;
+  }
+  return n;
+}
+
+int32_t layered_configure() {
+  LMB_TRY(latent_configure());
+  return retention_configure();
+}
+
+}  // namespace lmb
+
+using namespace lmb;
+
+extern "C" int32_t lmb200_model_create_layered(lmb200_ctx hctx, const lmb200_layered_config* cfg, const lmb200_layer_config* layers,
+                                               lmb200_model* out) {
+  Ctx* ctx = ctx_from(hctx);
+  if (!ctx) return LMB200_EINVAL;
+  LMB_REQUIRE(cfg && layers && out, "model_create_layered: null argument");
+  LMB_REQUIRE(cfg->n_layers >= 1 && cfg->width >= 1 && cfg->vocab >= 1, "model_create_layered: non-positive size");
+  LMB_REQUIRE(cfg->width <= 12288, "model_create_layered: width %d (at most 12288)", cfg->width);
+  LMB_REQUIRE(cfg->dtype == LMB200_F32 || cfg->dtype == LMB200_BF16, "model_create_layered: dtype %d", cfg->dtype);
+  LMB_REQUIRE(cfg->softcap >= 0.f && cfg->eps >= 0.f, "model_create_layered: softcap %g, eps %g", cfg->softcap, cfg->eps);
+  std::vector<LayerSpec> specs;
+  for (int l = 0; l < cfg->n_layers; ++l) {
+    LMB_TRY(check_layer(layers[l], specs, l));
+    LayerSpec s;
+    s.c = layers[l];
+    if (s.c.mixer == LMB200_MIXER_RETENTION) {
+      s.decay.assign(layers[l].decay, layers[l].decay + s.c.heads);
+      s.c.kv_from = -1; s.c.q_rank = s.c.kv_rank = s.c.rot_dim = 0;
+    }
+    s.c.decay = nullptr;
+    if (s.c.kv_from < 0) s.c.kv_from = -1;
+    derive_layer(s, cfg->width);
+    specs.push_back(s);
+  }
+  LMB_CUDA(cudaSetDevice(ctx->device));
+  Model* M = new Model();
+  M->ctx = ctx;
+  lmb200_model_config& c = M->cfg;
+  c.n_layers = cfg->n_layers; c.hidden = cfg->width; c.vocab = cfg->vocab; c.rms_eps = cfg->eps; c.dtype = cfg->dtype;
+  c.tp_size = 1; c.arch = LMB200_ARCH_LAYERED;
+  M->esz = c.dtype == LMB200_BF16 ? 2 : 4;
+  M->softcap = cfg->softcap;
+  M->specs = specs;
+  M->lw.resize(c.n_layers);
+  M->m_head.kind = MAP_PLAIN;
+  M->m_head.rows = c.vocab; M->m_head.K = c.hidden; M->m_head.src_rows[0] = c.vocab; M->m_head.src_cols[0] = c.hidden;
+  finish_map(M->m_head);
+  int32_t rc = LMB200_OK;
+  auto alloc = [&](void** p, int64_t bytes) {
+    if (rc != LMB200_OK) return;
+    rc = dmalloc(p, bytes, true, ctx->stream);
+    if (rc == LMB200_OK) M->weight_bytes += bytes;
+  };
+  auto upload = [&](float** p, const std::vector<float>& h) {
+    alloc((void**)p, (int64_t)h.size() * 4);
+    if (rc == LMB200_OK && !h.empty() && (cudaMemcpyAsync(*p, h.data(), h.size() * 4, cudaMemcpyHostToDevice, ctx->stream) != cudaSuccess ||
+                                          cudaStreamSynchronize(ctx->stream) != cudaSuccess))
+      rc = fail(LMB200_ECUDA, "model_create_layered: upload failed");
+  };
+  for (int l = 0; l < c.n_layers; ++l) {
+    const LayerSpec& s = M->specs[l];
+    LayeredWeights& w = M->lw[l];
+    alloc(&w.w_in, tiled_elems(s.m_in, c.dtype) * M->esz);
+    alloc(&w.w_out, tiled_elems(s.m_out, c.dtype) * M->esz);
+    alloc((void**)&w.norm, (int64_t)c.hidden * 4);
+    std::vector<float> f(s.c.rot_dims / 2);
+    for (int i = 0; i < s.c.rot_dims / 2; ++i) f[i] = (float)pow(s.c.rot_base, -2.0 * i / s.c.rot_dims);
+    upload(&w.inv_freq, f);
+    if (is_latent(s)) {
+      alloc(&w.w_uq, tiled_elems(s.m_uq, c.dtype) * M->esz);
+      alloc(&w.w_ukv, tiled_elems(s.m_ukv, c.dtype) * M->esz);
+      alloc(&w.w_uk, (int64_t)s.c.heads * s.c.dim * s.c.kv_rank * M->esz);
+      alloc(&w.w_uv, (int64_t)s.c.heads * s.c.vdim * s.c.kv_rank * M->esz);
+      alloc((void**)&w.q_norm, (int64_t)s.c.q_rank * 4);
+      if (s.c.kv_from < 0) alloc((void**)&w.kv_norm, (int64_t)s.c.kv_rank * 4);
+    } else {
+      std::vector<float> d((size_t)s.c.heads * kDecayPow);
+      for (int h = 0; h < s.c.heads; ++h)
+        for (int i = 0; i < kDecayPow; ++i) d[(size_t)h * kDecayPow + i] = (float)pow(s.decay[h], i);
+      upload(&w.decay, d);
+    }
+  }
+  alloc(&M->embed, (int64_t)c.vocab * c.hidden * M->esz);
+  alloc((void**)&M->final_norm, (int64_t)c.hidden * 4);
+  alloc(&M->lm_head, tiled_elems(M->m_head, c.dtype) * M->esz);
+  if (rc == LMB200_OK && cudaStreamSynchronize(ctx->stream) != cudaSuccess) rc = fail(LMB200_ECUDA, "model_create_layered: sync failed");
+  if (rc != LMB200_OK) { lmb200_model_destroy(reinterpret_cast<lmb200_model>(M)); return rc; }
+  *out = reinterpret_cast<lmb200_model>(M);
+  return LMB200_OK;
+}

@@ -60,17 +60,18 @@ __host__ __device__ inline bool wmap_resolve(const WMap& m, int i, int k, int* s
     case MAP_DOWN:
       *slot = 0; *lrow = i; *lcol = m.inter_off + k;
       return true;
+    case MAP_STACK:
+      for (int s = 0; s < m.n_src; ++s) {
+        const int r = i - m.row_off[s], c = k - m.col_off[s];
+        if (r >= 0 && r < m.src_rows[s] && c >= 0 && c < m.src_cols[s]) {
+          *slot = s; *lrow = r; *lcol = c;
+          return true;
+        }
+      }
+      return false;
   }
   return false;
 }
-
-struct FillSrc {
-  uint64_t key[3];
-  const float* src[3];     // staged logical tensors (NULL -> generator)
-  int colmajor;
-  int only_slot;           // -1: all
-  float scale;             // sigma / 131072
-};
 
 template <typename WT>
 __global__ void fill_tiled_kernel(WT* dst, WMap m, FillSrc f) {
@@ -750,12 +751,14 @@ enum Slot { S_ATTN_NORM = 0, S_Q = 1, S_K = 2, S_V = 3, S_O = 4, S_FFN_NORM = 5,
 constexpr uint64_t kIdEmbed = 0xFFFF0, kIdFinalNorm = 0xFFFF1, kIdHead = 0xFFFF2;
 constexpr uint64_t kIdKvBase = 0x100000;
 
+}  // namespace
+
 int64_t tiled_elems(const WMap& m, int dtype) {
   return dtype == LMB200_BF16 ? Layout<__nv_bfloat16>::w_elems(m.rows, m.K) : Layout<float>::w_elems(m.rows, m.K);
 }
 
 template <typename WT>
-int32_t fill_tiled(Ctx* ctx, void* dst, const WMap& m, const FillSrc& f) {
+static int32_t fill_tiled(Ctx* ctx, void* dst, const WMap& m, const FillSrc& f) {
   fill_tiled_kernel<WT><<<fill_grid((int64_t)m.rows * m.K), 256, 0, ctx->stream>>>(reinterpret_cast<WT*>(dst), m, f);
   ctx->launches++;
   LMB_CUDA(cudaGetLastError());
@@ -766,13 +769,19 @@ int32_t fill_tiled_dt(Model* M, void* dst, const WMap& m, const FillSrc& f) {
                                      : fill_tiled<float>(M->ctx, dst, m, f);
 }
 template <typename WT>
-int32_t fill_plain(Ctx* ctx, void* dst, int64_t rows, int64_t cols, uint64_t key, const float* src,
+static int32_t fill_plain(Ctx* ctx, void* dst, int64_t rows, int64_t cols, uint64_t key, const float* src,
                    int colmajor, float scale, float offset) {
   fill_plain_kernel<WT><<<fill_grid(rows * cols), 256, 0, ctx->stream>>>(reinterpret_cast<WT*>(dst), rows, cols, key,
                                                                          src, colmajor, scale, offset);
   ctx->launches++;
   LMB_CUDA(cudaGetLastError());
   return LMB200_OK;
+}
+
+int32_t fill_plain_dt(Model* M, int dtype, void* dst, int64_t rows, int64_t cols, uint64_t key, const float* src, int colmajor, float scale,
+                      float offset) {
+  return dtype == LMB200_BF16 ? fill_plain<__nv_bfloat16>(M->ctx, dst, rows, cols, key, src, colmajor, scale, offset)
+                              : fill_plain<float>(M->ctx, dst, rows, cols, key, src, colmajor, scale, offset);
 }
 
 void finish_map(WMap& m) {
@@ -792,7 +801,6 @@ int32_t dmalloc(void** p, int64_t bytes, bool zero, cudaStream_t st) {
   return LMB200_OK;
 }
 
-}  // namespace
 }  // namespace lmb
 
 using namespace lmb;
@@ -818,7 +826,8 @@ static int32_t derive_model(const lmb200_model_config& c, Model* M) {
   LMB_REQUIRE(c.intermediate % c.tp_size == 0 && (c.intermediate / c.tp_size) % 8 == 0,
               "model_create: intermediate %d / tp %d must be a multiple of 8", c.intermediate, c.tp_size);
   LMB_REQUIRE(c.hidden % 4 == 0, "model_create: hidden %d must be a multiple of 4", c.hidden);
-  LMB_REQUIRE(c.arch == LMB200_ARCH_LLAMA || c.arch == LMB200_ARCH_WHISPER_DECODER, "model_create: arch %d", c.arch);
+  LMB_REQUIRE(c.arch == LMB200_ARCH_LLAMA || c.arch == LMB200_ARCH_WHISPER_DECODER,
+              "model_create: arch %d (a decoder described layer by layer is created with lmb200_model_create_layered)", c.arch);
   if (c.arch == LMB200_ARCH_WHISPER_DECODER) {
     LMB_REQUIRE(c.n_kv_heads == c.n_heads && c.tp_size == 1, "model_create: the Whisper decoder has no GQA and no tensor parallelism");
     LMB_REQUIRE(c.max_positions >= 1 && c.cross_len >= 1, "model_create: Whisper needs max_positions and cross_len");
@@ -987,6 +996,7 @@ extern "C" int32_t lmb200_model_destroy(lmb200_model h) {
     cudaFree(L.b_o_cross); cudaFree(L.b_fc1); cudaFree(L.b_fc2);
     cudaFree(L.wg_qkv); cudaFree(L.bf_qkv); cudaFree(L.wg_qc); cudaFree(L.bf_qc); cudaFree(L.wg_fc1); cudaFree(L.bf_fc1);
   }
+  layered_free_model(M);
   cudaFree(M->final_norm_b); cudaFree(M->pos_emb); cudaFree(M->embed_tiled); cudaFree(M->wg_head); cudaFree(M->bf_head);
   cudaFree(M->embed); cudaFree(M->final_norm); cudaFree(M->lm_head); cudaFree(M->inv_freq);
   M->magic = 0;
@@ -1004,6 +1014,7 @@ extern "C" int32_t lmb200_model_weight_bytes(lmb200_model h, int64_t* bytes) {
 extern "C" int32_t lmb200_model_init_random(lmb200_model h, uint64_t seed, float sigma) {
   Model* M = model_from(h);
   if (!M) return LMB200_EINVAL;
+  if (M->cfg.arch == LMB200_ARCH_LAYERED) return layered_init_random(M, seed, sigma);
   LMB_REQUIRE(M->cfg.arch == LMB200_ARCH_LLAMA, "init_random: only for Llama-shaped models; set Whisper weights by name");
   Ctx* ctx = M->ctx;
   LMB_CUDA(cudaSetDevice(ctx->device));
@@ -1046,7 +1057,7 @@ extern "C" int32_t lmb200_model_init_random(lmb200_model h, uint64_t seed, float
 // The caller states the shape of what `host` points to; it must be the logical shape the model's
 // configuration gives the tensor (matrices [out, in]; vectors [n], [1, n] or [n, 1]), so that a
 // checkpoint of another width is refused instead of being read out of bounds.
-static int32_t check_weight_shape(const char* name, int32_t rank, const int64_t* dims, int64_t rows, int64_t cols) {
+int32_t lmb::check_weight_shape(const char* name, int32_t rank, const int64_t* dims, int64_t rows, int64_t cols) {
   LMB_REQUIRE(rank >= 1 && rank <= 2 && dims, "set_weight: '%s': rank %d (expected 1 or 2 with the dimensions given)", name, rank);
   const int64_t d0 = dims[0], d1 = rank == 2 ? dims[1] : 1;
   bool ok;
@@ -1071,6 +1082,7 @@ extern "C" int32_t lmb200_model_set_weight(lmb200_model h, const char* name, con
   Ctx* ctx = M->ctx;
   LMB_CUDA(cudaSetDevice(ctx->device));
   const lmb200_model_config& c = M->cfg;
+  if (c.arch == LMB200_ARCH_LAYERED) return layered_set_weight(M, name, host, rank, dims, layout);
   const std::string n(name);
   // resolve the name
   void* dst = nullptr;
@@ -1186,6 +1198,7 @@ extern "C" int32_t lmb200_model_set_weight(lmb200_model h, const char* name, con
 static std::vector<std::string> expected_weight_names(const Model* M) {
   std::vector<std::string> v;
   const lmb200_model_config& c = M->cfg;
+  if (c.arch == LMB200_ARCH_LAYERED) return layered_weight_names(M);
   char buf[160];
   if (c.arch == LMB200_ARCH_WHISPER_DECODER) {
     v = {"model.decoder.embed_tokens.weight", "model.decoder.embed_positions.weight", "model.decoder.layer_norm.weight",
@@ -1238,7 +1251,6 @@ extern "C" int32_t lmb200_model_missing_weights(lmb200_model h, char* names_out,
 // session
 // =============================================================================================
 namespace lmb {
-namespace {
 
 GemvParams gemv_params(Session* S, const void* W, const WMap& m, const GemvPlan& pl, const void* x) {
   GemvParams p;
@@ -1248,6 +1260,8 @@ GemvParams gemv_params(Session* S, const void* W, const WMap& m, const GemvPlan&
   p.partials = S->gemv_partials; p.counters = S->gemv_counters;
   return p;
 }
+
+namespace {
 
 // Partial-sum exchange of the two row-parallel projections of a layer (index 2l: o_proj, 2l + 1:
 // down_proj).  With the peer regions mapped, the projection writes this rank's partial into its
@@ -1414,6 +1428,34 @@ PeerPush peer_push(Session* S, int index) {
   return pp;
 }
 
+}  // namespace
+
+// first launch of a fused step: residual stream, first norm's input and its sums of squares from the embedding rows
+int32_t embed_prep_launch(Session* S, const float* gain, cudaStream_t st) {
+  const Model* M = S->m;
+  const int rows_per = S->embed_rows_per_cta, hid = M->cfg.hidden;
+  const dim3 grid((unsigned)ceil_div(hid, rows_per));
+  LMB_CUDA(launch_k(S->Bp == 16 ? embed_prep_kernel<16> : embed_prep_kernel<32>, grid, dim3(128), 0, st, (const int*)S->tokens,
+                    reinterpret_cast<const __nv_bfloat16*>(M->embed), M->cfg.vocab, hid, S->B, gain, S->xT,
+                    reinterpret_cast<__nv_bfloat16*>(S->xn), S->ssq, rows_per));
+  M->ctx->launches++;
+  return LMB200_OK;
+}
+
+int32_t argmax_launch(Session* S, cudaStream_t st) {
+  LMB_CUDA(launch_k(argmax_step_kernel, dim3(S->B), dim3(kArgmaxThreads), 0, st, (const float*)S->logits, S->logits_pitch, S->m->cfg.vocab,
+                    S->tokens, S->tok_hist, (const int*)S->step_ctr, S->B, S->stop));
+  S->m->ctx->launches++;
+  return LMB200_OK;
+}
+int32_t advance_launch(Session* S, cudaStream_t st) {
+  LMB_CUDA(launch_k(advance_kernel, dim3(1), dim3(32), 0, st, S->pos, (const int*)S->limit, S->B, S->step_ctr, (unsigned long long*)nullptr));
+  S->m->ctx->launches++;
+  return LMB200_OK;
+}
+
+namespace {
+
 // The fused decode step of a bf16 Llama / Phi-3: five launches per layer.  The residual add and the
 // RMSNorm around every Linear (src/NN.jl:406-414, 149-161) are carried by the projections themselves:
 // o_proj and down_proj finish with EPI_RESID_NORM (under tensor parallelism including the all-reduce of
@@ -1427,19 +1469,7 @@ int32_t enqueue_step_fused(Session* S, cudaStream_t st, int head) {
   const lmb200_model_config& c = M->cfg;
   const int dt = LMB200_BF16;
   const int B = S->B, hid = c.hidden, L = c.n_layers;
-  {
-    const int rows_per = S->embed_rows_per_cta;
-    const int grid = (int)ceil_div(hid, rows_per);
-    if (S->Bp == 16)
-      LMB_CUDA(launch_k(embed_prep_kernel<16>, dim3(grid), dim3(128), 0, st, (const int*)S->tokens,
-                        reinterpret_cast<const __nv_bfloat16*>(M->embed), c.vocab, hid, B, (const float*)M->layers[0].attn_norm,
-                        S->xT, reinterpret_cast<__nv_bfloat16*>(S->xn), S->ssq, rows_per));
-    else
-      LMB_CUDA(launch_k(embed_prep_kernel<32>, dim3(grid), dim3(128), 0, st, (const int*)S->tokens,
-                        reinterpret_cast<const __nv_bfloat16*>(M->embed), c.vocab, hid, B, (const float*)M->layers[0].attn_norm,
-                        S->xT, reinterpret_cast<__nv_bfloat16*>(S->xn), S->ssq, rows_per));
-    ctx->launches++;
-  }
+  LMB_TRY(embed_prep_launch(S, M->layers[0].attn_norm, st));
   int tiles = (int)ceil_div(hid, S->embed_rows_per_cta);        // slots of S->ssq the last producer wrote
   auto inv_scale = [&]() { InvScale iv; iv.ssq = S->ssq; iv.tiles = tiles; iv.n = hid; iv.eps = c.rms_eps; return iv; };
   for (int l = 0; l < L; ++l) {
@@ -1756,6 +1786,7 @@ int32_t enqueue_whisper_step_fused(Session* S, cudaStream_t st, bool with_head) 
 
 int32_t enqueue_step(Session* S, cudaStream_t st, int head) {
   const bool with_head = head != 0;
+  if (S->m->cfg.arch == LMB200_ARCH_LAYERED) return layered_enqueue_step(S, st, with_head);
   if (S->fused && S->m->cfg.arch == LMB200_ARCH_WHISPER_DECODER) return enqueue_whisper_step_fused(S, st, with_head);
   if (S->fused) return enqueue_step_fused(S, st, head);
   if (S->m->cfg.arch == LMB200_ARCH_WHISPER_DECODER)
@@ -1823,9 +1854,12 @@ int32_t ensure_graphs(Session* S) {
   return LMB200_OK;
 }
 
+}  // namespace
+}  // namespace lmb
+
 // with_head: the step ends in the head and the greedy token; want_logits: a caller will read the full logits after it
 // (under tensor parallelism the step otherwise computes only this rank's slice of them)
-int32_t run_step(Session* S, bool with_head, bool want_logits = true) {
+int32_t lmb::run_step(Session* S, bool with_head, bool want_logits) {
   Ctx* ctx = S->m->ctx;
   if (S->fused && S->m->cfg.arch == LMB200_ARCH_WHISPER_DECODER && !S->m->fold_valid) LMB_TRY(whisper_fold(S->m));
   LMB_TRY(ensure_graphs(S));
@@ -1839,12 +1873,9 @@ int32_t run_step(Session* S, bool with_head, bool want_logits = true) {
   return LMB200_OK;
 }
 
-}  // namespace
-}  // namespace lmb
-
 // Positions live on the device, one per sequence; the host keeps a copy for its bounds checks.  `ragged`
 // (the positions differ) selects the per-sequence RoPE path of the kernels, so changing it drops the graphs.
-static int32_t push_positions(Session* S) {
+int32_t lmb::push_positions(Session* S) {
   Ctx* ctx = S->m->ctx;
   bool ragged = false;
   int mx = 0;
@@ -1861,10 +1892,17 @@ static int32_t push_positions(Session* S) {
   }
   return LMB200_OK;
 }
-static int32_t set_all_positions(Session* S, int pos) {
-  S->host_pos_v.assign(S->B, pos);
+// Where the caller puts the sequences.  A recurrent state cannot be moved along with a position: only an empty state
+// (position 0) or the state as it is exists.
+static int32_t move_positions(Session* S, const std::vector<int>& pos) {
+  if (S->m->cfg.arch == LMB200_ARCH_LAYERED) {
+    LMB_TRY(layered_check_positions(S, pos.data()));
+    LMB_TRY(layered_clear_state(S, pos.data()));
+  }
+  S->host_pos_v = pos;
   return push_positions(S);
 }
+static int32_t set_all_positions(Session* S, int pos) { return move_positions(S, std::vector<int>(S->B, pos)); }
 // limits == NULL: no limit (decoding)
 static int32_t set_limits(Session* S, const int* limits) {
   Ctx* ctx = S->m->ctx;
@@ -1882,6 +1920,7 @@ extern "C" int32_t lmb200_session_create(lmb200_model hm, int32_t batch, int32_t
   LMB_REQUIRE(batch >= 1, "session_create: batch %d", batch);
   LMB_REQUIRE(max_ctx >= 1, "session_create: max_ctx %d", max_ctx);
   if (batch > 32) return wide_create(M, batch, max_ctx, out);
+  if (M->cfg.arch == LMB200_ARCH_LAYERED) return layered_session_create(M, batch, max_ctx, out);
   Ctx* ctx = M->ctx;
   LMB_CUDA(cudaSetDevice(ctx->device));
   const lmb200_model_config& c = M->cfg;
@@ -2009,6 +2048,7 @@ extern "C" int32_t lmb200_session_destroy(lmb200_session h) {
   cudaSetDevice(S->m->ctx->device);
   cudaStreamSynchronize(S->m->ctx->stream);
   drop_graphs(S);
+  layered_session_free(S);
   cudaFree(S->cross_kv);
   cudaFree(S->kv); cudaFree(S->x); cudaFree(S->delta); cudaFree(S->logits); cudaFree(S->xn); cudaFree(S->qbuf);
   cudaFree(S->attn_out); cudaFree(S->act); cudaFree(S->tokens); cudaFree(S->pos); cudaFree(S->limit); cudaFree(S->step_ctr); cudaFree(S->ragged_logits);
@@ -2056,8 +2096,7 @@ extern "C" int32_t lmb200_session_set_positions(lmb200_session h, const int32_t*
   for (int b = 0; b < S->B; ++b)
     LMB_REQUIRE(pos[b] >= 0 && pos[b] <= S->max_ctx, "set_positions: sequence %d at %d, outside 0..%d", b, pos[b], S->max_ctx);
   LMB_CUDA(cudaSetDevice(S->m->ctx->device));
-  S->host_pos_v.assign(pos, pos + S->B);
-  return push_positions(S);
+  return move_positions(S, std::vector<int>(pos, pos + S->B));
 }
 
 extern "C" int32_t lmb200_session_positions(lmb200_session h, int32_t* pos_out) {
@@ -2113,6 +2152,11 @@ extern "C" int32_t lmb200_session_fill_kv_random(lmb200_session h, int32_t n_pos
   Ctx* ctx = M->ctx;
   LMB_REQUIRE(n_pos >= 0 && n_pos <= S->max_ctx, "fill_kv_random: n_pos %d outside 0..%d", n_pos, S->max_ctx);
   LMB_CUDA(cudaSetDevice(ctx->device));
+  if (M->cfg.arch == LMB200_ARCH_LAYERED) {
+    LMB_TRY(layered_fill_random(S, n_pos, seed));
+    S->host_pos_v.assign(S->B, n_pos);
+    return push_positions(S);
+  }
   if (n_pos > 0) {
     for (int l = 0; l < M->cfg.n_layers; ++l) {
       const uint64_t kk = stream_key(seed, kIdKvBase + 2 * l), kvv = stream_key(seed, kIdKvBase + 2 * l + 1);
@@ -2180,6 +2224,14 @@ static int32_t copy_logits_out(Session* S, float* logits_out) {
   return LMB200_OK;
 }
 
+// every sequence's next lens[b] >= 1 tokens (packed one after the other), the logits of each one's last
+static int32_t extend_last(Session* S, const int32_t* tokens, const std::vector<int32_t>& lens, float* logits_out) {
+  std::vector<int32_t> want;
+  int32_t at = -1;
+  for (int32_t n : lens) want.push_back(at += n);
+  return layered_extend(S, tokens, lens.data(), (int32_t)want.size(), want.data(), logits_out, true);
+}
+
 extern "C" int32_t lmb200_prefill(lmb200_session h, const int32_t* tokens, int32_t n, float* logits_out) {
   Session* S = session_from(h);
   if (!S) return LMB200_EINVAL;
@@ -2192,6 +2244,10 @@ extern "C" int32_t lmb200_prefill(lmb200_session h, const int32_t* tokens, int32
   Ctx* ctx = S->m->ctx;
   LMB_CUDA(cudaSetDevice(ctx->device));
   const int B = S->B;
+  if (S->m->cfg.arch == LMB200_ARCH_LAYERED) {
+    const std::vector<int32_t> lens(B, n);
+    return extend_last(S, tokens, lens, logits_out);
+  }
   if ((int64_t)n * B > S->prompt_cap) {
     cudaFree(S->prompt);
     S->prompt = nullptr;
@@ -2248,6 +2304,11 @@ extern "C" int32_t lmb200_prefill_ragged(lmb200_session h, const int32_t* tokens
   }
   Ctx* ctx = S->m->ctx;
   LMB_CUDA(cudaSetDevice(ctx->device));
+  if (S->m->cfg.arch == LMB200_ARCH_LAYERED) {
+    std::vector<int32_t> packed;
+    for (int b = 0; b < B; ++b) packed.insert(packed.end(), tokens + (size_t)b * n_max, tokens + (size_t)b * n_max + lengths[b]);
+    return extend_last(S, packed.data(), std::vector<int32_t>(lengths, lengths + B), logits_out);
+  }
   if ((int64_t)longest * B > S->prompt_cap) {
     cudaFree(S->prompt);
     S->prompt = nullptr;
@@ -2326,6 +2387,72 @@ extern "C" int32_t lmb200_prefill_ragged(lmb200_session h, const int32_t* tokens
   return check_device_error(ctx);
 }
 
+// The next lengths[b] >= 0 tokens of every sequence, and the logits at any of their places.  A layered session takes them
+// in one pass; the other models have no such pass at a position other than 0, so they go through the decode step
+// one token per sequence at a time, a sequence whose tokens are over standing still.
+extern "C" int32_t lmb200_extend(lmb200_session h, const int32_t* tokens, const int32_t* lengths, int32_t n_want, const int32_t* want,
+                                 float* logits_out) {
+  Session* S = session_from(h);
+  if (!S) return LMB200_EINVAL;
+  LMB_REQUIRE(tokens && lengths && n_want >= 0 && (n_want == 0 || (want && logits_out)), "extend: null argument");
+  const int B = S->B;
+  int64_t total = 0;
+  int longest = 0;
+  for (int b = 0; b < B; ++b) {
+    LMB_REQUIRE(lengths[b] >= 0, "extend: sequence %d has length %d", b, lengths[b]);
+    total += lengths[b];
+    if (lengths[b] > longest) longest = lengths[b];
+  }
+  LMB_REQUIRE(total >= 1 && total <= 0x7fffffff, "extend: no tokens");
+  for (int i = 0; i < n_want; ++i)
+    LMB_REQUIRE(want[i] >= 0 && want[i] < total && (i == 0 || want[i] > want[i - 1]), "extend: wanted places must ascend inside 0..%lld",
+                (long long)total - 1);
+  if (!S->parts.empty()) return wide_extend(S, tokens, lengths, n_want, want, logits_out);
+  for (int b = 0; b < B; ++b)
+    if (S->host_pos_v[b] + lengths[b] > S->max_ctx)
+      return fail(LMB200_ESTATE, "extend: sequence %d: %d + %d tokens exceed max_ctx %d", b, S->host_pos_v[b], lengths[b], S->max_ctx);
+  Ctx* ctx = S->m->ctx;
+  LMB_CUDA(cudaSetDevice(ctx->device));
+  if (S->m->cfg.arch == LMB200_ARCH_LAYERED) return layered_extend(S, tokens, lengths, n_want, want, logits_out);
+  LMB_TRY(tp_guard(S, "extend"));
+  for (int b = 0; b < B; ++b)
+    LMB_REQUIRE(lengths[b] == longest || S->host_pos_v[b] + lengths[b] < S->cap, "extend: sequence %d is full and cannot stand by", b);
+  std::vector<int32_t> start(B, 0), limits(B), step_tok(B);
+  for (int b = 1; b < B; ++b) start[b] = start[b - 1] + lengths[b - 1];
+  for (int b = 0; b < B; ++b) limits[b] = S->host_pos_v[b] + lengths[b];
+  if (!S->ragged && B > 1) {
+    LMB_CUDA(cudaStreamSynchronize(ctx->stream));
+    drop_graphs(S);
+    S->ragged = true;
+  }
+  LMB_TRY(set_limits(S, limits.data()));
+  LMB_CUDA(cudaMemsetAsync(S->step_ctr, 0, 4, ctx->stream));
+  S->in_ragged_prefill = true;
+  int32_t rc = LMB200_OK;
+  for (int i = 0; i < longest && rc == LMB200_OK; ++i) {
+    bool head = i + 1 == longest;
+    for (int b = 0; b < B; ++b) step_tok[b] = i < lengths[b] ? tokens[start[b] + i] : 0;
+    for (int k = 0; k < n_want; ++k)
+      for (int b = 0; b < B; ++b) head = head || (i < lengths[b] && want[k] == start[b] + i);
+    if (cudaMemcpyAsync(S->tokens, step_tok.data(), (size_t)B * 4, cudaMemcpyHostToDevice, ctx->stream) != cudaSuccess) rc = fail(LMB200_ECUDA, "extend: token copy failed");
+    if (rc == LMB200_OK) rc = run_step(S, head, true);
+    for (int k = 0; k < n_want && rc == LMB200_OK; ++k)
+      for (int b = 0; b < B && rc == LMB200_OK; ++b)
+        if (i < lengths[b] && want[k] == start[b] + i &&
+            cudaMemcpyAsync(logits_out + (int64_t)k * S->m->cfg.vocab, S->logits + (int64_t)b * S->logits_pitch, (size_t)S->m->cfg.vocab * 4,
+                            cudaMemcpyDeviceToHost, ctx->stream) != cudaSuccess)
+          rc = fail(LMB200_ECUDA, "extend: logits copy failed");
+    cudaStreamSynchronize(ctx->stream);              // the staging array is reused
+  }
+  S->in_ragged_prefill = false;
+  const int32_t rc2 = set_limits(S, nullptr);
+  LMB_TRY(rc);
+  LMB_TRY(rc2);
+  S->host_pos_v.assign(limits.begin(), limits.end());
+  LMB_TRY(push_positions(S));
+  return check_device_error(ctx);
+}
+
 extern "C" int32_t lmb200_decode_step(lmb200_session h, const int32_t* tokens_in, int32_t* next_tokens_out,
                                       float* logits_out) {
   Session* S = session_from(h);
@@ -2400,7 +2527,8 @@ extern "C" int32_t lmb200_decode_until(lmb200_session h, const int32_t* first_to
   LMB_CUDA(cudaMemsetAsync(S->step_ctr, 0, 4, ctx->stream));
   int32_t rc = LMB200_OK;
   int done = 0;
-  const int kRun = 8;                                     // replays between two looks at the count
+  // replays between two looks at the count; a recurrent state cannot be put back, so it must not run past the end
+  const int kRun = layered_has_state(S->m) ? 1 : 8;
   while (done < budget && rc == LMB200_OK) {
     const int n = budget - done < kRun ? budget - done : kRun;
     for (int i = 0; i < n && rc == LMB200_OK; ++i) rc = run_step(S, true, false);
@@ -2428,7 +2556,7 @@ extern "C" int32_t lmb200_decode_until(lmb200_session h, const int32_t* first_to
     if (!all_eot) break;
     --keep;
   }
-  if (keep < done) {                                      // the session goes back to the step after the last useful one
+  if (keep < done && !layered_has_state(S->m)) {          // the session goes back to the step after the last useful one
     for (int& v : S->host_pos_v) v -= done - keep;
     LMB_TRY(push_positions(S));
   }
@@ -2454,6 +2582,7 @@ extern "C" int32_t lmb200_session_step_bytes(lmb200_session h, int32_t T, int64_
   if (!S->parts.empty()) return wide_step_bytes(S, T, bytes);
   Model* M = S->m;
   const lmb200_model_config& c = M->cfg;
+  if (c.arch == LMB200_ARCH_LAYERED) { *bytes = layered_step_bytes(S, T); return LMB200_OK; }
   const int64_t e = M->esz;
   int64_t per_layer = ((int64_t)M->m_qkv.rows * c.hidden + (int64_t)c.hidden * M->Hl * M->D +
                        (int64_t)2 * M->inter_l * c.hidden + (int64_t)c.hidden * M->inter_l) * e +
@@ -2593,6 +2722,7 @@ extern "C" int32_t lmb200_session_kv_layer(lmb200_session h, int32_t layer, void
   Session* S = session_from(h);
   if (!S) return LMB200_EINVAL;
   LMB_REQUIRE(kv_dptr && batch_stride && head_stride, "session_kv_layer: null argument");
+  LMB_REQUIRE(S->m->cfg.arch != LMB200_ARCH_LAYERED, "session_kv_layer: a layered decoder has no tiled key / value cache");
   LMB_REQUIRE(S->parts.empty(), "session_kv_layer: a session of more than 32 sequences has one cache per 32 sequences");
   LMB_REQUIRE(layer >= 0 && layer < S->m->cfg.n_layers, "session_kv_layer: layer %d", layer);
   *kv_dptr = reinterpret_cast<char*>(S->kv) + (int64_t)layer * S->kv_layer_stride * S->m->esz;
@@ -2607,6 +2737,7 @@ extern "C" int32_t lmb200_decode_attention_splitkv(lmb200_session h, int32_t lay
   if (!S) return LMB200_EINVAL;
   Model* M = S->m;
   LMB_REQUIRE(q_dptr && out_dptr, "decode_attention: null pointer");
+  LMB_REQUIRE(M->cfg.arch != LMB200_ARCH_LAYERED, "decode_attention: a layered decoder has no tiled key / value cache");
   LMB_REQUIRE(S->parts.empty(), "decode_attention: not built for a session of more than 32 sequences");
   LMB_REQUIRE(layer >= 0 && layer < M->cfg.n_layers, "decode_attention: layer %d", layer);
   LMB_REQUIRE(T >= 1 && T <= S->max_ctx, "decode_attention: T %d outside 1..%d", T, S->max_ctx);

@@ -11,9 +11,10 @@
 
 namespace lmb {
 
-enum MapKind { MAP_PLAIN = 0, MAP_QKV = 1, MAP_O = 2, MAP_GATEUP = 3, MAP_DOWN = 4 };
+enum MapKind { MAP_PLAIN = 0, MAP_QKV = 1, MAP_O = 2, MAP_GATEUP = 3, MAP_DOWN = 4, MAP_STACK = 5 };
+constexpr int kMaxSrc = 5;             // logical tensors one internal matrix can hold
 
-// How one internal (tiled) matrix maps onto up to three logical [out,in] tensors of the
+// How one internal (tiled) matrix maps onto up to kMaxSrc logical [out,in] tensors of the
 // reference (src/NN.jl:330-341, 238-244) -- including the head split f = h + H*d that the
 // reference's column-major reshape implies (src/NN.jl:347-354), the GQA mapping q = kv + KV*g
 // (src/NN.jl:305-317), the RoPE pairing (d, d + D/2) (src/NN.jl:274-276) and the tensor-parallel
@@ -24,8 +25,12 @@ struct WMap {
   int RB = 0, KC = 0;        // padded extent in 16-row blocks / 32-k chunks
   int H = 0, KV = 0, D = 0, G = 0, Hl = 0, KVl = 0, kv_off = 0;
   int inter_l = 0, inter_off = 0;
-  int src_rows[3] = {0, 0, 0};
-  int src_cols[3] = {0, 0, 0};
+  int src_rows[kMaxSrc] = {0, 0, 0, 0, 0};
+  int src_cols[kMaxSrc] = {0, 0, 0, 0, 0};
+  // MAP_STACK: tensor s occupies rows row_off[s] .. + src_rows[s] and columns col_off[s] .. + src_cols[s], the rest is zero
+  int n_src = 0;
+  int row_off[kMaxSrc] = {0, 0, 0, 0, 0};
+  int col_off[kMaxSrc] = {0, 0, 0, 0, 0};
 };
 
 struct LayerWeights {
@@ -53,6 +58,30 @@ struct LayerWeights {
   float *wg_qkv = nullptr, *bf_qkv = nullptr, *wg_qc = nullptr, *bf_qc = nullptr, *wg_fc1 = nullptr, *bf_fc1 = nullptr;
 };
 
+// One layer of a decoder whose layers are described one by one (LMB200_ARCH_LAYERED, csrc/layered.cu): its sizes and
+// constants, and how its tensors are stacked into the matrices the step multiplies with.
+struct LayerSpec {
+  lmb200_layer_config c{};
+  std::vector<double> decay;
+  // input projections, all reading the layer's norm: latent attention [dq | dkv | g | up], retention [q | k | v | g | up].
+  // Every part starts on a multiple of 32 rows.  The first n_store rows are mixer inputs, the rest the feed-forward's.
+  WMap m_in;
+  int row0[kMaxSrc] = {0, 0, 0, 0, 0};
+  int n_store = 0;
+  WMap m_uq, m_ukv;          // latent attention: queries from their latent; [uk | uv], per-head keys and values from the latent
+  WMap m_out;                // [o | down] side by side: mixer output columns from 0, feed-forward columns from cat0
+  int cat0 = 0;
+  int lat_rot = 0, lat_ld = 0;   // latent cache row: latent from 0, rotated key part from lat_rot, lat_ld elements in all
+};
+struct LayeredWeights {
+  void *w_in = nullptr, *w_out = nullptr, *w_uq = nullptr, *w_ukv = nullptr;
+  void *w_uk = nullptr, *w_uv = nullptr;      // row-major [heads * dim, kv_rank] and [heads * vdim, kv_rank] (absorbed attention)
+  float *norm = nullptr, *q_norm = nullptr, *kv_norm = nullptr;
+  float *inv_freq = nullptr;                  // [rot_dims / 2]
+  float *decay = nullptr;                     // retention: [heads][kDecayPow]: decay^0 .. decay^(kDecayPow - 1)
+};
+constexpr int kDecayPow = 72;
+
 struct Model {
   bool tp_solo = false;        // profiling aid: shard of one rank, no all-reduce
   uint32_t magic = 0x4D4F444C;
@@ -73,6 +102,10 @@ struct Model {
   void* lm_head = nullptr;
   float* inv_freq = nullptr;    // [D/2]
   int64_t weight_bytes = 0;
+  // LMB200_ARCH_LAYERED
+  std::vector<LayerSpec> specs;
+  std::vector<LayeredWeights> lw;
+  float softcap = 0.f;
   std::set<std::string> weights_set;   // registry names given through lmb200_model_set_weight
   bool all_weights_set = false;        // lmb200_model_init_random filled everything
 };
@@ -143,6 +176,11 @@ struct Session {
   cudaGraphExec_t graph_tok = nullptr;    // sliced head, tokens only (head_sliced)
   cudaStream_t graph_stream = nullptr;
   int graph_nodes_full = 0, graph_nodes_body = 0, graph_nodes_tok = 0;
+  // LMB200_ARCH_LAYERED (csrc/layered.cu): per layer a latent cache [B][cap][lat_ld], a recurrent state
+  // [B][heads][dim][round_up(vdim, 4)] float32, or NULL (a layer that reads another layer's latent cache)
+  std::vector<void*> latent;
+  std::vector<float*> state;
+  struct LayeredScratch* lay = nullptr;
   // a batch above 32: this session owns nothing on the device, it is a row of sub-sessions of at most 32 sequences
   std::vector<uint64_t> parts;
 };
@@ -160,6 +198,7 @@ int32_t wide_set_capture(Session* S, int32_t enable);
 int32_t wide_read_layer_output(Session* S, int32_t layer, float* host);
 int32_t wide_prefill(Session* S, const int32_t* tokens, int32_t n, float* logits_out);
 int32_t wide_prefill_ragged(Session* S, const int32_t* tokens, const int32_t* lengths, int32_t n_max, float* logits_out);
+int32_t wide_extend(Session* S, const int32_t* tokens, const int32_t* lengths, int32_t n_want, const int32_t* want, float* logits_out);
 int32_t wide_decode_step(Session* S, const int32_t* tokens_in, int32_t* next_tokens_out, float* logits_out);
 int32_t wide_decode_n(Session* S, const int32_t* first_tokens, int32_t n_steps, int32_t* tokens_out);
 int32_t wide_decode_until(Session* S, const int32_t* first_tokens, int32_t max_steps, int32_t eot_token, int32_t* tokens_out,
@@ -167,6 +206,72 @@ int32_t wide_decode_until(Session* S, const int32_t* first_tokens, int32_t max_s
 int32_t wide_step_bytes(Session* S, int32_t T, int64_t* bytes);
 
 int32_t step_kernels_configure();
+
+// decoders described layer by layer (csrc/layered.cu): what the model and session entry points hand over to
+void layered_free_model(Model* M);
+int32_t layered_init_random(Model* M, uint64_t seed, float sigma);
+int32_t layered_set_weight(Model* M, const char* name, const float* host, int32_t rank, const int64_t* dims, int32_t layout);
+std::vector<std::string> layered_weight_names(const Model* M);
+int32_t layered_session_create(Model* M, int batch, int max_ctx, lmb200_session* out);
+void layered_session_free(Session* S);
+// sequences whose position goes back to 0 start from an empty state; a position other than 0 or the present one needs
+// `forced` (synthetic contexts) where the model has recurrent layers
+int32_t layered_check_positions(const Session* S, const int32_t* pos);
+int32_t layered_clear_state(Session* S, const int32_t* new_pos);
+int32_t layered_fill_random(Session* S, int32_t n_pos, uint64_t seed);
+bool layered_has_state(const Model* M);
+int32_t layered_enqueue_step(Session* S, cudaStream_t st, bool with_head);
+// the next lengths[b] >= 0 tokens of every sequence (packed), logits of the packed places want[0 .. n_want) (logits_out may be
+// NULL).  greedy: want holds every sequence's last place, and the best tokens there become the next step's input
+int32_t layered_extend(Session* S, const int32_t* tokens, const int32_t* lengths, int32_t n_want, const int32_t* want, float* logits_out,
+                       bool greedy = false);
+int64_t layered_step_bytes(const Session* S, int32_t T);
+int32_t layered_configure();
+
+// pieces of model.cu and prefill.cu that layered.cu builds on
+struct FillSrc {
+  uint64_t key[kMaxSrc];
+  const float* src[kMaxSrc];     // staged logical tensors (NULL -> generator)
+  int colmajor;
+  int only_slot;           // -1: all
+  float scale;             // sigma / 131072
+};
+int32_t fill_tiled_dt(Model* M, void* dst, const WMap& m, const FillSrc& f);
+int32_t fill_plain_dt(Model* M, int dtype, void* dst, int64_t rows, int64_t cols, uint64_t key, const float* src, int colmajor, float scale,
+                      float offset);
+int32_t check_weight_shape(const char* name, int32_t rank, const int64_t* dims, int64_t rows, int64_t cols);
+int64_t tiled_elems(const WMap& m, int dtype);
+void finish_map(WMap& m);
+int32_t dmalloc(void** p, int64_t bytes, bool zero, cudaStream_t st);
+int32_t push_positions(Session* S);
+int32_t embed_prep_launch(Session* S, const float* gain, cudaStream_t st);
+GemvParams gemv_params(Session* S, const void* W, const WMap& m, const GemvPlan& pl, const void* x);
+int32_t argmax_launch(Session* S, cudaStream_t st);       // greedy tokens of S->logits into S->tokens
+int32_t advance_launch(Session* S, cudaStream_t st);      // end of a step on one GPU
+int32_t run_step(Session* S, bool with_head, bool want_logits = true);
+
+// Destination of a run of output rows of a GEMM over many tokens: element (token t, row row0 + r), r < rows, goes to
+// dst[t * pitch + r] after the activation.
+enum RowSegKind {
+  SEG_F32 = 0,        // float32
+  SEG_ACT = 1,        // model dtype
+  SEG_RELU2 = 2,      // relu(v)^2, model dtype
+  SEG_SILU = 3,       // silu(v), model dtype
+  SEG_SOFTCAP = 4     // softcap * tanh(v / softcap), float32 (softcap 0: v)
+};
+struct RowSeg {
+  int row0 = 0, rows = 0, kind = SEG_F32, pitch = 0;
+  void* dst = nullptr;
+};
+constexpr int kMaxSegs = 5;
+struct RowSegs {
+  RowSeg s[kMaxSegs];
+  int n = 0;
+  float softcap = 0.f;
+  void add(int row0, int rows, int kind, void* dst, int pitch) { s[n].row0 = row0; s[n].rows = rows; s[n].kind = kind; s[n].dst = dst; s[n].pitch = pitch; ++n; }
+};
+// rows of W (bf16 weight layout) times X [T, ldx] row-major bf16 (columns past K are not read), each row to its segment
+int32_t gemm_segments_bf16(Ctx* ctx, const void* W, const void* X, int ldx, int T, int rows, int K, const RowSegs& segs, cudaStream_t st);
 // prompt phase as GEMMs + flash attention (csrc/prefill.cu)
 int32_t prefill_configure();
 bool prefill_gemm_ok(const Session* S, int n);

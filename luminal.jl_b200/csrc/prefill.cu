@@ -38,7 +38,7 @@ constexpr int kEpiStageBytes = 32 * 80;        // per epilogue warp: 32 tokens x
 constexpr float kInvLn2 = 1.4426950408889634f;
 constexpr float kHalfPi = 1.5707963267948966f;
 
-enum GemmEpilogue { GEMM_STORE_F32 = 0, GEMM_SILU_GATE = 1, GEMM_QKV_ROPE = 2, GEMM_AFFINE = 3, GEMM_CROSS_KV = 4 };
+enum GemmEpilogue { GEMM_STORE_F32 = 0, GEMM_SILU_GATE = 1, GEMM_QKV_ROPE = 2, GEMM_AFFINE = 3, GEMM_CROSS_KV = 4, GEMM_SEGMENTS = 5 };
 
 struct GemmParams {
   const __nv_bfloat16* W = nullptr;     // canonical 128 x 128 units, unit (row group, k step) at (rg * KS + ks) * 16384
@@ -62,6 +62,7 @@ struct GemmParams {
   float out_scale = 1.f;
   int gelu = 0, out_bf16 = 0, is_v = 0;
   void* out_any = nullptr;
+  RowSegs segs;                         // GEMM_SEGMENTS
   const float2* rope = nullptr;         // [n_seq, D/2]: (sin, cos) of position pos0 + s times inv_freq[d0]
   int pos0 = 0, n_seq = 1, Hl = 0, KVl = 0, D = 0;
   // Implicit 1-D convolution (conv_taps > 0; src/NN.jl:55-104 without the unfolded buffer): X is the token-major input
@@ -79,6 +80,50 @@ __device__ __forceinline__ float gelu_ref(float a) {
   const float sg = 1.0f / (1.0f + exp2f((z * -1.0f) * kInvLn2));
   const float th = sg * 2.0f + -1.0f;
   return (a * 0.5f) * (1.0f + th);
+}
+
+// GEMM_SEGMENTS: segments start on multiples of 32 rows, so a warp's 32 rows lie in one segment (or in none)
+__device__ __forceinline__ void segment_epilogue(const GemmParams& p, float (&v)[32], int row, int t0, int t_end, unsigned char* stage) {
+  const int row0 = row & ~31, lane = threadIdx.x & 31;
+  RowSeg sg;
+  sg.rows = 0;
+#pragma unroll
+  for (int i = 0; i < kMaxSegs; ++i)
+    if (i < p.segs.n && row0 >= p.segs.s[i].row0 && row0 < p.segs.s[i].row0 + p.segs.s[i].rows) sg = p.segs.s[i];
+  if (sg.rows == 0) return;                              // padding between segments
+  const int r = row - sg.row0;
+  if (sg.kind == SEG_F32 || sg.kind == SEG_SOFTCAP) {
+    if (r >= sg.rows) return;
+    float* out = reinterpret_cast<float*>(sg.dst);
+    const float cap = sg.kind == SEG_SOFTCAP ? p.segs.softcap : 0.f;
+#pragma unroll
+    for (int i = 0; i < 32; ++i)
+      if (t0 + i < t_end) out[(int64_t)(t0 + i) * sg.pitch + r] = cap > 0.f ? cap * tanhf(v[i] / cap) : v[i];
+    return;
+  }
+  // bf16: the warp's 32 x 32 block is turned through shared memory, lane L then stores 32 consecutive features of token t0 + L
+  __nv_bfloat16* st = reinterpret_cast<__nv_bfloat16*>(stage);
+  constexpr int kPitch = 40;
+#pragma unroll
+  for (int i = 0; i < 32; ++i) {
+    float y = v[i];
+    if (sg.kind == SEG_RELU2) { y = fmaxf(y, 0.f); y = y * y; }
+    else if (sg.kind == SEG_SILU) y = y / (1.0f + expf(-y));
+    st[i * kPitch + lane] = __float2bfloat16_rn(y);
+  }
+  __syncwarp();
+  const int tL = t0 + lane, r0 = row0 - sg.row0;
+  if (tL < t_end) {
+    __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(sg.dst) + (int64_t)tL * sg.pitch + r0;
+    if (r0 + 32 <= sg.rows && (reinterpret_cast<uintptr_t>(dst) & 15) == 0) {
+      const uint4* src = reinterpret_cast<const uint4*>(st + lane * kPitch);
+#pragma unroll
+      for (int c = 0; c < 4; ++c) reinterpret_cast<uint4*>(dst)[c] = src[c];
+    } else {
+      for (int c = 0; c < 32 && r0 + c < sg.rows; ++c) dst[c] = st[lane * kPitch + c];
+    }
+  }
+  __syncwarp();
 }
 
 // v[i] = accumulator of (row, token t0 + i).  Rows g and g+8 of a 16-row block, which the fused
@@ -114,6 +159,10 @@ __device__ __forceinline__ void gemm_epilogue(const GemmParams& p, float (&v)[32
         reinterpret_cast<float*>(p.out_any)[(int64_t)t * p.ldo + row] = y;
       }
     }
+    return;
+  }
+  if (p.epi == GEMM_SEGMENTS) {
+    segment_epilogue(p, v, row, t0, t_end, stage);
     return;
   }
   // The fused epilogues below give every thread (one row) 32 tokens of one column of the output: stored directly,
@@ -564,7 +613,7 @@ EncodeTiledFn encode_tiled_fn() {
 }
 
 int32_t gemm_launch(Ctx* ctx, const GemmParams& p, cudaStream_t st) {
-  LMB_REQUIRE(p.K % 8 == 0 && p.ldx % 8 == 0 && (reinterpret_cast<uintptr_t>(p.X) & 15) == 0, "prefill gemm: K %d, row pitch %d", p.K, p.ldx);
+  LMB_REQUIRE(p.ldx % 8 == 0 && (reinterpret_cast<uintptr_t>(p.X) & 15) == 0, "prefill gemm: K %d, row pitch %d", p.K, p.ldx);
   EncodeTiledFn enc = encode_tiled_fn();
   if (!enc) return fail(LMB200_ECUDA, "prefill gemm: cuTensorMapEncodeTiled is not available");
   // 256-token tiles once there are enough tokens to fill them (LMB200_GEMM_BN=128 keeps the narrow tile for A/B runs)
@@ -783,6 +832,14 @@ int32_t gemm_conv1d(Ctx* ctx, const void* W, const __nv_bfloat16* X, int ldx, in
   p.epi = GEMM_AFFINE; p.bias = bias; p.out_scale = 1.0f; p.gelu = gelu; p.out_bf16 = out_bf16; p.out_any = out; p.ldo = ldo;
   p.conv_taps = taps; p.conv_P = stride; p.conv_pad = pad; p.conv_C = C; p.conv_cpad = cpad; p.conv_B = batch;
   p.conv_rows_in = rows_in; p.conv_Lout = Lout; p.conv_out_rpb = out_rpb;
+  return gemm_launch(ctx, p, st);
+}
+
+int32_t gemm_segments_bf16(Ctx* ctx, const void* W, const void* X, int ldx, int T, int rows, int K, const RowSegs& segs, cudaStream_t st) {
+  GemmParams p;
+  p.W = reinterpret_cast<const __nv_bfloat16*>(W); p.X = reinterpret_cast<const __nv_bfloat16*>(X); p.ldx = ldx; p.T = T; p.rows = rows; p.K = K;
+  p.epi = GEMM_SEGMENTS; p.segs = segs;
+  for (int i = 0; i < segs.n; ++i) LMB_REQUIRE(segs.s[i].row0 % 32 == 0, "gemm: a segment starts at row %d", segs.s[i].row0);
   return gemm_launch(ctx, p, st);
 }
 

@@ -1,0 +1,35 @@
+// Retention: linear attention with a fixed decay per head.  Per head, with R_t the rotation of position t,
+//   S_t = decay S_{t-1} + (R_t k_t / sqrt(dim)) v_t^T,   o_t = S_t^T R_t q_t,   y_t = o_t / rms(o_t) * silu(g_t)
+// over a float32 state S [dim, vdim] that a sequence carries from token to token.  Not in the reference (all of its attention
+// is softmax attention, src/NN.jl:343-387).
+#pragma once
+#include "common.cuh"
+
+namespace lmb {
+
+// Tokens start[b] .. start[b] + len[b] - 1 of the packed rows are positions pos0[b] .. of sequence b.
+struct RetentionView {
+  int B = 0;
+  const int* start = nullptr;
+  const int* len = nullptr;
+  const int* pos0 = nullptr;
+  int max_len = 1;                    // the longest len (grid sizing)
+  int H = 0, dim = 0, vdim = 0, rot_dims = 0, rot_interleaved = 0;
+  const float* inv_freq = nullptr;    // [rot_dims / 2]
+  const float* decay = nullptr;       // [H][decay_pitch]: powers 0 .. decay_pitch - 1
+  int decay_pitch = 0;
+  float eps = 0.f;
+  float* state = nullptr;             // [B][H][dim][round_up(vdim, 4)]
+  // rows [T, pitch] of the projections: head a of q at column a * dim and so on; g with silu still to be applied if raw_gate
+  const void *q = nullptr, *k = nullptr, *v = nullptr, *g = nullptr;
+  int q_pitch = 0, k_pitch = 0, v_pitch = 0, g_pitch = 0;
+  int in_f32 = 1, raw_gate = 1;
+  void* out = nullptr;                // model dtype: [T, ldo] row-major, or GEMV activations of padding bp
+  int ldo = 0, bp = 0;
+};
+
+int32_t retention_configure();
+// token after token: decoding, short portions, float32
+int32_t retention_steps(Ctx* ctx, int dtype, const RetentionView& v, cudaStream_t st);
+
+}  // namespace lmb

@@ -106,6 +106,23 @@ int32_t wide_prefill_ragged(Session* S, const int32_t* tokens, const int32_t* le
   });
 }
 
+int32_t wide_extend(Session* S, const int32_t* tokens, const int32_t* lengths, int32_t n_want, const int32_t* want, float* logits_out) {
+  const int64_t vocab = S->m->cfg.vocab;
+  int32_t t0 = 0, w0 = 0;
+  return each_part(S, [&](uint64_t h, int b0, int nb) {
+    int32_t n = 0;
+    for (int b = 0; b < nb; ++b) n += lengths[b0 + b];
+    std::vector<int32_t> w;
+    int32_t w1 = w0;
+    while (w1 < n_want && want[w1] < t0 + n) w.push_back(want[w1++] - t0);
+    const int32_t rc = n == 0 ? LMB200_OK
+                              : lmb200_extend(h, tokens + t0, lengths + b0, (int32_t)w.size(), w.data(), logits_out ? logits_out + w0 * vocab : nullptr);
+    t0 += n;
+    w0 = w1;
+    return rc;
+  });
+}
+
 int32_t wide_decode_step(Session* S, const int32_t* tokens_in, int32_t* next_tokens_out, float* logits_out) {
   const int64_t vocab = S->m->cfg.vocab;
   return each_part(S, [&](uint64_t h, int b0, int) {

@@ -88,6 +88,45 @@ def WhisperDecoderModel(device, *, d_model, heads, layers, ffn, vocab, max_posit
                  cross_len=cross_len)
 
 
+MIXERS = {"latent_attention": 0, "retention": 1}
+ROTATIONS = {"half": 0, "interleaved": 1}
+
+
+class LayeredModel(Model):
+    """A decoder described layer by layer (lmb200_model_create_layered).  `layers`: one dict per layer with `mixer`
+    ('latent_attention' or 'retention'), heads, dim, vdim, ff (0: no feed-forward), rot_dims, rot_base, rot_layout ('half' or
+    'interleaved'); latent attention also q_rank, kv_rank, rot_dim, scale, kv_from (None, or the layer whose latent cache it
+    reads); retention also decay (one value per head)."""
+
+    def __init__(self, device, *, width, vocab, layers, eps, softcap=0.0, dtype="bf16"):
+        self.device = device
+        code = _dtype_code(dtype)
+        arr = (_lib.LayerConfig * len(layers))()
+        keep = []
+        for c, layer in zip(arr, layers):
+            c.mixer = MIXERS[layer["mixer"]]
+            for k in ("heads", "dim", "vdim"):
+                setattr(c, k, int(layer[k]))
+            for k in ("q_rank", "kv_rank", "rot_dim", "rot_dims", "ff"):
+                setattr(c, k, int(layer.get(k) or 0))
+            c.kv_from = -1 if layer.get("kv_from") is None else int(layer["kv_from"])
+            c.rot_layout = ROTATIONS[layer.get("rot_layout", "half")]
+            c.rot_base = float(layer.get("rot_base") or 1.0)
+            c.scale = float(layer.get("scale", 1.0))
+            if "decay" in layer:
+                if len(layer["decay"]) != c.heads:
+                    raise ValueError(f"{len(layer['decay'])} decays for {c.heads} heads")
+                keep.append((C.c_double * c.heads)(*[float(d) for d in layer["decay"]]))
+                c.decay = C.cast(keep[-1], C.POINTER(C.c_double))
+        cfg = _lib.LayeredConfig(n_layers=len(layers), width=int(width), vocab=int(vocab), dtype=code, eps=float(eps),
+                                 softcap=float(softcap or 0.0))
+        h = C.c_uint64(0)
+        _lib.call("lmb200_model_create_layered", device.handle, C.byref(cfg), arr, C.byref(h))
+        self.handle = h
+        self.layers = [dict(layer) for layer in layers]
+        self.cfg = ModelConfig(n_layers=len(layers), hidden=int(width), vocab=int(vocab), rms_eps=float(eps), dtype=code, tp_size=1, arch=2)
+
+
 class Session:
     def __init__(self, model, batch, max_ctx):
         self.model, self.batch, self.max_ctx = model, int(batch), int(max_ctx)
@@ -172,6 +211,25 @@ class Session:
         _lib.call("lmb200_prefill", self.handle, t.ctypes.data_as(C.c_void_p), t.shape[1],
                   logits.ctypes.data_as(C.c_void_p) if want_logits else None)
         return logits
+
+    def extend(self, tokens, want=None):
+        """Appends the next tokens of every sequence: `tokens` is one id list per sequence (an empty one stands still), `want`
+        one list of places per sequence whose logits are asked for.  Returns them in order, [places, vocab].  Prompts,
+        portions of prompts and single tokens can be mixed."""
+        assert len(tokens) == self.batch
+        lens = np.array([len(t) for t in tokens], dtype=np.int32)
+        packed = np.concatenate([np.asarray(t, dtype=np.int32).reshape(-1) for t in tokens]).astype(np.int32)
+        start = np.concatenate([[0], np.cumsum(lens)[:-1]])
+        places = np.array([start[b] + int(p) for b, ps in enumerate(want or []) for p in ps], dtype=np.int32)
+        order = np.argsort(places, kind="stable")
+        uniq, back = np.unique(places[order], return_inverse=True)
+        uniq = np.ascontiguousarray(uniq, dtype=np.int32)
+        logits = np.empty((len(uniq), self.vocab), dtype=np.float32)
+        _lib.call("lmb200_extend", self.handle, packed.ctypes.data_as(C.c_void_p), lens.ctypes.data_as(C.c_void_p), len(uniq),
+                  uniq.ctypes.data_as(C.c_void_p) if len(uniq) else None, logits.ctypes.data_as(C.c_void_p) if len(uniq) else None)
+        out = np.empty((len(places), self.vocab), dtype=np.float32)
+        out[order] = logits[back]
+        return out
 
     def decode_step(self, tokens, want_logits=False):
         t = np.ascontiguousarray(np.asarray(tokens, dtype=np.int32).reshape(self.batch))
@@ -263,7 +321,7 @@ def _step_logits(session, tokens):
     return nxt, logits
 
 
-__all__ = ["Model", "Session", "greedy_generate", "decode_attention_noalloc", "shard_layout", "linear_gemv",
+__all__ = ["Model", "LayeredModel", "Session", "greedy_generate", "decode_attention_noalloc", "shard_layout", "linear_gemv",
            "WhisperDecoderModel"]
 
 
