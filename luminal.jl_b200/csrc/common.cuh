@@ -176,6 +176,17 @@ struct FlashView {
   int64_t k_b = 0, k_h = 0, k_s = 0;    // k and v
 };
 
+// Attention whose keys are wider than its values and come in two parts: dn features per head (k) and dr features that all heads
+// share (kr), queries [dn | dr] per head; the S queries are the last of Sk positions.  A row of the output may be multiplied by
+// sigmoid(gate[row * gate_pitch + head]), row = batch * S + position.
+struct FlashSplitView {
+  int H = 1, dn = 0, dr = 0, dv = 0;
+  int64_t q_b = 0, q_h = 0, q_s = 0, o_b = 0, o_h = 0, o_s = 0;
+  int64_t k_b = 0, k_h = 0, k_s = 0, v_b = 0, v_h = 0, v_s = 0, kr_b = 0, kr_s = 0;
+  const float* gate = nullptr;
+  int gate_pitch = 0;
+};
+
 static inline int64_t ceil_div(int64_t a, int64_t b) { return (a + b - 1) / b; }
 static inline int64_t round_up(int64_t a, int64_t b) { return ceil_div(a, b) * b; }
 

@@ -92,18 +92,31 @@ __device__ __forceinline__ uint64_t add2(uint64_t a, uint64_t b) {
   return d;
 }
 
-constexpr int kBN = 128, kStages = 2;
+constexpr int kBN = 128;
 constexpr int kMmaWarp = 16;                       // warps 0-15 softmax (two per query row), 16 MMA issue, 17-18 loaders
 constexpr int kThreads = (kMmaWarp + 1) * 32 + kLoaders;
 
-template <int D>
+// Head dims of a key: DN of its own and DR that all heads share (0: an ordinary head); DV of a value
+template <int DN, int DR, int DV>
 struct Smem {
+  static constexpr int D = DN + DR;
   static constexpr int kQ = kBM * D * 2;
-  static constexpr int kKV = kBN * D * 2;
+  static constexpr int kK = kBN * D * 2, kV = kBN * DV * 2;
+  static constexpr int vStages = 2;
+  static constexpr int kStages = 2 * kQ + 2 * kK + vStages * kV + 8192 <= 227 * 1024 ? 2 : 1;    // wide keys: one stage
   static constexpr int offQ = 0;                              // two query tiles
   static constexpr int offK = offQ + 2 * kQ;
-  static constexpr int offV = offK + kStages * kKV;
-  static constexpr int total = offV + kStages * kKV;
+  static constexpr int offV = offK + kStages * kK;
+  static constexpr int total = offV + vStages * kV;
+};
+
+// what the general launch (FlashSplitView) adds to a FlashView: the keys' count, the first query's position, the valid widths of the
+// padded parts, the output's strides and the gate
+struct FlashExtra {
+  int Sk = 0, q_off = 0, dn = 0, dr = 0, dv = 0;
+  int64_t o_b = 0, o_h = 0, o_s = 0;
+  const float* gate = nullptr;
+  int gate_pitch = 0;
 };
 
 __device__ __forceinline__ void mma_f16_ts(uint32_t tmem_d, uint32_t tmem_a, uint64_t bdesc, uint32_t idesc, uint32_t accumulate) {
@@ -112,17 +125,21 @@ __device__ __forceinline__ void mma_f16_ts(uint32_t tmem_d, uint32_t tmem_a, uin
       "r"(tmem_a), "l"(bdesc), "r"(idesc), "r"(accumulate)
       : "memory");
 }
-template <int D>
+template <int DN, int DR, int DV>
 __global__ void __launch_bounds__(kThreads, 1)
 flash_tc_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict__ q, const __grid_constant__ CUtensorMap kmap,
-                   const __grid_constant__ CUtensorMap vmap, const FlashView fv, int S, float scale, int causal, int* err) {
-  constexpr int W = D % 64 == 0 ? 64 : 32;            // head dims per swizzled sub-tile
+                   const __grid_constant__ CUtensorMap vmap, const __grid_constant__ CUtensorMap rmap, const FlashView fv, const FlashExtra ex, int S,
+                   float scale, int causal, int* err) {
+  constexpr int D = DN + DR;
+  constexpr int W = DN % 64 == 0 ? 64 : 32;           // head dims per swizzled sub-tile
+  static_assert(DN % W == 0 && DR % W == 0 && DV % W == 0, "whole sub-tiles");
   constexpr int kSub = kBN * W * 2;                  // bytes of one sub-tile [128 keys][W]
   constexpr uint32_t kSwz = W == 64 ? 2u : 4u;
   using namespace tc;
-  typedef Smem<D> SM;
+  typedef Smem<DN, DR, DV> SM;
+  constexpr int kStages = SM::kStages, vStages = SM::vStages;
   extern __shared__ __align__(1024) unsigned char smem[];
-  __shared__ __align__(8) uint64_t q_full, k_full[kStages], k_empty[kStages], v_full[kStages], v_empty[kStages];
+  __shared__ __align__(8) uint64_t q_full, k_full[kStages], k_empty[kStages], v_full[vStages], v_empty[vStages];
   __shared__ __align__(8) uint64_t s_full[2], p_full[2], o_done[2];
   __shared__ float xch[2][2][kBM];                    // [tile][column half][row]: the halves' row maxima, later their sums
   __shared__ uint32_t tmem_slot;
@@ -135,23 +152,22 @@ flash_tc_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict
   const int bi = (int)blockIdx.y / fv.H, hi = (int)blockIdx.y - bi * fv.H;
   const __nv_bfloat16* qb = q + bi * fv.q_b + hi * fv.q_h;
   const int kvh = hi / fv.G;
-  __nv_bfloat16* ob_base = out + bi * fv.q_b + hi * fv.q_h;
+  __nv_bfloat16* ob_base = out + bi * ex.o_b + hi * ex.o_h;
   const int64_t q_s = fv.q_s;
+  const int Sk = ex.Sk, q_off = ex.q_off;
   int n_tiles[2];
 #pragma unroll
   for (int t = 0; t < 2; ++t) {
     const int qt0 = q0 + t * kBM;
-    const int k_stop = qt0 >= S ? 0 : (causal ? min(S, qt0 + kBM) : S);
+    const int k_stop = qt0 >= S ? 0 : (causal ? min(Sk, q_off + qt0 + kBM) : Sk);
     n_tiles[t] = (k_stop + kBN - 1) / kBN;
   }
   const int n_max = max(n_tiles[0], n_tiles[1]);
 
   if (tid == 0) {
     mbar_init(&q_full, kLoaders / 32);
-    for (int s = 0; s < kStages; ++s) {
-      mbar_init(&k_full[s], 1); mbar_init(&k_empty[s], 1);
-      mbar_init(&v_full[s], 1); mbar_init(&v_empty[s], 1);
-    }
+    for (int s = 0; s < kStages; ++s) { mbar_init(&k_full[s], 1); mbar_init(&k_empty[s], 1); }
+    for (int s = 0; s < vStages; ++s) { mbar_init(&v_full[s], 1); mbar_init(&v_empty[s], 1); }
     for (int t = 0; t < 2; ++t) { mbar_init(&s_full[t], 1); mbar_init(&p_full[t], 8); mbar_init(&o_done[t], 1); }
     mbar_init_fence();
   }
@@ -169,7 +185,10 @@ flash_tc_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict
     for (int i = lt; i < 2 * kBM * (D / 8); i += kLoaders) {
       const int row = i / (D / 8), c8 = i - row * (D / 8);
       const int qi = q0 + row;
-      cp_async16(sQ + (row >> 7) * SM::kQ + canon(row & 127, c8, kBM), qb + (int64_t)min(qi, S - 1) * q_s + c8 * 8, qi < S ? 16u : 0u);
+      const int d = c8 * 8;                                  // the padding behind either part of a query is zero
+      const bool valid = qi < S && (DR == 0 || (d < DN ? d < ex.dn : d - DN < ex.dr));
+      const int src = DR == 0 || d < DN ? d : ex.dn + d - DN;
+      cp_async16(sQ + (row >> 7) * SM::kQ + canon(row & 127, c8, kBM), qb + (int64_t)min(qi, S - 1) * q_s + (valid ? src : 0), valid ? 16u : 0u);
     }
     cp_async_commit();
     cp_async_wait<0>();
@@ -180,25 +199,28 @@ flash_tc_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict
     uint64_t* empty = lw == 0 ? k_empty : v_empty;
     const CUtensorMap* map = lw == 0 ? &kmap : &vmap;
     const int off = lw == 0 ? SM::offK : SM::offV;
+    const int stages = lw == 0 ? kStages : vStages, stage_bytes = lw == 0 ? SM::kK : SM::kV, subs = (lw == 0 ? DN : DV) / W;
     for (int j = 0; j < n_max; ++j) {
-      const int s = j % kStages;
-      mbar_wait(&empty[s], ((j / kStages) & 1) ^ 1, dead, err);
+      const int s = j % stages;
+      mbar_wait(&empty[s], ((j / stages) & 1) ^ 1, dead, err);
       if (lane == 0) {
-        mbar_expect_tx(&full[s], (uint32_t)SM::kKV);
-#pragma unroll
-        for (int sub = 0; sub < D / W; ++sub) tma_load_4d(smem + off + s * SM::kKV + sub * kSub, map, sub * W, j * kBN, kvh, bi, &full[s]);
+        mbar_expect_tx(&full[s], (uint32_t)stage_bytes);
+        unsigned char* at = smem + off + s * stage_bytes;
+        for (int sub = 0; sub < subs; ++sub) tma_load_4d(at + sub * kSub, map, sub * W, j * kBN, kvh, bi, &full[s]);
+        if (DR > 0 && lw == 0)
+          for (int sub = 0; sub < DR / W; ++sub) tma_load_4d(at + (DN / W + sub) * kSub, &rmap, sub * W, j * kBN, 0, bi, &full[s]);
       }
       __syncwarp();
     }
   } else if (warp == kMmaWarp) {
     // ------------------------------ MMA issue ------------------------------
     constexpr uint32_t kIdescS = idesc_bf16(kBM, kBN, false, false);
-    constexpr uint32_t kIdescPV = idesc_bf16(kBM, D, false, true);          // V is read MN-major
+    constexpr uint32_t kIdescPV = idesc_bf16(kBM, DV, false, true);          // V is read MN-major
     mbar_wait(&q_full, 0, dead, err);
     auto issue_s = [&](int j, int t) {                // S[t] = Q[t] K(j)^T
       if (lane == 0) {
         const uint64_t adesc = smem_desc(smem_u32(smem + SM::offQ + t * SM::kQ), kBM * 16, 128);
-        const uint32_t sK = smem_u32(smem + SM::offK + (j % kStages) * SM::kKV);
+        const uint32_t sK = smem_u32(smem + SM::offK + (j % kStages) * SM::kK);
 #pragma unroll
         for (int ks = 0; ks < D / 16; ++ks) {
           const uint64_t bdesc = smem_desc_swz(sK + ((16 * ks) / W) * kSub + ((16 * ks) % W) * 2, 16, 16 * W, kSwz);
@@ -210,10 +232,10 @@ flash_tc_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict
     };
     auto issue_pv = [&](int j, int t) {               // O[t] += P[t] V(j), P read from tensor memory
       if (lane == 0) {
-        const uint64_t bdesc = smem_desc_swz(smem_u32(smem + SM::offV + (j % kStages) * SM::kKV), kSub, 16 * W, kSwz);
+        const uint64_t bdesc = smem_desc_swz(smem_u32(smem + SM::offV + (j % vStages) * SM::kV), kSub, 16 * W, kSwz);
 #pragma unroll
         for (int ks = 0; ks < kBN / 16; ++ks)
-          mma_f16_ts(tmem + kColO + t * D, tmem + kColS + t * kBN + ks * 8, bdesc + (uint64_t)(ks * ((32 * W) >> 4)), kIdescPV,
+          mma_f16_ts(tmem + kColO + t * DV, tmem + kColS + t * kBN + ks * 8, bdesc + (uint64_t)(ks * ((32 * W) >> 4)), kIdescPV,
                      (j > 0 || ks > 0) ? 1u : 0u);
         if (j == n_tiles[t] - 1) commit(&o_done[t]);
       }
@@ -229,8 +251,8 @@ flash_tc_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict
       __syncwarp();
     }
     for (int j = 0; j < n_max; ++j) {
-      const int s = j % kStages, s1 = (j + 1) % kStages;
-      mbar_wait(&v_full[s], (j / kStages) & 1, dead, err);
+      const int s = j % vStages, s1 = (j + 1) % kStages;
+      mbar_wait(&v_full[s], (j / vStages) & 1, dead, err);
       if (j + 1 < n_max) mbar_wait(&k_full[s1], ((j + 1) / kStages) & 1, dead, err);
 #pragma unroll
       for (int t = 0; t < 2; ++t) {
@@ -256,7 +278,7 @@ flash_tc_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict
     const int r = 32 * wq + lane;
     const int qi = q0 + t * kBM + r;
     const uint32_t lane_base = (uint32_t)(32 * wq) << 16;
-    const uint32_t colS = kColS + t * kBN + h * 64, colP = kColS + t * kBN + h * 32, colO = kColO + t * D + h * (D / 2);
+    const uint32_t colS = kColS + t * kBN + h * 64, colP = kColS + t * kBN + h * 32, colO = kColO + t * DV + h * (DV / 2);
     const int pair_bar = 1 + t * 4 + wq;              // named barrier of the two warps that share these rows
     const float c = scale * kLog2e;
     const int nt = n_tiles[t];
@@ -265,7 +287,7 @@ flash_tc_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict
       mbar_wait(&s_full[t], j & 1, dead, err);          // S(j) is complete, and with it (pipe order) P V(j - 1): O is at rest
       fence_after();
       const int key0 = j * kBN + h * 64;
-      const bool inside = (j + 1) * kBN <= S && (!causal || (j + 1) * kBN - 1 <= q0 + t * kBM);   // no key of the tile is masked
+      const bool inside = (j + 1) * kBN <= Sk && (!causal || (j + 1) * kBN - 1 <= q_off + q0 + t * kBM);   // no key of the tile is masked
       // pass 1: the maximum of this thread's 64 scores
       float mx4[4] = {-CUDART_INF_F, -CUDART_INF_F, -CUDART_INF_F, -CUDART_INF_F};
 #pragma unroll
@@ -279,7 +301,7 @@ flash_tc_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict
 #pragma unroll
           for (int i = 0; i < 32; ++i) {
             const int key = key0 + qd * 32 + i;
-            if (!(key >= S || (causal && key > qi))) mx4[i & 3] = fmaxf(mx4[i & 3], sv[i]);
+            if (!(key >= Sk || (causal && key > q_off + qi))) mx4[i & 3] = fmaxf(mx4[i & 3], sv[i]);
           }
         }
       }
@@ -293,7 +315,7 @@ flash_tc_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict
       if (__any_sync(0xffffffffu, raise) && j > 0) {      // both halves decide alike; each rescales its half of O's columns
         const float alpha = raise ? exp2f(m - mx) : 1.0f;
 #pragma unroll
-        for (int ch = 0; ch < D / 32; ++ch) {
+        for (int ch = 0; ch < DV / 32; ++ch) {
           float o[16];
           tmem_ld16(o, tmem + lane_base + colO + ch * 16);
 #pragma unroll
@@ -320,8 +342,8 @@ flash_tc_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict
           float a0 = sv[i], a1 = sv[i + 1];
           if (!inside) {
             const int key = key0 + qd * 16 + i;
-            if (key >= S || (causal && key > qi)) a0 = -CUDART_INF_F;
-            if (key + 1 >= S || (causal && key + 1 > qi)) a1 = -CUDART_INF_F;
+            if (key >= Sk || (causal && key > q_off + qi)) a0 = -CUDART_INF_F;
+            if (key + 1 >= Sk || (causal && key + 1 > q_off + qi)) a1 = -CUDART_INF_F;
           }
           float x0, x1;
           unpack2(fma2(pack2(a0, a1), c2, negm2), x0, x1);
@@ -355,15 +377,17 @@ flash_tc_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict
       l += xch[t][h ^ 1][r];
       mbar_wait(&o_done[t], 0, dead, err);            // the last P V has landed
       fence_after();
-      const float inv = 1.0f / l;
-      __nv_bfloat16* ob = ob_base + (int64_t)qi * q_s + h * (D / 2);
+      float inv = 1.0f / l;
+      if (DR > 0 && ex.gate && qi < S) inv *= 1.0f / (1.0f + expf(-ex.gate[((int64_t)bi * S + qi) * ex.gate_pitch + hi]));
+      __nv_bfloat16* ob = ob_base + (int64_t)qi * ex.o_s + h * (DV / 2);
 #pragma unroll
-      for (int ch = 0; ch < D / 32; ++ch) {
+      for (int ch = 0; ch < DV / 32; ++ch) {
         float o[16];
         tmem_ld16(o, tmem + lane_base + colO + ch * 16);
         if (qi < S) {
 #pragma unroll
           for (int i = 0; i < 16; i += 8) {
+            if (DR > 0 && h * (DV / 2) + ch * 16 + i >= ex.dv) continue;      // padding behind the value's width
             uint4 w;
             __nv_bfloat162 a0 = __floats2bfloat162_rn(o[i] * inv, o[i + 1] * inv), a1 = __floats2bfloat162_rn(o[i + 2] * inv, o[i + 3] * inv);
             __nv_bfloat162 a2 = __floats2bfloat162_rn(o[i + 4] * inv, o[i + 5] * inv), a3 = __floats2bfloat162_rn(o[i + 6] * inv, o[i + 7] * inv);
@@ -387,9 +411,16 @@ flash_tc_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict
 }  // namespace
 
 int32_t flash_tc_configure() {
-  LMB_CUDA(cudaFuncSetAttribute(flash_tc_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, Smem<128>::total + 1024));
-  LMB_CUDA(cudaFuncSetAttribute(flash_tc_kernel<96>, cudaFuncAttributeMaxDynamicSharedMemorySize, Smem<96>::total + 1024));
-  LMB_CUDA(cudaFuncSetAttribute(flash_tc_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, Smem<64>::total + 1024));
+#define LMB_CFG(...) \
+  LMB_CUDA(cudaFuncSetAttribute(flash_tc_kernel<__VA_ARGS__>, cudaFuncAttributeMaxDynamicSharedMemorySize, Smem<__VA_ARGS__>::total + 1024))
+  LMB_CFG(128, 0, 128);
+  LMB_CFG(96, 0, 96);
+  LMB_CFG(64, 0, 64);
+  LMB_CFG(64, 64, 64);
+  LMB_CFG(64, 64, 128);
+  LMB_CFG(128, 64, 64);
+  LMB_CFG(128, 64, 128);
+#undef LMB_CFG
   return LMB200_OK;
 }
 
@@ -412,20 +443,18 @@ EncodeTiledFn flash_encode_fn() {
   }
   return fn;
 }
-// 4-D map over K or V: dims {d, key, kv head, batch}; a box is [box_keys keys][W head dims], swizzled over its W * 2 bytes.
-// Keys past S arrive as zeros (the softmax masks them).
-int32_t kv_tensor_map(CUtensorMap* map, const void* base, const FlashView& fv, int64_t B, int64_t S, int64_t D, int box_keys) {
+// 4-D map over K or V: dims {d, key, kv head, batch}; a box is [kBN keys][W head dims], swizzled over its W * 2 bytes.  Keys past S and
+// features past D arrive as zeros (the softmax masks the former).
+int32_t kv_tensor_map(CUtensorMap* map, const void* base, int64_t n_kv, int64_t B, int64_t S, int64_t D, int64_t k_s, int64_t k_h, int64_t k_b, int W) {
   EncodeTiledFn enc = flash_encode_fn();
   if (!enc) return fail(LMB200_ECUDA, "flash attention: cuTensorMapEncodeTiled is not available");
-  const int W = D % 64 == 0 ? 64 : 32;
-  const int64_t n_kv = fv.H / fv.G;
-  const int64_t head_stride = n_kv > 1 ? fv.k_h : S * fv.k_s;           // a dimension of extent 1 still needs a valid stride
-  const int64_t batch_stride = B > 1 ? fv.k_b : S * fv.k_s * n_kv;
-  LMB_REQUIRE((reinterpret_cast<uintptr_t>(base) & 15) == 0 && fv.k_s % 8 == 0 && head_stride % 8 == 0 && batch_stride % 8 == 0,
+  const int64_t head_stride = n_kv > 1 ? k_h : S * k_s;           // a dimension of extent 1 still needs a valid stride
+  const int64_t batch_stride = B > 1 ? k_b : S * k_s * n_kv;
+  LMB_REQUIRE((reinterpret_cast<uintptr_t>(base) & 15) == 0 && k_s % 8 == 0 && head_stride % 8 == 0 && batch_stride % 8 == 0,
               "flash attention: K / V base and strides must be multiples of 16 bytes");
   const cuuint64_t dims[4] = {(cuuint64_t)D, (cuuint64_t)S, (cuuint64_t)n_kv, (cuuint64_t)B};
-  const cuuint64_t strides[3] = {(cuuint64_t)fv.k_s * 2, (cuuint64_t)head_stride * 2, (cuuint64_t)batch_stride * 2};
-  const cuuint32_t box[4] = {(cuuint32_t)W, (cuuint32_t)box_keys, 1, 1};
+  const cuuint64_t strides[3] = {(cuuint64_t)k_s * 2, (cuuint64_t)head_stride * 2, (cuuint64_t)batch_stride * 2};
+  const cuuint32_t box[4] = {(cuuint32_t)W, (cuuint32_t)kBN, 1, 1};
   const cuuint32_t estr[4] = {1, 1, 1, 1};
   const CUresult r = enc(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 4, const_cast<void*>(base), dims, strides, box, estr,
                          CU_TENSOR_MAP_INTERLEAVE_NONE, W == 64 ? CU_TENSOR_MAP_SWIZZLE_128B : CU_TENSOR_MAP_SWIZZLE_64B,
@@ -440,15 +469,58 @@ int32_t flash_tc_launch_view(Ctx* ctx, void* out, const void* q, const void* k, 
                              int64_t S, int64_t D, float scale, int causal, cudaStream_t stream) {
   dim3 grid((unsigned)ceil_div(S, 2 * kBM), (unsigned)(B * fv.H));
   CUtensorMap kmap, vmap;
-  LMB_TRY(kv_tensor_map(&kmap, k, fv, B, S, D, kBN));
-  LMB_TRY(kv_tensor_map(&vmap, v, fv, B, S, D, kBN));
+  const int W = D % 64 == 0 ? 64 : 32;
+  const int64_t n_kv = fv.H / fv.G;
+  LMB_TRY(kv_tensor_map(&kmap, k, n_kv, B, S, D, fv.k_s, fv.k_h, fv.k_b, W));
+  LMB_TRY(kv_tensor_map(&vmap, v, n_kv, B, S, D, fv.k_s, fv.k_h, fv.k_b, W));
+  FlashExtra ex;
+  ex.Sk = (int)S; ex.dn = ex.dv = (int)D;
+  ex.o_b = fv.q_b; ex.o_h = fv.q_h; ex.o_s = fv.q_s;
 #define LMB_FLASH(DD)                                                                                                   \
-  flash_tc_kernel<DD><<<grid, kThreads, Smem<DD>::total + 1024, stream>>>(                                        \
-      (__nv_bfloat16*)out, (const __nv_bfloat16*)q, kmap, vmap, fv, (int)S, scale, causal, ctx->dev_err)
+  flash_tc_kernel<DD, 0, DD><<<grid, kThreads, Smem<DD, 0, DD>::total + 1024, stream>>>(                          \
+      (__nv_bfloat16*)out, (const __nv_bfloat16*)q, kmap, vmap, kmap, fv, ex, (int)S, scale, causal, ctx->dev_err)
   if (D == 128) LMB_FLASH(128);
   else if (D == 96) LMB_FLASH(96);
   else if (D == 64) LMB_FLASH(64);
   else return fail(LMB200_EINVAL, "flash attention: head_dim %lld has no tensor-core kernel", (long long)D);
+#undef LMB_FLASH
+  ctx->launches++;
+  LMB_CUDA(cudaGetLastError());
+  return LMB200_OK;
+}
+
+bool flash_tc_split_supported(int dn, int dr, int dv) {
+  return dn >= 1 && dn <= 128 && dn % 8 == 0 && dr >= 8 && dr <= 64 && dr % 8 == 0 && dv >= 1 && dv <= 128 && dv % 8 == 0;
+}
+
+// causal attention of the last Sq of Sk positions with keys in two parts (FlashSplitView); widths are padded to whole sub-tiles of
+// 64 by the tensor maps' out-of-range fill
+int32_t flash_tc_launch_split(Ctx* ctx, void* out, const void* q, const void* k, const void* kr, const void* v, const FlashSplitView& f, int64_t B,
+                              int64_t Sq, int64_t Sk, float scale, cudaStream_t stream) {
+  LMB_REQUIRE(flash_tc_split_supported(f.dn, f.dr, f.dv), "flash attention: head widths %d + %d, %d", f.dn, f.dr, f.dv);
+  LMB_REQUIRE(Sq >= 1 && Sk >= Sq && B * f.H <= 65535, "flash attention: %lld queries, %lld keys", (long long)Sq, (long long)Sk);
+  LMB_REQUIRE((reinterpret_cast<uintptr_t>(q) & 15) == 0 && (reinterpret_cast<uintptr_t>(out) & 15) == 0 && f.q_s % 8 == 0 && f.q_h % 8 == 0 &&
+                  f.q_b % 8 == 0 && f.o_s % 8 == 0 && f.o_h % 8 == 0 && f.o_b % 8 == 0,
+              "flash attention: query and output rows must start on 16 bytes");
+  CUtensorMap kmap, vmap, rmap;
+  LMB_TRY(kv_tensor_map(&kmap, k, f.H, B, Sk, f.dn, f.k_s, f.k_h, f.k_b, 64));
+  LMB_TRY(kv_tensor_map(&vmap, v, f.H, B, Sk, f.dv, f.v_s, f.v_h, f.v_b, 64));
+  LMB_TRY(kv_tensor_map(&rmap, kr, 1, B, Sk, f.dr, f.kr_s, 0, f.kr_b, 64));
+  FlashView fv;
+  fv.H = f.H; fv.G = 1;
+  fv.q_b = f.q_b; fv.q_h = f.q_h; fv.q_s = f.q_s;
+  FlashExtra ex;
+  ex.Sk = (int)Sk; ex.q_off = (int)(Sk - Sq); ex.dn = f.dn; ex.dr = f.dr; ex.dv = f.dv;
+  ex.o_b = f.o_b; ex.o_h = f.o_h; ex.o_s = f.o_s;
+  ex.gate = f.gate; ex.gate_pitch = f.gate_pitch;
+  const dim3 grid((unsigned)ceil_div(Sq, 2 * kBM), (unsigned)(B * f.H));
+#define LMB_FLASH(DN, DV)                                                                                              \
+  flash_tc_kernel<DN, 64, DV><<<grid, kThreads, Smem<DN, 64, DV>::total + 1024, stream>>>(                       \
+      (__nv_bfloat16*)out, (const __nv_bfloat16*)q, kmap, vmap, rmap, fv, ex, (int)Sq, scale, 1, ctx->dev_err)
+  if (f.dn <= 64 && f.dv <= 64) LMB_FLASH(64, 64);
+  else if (f.dn <= 64) LMB_FLASH(64, 128);
+  else if (f.dv <= 64) LMB_FLASH(128, 64);
+  else LMB_FLASH(128, 128);
 #undef LMB_FLASH
   ctx->launches++;
   LMB_CUDA(cudaGetLastError());

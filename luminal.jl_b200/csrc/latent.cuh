@@ -26,15 +26,16 @@ int32_t latent_configure();
 
 // proj [T, pitch] float32 holds the projections of one layer: the query latent from column q0 and, if cache != NULL, latent and
 // key part from column kv0.  xq <- RMSNorm(query latent) in the model dtype, row-major [T, ldxq] or, bp > 0, a GEMV activation
-// buffer of that padding; the normed latent and the rotated key part go to the cache rows of the tokens.
+// buffer of that padding; the normed latent and the rotated key part go to the cache rows of the tokens and, if packed != NULL,
+// also to row t of packed [T, ld].
 int32_t latent_prep(Ctx* ctx, int dtype, const LatentView& v, const float* proj, int pitch, int q0, int kv0, const float* q_norm,
-                    const float* kv_norm, void* xq, int ldxq, int bp, void* cache, cudaStream_t st);
+                    const float* kv_norm, void* xq, int ldxq, int bp, void* cache, void* packed, cudaStream_t st);
 // q [T, H * (dim + rot_dim)] (float32 if q_f32, else the model dtype) -> qa [T, H, ld] in the model dtype, ordered like a cache
 // row: the absorbed part and the rotated part
 int32_t latent_absorb(Ctx* ctx, int dtype, const LatentView& v, const void* q, int q_f32, const void* w_uk, void* qa, cudaStream_t st);
 // softmax over positions 0 .. pos[t] of the token's sequence: olat [T, H, kv_rank] float32
-struct LatentAttnPlan { int keys_per_cta = 0, nsplit = 0; int64_t part_floats = 0, counters = 0; };
-LatentAttnPlan latent_attn_plan(const Ctx* ctx, int dtype, int T, int H, int kv_rank, int ctx_len);
+struct LatentAttnPlan { int nsplit = 0; int64_t part_floats = 0, counters = 0; };      // nsplit 0: the CUDA-core kernel
+LatentAttnPlan latent_attn_plan(const Ctx* ctx, int dtype, int T, int H, int kv_rank, int rot_dim, int ctx_len);
 int32_t latent_attend(Ctx* ctx, int dtype, const LatentView& v, const void* qa, const void* cache, const LatentAttnPlan& plan, float* part,
                       unsigned* counters, float* olat, cudaStream_t st);
 // out[t, a * vdim + i] = sigmoid(gate[t, a]) (Wuv_a olat[t, a])_i in the model dtype, row-major [T, ldo] or GEMV activations (bp > 0)

@@ -18,13 +18,18 @@
 
 namespace lmb {
 
+bool flash_tc_split_supported(int dn, int dr, int dv);
+int32_t flash_tc_launch_split(Ctx* ctx, void* out, const void* q, const void* k, const void* kr, const void* v, const FlashSplitView& f, int64_t B,
+                              int64_t Sq, int64_t Sk, float scale, cudaStream_t stream);
+
 // device buffers of a rows step over up to `cap_T` tokens
 struct RowsBuf {
   int64_t cap_T = 0;
   void* base = nullptr;
   int64_t bytes = 0;
   float *x = nullptr, *delta = nullptr, *proj = nullptr, *olat = nullptr;
-  void *xn = nullptr, *xq = nullptr, *q = nullptr, *qa = nullptr, *cat = nullptr;
+  void *xn = nullptr, *xq = nullptr, *q = nullptr, *qa = nullptr, *cat = nullptr, *packed = nullptr;
+  int packed_layer = -1;        // whose latent rows `packed` holds in this step
   int* meta = nullptr;          // tokens | seq | pos | last (sequence whose last token this is, or -1), cap_T each; then start | len | pos0, B each; want
 };
 
@@ -34,7 +39,7 @@ struct LayeredScratch {
   void *xq = nullptr, *qa = nullptr;
   std::vector<GemvPlan> p_in, p_out, p_uq;
   int *iota = nullptr, *ones = nullptr;          // [B]
-  LatentAttnPlan attn;
+  std::vector<LatentAttnPlan> attn;              // per layer, one token per sequence at the session's capacity
   float* attn_part = nullptr;
   unsigned* attn_counters = nullptr;
   RowsBuf step, prompt;                          // float32 decode step; everything longer
@@ -44,10 +49,13 @@ struct LayeredScratch {
   float* prompt_part = nullptr;                  // split partials of the absorbed attention in a rows step
   unsigned* prompt_counters = nullptr;
   int64_t prompt_part_floats = 0, prompt_counter_cap = 0;
+  void* expanded = nullptr;                      // keys and values multiplied out of the latents (long portions)
+  int64_t expanded_bytes = 0;
 };
 
 namespace {
 
+constexpr int kFlashMin = 32;           // shortest portion whose context is expanded to keys and values
 constexpr int kBlockTokens = 2048;      // tokens per round of the absorbed attention in a rows step (bounds its scratch)
 constexpr uint64_t kIdLayered = 0x200000, kIdLayeredState = 0x300000;
 enum LatentSlot { L_DQ = 0, L_DKV = 1, L_G = 2, L_UP = 3 };
@@ -294,6 +302,7 @@ int32_t ensure_rows(Session* S, RowsBuf& r, int64_t T, int64_t n_want) {
       {&r.qa, blk * max_over(M, [](const LayerSpec& s) { return is_latent(s) ? (int64_t)s.c.heads * s.lat_ld : 0; }) * e},
       {(void**)&r.olat, blk * max_over(M, [](const LayerSpec& s) { return is_latent(s) ? (int64_t)s.c.heads * s.c.kv_rank : 0; }) * 4},
       {&r.cat, T * max_over(M, [](const LayerSpec& s) { return row_ld(s.m_out.K); }) * e},
+      {&r.packed, T * max_over(M, [](const LayerSpec& s) { return is_latent(s) ? s.lat_ld : 0; }) * e},
       {(void**)&r.meta, (5 * T + 3 * S->B) * 4},
   };
   int64_t total = 0;
@@ -450,6 +459,25 @@ int32_t norm_rows(Session* S, RowsBuf& r, const RowsRun& run, int n_rows, const 
   return LMB200_OK;
 }
 
+// split scratch of the absorbed attention in a rows step (the counters are zero between launches)
+int32_t ensure_attn_scratch(Session* S, const LatentAttnPlan& plan) {
+  LayeredScratch& Z = *S->lay;
+  cudaStream_t st = S->m->ctx->stream;
+  if (plan.part_floats > Z.prompt_part_floats) {
+    cudaFree(Z.prompt_part);
+    Z.prompt_part = nullptr; Z.prompt_part_floats = 0;
+    LMB_TRY(dmalloc((void**)&Z.prompt_part, plan.part_floats * 4, false, st));
+    Z.prompt_part_floats = plan.part_floats;
+  }
+  if (plan.counters > Z.prompt_counter_cap) {
+    cudaFree(Z.prompt_counters);
+    Z.prompt_counters = nullptr; Z.prompt_counter_cap = 0;
+    LMB_TRY(dmalloc((void**)&Z.prompt_counters, plan.counters * 4, true, st));
+    Z.prompt_counter_cap = plan.counters;
+  }
+  return LMB200_OK;
+}
+
 int32_t latent_rows(Session* S, RowsBuf& r, const RowsRun& run, int l, bool graph, cudaStream_t st) {
   Model* M = S->m;
   Ctx* ctx = M->ctx;
@@ -468,23 +496,76 @@ int32_t latent_rows(Session* S, RowsBuf& r, const RowsRun& run, int l, bool grap
   v.T = T; v.seq = run.seq; v.pos = run.pos;
   void* cache = S->latent[cache_layer(M, l)];
   LMB_TRY(latent_prep(ctx, dt, v, r.proj, s.n_store, s.row0[L_DQ], own ? s.row0[L_DKV] : 0, w.q_norm, w.kv_norm, r.xq, ldq, 0,
-                      own ? cache : nullptr, st));
+                      own ? cache : nullptr, own ? r.packed : nullptr, st));
+  if (own) r.packed_layer = l;
   RowSegs qs;
   qs.add(0, q_width(s), SEG_ACT, r.q, q_width(s));
   LMB_TRY(rows_gemm(M, w.w_uq, s.m_uq, r.xq, ldq, T, qs, st));
-  for (int t0 = 0; t0 < T; t0 += kBlockTokens) {
+  const float* gate = r.proj + s.row0[L_G];
+  auto absorbed = [&](int t0, int t1) -> int32_t {
+    for (; t0 < t1; t0 += kBlockTokens) {
+      LatentView b = v;
+      b.T = std::min(kBlockTokens, t1 - t0); b.seq = run.seq + t0; b.pos = run.pos + t0;
+      LMB_TRY(latent_absorb(ctx, dt, b, (const char*)r.q + (int64_t)t0 * q_width(s) * e, 0, w.w_uk, r.qa, st));
+      const LatentAttnPlan plan = graph ? Z.attn[l] : latent_attn_plan(ctx, dt, b.T, b.H, b.kv_rank, b.rot_dim, run.ctx_len);
+      if (!graph) LMB_TRY(ensure_attn_scratch(S, plan));
+      LMB_TRY(latent_attend(ctx, dt, b, r.qa, cache, plan, graph ? Z.attn_part : Z.prompt_part, graph ? Z.attn_counters : Z.prompt_counters, r.olat, st));
+      LMB_TRY(latent_expand(ctx, dt, b, r.olat, w.w_uv, gate + (int64_t)t0 * s.n_store, s.n_store, (char*)r.cat + (int64_t)t0 * ldc * e, ldc, 0, st));
+    }
+    return LMB200_OK;
+  };
+  const bool flash = dt == LMB200_BF16 && !graph && flash_tc_split_supported(s.c.dim, s.c.rot_dim, s.c.vdim);
+  // keys and values of `rows` latent rows, then the attention of n queries per sequence over them
+  auto expanded = [&](int t0, const void* lat, int64_t rows, int n_batch, int n, int64_t ctx_rows) -> int32_t {
+    const int64_t kw = (int64_t)s.c.heads * s.c.dim, vw = out_width(s);
+    const int64_t bytes = round_up(rows * kw * 2, 256) + rows * vw * 2;
+    if (bytes > Z.expanded_bytes) {
+      LMB_CUDA(cudaStreamSynchronize(st));
+      cudaFree(Z.expanded);
+      Z.expanded = nullptr; Z.expanded_bytes = 0;
+      LMB_TRY(dmalloc(&Z.expanded, bytes, false, st));
+      Z.expanded_bytes = bytes;
+    }
+    void* kx = Z.expanded;
+    void* vx = (char*)Z.expanded + round_up(rows * kw * 2, 256);
+    RowSegs kv;
+    kv.add(s.m_ukv.row_off[0], (int)kw, SEG_ACT, kx, (int)kw);
+    kv.add(s.m_ukv.row_off[1], (int)vw, SEG_ACT, vx, (int)vw);
+    LMB_TRY(rows_gemm(M, w.w_ukv, s.m_ukv, lat, s.lat_ld, (int)rows, kv, st));
+    FlashSplitView f;
+    f.H = s.c.heads; f.dn = s.c.dim; f.dr = s.c.rot_dim; f.dv = s.c.vdim;
+    f.q_s = q_width(s); f.q_h = s.c.dim + s.c.rot_dim; f.q_b = (int64_t)n * f.q_s;
+    f.o_s = ldc; f.o_h = s.c.vdim; f.o_b = (int64_t)n * ldc;
+    f.k_s = kw; f.k_h = s.c.dim; f.k_b = ctx_rows * kw;
+    f.v_s = vw; f.v_h = s.c.vdim; f.v_b = ctx_rows * vw;
+    f.kr_s = s.lat_ld; f.kr_b = ctx_rows * s.lat_ld;
+    f.gate = gate + (int64_t)t0 * s.n_store; f.gate_pitch = s.n_store;
+    return flash_tc_launch_split(ctx, (char*)r.cat + (int64_t)t0 * ldc * e, (const char*)r.q + (int64_t)t0 * q_width(s) * e, kx,
+                                 (const char*)lat + (int64_t)s.lat_rot * e, vx, f, n_batch, n, ctx_rows, s.c.scale, st);
+  };
+  auto rotate = [&](int t0, int n) -> int32_t {
     LatentView b = v;
-    b.T = std::min(kBlockTokens, T - t0); b.seq = run.seq + t0; b.pos = run.pos + t0;
-    LMB_TRY(latent_absorb(ctx, dt, b, (const char*)r.q + (int64_t)t0 * q_width(s) * e, 0, w.w_uk, r.qa, st));
-    LatentAttnPlan plan = graph ? Z.attn : latent_attn_plan(ctx, dt, b.T, b.H, b.kv_rank, run.ctx_len);
-    float* part = graph ? Z.attn_part : Z.prompt_part;
-    unsigned* counters = graph ? Z.attn_counters : Z.prompt_counters;
-    LMB_REQUIRE(graph || (plan.part_floats <= Z.prompt_part_floats && plan.counters <= Z.prompt_counter_cap), "layered: attention scratch");
-    LMB_TRY(latent_attend(ctx, dt, b, r.qa, cache, plan, part, counters, r.olat, st));
-    LMB_TRY(latent_expand(ctx, dt, b, r.olat, w.w_uv, r.proj + (int64_t)t0 * s.n_store + s.row0[L_G], s.n_store,
-                          (char*)r.cat + (int64_t)t0 * ldc * e, ldc, 0, st));
+    b.T = n; b.pos = run.pos + t0;
+    return latent_rotate_q(ctx, b, (char*)r.q + (int64_t)t0 * q_width(s) * e, st);
+  };
+  if (!flash) return absorbed(0, T);
+  bool uniform = S->B > 1 && r.packed_layer == cache_layer(M, l);
+  for (int b = 0; b < S->B; ++b) uniform = uniform && run.h_pos0[b] == 0 && run.h_len[b] == run.h_len[0];
+  if (uniform && run.h_len[0] >= kFlashMin && (int64_t)S->B * s.c.heads <= 65535) {       // fresh prompts of one length: all at once
+    LMB_TRY(rotate(0, T));
+    return expanded(0, r.packed, T, S->B, run.h_len[0], run.h_len[0]);
   }
-  return LMB200_OK;
+  int pending = 0;                                      // first token of the run of short portions not yet attended
+  for (int b = 0; b < S->B; ++b) {
+    const int t0 = run.h_start[b], n = run.h_len[b];
+    if (n < kFlashMin) continue;
+    LMB_TRY(absorbed(pending, t0));
+    pending = t0 + n;
+    LMB_TRY(rotate(t0, n));
+    const char* lat = (const char*)cache + (int64_t)b * S->cap * s.lat_ld * e;
+    LMB_TRY(expanded(t0, lat, run.h_pos0[b] + n, 1, n, run.h_pos0[b] + n));
+  }
+  return absorbed(pending, T);
 }
 
 int32_t retention_rows(Session* S, RowsBuf& r, const RowsRun& run, int l, cudaStream_t st) {
@@ -515,6 +596,7 @@ int32_t retention_rows(Session* S, RowsBuf& r, const RowsRun& run, int l, cudaSt
 int32_t rows_step(Session* S, RowsBuf& r, const RowsRun& run, bool graph, cudaStream_t st) {
   Model* M = S->m;
   const int W = M->cfg.hidden, L = M->cfg.n_layers, bf = M->cfg.dtype == LMB200_BF16;
+  r.packed_layer = -1;
   for (int l = 0; l < L; ++l) {
     float* cap = S->capture_on && l > 0 ? S->capture + (int64_t)(l - 1) * S->B * W : nullptr;
     const float* delta = l ? r.delta : nullptr;
@@ -572,13 +654,13 @@ int32_t fused_step(Session* S, cudaStream_t st, bool with_head) {
       v.T = B; v.seq = Z.iota; v.pos = S->pos;
       void* cache = S->latent[cache_layer(M, l)];
       LMB_TRY(latent_prep(ctx, dt, v, Z.proj, s.n_store, s.row0[L_DQ], own ? s.row0[L_DKV] : 0, w.q_norm, w.kv_norm, Z.xq, 0, S->Bp,
-                          own ? cache : nullptr, st));
+                          own ? cache : nullptr, nullptr, st));
       GemvParams p = gemv_params(S, w.w_uq, s.m_uq, Z.p_uq[l], Z.xq);
       p.epi = EPI_STORE_F32; p.out = Z.qf; p.out_pitch = q_width(s);
       gemv_prefetch_next(p, ctx, dt, w.w_out, s.m_out.rows, s.m_out.K, Z.p_out[l]);
       LMB_TRY(gemv_launch(ctx, dt, p, st));
       LMB_TRY(latent_absorb(ctx, dt, v, Z.qf, 1, w.w_uk, Z.qa, st));
-      LMB_TRY(latent_attend(ctx, dt, v, Z.qa, cache, Z.attn, Z.attn_part, Z.attn_counters, Z.olat, st));
+      LMB_TRY(latent_attend(ctx, dt, v, Z.qa, cache, Z.attn[l], Z.attn_part, Z.attn_counters, Z.olat, st));
       LMB_TRY(latent_expand(ctx, dt, v, Z.olat, w.w_uv, Z.proj + s.row0[L_G], s.n_store, S->act, 0, S->Bp, st));
     } else {
       RetentionView v = retention_view(S, l);
@@ -660,23 +742,19 @@ int32_t layered_session_create(Model* M, int batch, int max_ctx, lmb200_session*
   auto alloc = [&](void** p, int64_t bytes) { if (rc == LMB200_OK) rc = dmalloc(p, bytes, true, ctx->stream); };
   S->latent.assign(c.n_layers, nullptr);
   S->state.assign(c.n_layers, nullptr);
-  int64_t lat_parts = 0, lat_counters = 0, prompt_parts = 0, prompt_counters = 0;
+  int64_t lat_parts = 0, lat_counters = 0;
   for (int l = 0; l < c.n_layers; ++l) {
     const LayerSpec& s = M->specs[l];
     if (!is_latent(s)) { alloc((void**)&S->state[l], (int64_t)batch * s.c.heads * s.c.dim * state_ld(s) * 4); continue; }
     if (s.c.kv_from < 0) alloc(&S->latent[l], (int64_t)batch * S->cap * s.lat_ld * M->esz);
   }
-  // one plan serves every latent layer: sized for the widest of them
-  const int heads = (int)max_over(M, [](const LayerSpec& s) { return is_latent(s) ? s.c.heads : 0; });
-  const int kvr = (int)max_over(M, [](const LayerSpec& s) { return is_latent(s) ? s.c.kv_rank : 0; });
-  if (heads) {
-    Z.attn = latent_attn_plan(ctx, c.dtype, batch, heads, kvr, S->cap);
-    lat_parts = Z.attn.part_floats; lat_counters = Z.attn.counters;
-    for (int T = 1; T <= kBlockTokens; T *= 2) {
-      const LatentAttnPlan p = latent_attn_plan(ctx, c.dtype, T, heads, kvr, S->cap);
-      prompt_parts = std::max(prompt_parts, 2 * p.part_floats); prompt_counters = std::max(prompt_counters, 2 * p.counters);
-    }
-    Z.prompt_part_floats = prompt_parts; Z.prompt_counter_cap = prompt_counters;
+  Z.attn.resize(c.n_layers);
+  for (int l = 0; l < c.n_layers; ++l) {
+    const LayerSpec& s = M->specs[l];
+    if (!is_latent(s)) continue;
+    Z.attn[l] = latent_attn_plan(ctx, c.dtype, batch, s.c.heads, s.c.kv_rank, s.c.rot_dim, S->cap);
+    lat_parts = std::max(lat_parts, Z.attn[l].part_floats);
+    lat_counters = std::max(lat_counters, Z.attn[l].counters);
   }
   if (bf) {
     int64_t max_part = 0;
@@ -708,8 +786,6 @@ int32_t layered_session_create(Model* M, int batch, int max_ctx, lmb200_session*
   }
   alloc((void**)&Z.attn_part, lat_parts * 4);
   alloc((void**)&Z.attn_counters, lat_counters * 4);
-  alloc((void**)&Z.prompt_part, prompt_parts * 4);
-  alloc((void**)&Z.prompt_counters, prompt_counters * 4);
   alloc((void**)&S->logits, (int64_t)batch * S->logits_pitch * 4);
   alloc((void**)&S->tokens, (int64_t)batch * 4);
   alloc((void**)&S->pos, (int64_t)batch * 4);
@@ -745,7 +821,7 @@ void layered_session_free(Session* S) {
   LayeredScratch& Z = *S->lay;
   cudaFree(Z.proj); cudaFree(Z.qf); cudaFree(Z.olat); cudaFree(Z.xq); cudaFree(Z.qa); cudaFree(Z.iota); cudaFree(Z.ones);
   cudaFree(Z.attn_part); cudaFree(Z.attn_counters); cudaFree(Z.prompt_part); cudaFree(Z.prompt_counters);
-  cudaFree(Z.want_logits); cudaFree(Z.want_xn);
+  cudaFree(Z.want_logits); cudaFree(Z.want_xn); cudaFree(Z.expanded);
   free_rows(Z.step);
   free_rows(Z.prompt);
   delete S->lay;
