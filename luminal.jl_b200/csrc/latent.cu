@@ -115,7 +115,7 @@ __global__ void __launch_bounds__(256) latent_absorb_kernel(const LatentView v, 
     const int t = i / v.rot_dim, d = i - t * v.rot_dim;
     const QT* qr = q + (t0 + t) * pitch + h * qd + v.dim;
     qa[((int64_t)(t0 + t) * v.H + h) * v.ld + v.rot + d] =
-        from_f32<WT>(rotated([&](int j) { return to_f32(qr[j]); }, d, v.rot_dims, v.rot_interleaved, v.pos[t0 + t], v.inv_freq));
+        from_f32<WT>(rotated([&](int j) { return to_f32(qr[j]); }, d, v.q_rotated ? 0 : v.rot_dims, v.rot_interleaved, v.pos[t0 + t], v.inv_freq));
   }
   __syncthreads();
   for (int r = 2 * tid; r < v.kv_rank; r += 512) {     // two latent columns per thread

@@ -16,6 +16,7 @@ struct LatentView {
   const int* seq = nullptr;
   const int* pos = nullptr;
   int H = 0, dim = 0, vdim = 0, q_rank = 0, kv_rank = 0, rot_dim = 0, rot_dims = 0, rot_interleaved = 1;
+  int q_rotated = 0;                // latent_absorb: the queries' positional parts are rotated already
   int rot = 0, ld = 0;              // cache row: latent from 0, rotated part from `rot`, `ld` elements (the gaps are zero)
   int64_t seq_stride = 0;           // cache elements per sequence
   const float* inv_freq = nullptr;  // [rot_dims / 2]
@@ -41,7 +42,7 @@ int32_t latent_attend(Ctx* ctx, int dtype, const LatentView& v, const void* qa, 
 // out[t, a * vdim + i] = sigmoid(gate[t, a]) (Wuv_a olat[t, a])_i in the model dtype, row-major [T, ldo] or GEMV activations (bp > 0)
 int32_t latent_expand(Ctx* ctx, int dtype, const LatentView& v, const float* olat, const void* w_uv, const float* gate, int gate_pitch,
                       void* out, int ldo, int bp, cudaStream_t st);
-// rotates the positional part of q [T, H * (dim + rot_dim)] in place (bf16)
+// rotates the positional part of q [T, H * (dim + rot_dim)] in place (bf16; where the projection's epilogue could not)
 int32_t latent_rotate_q(Ctx* ctx, const LatentView& v, void* q, cudaStream_t st);
 
 }  // namespace lmb

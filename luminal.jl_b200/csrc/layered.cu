@@ -29,6 +29,9 @@ struct RowsBuf {
   int64_t bytes = 0;
   float *x = nullptr, *delta = nullptr, *proj = nullptr, *olat = nullptr;
   void *xn = nullptr, *xq = nullptr, *q = nullptr, *qa = nullptr, *cat = nullptr, *packed = nullptr;
+  float2* angles = nullptr;     // [Model::rot_freqs][cap_T][max_half] (cos, sin) of the tokens' positions
+  int max_half = 0;
+  std::vector<bool> angles_valid;
   int packed_layer = -1;        // whose latent rows `packed` holds in this step
   int* meta = nullptr;          // tokens | seq | pos | last (sequence whose last token this is, or -1), cap_T each; then start | len | pos0, B each; want
 };
@@ -55,6 +58,7 @@ struct LayeredScratch {
 
 namespace {
 
+constexpr int kChunkMin = 8;            // longest portion from which retention runs in chunks
 constexpr int kFlashMin = 32;           // shortest portion whose context is expanded to keys and values
 constexpr int kBlockTokens = 2048;      // tokens per round of the absorbed attention in a rows step (bounds its scratch)
 constexpr uint64_t kIdLayered = 0x200000, kIdLayeredState = 0x300000;
@@ -128,6 +132,8 @@ void derive_layer(LayerSpec& s, int width) {
   } else {
     part(R_Q, c.heads * c.dim);
     part(R_K, c.heads * c.dim);
+    if (c.rot_layout == LMB200_ROT_HALF)
+      for (int slot : {(int)R_Q, (int)R_K}) { s.m_in.pair_head[slot] = c.dim; s.m_in.pair_dims[slot] = c.rot_dims; }
     part(R_V, out_width(s));
     part(R_G, out_width(s));
     s.n_store = at;
@@ -291,6 +297,7 @@ int32_t ensure_rows(Session* S, RowsBuf& r, int64_t T, int64_t n_want) {
   T = std::max<int64_t>(T, r.cap_T);
   free_rows(r);
   const int64_t blk = std::min<int64_t>(T, kBlockTokens);
+  r.max_half = (int)max_over(M, [](const LayerSpec& s) { return s.c.rot_dims / 2; });
   struct Piece { void** p; int64_t bytes; };
   const Piece pieces[] = {
       {(void**)&r.x, T * W * 4},
@@ -303,6 +310,7 @@ int32_t ensure_rows(Session* S, RowsBuf& r, int64_t T, int64_t n_want) {
       {(void**)&r.olat, blk * max_over(M, [](const LayerSpec& s) { return is_latent(s) ? (int64_t)s.c.heads * s.c.kv_rank : 0; }) * 4},
       {&r.cat, T * max_over(M, [](const LayerSpec& s) { return row_ld(s.m_out.K); }) * e},
       {&r.packed, T * max_over(M, [](const LayerSpec& s) { return is_latent(s) ? s.lat_ld : 0; }) * e},
+      {(void**)&r.angles, M->cfg.dtype == LMB200_BF16 ? (int64_t)M->rot_freqs.size() * T * r.max_half * 8 : 0},
       {(void**)&r.meta, (5 * T + 3 * S->B) * 4},
   };
   int64_t total = 0;
@@ -432,7 +440,6 @@ RetentionView retention_view(const Session* S, int l) {
   RetentionView v;
   v.B = S->B;
   v.H = s.c.heads; v.dim = s.c.dim; v.vdim = s.c.vdim; v.rot_dims = s.c.rot_dims;
-  v.rot_interleaved = s.c.rot_layout == LMB200_ROT_INTERLEAVED;
   v.inv_freq = M->lw[l].inv_freq; v.decay = M->lw[l].decay; v.decay_pitch = kDecayPow;
   v.eps = M->cfg.rms_eps;
   v.state = S->state[l];
@@ -456,6 +463,20 @@ int32_t norm_rows(Session* S, RowsBuf& r, const RowsRun& run, int n_rows, const 
   LMB_CUDA(launch_k(rows_norm_kernel<WT>, dim3((unsigned)n_rows), dim3(256), (size_t)W * 4, st, r.x, delta, embed ? run.tokens : (const int*)nullptr,
                     (const WT*)M->embed, M->cfg.vocab, pick, w, (WT*)xn, row_ld(W), W, M->cfg.rms_eps, capture, run.last));
   M->ctx->launches++;
+  return LMB200_OK;
+}
+
+// Makes `sg` a SEG_ROT segment of layer l: heads of `head` rows whose features from `off` on rotate.  The angles of this step's tokens
+// are computed once for all layers with the same frequencies.
+int32_t rotate_segment(Session* S, RowsBuf& r, const RowsRun& run, int l, RowSeg& sg, int head, int off, cudaStream_t st) {
+  Model* M = S->m;
+  const int id = M->lw[l].rot_id, n = M->specs[l].c.rot_dims / 2;
+  float2* tab = r.angles + (int64_t)id * r.cap_T * r.max_half;
+  if (!r.angles_valid[id]) {
+    LMB_TRY(angle_table(M->ctx, tab, M->lw[l].inv_freq, n, run.pos, run.T, st));
+    r.angles_valid[id] = true;
+  }
+  sg.rot = tab; sg.rot_head = head; sg.rot_off = off; sg.rot_dims = 2 * n;
   return LMB200_OK;
 }
 
@@ -499,7 +520,12 @@ int32_t latent_rows(Session* S, RowsBuf& r, const RowsRun& run, int l, bool grap
                       own ? cache : nullptr, own ? r.packed : nullptr, st));
   if (own) r.packed_layer = l;
   RowSegs qs;
-  qs.add(0, q_width(s), SEG_ACT, r.q, q_width(s));
+  const bool rot = dt == LMB200_BF16 && s.c.rot_dims > 0 && v.rot_interleaved && s.c.dim % 2 == 0 && s.c.rot_dim % 2 == 0;
+  qs.add(0, q_width(s), rot ? SEG_ROT : SEG_ACT, r.q, q_width(s));
+  if (rot) {
+    LMB_TRY(rotate_segment(S, r, run, l, qs.s[0], s.c.dim + s.c.rot_dim, s.c.dim, st));
+    v.q_rotated = 1;
+  }
   LMB_TRY(rows_gemm(M, w.w_uq, s.m_uq, r.xq, ldq, T, qs, st));
   const float* gate = r.proj + s.row0[L_G];
   auto absorbed = [&](int t0, int t1) -> int32_t {
@@ -544,6 +570,7 @@ int32_t latent_rows(Session* S, RowsBuf& r, const RowsRun& run, int l, bool grap
                                  (const char*)lat + (int64_t)s.lat_rot * e, vx, f, n_batch, n, ctx_rows, s.c.scale, st);
   };
   auto rotate = [&](int t0, int n) -> int32_t {
+    if (rot) return LMB200_OK;
     LatentView b = v;
     b.T = n; b.pos = run.pos + t0;
     return latent_rotate_q(ctx, b, (char*)r.q + (int64_t)t0 * q_width(s) * e, st);
@@ -574,11 +601,15 @@ int32_t retention_rows(Session* S, RowsBuf& r, const RowsRun& run, int l, cudaSt
   const LayerSpec& s = M->specs[l];
   LayeredWeights& w = M->lw[l];
   const int dt = M->cfg.dtype, T = run.T, e = M->esz, ldc = row_ld(s.m_out.K);
+  // bf16: the projection's epilogue rotates q and k (pairs are neighbouring rows; heads of odd width are rotated by the consumer)
+  const bool rot = dt == LMB200_BF16 && s.c.rot_dims > 0 && s.c.dim % 2 == 0;
   char* proj = reinterpret_cast<char*>(r.proj);
   auto at = [&](int slot) { return (void*)(proj + (int64_t)s.row0[slot] * e); };
   RowSegs in;
-  in.add(s.row0[R_Q], s.c.heads * s.c.dim, SEG_ACT, at(R_Q), s.n_store);
-  in.add(s.row0[R_K], s.c.heads * s.c.dim, SEG_ACT, at(R_K), s.n_store);
+  in.add(s.row0[R_Q], s.c.heads * s.c.dim, rot ? SEG_ROT : SEG_ACT, at(R_Q), s.n_store);
+  in.add(s.row0[R_K], s.c.heads * s.c.dim, rot ? SEG_ROT : SEG_ACT, at(R_K), s.n_store);
+  if (rot)
+    for (int i = 0; i < 2; ++i) LMB_TRY(rotate_segment(S, r, run, l, in.s[i], s.c.dim, 0, st));
   in.add(s.row0[R_V], out_width(s), SEG_ACT, at(R_V), s.n_store);
   in.add(s.row0[R_G], out_width(s), SEG_SILU, at(R_G), s.n_store);
   if (s.c.ff) in.add(s.row0[R_UP], s.c.ff, SEG_RELU2, (char*)r.cat + (int64_t)s.cat0 * e, ldc);
@@ -589,6 +620,8 @@ int32_t retention_rows(Session* S, RowsBuf& r, const RowsRun& run, int l, cudaSt
   v.q_pitch = v.k_pitch = v.v_pitch = v.g_pitch = s.n_store;
   v.in_f32 = dt != LMB200_BF16; v.raw_gate = 0;
   v.out = r.cat; v.ldo = ldc; v.bp = 0;
+  if (rot) v.rot_dims = 0;
+  if (run.max_len >= kChunkMin && retention_chunks_ok(v)) return retention_chunks(ctx, v, st);
   return retention_steps(ctx, dt, v, st);
 }
 
@@ -597,6 +630,7 @@ int32_t rows_step(Session* S, RowsBuf& r, const RowsRun& run, bool graph, cudaSt
   Model* M = S->m;
   const int W = M->cfg.hidden, L = M->cfg.n_layers, bf = M->cfg.dtype == LMB200_BF16;
   r.packed_layer = -1;
+  r.angles_valid.assign(M->rot_freqs.size(), false);
   for (int l = 0; l < L; ++l) {
     float* cap = S->capture_on && l > 0 ? S->capture + (int64_t)(l - 1) * S->B * W : nullptr;
     const float* delta = l ? r.delta : nullptr;
@@ -1019,6 +1053,12 @@ extern "C" int32_t lmb200_model_create_layered(lmb200_ctx hctx, const lmb200_lay
     std::vector<float> f(s.c.rot_dims / 2);
     for (int i = 0; i < s.c.rot_dims / 2; ++i) f[i] = (float)pow(s.c.rot_base, -2.0 * i / s.c.rot_dims);
     upload(&w.inv_freq, f);
+    if (!f.empty()) {
+      size_t id = 0;
+      while (id < M->rot_freqs.size() && M->rot_freqs[id] != f) ++id;
+      if (id == M->rot_freqs.size()) M->rot_freqs.push_back(f);
+      w.rot_id = (int)id;
+    }
     if (is_latent(s)) {
       alloc(&w.w_uq, tiled_elems(s.m_uq, c.dtype) * M->esz);
       alloc(&w.w_ukv, tiled_elems(s.m_ukv, c.dtype) * M->esz);

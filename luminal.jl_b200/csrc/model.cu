@@ -65,6 +65,10 @@ __host__ __device__ inline bool wmap_resolve(const WMap& m, int i, int k, int* s
         const int r = i - m.row_off[s], c = k - m.col_off[s];
         if (r >= 0 && r < m.src_rows[s] && c >= 0 && c < m.src_cols[s]) {
           *slot = s; *lrow = r; *lcol = c;
+          if (m.pair_dims[s] > 0) {
+            const int h = r / m.pair_head[s], f = r - h * m.pair_head[s];
+            if (f < m.pair_dims[s]) *lrow = h * m.pair_head[s] + (f >> 1) + (f & 1) * (m.pair_dims[s] >> 1);
+          }
           return true;
         }
       }

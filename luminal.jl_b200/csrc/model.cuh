@@ -31,6 +31,10 @@ struct WMap {
   int n_src = 0;
   int row_off[kMaxSrc] = {0, 0, 0, 0, 0};
   int col_off[kMaxSrc] = {0, 0, 0, 0, 0};
+  // rows of heads pair_head[s] wide whose first pair_dims[s] features rotate in half-split pairs (i, i + dims / 2): internal rows 2i and
+  // 2i + 1 hold pair i.  Applied to queries and keys alike it changes no product, and a pair always sits in neighbouring rows.
+  int pair_head[kMaxSrc] = {0, 0, 0, 0, 0};
+  int pair_dims[kMaxSrc] = {0, 0, 0, 0, 0};
 };
 
 struct LayerWeights {
@@ -78,6 +82,7 @@ struct LayeredWeights {
   void *w_uk = nullptr, *w_uv = nullptr;      // row-major [heads * dim, kv_rank] and [heads * vdim, kv_rank] (absorbed attention)
   float *norm = nullptr, *q_norm = nullptr, *kv_norm = nullptr;
   float *inv_freq = nullptr;                  // [rot_dims / 2]
+  int rot_id = -1;                            // layers with the same frequencies share an angle table (Model::rot_freqs)
   float *decay = nullptr;                     // retention: [heads][kDecayPow]: decay^0 .. decay^(kDecayPow - 1)
 };
 constexpr int kDecayPow = 72;
@@ -106,6 +111,7 @@ struct Model {
   std::vector<LayerSpec> specs;
   std::vector<LayeredWeights> lw;
   float softcap = 0.f;
+  std::vector<std::vector<float>> rot_freqs;   // the distinct frequency lists of the layers
   std::set<std::string> weights_set;   // registry names given through lmb200_model_set_weight
   bool all_weights_set = false;        // lmb200_model_init_random filled everything
 };
@@ -257,11 +263,15 @@ enum RowSegKind {
   SEG_ACT = 1,        // model dtype
   SEG_RELU2 = 2,      // relu(v)^2, model dtype
   SEG_SILU = 3,       // silu(v), model dtype
-  SEG_SOFTCAP = 4     // softcap * tanh(v / softcap), float32 (softcap 0: v)
+  SEG_SOFTCAP = 4,    // softcap * tanh(v / softcap), float32 (softcap 0: v)
+  SEG_ROT = 5         // bf16: neighbouring rows (2i, 2i + 1) of every head are rotated by angle i of the token's table row
 };
 struct RowSeg {
   int row0 = 0, rows = 0, kind = SEG_F32, pitch = 0;
   void* dst = nullptr;
+  // SEG_ROT: heads of rot_head rows, features rot_off .. rot_off + rot_dims - 1 rotate (all even); rot[token * rot_dims / 2 + i] = (cos, sin)
+  const float2* rot = nullptr;
+  int rot_head = 0, rot_off = 0, rot_dims = 0;
 };
 constexpr int kMaxSegs = 5;
 struct RowSegs {

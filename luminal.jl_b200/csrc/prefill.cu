@@ -101,6 +101,20 @@ __device__ __forceinline__ void segment_epilogue(const GemmParams& p, float (&v)
       if (t0 + i < t_end) out[(int64_t)(t0 + i) * sg.pitch + r] = cap > 0.f ? cap * tanhf(v[i] / cap) : v[i];
     return;
   }
+  if (sg.kind == SEG_ROT) {
+    const int f = r % sg.rot_head - sg.rot_off;         // partner rows are neighbouring lanes
+    const bool turn = f >= 0 && f < sg.rot_dims;
+    const float sign = (f & 1) ? 1.f : -1.f;
+    const float2* rot = sg.rot + (turn ? f >> 1 : 0);
+    float2 cs[32];                                      // all table reads first: between stores the compiler could not move them
+#pragma unroll
+    for (int i = 0; i < 32; ++i) cs[i] = turn && t0 + i < t_end ? __ldg(rot + (int64_t)(t0 + i) * (sg.rot_dims >> 1)) : make_float2(1.f, 0.f);
+#pragma unroll
+    for (int i = 0; i < 32; ++i) {
+      const float w = __shfl_xor_sync(0xffffffffu, v[i], 1);
+      v[i] = v[i] * cs[i].x + sign * (w * cs[i].y);
+    }
+  }
   // bf16: the warp's 32 x 32 block is turned through shared memory, lane L then stores 32 consecutive features of token t0 + L
   __nv_bfloat16* st = reinterpret_cast<__nv_bfloat16*>(stage);
   constexpr int kPitch = 40;

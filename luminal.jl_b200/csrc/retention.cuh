@@ -14,7 +14,8 @@ struct RetentionView {
   const int* len = nullptr;
   const int* pos0 = nullptr;
   int max_len = 1;                    // the longest len (grid sizing)
-  int H = 0, dim = 0, vdim = 0, rot_dims = 0, rot_interleaved = 0;
+  int H = 0, dim = 0, vdim = 0;
+  int rot_dims = 0;                   // features of q and k still to be rotated, in neighbouring pairs (2i, 2i + 1); 0: rotated already
   const float* inv_freq = nullptr;    // [rot_dims / 2]
   const float* decay = nullptr;       // [H][decay_pitch]: powers 0 .. decay_pitch - 1
   int decay_pitch = 0;
@@ -29,7 +30,12 @@ struct RetentionView {
 };
 
 int32_t retention_configure();
-// token after token: decoding, short portions, float32
+// token after token: decoding, short portions, float32, any sizes
 int32_t retention_steps(Ctx* ctx, int dtype, const RetentionView& v, cudaStream_t st);
+// chunks of 64 tokens on the tensor cores: bf16 rows, rotated, gated (raw_gate 0), row-major output
+bool retention_chunks_ok(const RetentionView& v);
+int32_t retention_chunks(Ctx* ctx, const RetentionView& v, cudaStream_t st);
+// angle tables of T tokens: tab[t * n + i] = (cos, sin) of pos[t] * inv_freq[i]
+int32_t angle_table(Ctx* ctx, float2* tab, const float* inv_freq, int n, const int* pos, int T, cudaStream_t st);
 
 }  // namespace lmb
