@@ -1,7 +1,7 @@
 #!/usr/bin/env python
 """Throughput of the B200 backend on the reference's benchmark configurations.
 
-    python bench.py [--config llama3_8b|phi3_mini|whisper_base|small_llama|flash]
+    python bench.py [--config llama3_8b|phi3_mini|whisper_base|small_llama|flash|gibutar]
                     [--gpus N] [--steps K] [--warmup W] [--repeats R] [--impl ours|reference]
 
 Default: the Llama-3-8B-shape decode (32 layers, hidden 4096, 32 q / 8 kv heads x 128, MLP 14336,
@@ -295,6 +295,9 @@ def run_reference(args):
         return
     if args.config == "small_llama":
         return run_reference_small_llama(args)
+    if args.config == "gibutar":
+        print(json.dumps({"impl": "reference", "unavailable": "the reference has no such model"}))
+        return
     name = args.config if args.config in DECODE else "llama3_8b"
     wl = DECODE[name]
     samples, base = [], None
@@ -751,9 +754,143 @@ def run_whisper(args):
     sess.close(); model.close(); enc.close()
 
 
+# -------------------------------------------------------------------------------------------------
+# gibutar: latent attention + retention layers at the sizes of real models' layers, beside Llama at equal width
+# -------------------------------------------------------------------------------------------------
+def gibutar_size(width, heads, ff, kv_rank, q_rank, layers, vocab=32064):
+    """One latent-attention layer to three retention layers, the second latent layer of a pair reading the first one's cache."""
+    dim = width // heads
+    out = []
+    for i in range(layers):
+        if i % 4 == 0:
+            mx = dict(heads=heads, dim=dim, rot_dim=64, vdim=dim, kv_rank=kv_rank, q_rank=q_rank, scale=(dim + 64) ** -0.5,
+                      rot=dict(base=500000.0, dims=64))
+            if i % 8 == 4:
+                mx["kv_from"] = i - 4
+            out.append(dict(type="latent_attention", mixer=mx, mlp=dict(kind="dense", ff=ff)))
+        else:
+            out.append(dict(type="retention", mixer=dict(heads=heads, dim=dim, vdim=dim, rot=dict(base=10000.0, dims=dim),
+                                                         decay=[1.0 - 2.0 ** -(5 + 4 * h / heads) for h in range(heads)]),
+                            mlp=dict(kind="dense", ff=ff)))
+    return dict(architecture="Gibutar", width=width, vocab=vocab, norm=dict(eps=1e-5), logit_softcap=30.0, layers=out)
+
+
+GIBUTAR_SIZES = {
+    "w4096": dict(width=4096, heads=32, ff=14336, kv_rank=512, q_rank=1536, layers=8),
+    "w2048": dict(width=2048, heads=16, ff=8192, kv_rank=512, q_rank=768, layers=8),
+}
+
+
+def gibutar_flops(cfg, n):
+    """Multiply-adds x 2 of one token's share of an n-token prompt (head left out: it runs on the last position only)."""
+    total = 0
+    for layer in cfg["layers"]:
+        mx, W = layer["mixer"], cfg["width"]
+        H, d, v = mx["heads"], mx["dim"], mx["vdim"]
+        total += 4 * W * layer["mlp"]["ff"] + 2 * W * H * v
+        if layer["type"] == "latent_attention":
+            total += 2 * W * (mx["q_rank"] + H) + 2 * mx["q_rank"] * H * (d + mx["rot_dim"]) + 2 * mx["kv_rank"] * H * (d + v)
+            total += 0 if "kv_from" in mx else 2 * W * (mx["kv_rank"] + mx["rot_dim"])
+            total += 2 * H * (d + mx["rot_dim"] + v) * n / 2
+        else:
+            total += 4 * W * H * (d + v) + 4 * H * d * v
+    return total
+
+
+def run_gibutar(args):
+    import numpy as np
+    import torch
+    import luminal_jl_b200 as L
+    D = Dist(1)
+    stream = torch.cuda.Stream()
+    dev = L.B200Device(0, stream=stream.cuda_stream)
+    peaks = load_peaks()
+    steps, warm, ctx = min(args.steps, 64), max(args.warmup, 3), 8192
+    batch, p_batch, p_len = 32, 16, 2048
+    rng = np.random.default_rng(5)
+    sampler = ClockSampler(0)
+    sampler.start()
+
+    def measure(model, flop_per_token):
+        vocab = model.cfg.vocab
+        out = {"weight_bytes": model.weight_bytes()}
+        launches = {}
+        for b in (batch, 1):
+            sess = L.Session(model, b, ctx)
+            first = torch.randint(0, vocab, (b,), dtype=torch.int32, device="cuda")
+            toks = torch.empty((max(steps, warm), b), dtype=torch.int32, device="cuda")
+
+            def prep(_r):
+                sess.fill_kv_random(ctx - steps, seed=3)
+                launches[b] = dev.launch_count()
+            with torch.cuda.stream(stream):
+                sess.fill_kv_random(ctx - steps - warm, seed=3)
+                sess.decode_n_device(first.data_ptr(), warm, toks.data_ptr())
+                ms = median(timed_regions(D, stream, args.repeats, prep, lambda: sess.decode_n_device(first.data_ptr(), steps, toks.data_ptr()))) / steps
+            launches[b] = dev.launch_count() - launches[b]
+            by = sess.step_bytes(ctx - steps // 2)
+            out[f"decode_b{b}"] = {"ms_per_step": ms, "tokens_per_s": b / ms * 1e3, "step_bytes": by, "gbs": by / ms / 1e6, "frac_of_hbm": by / ms / 1e6 / peaks["hbm"],
+                                   "launches_per_step": launches[b] / steps}
+            if b == batch:                                    # the same steps through host buffers
+                tin = torch.randint(0, vocab, (b,), dtype=torch.int32).pin_memory()
+                tout = torch.empty(b, dtype=torch.int32).pin_memory()
+
+                def e2e():
+                    for _ in range(steps):
+                        sess.decode_step_raw(tin.data_ptr(), tout.data_ptr())
+                        tin.copy_(tout)
+                with torch.cuda.stream(stream):
+                    out["e2e_ms_per_step"] = median(timed_regions(D, stream, 3, prep, e2e)) / steps
+            sess.close()
+        for b, n in ((p_batch, p_len), (1, 8192)):
+            sess = L.Session(model, b, n)
+            prompt = rng.integers(0, vocab, (b, n)).astype(np.int32)
+
+            def prompt_run():
+                sess.prefill(prompt, want_logits=False)
+            with torch.cuda.stream(stream):
+                for _ in range(2):
+                    sess.reset()
+                    prompt_run()
+                ms = median(timed_regions(D, stream, args.repeats, lambda _r: sess.reset(), prompt_run))
+            tf = flop_per_token(n) * b * n / ms / 1e9
+            out[f"prefill_{b}x{n}"] = {"ms": ms, "tokens_per_s": b * n / ms * 1e3, "tflops": tf, "frac_of_sustained_bf16": tf / peaks["tf_sustained"]}
+            sess.close()
+        return out, launches[batch]
+
+    variants, total_launches = {}, 0
+    for name, sz in GIBUTAR_SIZES.items():
+        cfg = gibutar_size(**sz)
+        model = L.models.build_model(dev, cfg, "bf16")
+        model.init_random(1234, 0.02)
+        ours, n_launch = measure(model, lambda n: gibutar_flops(cfg, n))
+        total_launches = total_launches or n_launch
+        model.close()
+        kv = max(1, sz["heads"] // 4)
+        lc = dict(n_layers=sz["layers"], hidden=sz["width"], n_heads=sz["heads"], n_kv_heads=kv, intermediate=sz["ff"], vocab=cfg["vocab"], eps=1e-5, rope_base=500000.0)
+        model = L.Model(dev, dtype="bf16", **lc)
+        model.init_random(1234, 0.02)
+        per_tok = 2 * (model_params(lc) - 2 * lc["vocab"] * lc["hidden"])
+        llama, _ = measure(model, lambda n: per_tok + 4 * lc["n_layers"] * lc["hidden"] * (n / 2.0))
+        model.close()
+        variants[name] = {"sizes": sz, "gibutar": ours, "llama_same_width": llama}
+    head = variants["w4096"]["gibutar"]
+    print(json.dumps({
+        "metric": METRIC, "value": head[f"decode_b{batch}"]["tokens_per_s"], "unit": "tokens/s", "n_gpus": 1, "steps": steps, "warmup": warm,
+        "ms_per_step": head[f"decode_b{batch}"]["ms_per_step"], "higher_is_better": True, "scaling": "weak", "vs_baseline": None, "dtype": "bf16",
+        "data": "synthetic",
+        "config": {"workload": f"Gibutar layers (1 latent attention : 3 retention, feed-forward on every layer), 8 layers, bf16, random weights; decode "
+                               f"batch {batch} and 1 with the context ending at {ctx}, prompts {p_batch} x {p_len} and 1 x 8192; Llama (8 layers, GQA 4:1) at equal width",
+                   "name": "gibutar", "batch": batch,
+                   "l2": "a step streams several GB of weights, latents and states: inputs larger than L2"},
+        "e2e": {"value": batch / head["e2e_ms_per_step"] * 1e3, "unit": "tokens/s", "h2d_bytes_per_step": batch * 4, "d2h_bytes_per_step": batch * 4},
+        "gpu_launches": int(total_launches), "clocks": sampler.stop(), "variants": variants, "roofline": None, "cpu_baseline": None,
+    }))
+
+
 def main():
     ap = argparse.ArgumentParser()
-    ap.add_argument("--config", default="llama3_8b", choices=["llama3_8b", "phi3_mini", "whisper_base", "small_llama", "flash"])
+    ap.add_argument("--config", default="llama3_8b", choices=["llama3_8b", "phi3_mini", "whisper_base", "small_llama", "flash", "gibutar"])
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=256)
     ap.add_argument("--warmup", type=int, default=3)
@@ -775,6 +912,8 @@ def main():
         run_small_llama(args)
     elif args.config == "flash":
         run_flash(args)
+    elif args.config == "gibutar":
+        run_gibutar(args)
     else:
         run_whisper(args)
 
