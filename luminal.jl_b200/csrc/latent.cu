@@ -5,6 +5,7 @@
 
 #include "latent.cuh"
 #include "pdl.cuh"
+#include "tc.cuh"
 
 namespace lmb {
 namespace {
@@ -99,7 +100,7 @@ __global__ void __launch_bounds__(128) latent_rotate_q_kernel(const LatentView v
 
 // one CTA: head blockIdx.x, tokens kTok * blockIdx.y ..
 template <typename WT, typename QT>
-__global__ void __launch_bounds__(256) latent_absorb_kernel(const LatentView v, const QT* __restrict__ q, const WT* __restrict__ w_uk,
+__global__ void __launch_bounds__(256) latent_absorb_kernel(const LatentView v, const QT* __restrict__ q, const WT* __restrict__ w_ukt,
                                                             WT* __restrict__ qa) {
   extern __shared__ float qs[];                        // [dim][kTok]
   pdl_launch_dependents();
@@ -120,13 +121,13 @@ __global__ void __launch_bounds__(256) latent_absorb_kernel(const LatentView v, 
   __syncthreads();
   for (int r = 2 * tid; r < v.kv_rank; r += 512) {     // two latent columns per thread
     const bool two = r + 1 < v.kv_rank;
-    const WT* w = w_uk + (int64_t)h * v.dim * v.kv_rank + r;
+    const WT* w = w_ukt + ((int64_t)h * v.kv_rank + r) * v.dim;
     float a0[kTok], a1[kTok];
 #pragma unroll
     for (int t = 0; t < kTok; ++t) a0[t] = a1[t] = 0.f;
 #pragma unroll 4
     for (int d = 0; d < v.dim; ++d) {
-      const float w0 = to_f32(w[(int64_t)d * v.kv_rank]), w1 = two ? to_f32(w[(int64_t)d * v.kv_rank + 1]) : 0.f;
+      const float w0 = to_f32(w[d]), w1 = two ? to_f32(w[v.dim + d]) : 0.f;
       const float4 x0 = *reinterpret_cast<const float4*>(qs + d * kTok), x1 = *reinterpret_cast<const float4*>(qs + d * kTok + 4);
       const float x[kTok] = {x0.x, x0.y, x0.z, x0.w, x1.x, x1.y, x1.z, x1.w};
 #pragma unroll
@@ -196,12 +197,13 @@ __global__ void __launch_bounds__(kSimple) latent_attend_simple_kernel(const Lat
 }
 
 // ---------------------------------------------------------------------------------------------
-// bf16 absorbed attention, split over the keys.  One CTA = 8 warps: the 16 MT heads of one group of one token against `keys_per_cta`
-// keys in tiles of 64.  The latent rows of a tile arrive once (cp.async, two stages, row pitch an odd number of 16-byte chunks) and serve
-// as keys (S = Q' C^T, 16 keys x 16 heads per warp) and as values (O += P C, every warp a slice of the latent's columns); the scores and
-// the running softmax stay float32.  Splits are merged by the last CTA of a (token, head group) to finish, in split order.
+// bf16 absorbed attention, split over the keys.  One CTA holds the 16 MT heads of one group of one token; its 16 warps are two teams of
+// 8 that take the 32-key tiles of the CTA's share in turn, so that one team's products run during the other's softmax.  A tile's
+// latent rows arrive by bulk copies (one per row, two stages per team; the row pitch is an odd number of 16-byte chunks) and serve as keys
+// (S = Q' C^T: 16 heads x 16 keys x half of the features per warp) and as values (O += P C: every warp a slice of the latent's columns).  Scores
+// and the running softmax stay float32.  Every team leaves (O, max, sum) of its keys; latent_expand merges them.
 // ---------------------------------------------------------------------------------------------
-constexpr int kLatThreads = 256, kLatKeys = 64, kLatStages = 2;
+constexpr int kTeams = 2, kTeamThreads = 256, kLatThreads = kTeams * kTeamThreads, kLatKeys = 32, kLatStages = 2;
 constexpr int kScorePitch = kLatKeys + 4, kProbPitch = kLatKeys + 8;
 
 __device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t addr) {
@@ -210,12 +212,16 @@ __device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t addr) {
 __device__ __forceinline__ void ldsm4_trans(uint32_t (&r)[4], uint32_t addr) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];\n" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
 }
-__device__ __forceinline__ void mma16816(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+__device__ __forceinline__ void mma16816(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
   asm volatile(
       "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
       : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+      : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
 }
+__device__ __forceinline__ void mma16816(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  mma16816(c, a[0], a[1], a[2], a[3], b0, b1);
+}
+__device__ __forceinline__ uint32_t smem_addr(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
 
 struct LatTile {                        // shared-memory shape of a row: latent padded to R16, rotated part padded to P16
   int R16, P16, pitch;                  // pitch in elements
@@ -229,89 +235,107 @@ __host__ __device__ inline LatTile lat_tile(int kv_rank, int rot_dim) {
 }
 size_t lat_smem(int MT, int kv_rank, int rot_dim) {
   const LatTile t = lat_tile(kv_rank, rot_dim);
-  return (size_t)(kLatStages * kLatKeys + MT * 16) * t.pitch * 2 + (size_t)2 * 16 * kScorePitch * 4 + (size_t)MT * 16 * kProbPitch * 2 +
-         (size_t)MT * 16 * 3 * 4;
+  return (size_t)(kTeams * kLatStages * kLatKeys + MT * 16) * t.pitch * 2 +
+         (size_t)kTeams * MT * 16 * (2 * kScorePitch * 4 + kProbPitch * 2 + 4);
 }
-
-__device__ __forceinline__ int lat_keys_per_cta(int n, int nsplit) { return (((n + nsplit - 1) / nsplit + kLatKeys - 1) / kLatKeys) * kLatKeys; }
+// keys per split: every sequence divides its own context by the same split count, in whole tiles of every team
+__host__ __device__ inline int lat_keys_per_cta(int n, int nsplit) {
+  constexpr int unit = kTeams * kLatKeys;
+  return (((n + nsplit - 1) / nsplit + unit - 1) / unit) * unit;
+}
+// partial results of (token, head group, split, team): O [16 MT][kv_rank], then max and sum per head (log2 units)
+__host__ __device__ inline int64_t lat_slot(int M, int kv_rank) { return (int64_t)M * (kv_rank + 2); }
 
 template <int NT, int MT>
 __global__ void __launch_bounds__(kLatThreads, 1) latent_attend_tc_kernel(const LatentView v, const __nv_bfloat16* __restrict__ qa,
-                                                                          const __nv_bfloat16* __restrict__ cache, int nsplit, float* __restrict__ part,
-                                                                          unsigned* __restrict__ counters, float* __restrict__ olat) {
+                                                                          const __nv_bfloat16* __restrict__ cache, int nsplit,
+                                                                          float* __restrict__ part, int* err) {
   extern __shared__ __align__(16) unsigned char sm_raw[];
-  __shared__ int is_last;
+  __shared__ __align__(8) uint64_t full[kTeams][kLatStages];
   const LatTile L = lat_tile(v.kv_rank, v.rot_dim);
   constexpr int M = MT * 16;
-  __nv_bfloat16* sK = reinterpret_cast<__nv_bfloat16*>(sm_raw);                    // [stage][key][pitch]
-  __nv_bfloat16* sQ = sK + kLatStages * kLatKeys * L.pitch;                        // [M][pitch]
-  float* sS = reinterpret_cast<float*>(sQ + M * L.pitch);                          // [2][16][kScorePitch]: head tiles (MT 2) or halves of the features (MT 1)
-  __nv_bfloat16* sP = reinterpret_cast<__nv_bfloat16*>(sS + 2 * 16 * kScorePitch); // [M][kProbPitch]
-  float* sA = reinterpret_cast<float*>(sP + M * kProbPitch);                       // [M] rescale, [M] max, [M] sum
-  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int tid = threadIdx.x, lane = tid & 31, team = tid / kTeamThreads, tt = tid - team * kTeamThreads, warp = tt >> 5;
+  __nv_bfloat16* sK = reinterpret_cast<__nv_bfloat16*>(sm_raw) + team * kLatStages * kLatKeys * L.pitch;        // [stage][key][pitch]
+  __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(sm_raw) + kTeams * kLatStages * kLatKeys * L.pitch;      // [M][pitch]
+  float* sS = reinterpret_cast<float*>(sQ + M * L.pitch) + team * 2 * M * kScorePitch;                          // [half of the features][M][kScorePitch]
+  __nv_bfloat16* sP = reinterpret_cast<__nv_bfloat16*>(reinterpret_cast<float*>(sQ + M * L.pitch) + kTeams * 2 * M * kScorePitch) +
+                      team * M * kProbPitch;                                                                    // [M][kProbPitch]
+  float* sA = reinterpret_cast<float*>(reinterpret_cast<__nv_bfloat16*>(reinterpret_cast<float*>(sQ + M * L.pitch) + kTeams * 2 * M * kScorePitch) +
+                                       kTeams * M * kProbPitch) + team * M;                                     // [M] rescale
   const int groups = (v.H + M - 1) / M;
   const int t = blockIdx.x / groups, hg = blockIdx.x - t * groups;
+  auto team_sync = [&]() { asm volatile("bar.sync %0, %1;\n" ::"r"(1 + team), "n"(kTeamThreads) : "memory"); };
+  if (tid == 0) {
+    for (int i = 0; i < kTeams; ++i)
+      for (int s = 0; s < kLatStages; ++s) tc::mbar_init(&full[i][s], 1);
+    tc::mbar_init_fence();
+  }
+  // the padding between and behind the parts, and rows past the context, are never written by a copy: zero everything once
+  for (int i = tid; i < (kTeams * kLatStages * kLatKeys + M) * L.pitch / 8; i += kLatThreads) reinterpret_cast<uint4*>(sm_raw)[i] = make_uint4(0, 0, 0, 0);
+  tc::fence_async_smem();
   pdl_launch_dependents();
   pdl_wait();
   const int n = v.pos[t] + 1;
   const int kpc = lat_keys_per_cta(n, nsplit);
   const int k_begin = blockIdx.y * kpc, k_end = min(n, k_begin + kpc);
   if (k_begin >= n) return;
-  const int tiles = (k_end - k_begin + kLatKeys - 1) / kLatKeys;
-  const __nv_bfloat16* base = cache + v.seq[t] * v.seq_stride;
-  const int chunks = v.ld >> 3, c_chunks = v.rot >> 3;
-
-  auto load_tile = [&](int j) {
-    __nv_bfloat16* dst = sK + (j & 1) * kLatKeys * L.pitch;
-    const int key0 = k_begin + j * kLatKeys;
-    for (int i = tid; i < kLatKeys * chunks; i += kLatThreads) {
-      const int key = i / chunks, c = i - key * chunks;
-      const int col = c < c_chunks ? c * 8 : L.R16 + (c - c_chunks) * 8;
-      const bool ok = key0 + key < k_end;
-      const uint32_t d = (uint32_t)__cvta_generic_to_shared(dst + key * L.pitch + col);
-      asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"(d), "l"(base + (int64_t)(ok ? key0 + key : k_begin) * v.ld + c * 8),
-                   "r"(ok ? 16 : 0)
-                   : "memory");
-    }
-    asm volatile("cp.async.commit_group;\n" ::: "memory");
-  };
-  // the padding between and behind the parts is never written by a copy: zero it once
-  for (int i = tid; i < (kLatStages * kLatKeys + M) * L.pitch / 8; i += kLatThreads) reinterpret_cast<uint4*>(sm_raw)[i] = make_uint4(0, 0, 0, 0);
   __syncthreads();
-  load_tile(0);
-  if (tiles > 1) load_tile(1);
-  for (int i = tid; i < M * chunks; i += kLatThreads) {
-    const int h = i / chunks, c = i - h * chunks;
-    const int col = c < c_chunks ? c * 8 : L.R16 + (c - c_chunks) * 8;
+  const int all_tiles = (k_end - k_begin + kLatKeys - 1) / kLatKeys;
+  const int tiles = (all_tiles - team + kTeams - 1) / kTeams;         // this team's: team, team + 2, ...
+  const __nv_bfloat16* base = cache + v.seq[t] * v.seq_stride;
+  const bool one_piece = v.rot == L.R16;
+  auto load_tile = [&](int j) {                        // warp 0 of the team: lane r copies row r
+    const int key0 = k_begin + (j * kTeams + team) * kLatKeys, valid = min(kLatKeys, k_end - key0);
+    uint64_t* bar = &full[team][j % kLatStages];
+    if (lane == 0) tc::mbar_expect_tx(bar, (uint32_t)(valid * v.ld * 2));
+    __syncwarp();
+    if (lane < valid) {
+      __nv_bfloat16* dst = sK + ((j % kLatStages) * kLatKeys + lane) * L.pitch;
+      const __nv_bfloat16* src = base + (int64_t)(key0 + lane) * v.ld;
+      if (one_piece) tc::bulk_g2s(dst, src, (uint32_t)(v.ld * 2), bar);
+      else {
+        tc::bulk_g2s(dst, src, (uint32_t)(v.rot * 2), bar);
+        if (v.ld > v.rot) tc::bulk_g2s(dst + L.R16, src + v.rot, (uint32_t)((v.ld - v.rot) * 2), bar);
+      }
+    }
+  };
+  if (warp == 0)
+    for (int j = 0; j < min(tiles, kLatStages); ++j) load_tile(j);
+  const int chunks = v.ld >> 3, c_chunks = v.rot >> 3;
+  for (int h = tid >> 5; h < M; h += kLatThreads / 32)
     if (hg * M + h < v.H)
-      *reinterpret_cast<uint4*>(sQ + h * L.pitch + col) = *reinterpret_cast<const uint4*>(qa + ((int64_t)t * v.H + hg * M + h) * v.ld + c * 8);
-  }
+      for (int c = lane; c < chunks; c += 32)
+        *reinterpret_cast<uint4*>(sQ + h * L.pitch + (c < c_chunks ? c * 8 : L.R16 + (c - c_chunks) * 8)) =
+            *reinterpret_cast<const uint4*>(qa + ((int64_t)t * v.H + hg * M + h) * v.ld + c * 8);
+  __syncthreads();
 
-  const int KS = (L.R16 + L.P16) >> 4;                 // 16-feature steps of the scores
-  const int half = warp & 1, kg = warp >> 1;           // MT 2: head tile; MT 1: which half of the steps
-  const int ks0 = MT == 2 ? 0 : (half ? (KS + 1) / 2 : 0), ks1 = MT == 2 ? KS : (half ? KS : (KS + 1) / 2);
+  // scores: warp = (half of the feature steps, head tile, 16-key group); MT 1: quarters of the steps instead of head tiles
+  const int KS = (L.R16 + L.P16) >> 4;
+  const int khalf = warp & 1, mt = MT == 2 ? (warp >> 1) & 1 : 0, kg = MT == 2 ? warp >> 2 : (warp >> 1) & 1;
+  const bool scorer = MT == 2 || warp < 4;
+  const int ks0 = khalf ? (KS + 1) / 2 : 0, ks1 = khalf ? KS : (KS + 1) / 2;
   float acc[MT][NT][4];
 #pragma unroll
   for (int m = 0; m < MT; ++m)
 #pragma unroll
     for (int i = 0; i < NT; ++i) acc[m][i][0] = acc[m][i][1] = acc[m][i][2] = acc[m][i][3] = 0.f;
-  constexpr int TPR = kLatThreads / M, KPT = kLatKeys / TPR;        // softmax: threads per head, keys per thread
-  const int srow = tid / TPR, spart = tid % TPR;
+  constexpr int TPR = kTeamThreads / M, KPT = kLatKeys / TPR;       // softmax: threads per head, keys per thread
+  const int srow = tt / TPR, spart = tt % TPR;
   const float cs = v.scale * kLog2e;
   float m_run = -CUDART_INF_F, l_run = 0.f;
-  const uint32_t qaddr = (uint32_t)__cvta_generic_to_shared(sQ + ((MT == 2 ? half * 16 : 0) + (lane & 15)) * L.pitch + (lane >> 4) * 8);
+  const uint32_t qaddr = smem_addr(sQ + (mt * 16 + (lane & 15)) * L.pitch + (lane >> 4) * 8);
   const int col0 = warp * NT * 8;                      // this warp's slice of the latent's columns
+  bool dead = false;
 
   for (int j = 0; j < tiles; ++j) {
-    if (j + 1 < tiles) asm volatile("cp.async.wait_group 1;\n" ::: "memory");
-    else asm volatile("cp.async.wait_group 0;\n" ::: "memory");
-    __syncthreads();
-    const __nv_bfloat16* K = sK + (j & 1) * kLatKeys * L.pitch;
-    {
+    tc::mbar_wait(&full[team][j % kLatStages], (j / kLatStages) & 1, dead, err);
+    const __nv_bfloat16* K = sK + (j % kLatStages) * kLatKeys * L.pitch;
+    const int key0 = k_begin + (j * kTeams + team) * kLatKeys;
+    if (scorer) {
       float s0[2][4], s1[2][4];                        // even and odd steps, two 8-key tiles
 #pragma unroll
       for (int i = 0; i < 4; ++i) s0[0][i] = s0[1][i] = s1[0][i] = s1[1][i] = 0.f;
-      const uint32_t kaddr = (uint32_t)__cvta_generic_to_shared(K + (kg * 16 + (lane & 7) + ((lane >> 4) << 3)) * L.pitch + ((lane >> 3) & 1) * 8);
+      const uint32_t kaddr = smem_addr(K + (kg * 16 + (lane & 7) + ((lane >> 4) << 3)) * L.pitch + ((lane >> 3) & 1) * 8);
       int ks = ks0;
 #pragma unroll 2
       for (; ks + 1 < ks1; ks += 2) {
@@ -332,23 +356,21 @@ __global__ void __launch_bounds__(kLatThreads, 1) latent_attend_tc_kernel(const 
         mma16816(s0[0], a, b[0], b[1]);
         mma16816(s0[1], a, b[2], b[3]);
       }
-      float* o = sS + half * 16 * kScorePitch + (lane >> 2) * kScorePitch + kg * 16 + (lane & 3) * 2;
+      float* o = sS + (khalf * M + mt * 16 + (lane >> 2)) * kScorePitch + kg * 16 + (lane & 3) * 2;
 #pragma unroll
       for (int i = 0; i < 2; ++i) {
         *reinterpret_cast<float2*>(o + i * 8) = make_float2(s0[i][0] + s1[i][0], s0[i][1] + s1[i][1]);
         *reinterpret_cast<float2*>(o + 8 * kScorePitch + i * 8) = make_float2(s0[i][2] + s1[i][2], s0[i][3] + s1[i][3]);
       }
     }
-    __syncthreads();
+    team_sync();
     {
       float s[KPT];
       float mx = -CUDART_INF_F;
-      const int key0 = k_begin + j * kLatKeys + spart * KPT;
 #pragma unroll
       for (int i = 0; i < KPT; ++i) {
-        float x = sS[srow * kScorePitch + spart * KPT + i];
-        if (MT == 1) x += sS[16 * kScorePitch + srow * kScorePitch + spart * KPT + i];
-        s[i] = key0 + i < k_end ? x * cs : -CUDART_INF_F;
+        const float x = sS[srow * kScorePitch + spart * KPT + i] + sS[(M + srow) * kScorePitch + spart * KPT + i];
+        s[i] = key0 + spart * KPT + i < k_end ? x * cs : -CUDART_INF_F;
         mx = fmaxf(mx, s[i]);
       }
 #pragma unroll
@@ -368,21 +390,22 @@ __global__ void __launch_bounds__(kLatThreads, 1) latent_attend_tc_kernel(const 
       m_run = mn;
       if (spart == 0) sA[srow] = alpha;
     }
-    __syncthreads();
+    team_sync();
     if (col0 < L.R16) {
 #pragma unroll
       for (int m = 0; m < MT; ++m) {
         const float a0 = sA[m * 16 + (lane >> 2)], a1 = sA[m * 16 + (lane >> 2) + 8];
+        if (__any_sync(0xffffffffu, a0 != 1.f || a1 != 1.f)) {
 #pragma unroll
-        for (int i = 0; i < NT; ++i) { acc[m][i][0] *= a0; acc[m][i][1] *= a0; acc[m][i][2] *= a1; acc[m][i][3] *= a1; }
+          for (int i = 0; i < NT; ++i) { acc[m][i][0] *= a0; acc[m][i][1] *= a0; acc[m][i][2] *= a1; acc[m][i][3] *= a1; }
+        }
       }
 #pragma unroll
       for (int ks = 0; ks < kLatKeys / 16; ++ks) {
         uint32_t p[MT][4];
 #pragma unroll
-        for (int m = 0; m < MT; ++m)
-          ldsm4(p[m], (uint32_t)__cvta_generic_to_shared(sP + (m * 16 + (lane & 15)) * kProbPitch + ks * 16 + (lane >> 4) * 8));
-        const uint32_t vaddr = (uint32_t)__cvta_generic_to_shared(K + (ks * 16 + (lane & 15)) * L.pitch + col0 + (lane >> 4) * 8);
+        for (int m = 0; m < MT; ++m) ldsm4(p[m], smem_addr(sP + (m * 16 + (lane & 15)) * kProbPitch + ks * 16 + (lane >> 4) * 8));
+        const uint32_t vaddr = smem_addr(K + (ks * 16 + (lane & 15)) * L.pitch + col0 + (lane >> 4) * 8);
 #pragma unroll
         for (int i = 0; i < NT; i += 2) {
           if (col0 + i * 8 >= L.R16) break;
@@ -396,15 +419,13 @@ __global__ void __launch_bounds__(kLatThreads, 1) latent_attend_tc_kernel(const 
         }
       }
     }
-    __syncthreads();                                   // the stage is free
-    if (j + 2 < tiles) load_tile(j + 2);
+    team_sync();                                       // the stage, the scores and the probabilities are free
+    if (warp == 0 && j + kLatStages < tiles) load_tile(j + kLatStages);
   }
-  if (spart == 0) { sA[M + srow] = m_run; sA[2 * M + srow] = l_run; }
-  __syncthreads();
   const int R = v.kv_rank;
-  const int nvalid = (n + kpc - 1) / kpc;
-  auto each = [&](auto f) {                            // f(head row, column, value) of this thread's accumulators
-    if (col0 >= L.R16) return;
+  float* mine = part + (((int64_t)blockIdx.x * nsplit + blockIdx.y) * kTeams + team) * lat_slot(M, R);
+  if (spart == 0) { mine[(int64_t)M * R + srow] = m_run; mine[(int64_t)M * R + M + srow] = l_run; }
+  if (col0 < L.R16) {
 #pragma unroll
     for (int m = 0; m < MT; ++m)
 #pragma unroll
@@ -412,50 +433,144 @@ __global__ void __launch_bounds__(kLatThreads, 1) latent_attend_tc_kernel(const 
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int row = m * 16 + (lane >> 2) + (e >> 1) * 8, col = col0 + i * 8 + (lane & 3) * 2 + (e & 1);
-          if (col < R && hg * M + row < v.H) f(row, col, acc[m][i][e]);
+          if (col < R) mine[(int64_t)row * R + col] = acc[m][i][e];
         }
-  };
-  if (nvalid == 1) {
-    each([&](int row, int col, float x) { olat[((int64_t)t * v.H + hg * M + row) * R + col] = x / sA[2 * M + row]; });
-    return;
-  }
-  const int64_t slot_floats = (int64_t)M * (R + 2);
-  float* mine = part + ((int64_t)blockIdx.x * nsplit + blockIdx.y) * slot_floats;
-  each([&](int row, int col, float x) { mine[(int64_t)row * R + col] = x; });
-  if (tid < M) { mine[(int64_t)M * R + tid] = sA[M + tid]; mine[(int64_t)M * R + M + tid] = sA[2 * M + tid]; }
-  __threadfence();
-  __syncthreads();
-  if (tid == 0) {
-    const unsigned prev = atomicAdd(&counters[blockIdx.x], 1u);
-    is_last = prev == (unsigned)nvalid - 1u;
-    if (is_last) counters[blockIdx.x] = 0u;
-  }
-  __syncthreads();
-  if (!is_last) return;
-  __threadfence();
-  const float* p0 = part + (int64_t)blockIdx.x * nsplit * slot_floats;
-  float* wgt = sS;                                     // [M]: 1 / denominator, then the weights split by split
-  if (tid < M) {
-    float mx = -CUDART_INF_F, den = 0.f;
-    for (int i = 0; i < nvalid; ++i) mx = fmaxf(mx, __ldcg(p0 + i * slot_floats + (int64_t)M * R + tid));
-    for (int i = 0; i < nvalid; ++i)
-      den += exp2f(__ldcg(p0 + i * slot_floats + (int64_t)M * R + tid) - mx) * __ldcg(p0 + i * slot_floats + (int64_t)M * R + M + tid);
-    wgt[tid] = mx;
-    wgt[M + tid] = 1.0f / den;
-  }
-  __syncthreads();
-  for (int i = tid; i < M * R; i += kLatThreads) {
-    const int row = i / R, col = i - row * R;
-    if (hg * M + row >= v.H) continue;
-    const float mx = wgt[row], inv = wgt[M + row];
-    float x = 0.f;
-#pragma unroll 4
-    for (int k = 0; k < nvalid; ++k) x += exp2f(__ldcg(p0 + k * slot_floats + (int64_t)M * R + row) - mx) * __ldcg(p0 + k * slot_floats + i);
-    olat[((int64_t)t * v.H + hg * M + row) * R + col] = x * inv;
   }
 }
 
-bool lat_tc_ok(int kv_rank, int rot_dim) { return kv_rank <= 512 && lat_smem(2, kv_rank, rot_dim) <= 220 * 1024; }
+// ---------------------------------------------------------------------------------------------
+// Products of one head's matrix W [N, K] (row-major, 16-byte rows) with up to 16 tokens: 8 warps share the N / 8 column tiles of the CTA's
+// slice.  Within 32 features lane tq takes the eight from 8 tq on for both operands, so every fragment is one 16-byte load.
+// ---------------------------------------------------------------------------------------------
+constexpr int kHeadTok = 16;
+
+// sA: [kHeadTok][pitch] bf16, zero behind K (pitch covers K rounded up to 32); f(token row, column n, value)
+template <typename F>
+__device__ __forceinline__ void head_product(const __nv_bfloat16* __restrict__ W, int N, int K, int n_begin, int n_end, const __nv_bfloat16* sA, int pitch, F f) {
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, tq = lane & 3;
+  for (int n0 = n_begin + warp * 16; n0 < n_end; n0 += 8 * 16) {          // two column tiles at a time
+    float c[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+    const __nv_bfloat16* w0 = W + (int64_t)min(n0 + g, N - 1) * K;
+    const __nv_bfloat16* w1 = W + (int64_t)min(n0 + 8 + g, N - 1) * K;
+#pragma unroll 4
+    for (int k = 8 * tq; k - 8 * tq < K; k += 32) {
+      const bool in = k < K;
+      const uint4 z = make_uint4(0, 0, 0, 0);
+      const uint4 b0 = in ? __ldg(reinterpret_cast<const uint4*>(w0 + k)) : z, b1 = in ? __ldg(reinterpret_cast<const uint4*>(w1 + k)) : z;
+      const uint4 a0 = *reinterpret_cast<const uint4*>(sA + g * pitch + k), a1 = *reinterpret_cast<const uint4*>(sA + (g + 8) * pitch + k);
+      mma16816(c[0], a0.x, a1.x, a0.y, a1.y, b0.x, b0.y);
+      mma16816(c[1], a0.x, a1.x, a0.y, a1.y, b1.x, b1.y);
+      mma16816(c[0], a0.z, a1.z, a0.w, a1.w, b0.z, b0.w);
+      mma16816(c[1], a0.z, a1.z, a0.w, a1.w, b1.z, b1.w);
+    }
+#pragma unroll
+    for (int i = 0; i < 2; ++i)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int n = n0 + 8 * i + 2 * tq + (e & 1);
+        if (n < n_end) f(g + 8 * (e >> 1), n, c[i][e]);
+      }
+  }
+}
+__host__ __device__ inline int head_pitch(int K) { return ((K + 31) & ~31) + 8; }
+
+// queries against the latents: head blockIdx.x, tokens 16 * blockIdx.y .., latent columns of slice blockIdx.z; W_uk as [H, kv_rank, dim]
+template <typename QT>
+__global__ void __launch_bounds__(256) latent_absorb_tc_kernel(const LatentView v, const QT* __restrict__ q, const __nv_bfloat16* __restrict__ w_ukt,
+                                                               __nv_bfloat16* __restrict__ qa) {
+  extern __shared__ __align__(16) unsigned char sm_raw[];
+  __nv_bfloat16* sA = reinterpret_cast<__nv_bfloat16*>(sm_raw);
+  pdl_launch_dependents();
+  pdl_wait();
+  const int h = blockIdx.x, t0 = blockIdx.y * kHeadTok, n = min(kHeadTok, v.T - t0), tid = threadIdx.x;
+  const int qd = v.dim + v.rot_dim, pitch = head_pitch(v.dim);
+  const int64_t qp = (int64_t)v.H * qd;
+  for (int t = tid >> 5; t < kHeadTok; t += 8)
+    for (int d = tid & 31; d < pitch; d += 32)
+      sA[t * pitch + d] = __float2bfloat16_rn(t < n && d < v.dim ? to_f32(q[(t0 + t) * qp + h * qd + d]) : 0.f);
+  if (blockIdx.z == 0)
+    for (int i = tid; i < v.rot_dim * n; i += 256) {
+      const int t = i / v.rot_dim, d = i - t * v.rot_dim;
+      const QT* qr = q + (t0 + t) * qp + h * qd + v.dim;
+      qa[((int64_t)(t0 + t) * v.H + h) * v.ld + v.rot + d] = __float2bfloat16_rn(
+          rotated([&](int j) { return to_f32(qr[j]); }, d, v.q_rotated ? 0 : v.rot_dims, v.rot_interleaved, v.pos[t0 + t], v.inv_freq));
+    }
+  __syncthreads();
+  const int R = v.kv_rank, per = (((R + gridDim.z - 1) / gridDim.z) + 15) & ~15, r0 = blockIdx.z * per;
+  head_product(w_ukt + (int64_t)h * R * v.dim, R, v.dim, r0, min(R, r0 + per), sA, pitch, [&](int t, int r, float x) {
+    if (t < n) qa[((int64_t)(t0 + t) * v.H + h) * v.ld + r] = __float2bfloat16_rn(x);
+  });
+}
+
+// merges the partial results of a head's keys, multiplies the weighted latents out to values and gates them
+__global__ void __launch_bounds__(256) latent_expand_tc_kernel(const LatentView v, const float* __restrict__ part, int nsplit, int M,
+                                                               const __nv_bfloat16* __restrict__ w_uv, const float* __restrict__ gate, int gate_pitch,
+                                                               __nv_bfloat16* __restrict__ out, int ldo, int bp) {
+  extern __shared__ __align__(16) unsigned char sm_raw[];
+  __nv_bfloat16* sA = reinterpret_cast<__nv_bfloat16*>(sm_raw);
+  __shared__ float s_gate[kHeadTok];
+  const int R = v.kv_rank, pitch = head_pitch(R);
+  float* s_w = reinterpret_cast<float*>(sA + kHeadTok * pitch);                // [kHeadTok][nsplit * kTeams] weights of the partial results
+  pdl_launch_dependents();
+  pdl_wait();
+  const int h = blockIdx.x, t0 = blockIdx.y * kHeadTok, n = min(kHeadTok, v.T - t0), tid = threadIdx.x, lane = tid & 31;
+  const int groups = (v.H + M - 1) / M, hg = h / M, row = h - hg * M, np = nsplit * kTeams;
+  const int64_t slot = lat_slot(M, R);
+  for (int t = tid >> 5; t < n; t += 8) {
+    const float* p = part + ((int64_t)(t0 + t) * groups + hg) * np * slot + (int64_t)M * R + row;
+    const int ctx = v.pos[t0 + t] + 1, kpc = lat_keys_per_cta(ctx, nsplit);
+    float mx = -CUDART_INF_F;
+    for (int i = lane; i < np; i += 32) {
+      const int first = (i / kTeams) * kpc + (i % kTeams) * kLatKeys;          // a team without a tile has left (-inf, 0)
+      const float m = first < ctx ? __ldcg(p + i * slot) : -CUDART_INF_F;
+      s_w[t * np + i] = m;
+      mx = fmaxf(mx, m);
+    }
+#pragma unroll
+    for (int off = 16; off > 0; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
+    float den = 0.f;
+    for (int i = lane; i < np; i += 32) {
+      const float m = s_w[t * np + i];
+      const float w = m == -CUDART_INF_F ? 0.f : exp2f(m - mx);
+      s_w[t * np + i] = w;
+      if (w > 0.f) den += w * __ldcg(p + i * slot + M);
+    }
+#pragma unroll
+    for (int off = 16; off > 0; off >>= 1) den += __shfl_xor_sync(0xffffffffu, den, off);
+    if (lane == 0) s_gate[t] = 1.0f / (den * (1.0f + expf(-gate[(int64_t)(t0 + t) * gate_pitch + h])));       // gate / denominator
+  }
+  __syncthreads();
+  for (int i = tid; i < kHeadTok * pitch; i += 256) {
+    const int t = i / pitch, r = i - t * pitch;
+    float x = 0.f;
+    if (t < n && r < R) {
+      const float* p = part + ((int64_t)(t0 + t) * groups + hg) * np * slot + (int64_t)row * R + r;
+#pragma unroll 4
+      for (int k = 0; k < np; ++k) {
+        const float w = s_w[t * np + k];
+        if (w > 0.f) x += w * __ldcg(p + k * slot);
+      }
+      x *= s_gate[t];
+    }
+    sA[i] = __float2bfloat16_rn(x);
+  }
+  __syncthreads();
+  const int V = v.vdim, per = (((V + gridDim.z - 1) / gridDim.z) + 15) & ~15, n0 = blockIdx.z * per;
+  head_product(w_uv + (int64_t)h * V * R, V, R, n0, min(V, n0 + per), sA, pitch, [&](int t, int d, float x) {
+    if (t < n) out[bp > 0 ? Layout<__nv_bfloat16>::x_offset(t0 + t, h * V + d, bp) : (int64_t)(t0 + t) * ldo + h * V + d] = __float2bfloat16_rn(x);
+  });
+}
+
+// column slices that give every SM a CTA, each at least 64 columns
+unsigned head_slices(const Ctx* ctx, int64_t ctas, int N) {
+  int64_t z = ctas >= ctx->sm_count ? 1 : ceil_div(ctx->sm_count, ctas);
+  return (unsigned)std::max<int64_t>(1, std::min<int64_t>(z, N / 64));
+}
+
+constexpr size_t kLatMaxSmem = 220 * 1024;
+bool lat_tc_ok(const LatentView& v) {
+  return v.kv_rank <= 512 && v.kv_rank % 8 == 0 && v.dim % 8 == 0 && lat_smem(2, v.kv_rank, v.rot_dim) <= kLatMaxSmem;
+}
 int lat_mt(int H) { return H > 16 ? 2 : 1; }
 int lat_nt(int kv_rank) { return kv_rank <= 128 ? 2 : (kv_rank <= 256 ? 4 : 8); }
 
@@ -503,8 +618,8 @@ __global__ void __launch_bounds__(256) latent_expand_kernel(const LatentView v, 
 
 int32_t latent_configure() {
 #define LMB_CFG(NT)                                                                                                                  \
-  LMB_CUDA(cudaFuncSetAttribute(latent_attend_tc_kernel<NT, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));           \
-  LMB_CUDA(cudaFuncSetAttribute(latent_attend_tc_kernel<NT, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024))
+  LMB_CUDA(cudaFuncSetAttribute(latent_attend_tc_kernel<NT, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kLatMaxSmem));           \
+  LMB_CUDA(cudaFuncSetAttribute(latent_attend_tc_kernel<NT, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kLatMaxSmem))
   LMB_CFG(2);
   LMB_CFG(4);
   LMB_CFG(8);
@@ -531,58 +646,65 @@ int32_t latent_rotate_q(Ctx* ctx, const LatentView& v, void* q, cudaStream_t st)
   return LMB200_OK;
 }
 
-int32_t latent_absorb(Ctx* ctx, int dtype, const LatentView& v, const void* q, int q_f32, const void* w_uk, void* qa, cudaStream_t st) {
+int32_t latent_absorb(Ctx* ctx, int dtype, const LatentView& v, const void* q, int q_f32, const void* w_ukt, void* qa, cudaStream_t st) {
+  if (dtype == LMB200_BF16 && lat_tc_ok(v)) {
+    const int64_t tg = ceil_div(v.T, kHeadTok);
+    const dim3 grid((unsigned)v.H, (unsigned)tg, head_slices(ctx, v.H * tg, v.kv_rank));
+    const size_t smem = (size_t)kHeadTok * head_pitch(v.dim) * 2;
+    if (q_f32) LMB_CUDA(launch_k(latent_absorb_tc_kernel<float>, grid, dim3(256), smem, st, v, (const float*)q, (const __nv_bfloat16*)w_ukt, (__nv_bfloat16*)qa));
+    else LMB_CUDA(launch_k(latent_absorb_tc_kernel<__nv_bfloat16>, grid, dim3(256), smem, st, v, (const __nv_bfloat16*)q, (const __nv_bfloat16*)w_ukt, (__nv_bfloat16*)qa));
+    ctx->launches++;
+    return LMB200_OK;
+  }
   const dim3 grid((unsigned)v.H, (unsigned)ceil_div(v.T, kTok));
   const size_t smem = (size_t)v.dim * kTok * 4;
   LMB_REQUIRE(smem <= 48 * 1024 && grid.y <= 65535, "latent attention: head width %d, %d tokens", v.dim, v.T);
   if (dtype != LMB200_BF16)
-    LMB_CUDA(launch_k(latent_absorb_kernel<float, float>, grid, dim3(256), smem, st, v, (const float*)q, (const float*)w_uk, (float*)qa));
+    LMB_CUDA(launch_k(latent_absorb_kernel<float, float>, grid, dim3(256), smem, st, v, (const float*)q, (const float*)w_ukt, (float*)qa));
   else if (q_f32)
-    LMB_CUDA(launch_k(latent_absorb_kernel<__nv_bfloat16, float>, grid, dim3(256), smem, st, v, (const float*)q, (const __nv_bfloat16*)w_uk,
+    LMB_CUDA(launch_k(latent_absorb_kernel<__nv_bfloat16, float>, grid, dim3(256), smem, st, v, (const float*)q, (const __nv_bfloat16*)w_ukt,
                       (__nv_bfloat16*)qa));
   else
     LMB_CUDA(launch_k(latent_absorb_kernel<__nv_bfloat16, __nv_bfloat16>, grid, dim3(256), smem, st, v, (const __nv_bfloat16*)q,
-                      (const __nv_bfloat16*)w_uk, (__nv_bfloat16*)qa));
+                      (const __nv_bfloat16*)w_ukt, (__nv_bfloat16*)qa));
   ctx->launches++;
   return LMB200_OK;
 }
 
 // The split whose CTAs fill whole waves of the SMs: cost = waves x (keys per CTA + a fixed share for the queries, the merge and the
 // first tile's latency).  Every sequence divides its own context by the same split count.
-LatentAttnPlan latent_attn_plan(const Ctx* ctx, int dtype, int T, int H, int kv_rank, int rot_dim, int ctx_len) {
+LatentAttnPlan latent_attn_plan(const Ctx* ctx, int dtype, const LatentView& v, int T, int ctx_len) {
   LatentAttnPlan p;
-  if (dtype != LMB200_BF16 || !lat_tc_ok(kv_rank, rot_dim)) return p;
-  const int M = 16 * lat_mt(H);
-  const int64_t pairs = (int64_t)T * ceil_div(H, M), resident = ctx->sm_count;
-  const int64_t max_split = std::min<int64_t>(64, ceil_div(ctx_len, 2 * kLatKeys));
+  p.part_floats = (int64_t)T * v.H * v.kv_rank;                  // the CUDA-core kernel's output
+  if (dtype != LMB200_BF16 || !lat_tc_ok(v)) return p;
+  const int M = 16 * lat_mt(v.H);
+  const int64_t pairs = (int64_t)T * ceil_div(v.H, M), resident = ctx->sm_count;
+  const int64_t max_split = std::max<int64_t>(1, std::min<int64_t>(64, ceil_div(ctx_len, 4 * kLatKeys)));
   int64_t best = 1, best_cost = -1;
-  for (int64_t ns = 1; ns <= std::max<int64_t>(1, max_split); ++ns) {
-    const int64_t keys = round_up(ceil_div(ctx_len, ns), kLatKeys);
-    const int64_t cost = ceil_div(pairs * ns, resident) * (keys + 192);
+  for (int64_t ns = 1; ns <= max_split; ++ns) {
+    const int64_t cost = ceil_div(pairs * ns, resident) * (lat_keys_per_cta(ctx_len, (int)ns) + 192);
     if (best_cost < 0 || cost < best_cost) { best_cost = cost; best = ns; }
   }
   p.nsplit = (int)best;
-  if (best > 1) {
-    p.part_floats = pairs * best * M * (kv_rank + 2);
-    p.counters = pairs;
-  }
+  p.part_floats = pairs * best * kTeams * lat_slot(M, v.kv_rank);
   return p;
 }
 
-int32_t latent_attend(Ctx* ctx, int dtype, const LatentView& v, const void* qa, const void* cache, const LatentAttnPlan& plan, float* part,
-                      unsigned* counters, float* olat, cudaStream_t st) {
-  if (dtype == LMB200_BF16 && plan.nsplit >= 1 && lat_tc_ok(v.kv_rank, v.rot_dim)) {
+int32_t latent_attend(Ctx* ctx, int dtype, const LatentView& v, const void* qa, const void* cache, const LatentAttnPlan& plan, float* part, cudaStream_t st) {
+  if (plan.nsplit >= 1) {
+    LMB_REQUIRE(dtype == LMB200_BF16 && lat_tc_ok(v), "latent attention: the plan is not this layer's");
     const int MT = lat_mt(v.H), NT = lat_nt(v.kv_rank);
     const dim3 grid((unsigned)(v.T * ceil_div(v.H, 16 * MT)), (unsigned)plan.nsplit);
     const size_t smem = lat_smem(MT, v.kv_rank, v.rot_dim);
     auto go = [&](auto kern) {
-      return launch_k(kern, grid, dim3(kLatThreads), smem, st, v, (const __nv_bfloat16*)qa, (const __nv_bfloat16*)cache, plan.nsplit, part, counters, olat);
+      return launch_k(kern, grid, dim3(kLatThreads), smem, st, v, (const __nv_bfloat16*)qa, (const __nv_bfloat16*)cache, plan.nsplit, part, ctx->dev_err);
     };
     if (MT == 1) LMB_CUDA(NT == 2 ? go(latent_attend_tc_kernel<2, 1>) : NT == 4 ? go(latent_attend_tc_kernel<4, 1>) : go(latent_attend_tc_kernel<8, 1>));
     else LMB_CUDA(NT == 2 ? go(latent_attend_tc_kernel<2, 2>) : NT == 4 ? go(latent_attend_tc_kernel<4, 2>) : go(latent_attend_tc_kernel<8, 2>));
     ctx->launches++;
     return LMB200_OK;
   }
+  float* olat = part;
   const size_t smem = (size_t)(v.ld + v.kv_rank + kSimple) * 4;
   LMB_REQUIRE(smem <= 48 * 1024, "latent attention: latent width %d", v.kv_rank);
   LMB_REQUIRE(v.T <= 65535, "latent attention: %d tokens in one absorbed launch", v.T);
@@ -596,8 +718,18 @@ int32_t latent_attend(Ctx* ctx, int dtype, const LatentView& v, const void* qa, 
   return LMB200_OK;
 }
 
-int32_t latent_expand(Ctx* ctx, int dtype, const LatentView& v, const float* olat, const void* w_uv, const float* gate, int gate_pitch,
-                      void* out, int ldo, int bp, cudaStream_t st) {
+int32_t latent_expand(Ctx* ctx, int dtype, const LatentView& v, const float* part, const LatentAttnPlan& plan, const void* w_uv, const float* gate,
+                      int gate_pitch, void* out, int ldo, int bp, cudaStream_t st) {
+  if (plan.nsplit >= 1) {
+    const int64_t tg = ceil_div(v.T, kHeadTok);
+    const dim3 grid((unsigned)v.H, (unsigned)tg, head_slices(ctx, v.H * tg, v.vdim));
+    const size_t smem = (size_t)kHeadTok * head_pitch(v.kv_rank) * 2 + (size_t)kHeadTok * plan.nsplit * kTeams * 4;
+    LMB_CUDA(launch_k(latent_expand_tc_kernel, grid, dim3(256), smem, st, v, part, plan.nsplit, 16 * lat_mt(v.H), (const __nv_bfloat16*)w_uv, gate,
+                      gate_pitch, (__nv_bfloat16*)out, ldo, bp));
+    ctx->launches++;
+    return LMB200_OK;
+  }
+  const float* olat = part;
   const dim3 grid((unsigned)v.H, (unsigned)ceil_div(v.T, kTok));
   const size_t smem = (size_t)kTok * v.kv_rank * 4;
   LMB_REQUIRE(smem <= 48 * 1024 && grid.y <= 65535, "latent attention: latent width %d, %d tokens", v.kv_rank, v.T);

@@ -33,15 +33,16 @@ int32_t latent_prep(Ctx* ctx, int dtype, const LatentView& v, const float* proj,
                     const float* kv_norm, void* xq, int ldxq, int bp, void* cache, void* packed, cudaStream_t st);
 // q [T, H * (dim + rot_dim)] (float32 if q_f32, else the model dtype) -> qa [T, H, ld] in the model dtype, ordered like a cache
 // row: the absorbed part and the rotated part
-int32_t latent_absorb(Ctx* ctx, int dtype, const LatentView& v, const void* q, int q_f32, const void* w_uk, void* qa, cudaStream_t st);
-// softmax over positions 0 .. pos[t] of the token's sequence: olat [T, H, kv_rank] float32
-struct LatentAttnPlan { int nsplit = 0; int64_t part_floats = 0, counters = 0; };      // nsplit 0: the CUDA-core kernel
-LatentAttnPlan latent_attn_plan(const Ctx* ctx, int dtype, int T, int H, int kv_rank, int rot_dim, int ctx_len);
-int32_t latent_attend(Ctx* ctx, int dtype, const LatentView& v, const void* qa, const void* cache, const LatentAttnPlan& plan, float* part,
-                      unsigned* counters, float* olat, cudaStream_t st);
+// (w_ukt: W_uk with every head transposed, [H, kv_rank, dim])
+int32_t latent_absorb(Ctx* ctx, int dtype, const LatentView& v, const void* q, int q_f32, const void* w_ukt, void* qa, cudaStream_t st);
+// softmax over positions 0 .. pos[t] of the token's sequence: the weighted latents, as partial results per share of the keys (nsplit >= 1)
+// or whole (nsplit 0, the CUDA-core kernel); part holds plan.part_floats
+struct LatentAttnPlan { int nsplit = 0; int64_t part_floats = 0; };
+LatentAttnPlan latent_attn_plan(const Ctx* ctx, int dtype, const LatentView& v, int T, int ctx_len);
+int32_t latent_attend(Ctx* ctx, int dtype, const LatentView& v, const void* qa, const void* cache, const LatentAttnPlan& plan, float* part, cudaStream_t st);
 // out[t, a * vdim + i] = sigmoid(gate[t, a]) (Wuv_a olat[t, a])_i in the model dtype, row-major [T, ldo] or GEMV activations (bp > 0)
-int32_t latent_expand(Ctx* ctx, int dtype, const LatentView& v, const float* olat, const void* w_uv, const float* gate, int gate_pitch,
-                      void* out, int ldo, int bp, cudaStream_t st);
+int32_t latent_expand(Ctx* ctx, int dtype, const LatentView& v, const float* part, const LatentAttnPlan& plan, const void* w_uv, const float* gate,
+                      int gate_pitch, void* out, int ldo, int bp, cudaStream_t st);
 // rotates the positional part of q [T, H * (dim + rot_dim)] in place (bf16; where the projection's epilogue could not)
 int32_t latent_rotate_q(Ctx* ctx, const LatentView& v, void* q, cudaStream_t st);
 

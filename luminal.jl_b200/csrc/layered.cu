@@ -27,7 +27,7 @@ struct RowsBuf {
   int64_t cap_T = 0;
   void* base = nullptr;
   int64_t bytes = 0;
-  float *x = nullptr, *delta = nullptr, *proj = nullptr, *olat = nullptr;
+  float *x = nullptr, *delta = nullptr, *proj = nullptr;
   void *xn = nullptr, *xq = nullptr, *q = nullptr, *qa = nullptr, *cat = nullptr, *packed = nullptr;
   float2* angles = nullptr;     // [Model::rot_freqs][cap_T][max_half] (cos, sin) of the tokens' positions
   int max_half = 0;
@@ -38,20 +38,18 @@ struct RowsBuf {
 
 struct LayeredScratch {
   // fused step
-  float *proj = nullptr, *qf = nullptr, *olat = nullptr;
+  float *proj = nullptr, *qf = nullptr;
   void *xq = nullptr, *qa = nullptr;
   std::vector<GemvPlan> p_in, p_out, p_uq;
   int *iota = nullptr, *ones = nullptr;          // [B]
   std::vector<LatentAttnPlan> attn;              // per layer, one token per sequence at the session's capacity
   float* attn_part = nullptr;
-  unsigned* attn_counters = nullptr;
   RowsBuf step, prompt;                          // float32 decode step; everything longer
   float* want_logits = nullptr;
   void* want_xn = nullptr;
   int64_t want_cap = 0;
-  float* prompt_part = nullptr;                  // split partials of the absorbed attention in a rows step
-  unsigned* prompt_counters = nullptr;
-  int64_t prompt_part_floats = 0, prompt_counter_cap = 0;
+  float* prompt_part = nullptr;                  // partial results of the absorbed attention in a rows step
+  int64_t prompt_part_floats = 0;
   void* expanded = nullptr;                      // keys and values multiplied out of the latents (long portions)
   int64_t expanded_bytes = 0;
 };
@@ -155,6 +153,7 @@ struct Target {
   int slot = 0;
   void* plain = nullptr;         // row-major copy in the model dtype (float32 for vectors)
   bool vec = false;
+  int head = 0;                  // the copy holds heads of this many rows transposed
   int64_t rows = 0, cols = 0;
 };
 
@@ -185,7 +184,7 @@ bool find_target(Model* M, const std::string& n, Target* t) {
     if (tail == "mix.g") return mat(w.w_in, s.m_in, L_G);
     if (s.c.kv_from < 0 && tail == "mix.dkv") return mat(w.w_in, s.m_in, L_DKV);
     if (s.c.kv_from < 0 && tail == "mix.dkv.norm") return vec(w.kv_norm, s.c.kv_rank);
-    if (tail == "mix.uk") { mat(w.w_ukv, s.m_ukv, 0); t->plain = w.w_uk; return true; }
+    if (tail == "mix.uk") { mat(w.w_ukv, s.m_ukv, 0); t->plain = w.w_ukt; t->head = s.c.dim; return true; }
     if (tail == "mix.uv") { mat(w.w_ukv, s.m_ukv, 1); t->plain = w.w_uv; return true; }
     return false;
   }
@@ -199,7 +198,7 @@ bool find_target(Model* M, const std::string& n, Target* t) {
 // fills a tensor from `src` (device float32) or, src == NULL, from the generator
 int32_t fill_target(Model* M, const Target& t, uint64_t key, const float* src, int layout, float scale) {
   if (t.vec) return fill_plain_dt(M, LMB200_F32, t.plain, t.rows, t.cols, key, src, 0, scale, src ? 0.f : 1.f);
-  if (t.plain) LMB_TRY(fill_plain_dt(M, M->cfg.dtype, t.plain, t.rows, t.cols, key, src, layout, scale, 0.f));
+  if (t.plain) LMB_TRY(fill_plain_dt(M, M->cfg.dtype, t.plain, t.rows, t.cols, key, src, layout, scale, 0.f, t.head));
   if (!t.tiled) return LMB200_OK;
   FillSrc f{};
   f.only_slot = t.slot; f.colmajor = layout; f.scale = scale;
@@ -211,7 +210,7 @@ int32_t fill_target(Model* M, const Target& t, uint64_t key, const float* src, i
 
 void layered_free_model(Model* M) {
   for (LayeredWeights& w : M->lw) {
-    cudaFree(w.w_in); cudaFree(w.w_out); cudaFree(w.w_uq); cudaFree(w.w_ukv); cudaFree(w.w_uk); cudaFree(w.w_uv);
+    cudaFree(w.w_in); cudaFree(w.w_out); cudaFree(w.w_uq); cudaFree(w.w_ukv); cudaFree(w.w_ukt); cudaFree(w.w_uv);
     cudaFree(w.norm); cudaFree(w.q_norm); cudaFree(w.kv_norm); cudaFree(w.inv_freq); cudaFree(w.decay);
   }
   M->lw.clear();
@@ -307,7 +306,6 @@ int32_t ensure_rows(Session* S, RowsBuf& r, int64_t T, int64_t n_want) {
       {&r.xq, T * row_ld((int)max_over(M, [](const LayerSpec& s) { return s.c.q_rank; })) * e},
       {&r.q, T * max_over(M, [](const LayerSpec& s) { return is_latent(s) ? q_width(s) : 0; }) * e},
       {&r.qa, blk * max_over(M, [](const LayerSpec& s) { return is_latent(s) ? (int64_t)s.c.heads * s.lat_ld : 0; }) * e},
-      {(void**)&r.olat, blk * max_over(M, [](const LayerSpec& s) { return is_latent(s) ? (int64_t)s.c.heads * s.c.kv_rank : 0; }) * 4},
       {&r.cat, T * max_over(M, [](const LayerSpec& s) { return row_ld(s.m_out.K); }) * e},
       {&r.packed, T * max_over(M, [](const LayerSpec& s) { return is_latent(s) ? s.lat_ld : 0; }) * e},
       {(void**)&r.angles, M->cfg.dtype == LMB200_BF16 ? (int64_t)M->rot_freqs.size() * T * r.max_half * 8 : 0},
@@ -480,7 +478,7 @@ int32_t rotate_segment(Session* S, RowsBuf& r, const RowsRun& run, int l, RowSeg
   return LMB200_OK;
 }
 
-// split scratch of the absorbed attention in a rows step (the counters are zero between launches)
+// scratch of the absorbed attention in a rows step
 int32_t ensure_attn_scratch(Session* S, const LatentAttnPlan& plan) {
   LayeredScratch& Z = *S->lay;
   cudaStream_t st = S->m->ctx->stream;
@@ -489,12 +487,6 @@ int32_t ensure_attn_scratch(Session* S, const LatentAttnPlan& plan) {
     Z.prompt_part = nullptr; Z.prompt_part_floats = 0;
     LMB_TRY(dmalloc((void**)&Z.prompt_part, plan.part_floats * 4, false, st));
     Z.prompt_part_floats = plan.part_floats;
-  }
-  if (plan.counters > Z.prompt_counter_cap) {
-    cudaFree(Z.prompt_counters);
-    Z.prompt_counters = nullptr; Z.prompt_counter_cap = 0;
-    LMB_TRY(dmalloc((void**)&Z.prompt_counters, plan.counters * 4, true, st));
-    Z.prompt_counter_cap = plan.counters;
   }
   return LMB200_OK;
 }
@@ -532,11 +524,12 @@ int32_t latent_rows(Session* S, RowsBuf& r, const RowsRun& run, int l, bool grap
     for (; t0 < t1; t0 += kBlockTokens) {
       LatentView b = v;
       b.T = std::min(kBlockTokens, t1 - t0); b.seq = run.seq + t0; b.pos = run.pos + t0;
-      LMB_TRY(latent_absorb(ctx, dt, b, (const char*)r.q + (int64_t)t0 * q_width(s) * e, 0, w.w_uk, r.qa, st));
-      const LatentAttnPlan plan = graph ? Z.attn[l] : latent_attn_plan(ctx, dt, b.T, b.H, b.kv_rank, b.rot_dim, run.ctx_len);
+      LMB_TRY(latent_absorb(ctx, dt, b, (const char*)r.q + (int64_t)t0 * q_width(s) * e, 0, w.w_ukt, r.qa, st));
+      const LatentAttnPlan plan = graph ? Z.attn[l] : latent_attn_plan(ctx, dt, b, b.T, run.ctx_len);
       if (!graph) LMB_TRY(ensure_attn_scratch(S, plan));
-      LMB_TRY(latent_attend(ctx, dt, b, r.qa, cache, plan, graph ? Z.attn_part : Z.prompt_part, graph ? Z.attn_counters : Z.prompt_counters, r.olat, st));
-      LMB_TRY(latent_expand(ctx, dt, b, r.olat, w.w_uv, gate + (int64_t)t0 * s.n_store, s.n_store, (char*)r.cat + (int64_t)t0 * ldc * e, ldc, 0, st));
+      float* part = graph ? Z.attn_part : Z.prompt_part;
+      LMB_TRY(latent_attend(ctx, dt, b, r.qa, cache, plan, part, st));
+      LMB_TRY(latent_expand(ctx, dt, b, part, plan, w.w_uv, gate + (int64_t)t0 * s.n_store, s.n_store, (char*)r.cat + (int64_t)t0 * ldc * e, ldc, 0, st));
     }
     return LMB200_OK;
   };
@@ -693,9 +686,9 @@ int32_t fused_step(Session* S, cudaStream_t st, bool with_head) {
       p.epi = EPI_STORE_F32; p.out = Z.qf; p.out_pitch = q_width(s);
       gemv_prefetch_next(p, ctx, dt, w.w_out, s.m_out.rows, s.m_out.K, Z.p_out[l]);
       LMB_TRY(gemv_launch(ctx, dt, p, st));
-      LMB_TRY(latent_absorb(ctx, dt, v, Z.qf, 1, w.w_uk, Z.qa, st));
-      LMB_TRY(latent_attend(ctx, dt, v, Z.qa, cache, Z.attn[l], Z.attn_part, Z.attn_counters, Z.olat, st));
-      LMB_TRY(latent_expand(ctx, dt, v, Z.olat, w.w_uv, Z.proj + s.row0[L_G], s.n_store, S->act, 0, S->Bp, st));
+      LMB_TRY(latent_absorb(ctx, dt, v, Z.qf, 1, w.w_ukt, Z.qa, st));
+      LMB_TRY(latent_attend(ctx, dt, v, Z.qa, cache, Z.attn[l], Z.attn_part, st));
+      LMB_TRY(latent_expand(ctx, dt, v, Z.attn_part, Z.attn[l], w.w_uv, Z.proj + s.row0[L_G], s.n_store, S->act, 0, S->Bp, st));
     } else {
       RetentionView v = retention_view(S, l);
       v.start = Z.iota; v.len = Z.ones; v.pos0 = S->pos;
@@ -776,7 +769,7 @@ int32_t layered_session_create(Model* M, int batch, int max_ctx, lmb200_session*
   auto alloc = [&](void** p, int64_t bytes) { if (rc == LMB200_OK) rc = dmalloc(p, bytes, true, ctx->stream); };
   S->latent.assign(c.n_layers, nullptr);
   S->state.assign(c.n_layers, nullptr);
-  int64_t lat_parts = 0, lat_counters = 0;
+  int64_t lat_parts = 0;
   for (int l = 0; l < c.n_layers; ++l) {
     const LayerSpec& s = M->specs[l];
     if (!is_latent(s)) { alloc((void**)&S->state[l], (int64_t)batch * s.c.heads * s.c.dim * state_ld(s) * 4); continue; }
@@ -786,9 +779,8 @@ int32_t layered_session_create(Model* M, int batch, int max_ctx, lmb200_session*
   for (int l = 0; l < c.n_layers; ++l) {
     const LayerSpec& s = M->specs[l];
     if (!is_latent(s)) continue;
-    Z.attn[l] = latent_attn_plan(ctx, c.dtype, batch, s.c.heads, s.c.kv_rank, s.c.rot_dim, S->cap);
+    Z.attn[l] = latent_attn_plan(ctx, c.dtype, latent_view(S, l), batch, S->cap);
     lat_parts = std::max(lat_parts, Z.attn[l].part_floats);
-    lat_counters = std::max(lat_counters, Z.attn[l].counters);
   }
   if (bf) {
     int64_t max_part = 0;
@@ -813,13 +805,11 @@ int32_t layered_session_create(Model* M, int batch, int max_ctx, lmb200_session*
     alloc((void**)&Z.qf, batch * max_over(M, [](const LayerSpec& s) { return is_latent(s) ? q_width(s) : 0; }) * 4);
     alloc(&Z.xq, x_bytes(std::max<int64_t>(1, max_over(M, [](const LayerSpec& s) { return s.c.q_rank; }))));
     alloc(&Z.qa, batch * max_over(M, [](const LayerSpec& s) { return is_latent(s) ? (int64_t)s.c.heads * s.lat_ld : 0; }) * 2);
-    alloc((void**)&Z.olat, batch * max_over(M, [](const LayerSpec& s) { return is_latent(s) ? (int64_t)s.c.heads * s.c.kv_rank : 0; }) * 4);
     S->fused = true;
   } else if (rc == LMB200_OK) {
     rc = ensure_rows(S, Z.step, batch, 0);
   }
   alloc((void**)&Z.attn_part, lat_parts * 4);
-  alloc((void**)&Z.attn_counters, lat_counters * 4);
   alloc((void**)&S->logits, (int64_t)batch * S->logits_pitch * 4);
   alloc((void**)&S->tokens, (int64_t)batch * 4);
   alloc((void**)&S->pos, (int64_t)batch * 4);
@@ -853,8 +843,8 @@ void layered_session_free(Session* S) {
   S->state.clear();
   if (!S->lay) return;
   LayeredScratch& Z = *S->lay;
-  cudaFree(Z.proj); cudaFree(Z.qf); cudaFree(Z.olat); cudaFree(Z.xq); cudaFree(Z.qa); cudaFree(Z.iota); cudaFree(Z.ones);
-  cudaFree(Z.attn_part); cudaFree(Z.attn_counters); cudaFree(Z.prompt_part); cudaFree(Z.prompt_counters);
+  cudaFree(Z.proj); cudaFree(Z.qf); cudaFree(Z.xq); cudaFree(Z.qa); cudaFree(Z.iota); cudaFree(Z.ones);
+  cudaFree(Z.attn_part); cudaFree(Z.prompt_part);
   cudaFree(Z.want_logits); cudaFree(Z.want_xn); cudaFree(Z.expanded);
   free_rows(Z.step);
   free_rows(Z.prompt);
@@ -1062,7 +1052,7 @@ extern "C" int32_t lmb200_model_create_layered(lmb200_ctx hctx, const lmb200_lay
     if (is_latent(s)) {
       alloc(&w.w_uq, tiled_elems(s.m_uq, c.dtype) * M->esz);
       alloc(&w.w_ukv, tiled_elems(s.m_ukv, c.dtype) * M->esz);
-      alloc(&w.w_uk, (int64_t)s.c.heads * s.c.dim * s.c.kv_rank * M->esz);
+      alloc(&w.w_ukt, (int64_t)s.c.heads * s.c.dim * s.c.kv_rank * M->esz);
       alloc(&w.w_uv, (int64_t)s.c.heads * s.c.vdim * s.c.kv_rank * M->esz);
       alloc((void**)&w.q_norm, (int64_t)s.c.q_rank * 4);
       if (s.c.kv_from < 0) alloc((void**)&w.kv_norm, (int64_t)s.c.kv_rank * 4);

@@ -107,7 +107,7 @@ __global__ void fill_tiled_kernel(WT* dst, WMap m, FillSrc f) {
 // plain row-major tensors (embedding table, norm gains)
 template <typename WT>
 __global__ void fill_plain_kernel(WT* dst, int64_t rows, int64_t cols, uint64_t key, const float* src,
-                                  int colmajor, float scale, float offset) {
+                                  int colmajor, float scale, float offset, int head) {
   const int64_t total = rows * cols;
   for (int64_t o = blockIdx.x * (int64_t)blockDim.x + threadIdx.x; o < total;
        o += (int64_t)gridDim.x * blockDim.x) {
@@ -118,7 +118,12 @@ __global__ void fill_plain_kernel(WT* dst, int64_t rows, int64_t cols, uint64_t 
     } else {
       v = synth_value(key, (uint64_t)o, scale, offset);
     }
-    dst[o] = from_f32<WT>(v);
+    int64_t at = o;
+    if (head > 0) {
+      const int64_t r = o / cols, c = o - r * cols, h = r / head;
+      at = (h * cols + c) * head + (r - h * head);
+    }
+    dst[at] = from_f32<WT>(v);
   }
 }
 
@@ -774,18 +779,18 @@ int32_t fill_tiled_dt(Model* M, void* dst, const WMap& m, const FillSrc& f) {
 }
 template <typename WT>
 static int32_t fill_plain(Ctx* ctx, void* dst, int64_t rows, int64_t cols, uint64_t key, const float* src,
-                   int colmajor, float scale, float offset) {
+                   int colmajor, float scale, float offset, int head = 0) {
   fill_plain_kernel<WT><<<fill_grid(rows * cols), 256, 0, ctx->stream>>>(reinterpret_cast<WT*>(dst), rows, cols, key,
-                                                                         src, colmajor, scale, offset);
+                                                                         src, colmajor, scale, offset, head);
   ctx->launches++;
   LMB_CUDA(cudaGetLastError());
   return LMB200_OK;
 }
 
 int32_t fill_plain_dt(Model* M, int dtype, void* dst, int64_t rows, int64_t cols, uint64_t key, const float* src, int colmajor, float scale,
-                      float offset) {
-  return dtype == LMB200_BF16 ? fill_plain<__nv_bfloat16>(M->ctx, dst, rows, cols, key, src, colmajor, scale, offset)
-                              : fill_plain<float>(M->ctx, dst, rows, cols, key, src, colmajor, scale, offset);
+                      float offset, int head) {
+  return dtype == LMB200_BF16 ? fill_plain<__nv_bfloat16>(M->ctx, dst, rows, cols, key, src, colmajor, scale, offset, head)
+                              : fill_plain<float>(M->ctx, dst, rows, cols, key, src, colmajor, scale, offset, head);
 }
 
 void finish_map(WMap& m) {

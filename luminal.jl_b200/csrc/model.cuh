@@ -79,7 +79,7 @@ struct LayerSpec {
 };
 struct LayeredWeights {
   void *w_in = nullptr, *w_out = nullptr, *w_uq = nullptr, *w_ukv = nullptr;
-  void *w_uk = nullptr, *w_uv = nullptr;      // row-major [heads * dim, kv_rank] and [heads * vdim, kv_rank] (absorbed attention)
+  void *w_ukt = nullptr, *w_uv = nullptr;     // row-major [heads, kv_rank, dim] and [heads * vdim, kv_rank] (absorbed attention)
   float *norm = nullptr, *q_norm = nullptr, *kv_norm = nullptr;
   float *inv_freq = nullptr;                  // [rot_dims / 2]
   int rot_id = -1;                            // layers with the same frequencies share an angle table (Model::rot_freqs)
@@ -243,8 +243,9 @@ struct FillSrc {
   float scale;             // sigma / 131072
 };
 int32_t fill_tiled_dt(Model* M, void* dst, const WMap& m, const FillSrc& f);
+// head > 0: every block of `head` rows is stored transposed, [rows / head, cols, head]
 int32_t fill_plain_dt(Model* M, int dtype, void* dst, int64_t rows, int64_t cols, uint64_t key, const float* src, int colmajor, float scale,
-                      float offset);
+                      float offset, int head = 0);
 int32_t check_weight_shape(const char* name, int32_t rank, const int64_t* dims, int64_t rows, int64_t cols);
 int64_t tiled_elems(const WMap& m, int dtype);
 void finish_map(WMap& m);
