@@ -200,11 +200,11 @@ __global__ void __launch_bounds__(kSimple) latent_attend_simple_kernel(const Lat
 // bf16 absorbed attention, split over the keys.  One CTA holds the 16 MT heads of one group of one token; its 16 warps are two teams of
 // 8 that take the 32-key tiles of the CTA's share in turn, so that one team's products run during the other's softmax.  A tile's
 // latent rows arrive by bulk copies (one per row, two stages per team; the row pitch is an odd number of 16-byte chunks) and serve as keys
-// (S = Q' C^T: 16 heads x 16 keys x half of the features per warp) and as values (O += P C: every warp a slice of the latent's columns).  Scores
+// (S = Q' C^T: all heads x 16 keys x a quarter of the features per warp) and as values (O += P C: every warp a slice of the latent's columns).  Scores
 // and the running softmax stay float32.  Every team leaves (O, max, sum) of its keys; latent_expand merges them.
 // ---------------------------------------------------------------------------------------------
 constexpr int kTeams = 2, kTeamThreads = 256, kLatThreads = kTeams * kTeamThreads, kLatKeys = 32, kLatStages = 2;
-constexpr int kScorePitch = kLatKeys + 4, kProbPitch = kLatKeys + 8;
+constexpr int kScorePitch = kLatKeys + 4, kProbPitch = kLatKeys + 8, kParts = 4;      // kParts: the features of a score are summed in four parts
 
 __device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t addr) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];\n" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
@@ -221,6 +221,11 @@ __device__ __forceinline__ void mma16816(float (&c)[4], uint32_t a0, uint32_t a1
 __device__ __forceinline__ void mma16816(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
   mma16816(c, a[0], a[1], a[2], a[3], b0, b1);
 }
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
+  return y;
+}
 __device__ __forceinline__ uint32_t smem_addr(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
 
 struct LatTile {                        // shared-memory shape of a row: latent padded to R16, rotated part padded to P16
@@ -236,7 +241,7 @@ __host__ __device__ inline LatTile lat_tile(int kv_rank, int rot_dim) {
 size_t lat_smem(int MT, int kv_rank, int rot_dim) {
   const LatTile t = lat_tile(kv_rank, rot_dim);
   return (size_t)(kTeams * kLatStages * kLatKeys + MT * 16) * t.pitch * 2 +
-         (size_t)kTeams * MT * 16 * (2 * kScorePitch * 4 + kProbPitch * 2 + 4);
+         (size_t)kTeams * MT * 16 * (kParts * kScorePitch * 4 + kProbPitch * 2 + 4);
 }
 // keys per split: every sequence divides its own context by the same split count, in whole tiles of every team
 __host__ __device__ inline int lat_keys_per_cta(int n, int nsplit) {
@@ -257,11 +262,11 @@ __global__ void __launch_bounds__(kLatThreads, 1) latent_attend_tc_kernel(const 
   const int tid = threadIdx.x, lane = tid & 31, team = tid / kTeamThreads, tt = tid - team * kTeamThreads, warp = tt >> 5;
   __nv_bfloat16* sK = reinterpret_cast<__nv_bfloat16*>(sm_raw) + team * kLatStages * kLatKeys * L.pitch;        // [stage][key][pitch]
   __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(sm_raw) + kTeams * kLatStages * kLatKeys * L.pitch;      // [M][pitch]
-  float* sS = reinterpret_cast<float*>(sQ + M * L.pitch) + team * 2 * M * kScorePitch;                          // [half of the features][M][kScorePitch]
-  __nv_bfloat16* sP = reinterpret_cast<__nv_bfloat16*>(reinterpret_cast<float*>(sQ + M * L.pitch) + kTeams * 2 * M * kScorePitch) +
-                      team * M * kProbPitch;                                                                    // [M][kProbPitch]
-  float* sA = reinterpret_cast<float*>(reinterpret_cast<__nv_bfloat16*>(reinterpret_cast<float*>(sQ + M * L.pitch) + kTeams * 2 * M * kScorePitch) +
-                                       kTeams * M * kProbPitch) + team * M;                                     // [M] rescale
+  float* scores = reinterpret_cast<float*>(sQ + M * L.pitch);
+  float* sS = scores + team * kParts * M * kScorePitch;                                                         // [part][M][kScorePitch]
+  __nv_bfloat16* probs = reinterpret_cast<__nv_bfloat16*>(scores + kTeams * kParts * M * kScorePitch);
+  __nv_bfloat16* sP = probs + team * M * kProbPitch;                                                            // [M][kProbPitch]
+  float* sA = reinterpret_cast<float*>(probs + kTeams * M * kProbPitch) + team * M;                             // [M] rescale
   const int groups = (v.H + M - 1) / M;
   const int t = blockIdx.x / groups, hg = blockIdx.x - t * groups;
   auto team_sync = [&]() { asm volatile("bar.sync %0, %1;\n" ::"r"(1 + team), "n"(kTeamThreads) : "memory"); };
@@ -284,14 +289,15 @@ __global__ void __launch_bounds__(kLatThreads, 1) latent_attend_tc_kernel(const 
   const int tiles = (all_tiles - team + kTeams - 1) / kTeams;         // this team's: team, team + 2, ...
   const __nv_bfloat16* base = cache + v.seq[t] * v.seq_stride;
   const bool one_piece = v.rot == L.R16;
-  auto load_tile = [&](int j) {                        // warp 0 of the team: lane r copies row r
-    const int key0 = k_begin + (j * kTeams + team) * kLatKeys, valid = min(kLatKeys, k_end - key0);
+  // every warp of the team issues the copies of four rows (one warp for all of them would hold the others up at the next barrier)
+  auto load_tile = [&](int j) {
+    constexpr int kRows = kLatKeys / (kTeamThreads / 32);
+    const int key0 = k_begin + (j * kTeams + team) * kLatKeys, valid = min(kLatKeys, k_end - key0), row = warp * kRows + lane;
     uint64_t* bar = &full[team][j % kLatStages];
-    if (lane == 0) tc::mbar_expect_tx(bar, (uint32_t)(valid * v.ld * 2));
-    __syncwarp();
-    if (lane < valid) {
-      __nv_bfloat16* dst = sK + ((j % kLatStages) * kLatKeys + lane) * L.pitch;
-      const __nv_bfloat16* src = base + (int64_t)(key0 + lane) * v.ld;
+    if (tt == 0) tc::mbar_expect_tx(bar, (uint32_t)(valid * v.ld * 2));
+    if (lane < kRows && row < valid) {
+      __nv_bfloat16* dst = sK + ((j % kLatStages) * kLatKeys + row) * L.pitch;
+      const __nv_bfloat16* src = base + (int64_t)(key0 + row) * v.ld;
       if (one_piece) tc::bulk_g2s(dst, src, (uint32_t)(v.ld * 2), bar);
       else {
         tc::bulk_g2s(dst, src, (uint32_t)(v.rot * 2), bar);
@@ -299,8 +305,7 @@ __global__ void __launch_bounds__(kLatThreads, 1) latent_attend_tc_kernel(const 
       }
     }
   };
-  if (warp == 0)
-    for (int j = 0; j < min(tiles, kLatStages); ++j) load_tile(j);
+  for (int j = 0; j < min(tiles, kLatStages); ++j) load_tile(j);
   const int chunks = v.ld >> 3, c_chunks = v.rot >> 3;
   for (int h = tid >> 5; h < M; h += kLatThreads / 32)
     if (hg * M + h < v.H)
@@ -309,11 +314,10 @@ __global__ void __launch_bounds__(kLatThreads, 1) latent_attend_tc_kernel(const 
             *reinterpret_cast<const uint4*>(qa + ((int64_t)t * v.H + hg * M + h) * v.ld + c * 8);
   __syncthreads();
 
-  // scores: warp = (half of the feature steps, head tile, 16-key group); MT 1: quarters of the steps instead of head tiles
+  // scores: warp = (16-key group, quarter of the feature steps), all heads
   const int KS = (L.R16 + L.P16) >> 4;
-  const int khalf = warp & 1, mt = MT == 2 ? (warp >> 1) & 1 : 0, kg = MT == 2 ? warp >> 2 : (warp >> 1) & 1;
-  const bool scorer = MT == 2 || warp < 4;
-  const int ks0 = khalf ? (KS + 1) / 2 : 0, ks1 = khalf ? KS : (KS + 1) / 2;
+  const int kg = warp & 1, part_i = warp >> 1;
+  const int ks0 = part_i * KS / kParts, ks1 = (part_i + 1) * KS / kParts;
   float acc[MT][NT][4];
 #pragma unroll
   for (int m = 0; m < MT; ++m)
@@ -323,7 +327,7 @@ __global__ void __launch_bounds__(kLatThreads, 1) latent_attend_tc_kernel(const 
   const int srow = tt / TPR, spart = tt % TPR;
   const float cs = v.scale * kLog2e;
   float m_run = -CUDART_INF_F, l_run = 0.f;
-  const uint32_t qaddr = smem_addr(sQ + (mt * 16 + (lane & 15)) * L.pitch + (lane >> 4) * 8);
+  const uint32_t qaddr = smem_addr(sQ + (lane & 15) * L.pitch + (lane >> 4) * 8), qnext = (uint32_t)(16 * L.pitch * 2);
   const int col0 = warp * NT * 8;                      // this warp's slice of the latent's columns
   bool dead = false;
 
@@ -331,56 +335,62 @@ __global__ void __launch_bounds__(kLatThreads, 1) latent_attend_tc_kernel(const 
     tc::mbar_wait(&full[team][j % kLatStages], (j / kLatStages) & 1, dead, err);
     const __nv_bfloat16* K = sK + (j % kLatStages) * kLatKeys * L.pitch;
     const int key0 = k_begin + (j * kTeams + team) * kLatKeys;
-    if (scorer) {
-      float s0[2][4], s1[2][4];                        // even and odd steps, two 8-key tiles
+    {
+      float sc[MT][2][4];                              // two 8-key tiles per head tile
 #pragma unroll
-      for (int i = 0; i < 4; ++i) s0[0][i] = s0[1][i] = s1[0][i] = s1[1][i] = 0.f;
+      for (int m = 0; m < MT; ++m)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) sc[m][0][i] = sc[m][1][i] = 0.f;
       const uint32_t kaddr = smem_addr(K + (kg * 16 + (lane & 7) + ((lane >> 4) << 3)) * L.pitch + ((lane >> 3) & 1) * 8);
-      int ks = ks0;
-#pragma unroll 2
-      for (; ks + 1 < ks1; ks += 2) {
-        uint32_t a[4], b[4], a2[4], b2[4];
-        ldsm4(a, qaddr + ks * 32);
+#pragma unroll 5
+      for (int ks = ks0; ks < ks1; ++ks) {
+        uint32_t a[MT][4], b[4];
         ldsm4(b, kaddr + ks * 32);
-        ldsm4(a2, qaddr + ks * 32 + 32);
-        ldsm4(b2, kaddr + ks * 32 + 32);
-        mma16816(s0[0], a, b[0], b[1]);
-        mma16816(s0[1], a, b[2], b[3]);
-        mma16816(s1[0], a2, b2[0], b2[1]);
-        mma16816(s1[1], a2, b2[2], b2[3]);
-      }
-      if (ks < ks1) {
-        uint32_t a[4], b[4];
-        ldsm4(a, qaddr + ks * 32);
-        ldsm4(b, kaddr + ks * 32);
-        mma16816(s0[0], a, b[0], b[1]);
-        mma16816(s0[1], a, b[2], b[3]);
-      }
-      float* o = sS + (khalf * M + mt * 16 + (lane >> 2)) * kScorePitch + kg * 16 + (lane & 3) * 2;
 #pragma unroll
-      for (int i = 0; i < 2; ++i) {
-        *reinterpret_cast<float2*>(o + i * 8) = make_float2(s0[i][0] + s1[i][0], s0[i][1] + s1[i][1]);
-        *reinterpret_cast<float2*>(o + 8 * kScorePitch + i * 8) = make_float2(s0[i][2] + s1[i][2], s0[i][3] + s1[i][3]);
+        for (int m = 0; m < MT; ++m) ldsm4(a[m], qaddr + m * qnext + ks * 32);
+#pragma unroll
+        for (int m = 0; m < MT; ++m) {
+          mma16816(sc[m][0], a[m], b[0], b[1]);
+          mma16816(sc[m][1], a[m], b[2], b[3]);
+        }
+      }
+#pragma unroll
+      for (int m = 0; m < MT; ++m) {
+        float* o = sS + (part_i * M + m * 16 + (lane >> 2)) * kScorePitch + kg * 16 + (lane & 3) * 2;
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          *reinterpret_cast<float2*>(o + i * 8) = make_float2(sc[m][i][0], sc[m][i][1]);
+          *reinterpret_cast<float2*>(o + 8 * kScorePitch + i * 8) = make_float2(sc[m][i][2], sc[m][i][3]);
+        }
       }
     }
-    team_sync();
+    team_sync();                                       // the scores are there; everyone is past the previous tile
     {
       float s[KPT];
       float mx = -CUDART_INF_F;
+      const float* sp = sS + srow * kScorePitch + spart * KPT;
 #pragma unroll
-      for (int i = 0; i < KPT; ++i) {
-        const float x = sS[srow * kScorePitch + spart * KPT + i] + sS[(M + srow) * kScorePitch + spart * KPT + i];
-        s[i] = key0 + spart * KPT + i < k_end ? x * cs : -CUDART_INF_F;
-        mx = fmaxf(mx, s[i]);
+      for (int i = 0; i < KPT; i += 2) {
+        const float2 a = *reinterpret_cast<const float2*>(sp + i), b = *reinterpret_cast<const float2*>(sp + M * kScorePitch + i);
+        const float2 c = *reinterpret_cast<const float2*>(sp + 2 * M * kScorePitch + i), d = *reinterpret_cast<const float2*>(sp + 3 * M * kScorePitch + i);
+        s[i] = ((a.x + b.x) + (c.x + d.x)) * cs;
+        s[i + 1] = ((a.y + b.y) + (c.y + d.y)) * cs;
       }
+      if (key0 + kLatKeys > k_end) {
+#pragma unroll
+        for (int i = 0; i < KPT; ++i)
+          if (key0 + spart * KPT + i >= k_end) s[i] = -CUDART_INF_F;
+      }
+#pragma unroll
+      for (int i = 0; i < KPT; ++i) mx = fmaxf(mx, s[i]);
 #pragma unroll
       for (int off = TPR / 2; off > 0; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
       const float mn = fmaxf(m_run, mx);               // finite: every tile holds at least one key
-      const float alpha = exp2f(m_run - mn);
+      const float alpha = ex2(m_run - mn);
       float sum = 0.f;
 #pragma unroll
       for (int i = 0; i < KPT; i += 2) {
-        const float p0 = exp2f(s[i] - mn), p1 = exp2f(s[i + 1] - mn);
+        const float p0 = ex2(s[i] - mn), p1 = ex2(s[i + 1] - mn);
         sum += p0 + p1;
         *reinterpret_cast<__nv_bfloat162*>(sP + srow * kProbPitch + spart * KPT + i) = __floats2bfloat162_rn(p0, p1);
       }
@@ -390,6 +400,7 @@ __global__ void __launch_bounds__(kLatThreads, 1) latent_attend_tc_kernel(const 
       m_run = mn;
       if (spart == 0) sA[srow] = alpha;
     }
+    if (j >= 1 && j + 1 < tiles) load_tile(j + 1);        // into the stage of tile j - 1
     team_sync();
     if (col0 < L.R16) {
 #pragma unroll
@@ -419,8 +430,6 @@ __global__ void __launch_bounds__(kLatThreads, 1) latent_attend_tc_kernel(const 
         }
       }
     }
-    team_sync();                                       // the stage, the scores and the probabilities are free
-    if (warp == 0 && j + kLatStages < tiles) load_tile(j + kLatStages);
   }
   const int R = v.kv_rank;
   float* mine = part + (((int64_t)blockIdx.x * nsplit + blockIdx.y) * kTeams + team) * lat_slot(M, R);
@@ -540,19 +549,25 @@ __global__ void __launch_bounds__(256) latent_expand_tc_kernel(const LatentView 
     if (lane == 0) s_gate[t] = 1.0f / (den * (1.0f + expf(-gate[(int64_t)(t0 + t) * gate_pitch + h])));       // gate / denominator
   }
   __syncthreads();
-  for (int i = tid; i < kHeadTok * pitch; i += 256) {
-    const int t = i / pitch, r = i - t * pitch;
-    float x = 0.f;
+  // four latent columns per thread; the loads do not depend on the weights (a share nobody wrote holds stale numbers, weight 0)
+  const int q4 = pitch >> 2;
+  for (int i = tid; i < kHeadTok * q4; i += 256) {
+    const int t = i / q4, r = (i - t * q4) * 4;
+    float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
     if (t < n && r < R) {
       const float* p = part + ((int64_t)(t0 + t) * groups + hg) * np * slot + (int64_t)row * R + r;
-#pragma unroll 4
+#pragma unroll 8
       for (int k = 0; k < np; ++k) {
+        const float4 y = __ldcg(reinterpret_cast<const float4*>(p + k * slot));
         const float w = s_w[t * np + k];
-        if (w > 0.f) x += w * __ldcg(p + k * slot);
+        if (w > 0.f) { x.x += w * y.x; x.y += w * y.y; x.z += w * y.z; x.w += w * y.w; }
       }
-      x *= s_gate[t];
+      const float s = s_gate[t];
+      x.x *= s; x.y *= s; x.z *= s; x.w *= s;
     }
-    sA[i] = __float2bfloat16_rn(x);
+    __nv_bfloat162* o = reinterpret_cast<__nv_bfloat162*>(sA + t * pitch + r);
+    o[0] = __floats2bfloat162_rn(x.x, x.y);
+    o[1] = __floats2bfloat162_rn(x.z, x.w);
   }
   __syncthreads();
   const int V = v.vdim, per = (((V + gridDim.z - 1) / gridDim.z) + 15) & ~15, n0 = blockIdx.z * per;
@@ -567,7 +582,7 @@ unsigned head_slices(const Ctx* ctx, int64_t ctas, int N) {
   return (unsigned)std::max<int64_t>(1, std::min<int64_t>(z, N / 64));
 }
 
-constexpr size_t kLatMaxSmem = 220 * 1024;
+constexpr size_t kLatMaxSmem = 226 * 1024;
 bool lat_tc_ok(const LatentView& v) {
   return v.kv_rank <= 512 && v.kv_rank % 8 == 0 && v.dim % 8 == 0 && lat_smem(2, v.kv_rank, v.rot_dim) <= kLatMaxSmem;
 }

@@ -56,7 +56,7 @@ struct LayeredScratch {
 
 namespace {
 
-constexpr int kChunkMin = 8;            // longest portion from which retention runs in chunks
+constexpr int kChunkMin = 8, kTcMin = 80;   // longest portion from which retention runs in chunks of 64, of 128 tokens
 constexpr int kFlashMin = 32;           // shortest portion whose context is expanded to keys and values
 constexpr int kBlockTokens = 2048;      // tokens per round of the absorbed attention in a rows step (bounds its scratch)
 constexpr uint64_t kIdLayered = 0x200000, kIdLayeredState = 0x300000;
@@ -608,12 +608,13 @@ int32_t retention_rows(Session* S, RowsBuf& r, const RowsRun& run, int l, cudaSt
   if (s.c.ff) in.add(s.row0[R_UP], s.c.ff, SEG_RELU2, (char*)r.cat + (int64_t)s.cat0 * e, ldc);
   LMB_TRY(rows_gemm(M, w.w_in, s.m_in, r.xn, row_ld(M->cfg.hidden), T, in, st));
   RetentionView v = retention_view(S, l);
-  v.start = run.start; v.len = run.len; v.pos0 = run.pos0; v.max_len = run.max_len;
+  v.start = run.start; v.len = run.len; v.pos0 = run.pos0; v.total = run.T;
   v.q = at(R_Q); v.k = at(R_K); v.v = at(R_V); v.g = at(R_G);
   v.q_pitch = v.k_pitch = v.v_pitch = v.g_pitch = s.n_store;
   v.in_f32 = dt != LMB200_BF16; v.raw_gate = 0;
   v.out = r.cat; v.ldo = ldc; v.bp = 0;
   if (rot) v.rot_dims = 0;
+  if (run.max_len >= kTcMin && retention_tc_ok(v)) return retention_tc(ctx, v, st);
   if (run.max_len >= kChunkMin && retention_chunks_ok(v)) return retention_chunks(ctx, v, st);
   return retention_steps(ctx, dt, v, st);
 }

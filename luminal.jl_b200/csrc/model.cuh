@@ -85,7 +85,7 @@ struct LayeredWeights {
   int rot_id = -1;                            // layers with the same frequencies share an angle table (Model::rot_freqs)
   float *decay = nullptr;                     // retention: [heads][kDecayPow]: decay^0 .. decay^(kDecayPow - 1)
 };
-constexpr int kDecayPow = 72;
+constexpr int kDecayPow = 136;
 
 struct Model {
   bool tp_solo = false;        // profiling aid: shard of one rank, no all-reduce

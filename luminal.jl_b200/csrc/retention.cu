@@ -5,14 +5,15 @@
 namespace lmb {
 namespace {
 
-constexpr int kStepThreads = 128;
+constexpr int kStepMax = 512;           // threads per CTA: 512 where few (head, sequence) pairs leave SMs idle, else 128
 
 // One CTA per (head, sequence).  Thread (c, w): four value columns 4 c .., rows w, w + W, ... of the state, where W = threads / column
 // groups; a thread owns its elements of the state for all tokens, so only q, k, v and the partial outputs go through shared memory.
 template <typename IT, typename OT>
-__global__ void __launch_bounds__(kStepThreads) retention_step_kernel(const RetentionView v) {
+__global__ void __launch_bounds__(kStepMax) retention_step_kernel(const RetentionView v) {
   extern __shared__ float sm[];
-  __shared__ float red[kStepThreads / 32];
+  __shared__ float red[kStepMax / 32];
+  const int kStepThreads = blockDim.x;
   const int h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x;
   const int D = v.dim, V = v.vdim, V4 = (V + 3) >> 2;         // state rows are V4 float4s
   const int cols = min(V4, kStepThreads), W = kStepThreads / cols;
@@ -76,7 +77,6 @@ __global__ void __launch_bounds__(kStepThreads) retention_step_kernel(const Rete
     if ((tid & 31) == 0) red[tid >> 5] = ss;
     __syncthreads();
     float tot = 0.f;
-#pragma unroll
     for (int j = 0; j < kStepThreads / 32; ++j) tot += red[j];
     const float inv = 1.0f / sqrtf(tot / (float)V + v.eps);
     const IT* g = reinterpret_cast<const IT*>(v.g) + t * v.g_pitch + h * V;
@@ -91,8 +91,8 @@ __global__ void __launch_bounds__(kStepThreads) retention_step_kernel(const Rete
   }
 }
 
-size_t step_smem(const RetentionView& v) {
-  const int V4 = (v.vdim + 3) >> 2, cols = V4 < kStepThreads ? V4 : kStepThreads, W = kStepThreads / cols;
+size_t step_smem(const RetentionView& v, int threads) {
+  const int V4 = (v.vdim + 3) >> 2, cols = V4 < threads ? V4 : threads, W = threads / cols;
   return (size_t)(2 * ((v.dim + 3) & ~3) + 4 * V4 + W * 4 * V4) * 4;
 }
 
@@ -449,7 +449,7 @@ int32_t retention_configure() {
   LMB_CFG(128, 64, 2);
   LMB_CFG(256, 32, 2);
 #undef LMB_CFG
-  return LMB200_OK;
+  return retention_tc_configure();
 }
 
 int32_t angle_table(Ctx* ctx, float2* tab, const float* inv_freq, int n, const int* pos, int T, cudaStream_t st) {
@@ -476,16 +476,17 @@ int32_t retention_chunks(Ctx* ctx, const RetentionView& v, cudaStream_t st) {
 }
 
 int32_t retention_steps(Ctx* ctx, int dtype, const RetentionView& v, cudaStream_t st) {
-  const size_t smem = step_smem(v);
+  const int threads = (int64_t)v.B * v.H < 2 * ctx->sm_count ? kStepMax : 128;
+  const size_t smem = step_smem(v, threads);
   LMB_REQUIRE(smem <= 48 * 1024, "retention: heads of %d x %d", v.dim, v.vdim);
   const dim3 grid((unsigned)v.H, (unsigned)v.B);
   if (dtype != LMB200_BF16) {
     LMB_REQUIRE(v.in_f32, "retention: float32 models have float32 projections");
-    LMB_CUDA(launch_k(retention_step_kernel<float, float>, grid, dim3(kStepThreads), smem, st, v));
+    LMB_CUDA(launch_k(retention_step_kernel<float, float>, grid, dim3(threads), smem, st, v));
   } else if (v.in_f32) {
-    LMB_CUDA(launch_k(retention_step_kernel<float, __nv_bfloat16>, grid, dim3(kStepThreads), smem, st, v));
+    LMB_CUDA(launch_k(retention_step_kernel<float, __nv_bfloat16>, grid, dim3(threads), smem, st, v));
   } else {
-    LMB_CUDA(launch_k(retention_step_kernel<__nv_bfloat16, __nv_bfloat16>, grid, dim3(kStepThreads), smem, st, v));
+    LMB_CUDA(launch_k(retention_step_kernel<__nv_bfloat16, __nv_bfloat16>, grid, dim3(threads), smem, st, v));
   }
   ctx->launches++;
   return LMB200_OK;

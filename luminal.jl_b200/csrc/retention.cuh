@@ -13,7 +13,7 @@ struct RetentionView {
   const int* start = nullptr;
   const int* len = nullptr;
   const int* pos0 = nullptr;
-  int max_len = 1;                    // the longest len (grid sizing)
+  int total = 0;                      // packed rows (bounds of the tensor maps)
   int H = 0, dim = 0, vdim = 0;
   int rot_dims = 0;                   // features of q and k still to be rotated, in neighbouring pairs (2i, 2i + 1); 0: rotated already
   const float* inv_freq = nullptr;    // [rot_dims / 2]
@@ -35,6 +35,10 @@ int32_t retention_steps(Ctx* ctx, int dtype, const RetentionView& v, cudaStream_
 // chunks of 64 tokens on the tensor cores: bf16 rows, rotated, gated (raw_gate 0), row-major output
 bool retention_chunks_ok(const RetentionView& v);
 int32_t retention_chunks(Ctx* ctx, const RetentionView& v, cudaStream_t st);
+// the same in chunks of 128 tokens with tcgen05 (csrc/retention_tc.cu)
+bool retention_tc_ok(const RetentionView& v);
+int32_t retention_tc(Ctx* ctx, const RetentionView& v, cudaStream_t st);
+int32_t retention_tc_configure();
 // angle tables of T tokens: tab[t * n + i] = (cos, sin) of pos[t] * inv_freq[i]
 int32_t angle_table(Ctx* ctx, float2* tab, const float* inv_freq, int n, const int* pos, int T, cudaStream_t st);
 
