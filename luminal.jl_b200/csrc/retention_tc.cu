@@ -31,6 +31,7 @@ constexpr int offQ = 0, offK = kTile, offKl = 3 * kTile, offV = 4 * kTile, offSh
 struct Tail {                                            // behind the tiles
   uint64_t q_full, q_empty, k_full[2], k_empty[2], v_full, v_empty, s_full, p_ready, kt_ready, st_ready, o_full, o_empty, m4_done, x_full;
   uint32_t tmem;
+  float pw[kT + 4];                                      // decay^0 .. decay^128
   float ssq[2][kT];                                      // sums of squares of the two column halves
   float peer[2][kT];                                     // the other CTA's rows, by chunk parity
 };
@@ -95,6 +96,7 @@ __global__ void __launch_bounds__(kThreads, 1) retention_tc_kernel(const Retenti
     mbar_init(&tl.x_full, kT);
     mbar_init_fence();
   }
+  for (int i = tid; i <= kT; i += kThreads) tl.pw[i] = v.decay[(int64_t)h * v.decay_pitch + i];      // constants of the model
   if (warp == 16) tmem_alloc(&tl.tmem, 512);
   fence_before();
   __syncthreads();
@@ -110,7 +112,7 @@ __global__ void __launch_bounds__(kThreads, 1) retention_tc_kernel(const Retenti
   const int n_all = v.len[b], t_first = v.start[b];
   const int chunks = (n_all + kT - 1) / kT;              // 0: nothing to do (uniform over the pair)
   const int D = v.dim, V = v.vdim, ld = (V + 3) & ~3, c0 = slice * 128;
-  const float* pw = v.decay + (int64_t)h * v.decay_pitch;
+  const float* pw = tl.pw;
   const float scale = 1.0f / sqrtf((float)D);
   const uint32_t lane_base = (uint32_t)(32 * (warp & 3)) << 16;
 
@@ -259,9 +261,13 @@ __global__ void __launch_bounds__(kThreads, 1) retention_tc_kernel(const Retenti
   } else {
     // ------------------------------ scores and outputs ------------------------------
     const int half = warp >> 2, row = 32 * (warp & 3) + lane, pair_bar = 1 + (warp & 3);
-    const float wi = pw[row + 1];
+    const float wi = pw[row + 1], g1 = pw[1];
     for (int c = 0; c < chunks; ++c) {
       const int n = min(kT, n_all - c * kT);
+      const int64_t t = t_first + (int64_t)c * kT + row;
+      const int col = h * V + c0 + half * 64, left = V - c0 - half * 64;       // valid columns: a multiple of 8, or <= 0
+      const __nv_bfloat16* gate = reinterpret_cast<const __nv_bfloat16*>(v.g) + t * v.g_pitch + col;
+      if (row < n && left > 0) asm volatile("prefetch.global.L2 [%0];\n" ::"l"(gate));
       mbar_wait(&tl.s_full, c & 1, dead, err);
       fence_after();
       uint32_t hi[32], lo[32];
@@ -271,13 +277,17 @@ __global__ void __launch_bounds__(kThreads, 1) retention_tc_kernel(const Retenti
         for (int ch = 0; ch < 4; ++ch) {
           float s[16];
           tmem_ld16(s, tmem + lane_base + kColP + half * 64 + ch * 16);
+          // weights from the nearest key of the sixteen outwards: one table entry, then one factor per key
+          const int d = row - (half * 64 + ch * 16 + 15);                      // distance to the last key
+          float w = scale * pw[max(d, 0)];
 #pragma unroll
-          for (int i = 0; i < 16; i += 2) {
-            const int d = row - (half * 64 + ch * 16 + i);                     // distance to the key
-            const float x = d >= 0 ? s[i] * (scale * __ldg(pw + d)) : 0.f;
-            const float y = d >= 1 ? s[i + 1] * (scale * __ldg(pw + d - 1)) : 0.f;
-            split2(x, y, hi[ch * 8 + i / 2], lo[ch * 8 + i / 2]);
+          for (int i = 15; i >= 0; --i) {
+            const bool seen = d + 15 - i >= 0;
+            s[i] = seen ? s[i] * w : 0.f;
+            if (seen) w *= g1;
           }
+#pragma unroll
+          for (int i = 0; i < 16; i += 2) split2(s[i], s[i + 1], hi[ch * 8 + i / 2], lo[ch * 8 + i / 2]);
         }
       } else {
 #pragma unroll
@@ -332,22 +342,25 @@ __global__ void __launch_bounds__(kThreads, 1) retention_tc_kernel(const Retenti
       }
       const float inv = 1.0f / sqrtf(ss / (float)V + v.eps);
       if (row < n) {
-        const int64_t t = t_first + (int64_t)c * kT + row;
-        const int col = h * V + c0 + half * 64, left = V - c0 - half * 64;     // a multiple of 8, or <= 0
-        const __nv_bfloat16* gate = reinterpret_cast<const __nv_bfloat16*>(v.g) + t * v.g_pitch + col;
         __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(v.out) + t * v.ldo + col;
 #pragma unroll
-        for (int q = 0; q < 8; ++q) {
-          if (q * 8 >= left) continue;
-          uint4 gu = __ldg(reinterpret_cast<const uint4*>(gate + q * 8));
-          uint32_t* gi = reinterpret_cast<uint32_t*>(&gu);
+        for (int q0 = 0; q0 < 8; q0 += 4) {                                    // four gate vectors in flight
+          uint4 gu[4];
 #pragma unroll
-          for (int e = 0; e < 4; ++e) {
-            const float2 g = unpack2bf(gi[e]);
-            const __nv_bfloat162 r = __floats2bfloat162_rn(o[q * 8 + 2 * e] * inv * g.x, o[q * 8 + 2 * e + 1] * inv * g.y);
-            gi[e] = *reinterpret_cast<const uint32_t*>(&r);
+          for (int q = 0; q < 4; ++q)
+            gu[q] = (q0 + q) * 8 < left ? __ldg(reinterpret_cast<const uint4*>(gate + (q0 + q) * 8)) : make_uint4(0, 0, 0, 0);
+#pragma unroll
+          for (int q = 0; q < 4; ++q) {
+            uint32_t* gi = reinterpret_cast<uint32_t*>(&gu[q]);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+              const float2 g = unpack2bf(gi[e]);
+              const int i = (q0 + q) * 8 + 2 * e;
+              const __nv_bfloat162 r = __floats2bfloat162_rn(o[i] * inv * g.x, o[i + 1] * inv * g.y);
+              gi[e] = *reinterpret_cast<const uint32_t*>(&r);
+            }
+            if ((q0 + q) * 8 < left) *reinterpret_cast<uint4*>(out + (q0 + q) * 8) = gu[q];
           }
-          *reinterpret_cast<uint4*>(out + q * 8) = gu;
         }
       }
     }
