@@ -201,7 +201,7 @@ __global__ void __launch_bounds__(kSimple) latent_attend_simple_kernel(const Lat
 // 8 that take the 32-key tiles of the CTA's share in turn, so that one team's products run during the other's softmax.  A tile's
 // latent rows arrive by bulk copies (one per row, two stages per team; the row pitch is an odd number of 16-byte chunks) and serve as keys
 // (S = Q' C^T: all heads x 16 keys x a quarter of the features per warp) and as values (O += P C: every warp a slice of the latent's columns).  Scores
-// and the running softmax stay float32.  Every team leaves (O, max, sum) of its keys; latent_expand merges them.
+// and the running softmax stay float32.  A CTA leaves (O, max, sum) of its keys; latent_expand merges the splits.
 // ---------------------------------------------------------------------------------------------
 constexpr int kTeams = 2, kTeamThreads = 256, kLatThreads = kTeams * kTeamThreads, kLatKeys = 32, kLatStages = 2;
 constexpr int kScorePitch = kLatKeys + 4, kProbPitch = kLatKeys + 8, kParts = 4;      // kParts: the features of a score are summed in four parts
@@ -248,7 +248,7 @@ __host__ __device__ inline int lat_keys_per_cta(int n, int nsplit) {
   constexpr int unit = kTeams * kLatKeys;
   return (((n + nsplit - 1) / nsplit + unit - 1) / unit) * unit;
 }
-// partial results of (token, head group, split, team): O [16 MT][kv_rank], then max and sum per head (log2 units)
+// partial results of (token, head group, split): O [16 MT][kv_rank], then max and sum per head (log2 units)
 __host__ __device__ inline int64_t lat_slot(int M, int kv_rank) { return (int64_t)M * (kv_rank + 2); }
 
 template <int NT, int MT>
@@ -431,20 +431,41 @@ __global__ void __launch_bounds__(kLatThreads, 1) latent_attend_tc_kernel(const 
       }
     }
   }
+  // The second team hands its accumulators over through shared memory (a thread's counterpart owns the same elements), and the
+  // first leaves the merged result of the CTA's keys.
   const int R = v.kv_rank;
-  float* mine = part + (((int64_t)blockIdx.x * nsplit + blockIdx.y) * kTeams + team) * lat_slot(M, R);
-  if (spart == 0) { mine[(int64_t)M * R + srow] = m_run; mine[(int64_t)M * R + M + srow] = l_run; }
-  if (col0 < L.R16) {
+  float* stat = reinterpret_cast<float*>(probs);       // [team][max, sum][M]
+  float* hand = reinterpret_cast<float*>(sm_raw);      // [MT * NT * 4][kTeamThreads], over the key stages (and, for narrow latents, the scores)
+  __syncthreads();
+  if (spart == 0) { stat[(2 * team) * M + srow] = m_run; stat[(2 * team + 1) * M + srow] = l_run; }
+  if (team == 1) {
 #pragma unroll
     for (int m = 0; m < MT; ++m)
 #pragma unroll
       for (int i = 0; i < NT; ++i)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const int row = m * 16 + (lane >> 2) + (e >> 1) * 8, col = col0 + i * 8 + (lane & 3) * 2 + (e & 1);
-          if (col < R) mine[(int64_t)row * R + col] = acc[m][i][e];
-        }
+        for (int e = 0; e < 4; ++e) hand[((m * NT + i) * 4 + e) * kTeamThreads + tt] = acc[m][i][e];
   }
+  __syncthreads();
+  if (team == 1) return;
+  float* mine = part + ((int64_t)blockIdx.x * nsplit + blockIdx.y) * lat_slot(M, R);
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int e2 = 0; e2 < 2; ++e2) {
+      const int row = m * 16 + (lane >> 2) + e2 * 8;
+      const float m0 = stat[row], m1 = stat[2 * M + row], mx = fmaxf(m0, m1);          // the first team has had a tile: m0 is finite
+      const float w0 = ex2(m0 - mx), w1 = ex2(m1 - mx);
+      if (warp == 0 && (lane & 3) == 0) { mine[(int64_t)M * R + row] = mx; mine[(int64_t)M * R + M + row] = stat[M + row] * w0 + stat[3 * M + row] * w1; }
+      if (col0 >= L.R16) continue;
+#pragma unroll
+      for (int i = 0; i < NT; ++i) {
+        const int col = col0 + i * 8 + (lane & 3) * 2;
+        const float* o = hand + ((m * NT + i) * 4 + e2 * 2) * kTeamThreads + tt;
+        const float x = acc[m][i][2 * e2] * w0 + o[0] * w1, y = acc[m][i][2 * e2 + 1] * w0 + o[kTeamThreads] * w1;
+        if (col < R) *reinterpret_cast<float2*>(mine + (int64_t)row * R + col) = make_float2(x, y);       // R is even
+      }
+    }
 }
 
 // ---------------------------------------------------------------------------------------------
@@ -511,27 +532,27 @@ __global__ void __launch_bounds__(256) latent_absorb_tc_kernel(const LatentView 
   });
 }
 
-// merges the partial results of a head's keys, multiplies the weighted latents out to values and gates them
+// merges the partial results of a head's keys, multiplies the weighted latents out to values and gates them: head blockIdx.x, tokens
+// tok * blockIdx.y .. (tok <= kHeadTok; few tokens per CTA spread the merging over the SMs), value columns of slice blockIdx.z
 __global__ void __launch_bounds__(256) latent_expand_tc_kernel(const LatentView v, const float* __restrict__ part, int nsplit, int M,
                                                                const __nv_bfloat16* __restrict__ w_uv, const float* __restrict__ gate, int gate_pitch,
-                                                               __nv_bfloat16* __restrict__ out, int ldo, int bp) {
+                                                               __nv_bfloat16* __restrict__ out, int ldo, int bp, int tok) {
   extern __shared__ __align__(16) unsigned char sm_raw[];
   __nv_bfloat16* sA = reinterpret_cast<__nv_bfloat16*>(sm_raw);
   __shared__ float s_gate[kHeadTok];
   const int R = v.kv_rank, pitch = head_pitch(R);
-  float* s_w = reinterpret_cast<float*>(sA + kHeadTok * pitch);                // [kHeadTok][nsplit * kTeams] weights of the partial results
+  float* s_w = reinterpret_cast<float*>(sA + kHeadTok * pitch);                // [kHeadTok][nsplit] weights of the partial results
   pdl_launch_dependents();
   pdl_wait();
-  const int h = blockIdx.x, t0 = blockIdx.y * kHeadTok, n = min(kHeadTok, v.T - t0), tid = threadIdx.x, lane = tid & 31;
-  const int groups = (v.H + M - 1) / M, hg = h / M, row = h - hg * M, np = nsplit * kTeams;
+  const int h = blockIdx.x, t0 = blockIdx.y * tok, n = min(tok, v.T - t0), tid = threadIdx.x, lane = tid & 31;
+  const int groups = (v.H + M - 1) / M, hg = h / M, row = h - hg * M, np = nsplit;
   const int64_t slot = lat_slot(M, R);
   for (int t = tid >> 5; t < n; t += 8) {
     const float* p = part + ((int64_t)(t0 + t) * groups + hg) * np * slot + (int64_t)M * R + row;
     const int ctx = v.pos[t0 + t] + 1, kpc = lat_keys_per_cta(ctx, nsplit);
     float mx = -CUDART_INF_F;
     for (int i = lane; i < np; i += 32) {
-      const int first = (i / kTeams) * kpc + (i % kTeams) * kLatKeys;          // a team without a tile has left (-inf, 0)
-      const float m = first < ctx ? __ldcg(p + i * slot) : -CUDART_INF_F;
+      const float m = i * kpc < ctx ? __ldcg(p + i * slot) : -CUDART_INF_F;
       s_w[t * np + i] = m;
       mx = fmaxf(mx, m);
     }
@@ -701,7 +722,7 @@ LatentAttnPlan latent_attn_plan(const Ctx* ctx, int dtype, const LatentView& v, 
     if (best_cost < 0 || cost < best_cost) { best_cost = cost; best = ns; }
   }
   p.nsplit = (int)best;
-  p.part_floats = pairs * best * kTeams * lat_slot(M, v.kv_rank);
+  p.part_floats = pairs * best * lat_slot(M, v.kv_rank);
   return p;
 }
 
@@ -736,11 +757,13 @@ int32_t latent_attend(Ctx* ctx, int dtype, const LatentView& v, const void* qa, 
 int32_t latent_expand(Ctx* ctx, int dtype, const LatentView& v, const float* part, const LatentAttnPlan& plan, const void* w_uv, const float* gate,
                       int gate_pitch, void* out, int ldo, int bp, cudaStream_t st) {
   if (plan.nsplit >= 1) {
-    const int64_t tg = ceil_div(v.T, kHeadTok);
+    int tok = kHeadTok;
+    while (tok > 2 && v.H * ceil_div(v.T, tok) < ctx->sm_count) tok >>= 1;
+    const int64_t tg = ceil_div(v.T, tok);
     const dim3 grid((unsigned)v.H, (unsigned)tg, head_slices(ctx, v.H * tg, v.vdim));
-    const size_t smem = (size_t)kHeadTok * head_pitch(v.kv_rank) * 2 + (size_t)kHeadTok * plan.nsplit * kTeams * 4;
+    const size_t smem = (size_t)kHeadTok * head_pitch(v.kv_rank) * 2 + (size_t)kHeadTok * plan.nsplit * 4;
     LMB_CUDA(launch_k(latent_expand_tc_kernel, grid, dim3(256), smem, st, v, part, plan.nsplit, 16 * lat_mt(v.H), (const __nv_bfloat16*)w_uv, gate,
-                      gate_pitch, (__nv_bfloat16*)out, ldo, bp));
+                      gate_pitch, (__nv_bfloat16*)out, ldo, bp, tok));
     ctx->launches++;
     return LMB200_OK;
   }
