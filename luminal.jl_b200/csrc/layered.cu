@@ -321,6 +321,13 @@ int32_t ensure_rows(Session* S, RowsBuf& r, int64_t T, int64_t n_want) {
   return LMB200_OK;
 }
 
+// four consecutive elements in one store
+__device__ __forceinline__ void store4(float* o, float a, float b, float c, float d) { *reinterpret_cast<float4*>(o) = make_float4(a, b, c, d); }
+__device__ __forceinline__ void store4(__nv_bfloat16* o, float a, float b, float c, float d) {
+  reinterpret_cast<__nv_bfloat162*>(o)[0] = __floats2bfloat162_rn(a, b);
+  reinterpret_cast<__nv_bfloat162*>(o)[1] = __floats2bfloat162_rn(c, d);
+}
+
 // x[t] <- embedding row (tokens given) or x[t] + delta[t]; xn[t] = RMSNorm(x[t]) w in the model dtype.  Rows in order, or the rows
 // `pick` chooses (then x itself is left alone).  capture [.., n]: the new row of every sequence's last token.
 template <typename WT>
@@ -328,7 +335,7 @@ __global__ void __launch_bounds__(256) rows_norm_kernel(float* __restrict__ x, c
                                                         const WT* __restrict__ embed, int vocab, const int* __restrict__ pick,
                                                         const float* __restrict__ w, WT* __restrict__ xn, int ldn, int n, float eps,
                                                         float* __restrict__ capture, const int* __restrict__ last) {
-  extern __shared__ float row[];
+  extern __shared__ __align__(16) float row[];
   __shared__ float red[8];
   pdl_launch_dependents();
   pdl_wait();
@@ -338,14 +345,29 @@ __global__ void __launch_bounds__(256) rows_norm_kernel(float* __restrict__ x, c
   const bool ok = tok >= 0 && tok < vocab;
   const int cap = capture && !pick ? last[t] : -1;
   float ss = 0.f;
-  for (int i = tid; i < n; i += 256) {
-    float v;
-    if (tokens) v = ok ? to_f32(embed[(int64_t)tok * n + i]) : 0.f;
-    else v = x[t * n + i] + (delta ? delta[t * n + i] : 0.f);
-    if (!pick) x[t * n + i] = v;
-    if (cap >= 0) capture[(int64_t)cap * n + i] = v;
-    row[i] = v;
-    ss += v * v;
+  // whole vectors where the rows allow it (residual rows: the embedding and the captured rows take the other loop)
+  if (!tokens && cap < 0 && (n & 3) == 0 && (ldn & 3) == 0) {
+    float4* x4 = reinterpret_cast<float4*>(x + t * n);
+    const float4* d4 = delta ? reinterpret_cast<const float4*>(delta + t * n) : nullptr;
+    float4* r4 = reinterpret_cast<float4*>(row);
+#pragma unroll 4
+    for (int i = tid; i < (n >> 2); i += 256) {
+      float4 v = x4[i];
+      if (d4) { const float4 d = d4[i]; v.x += d.x; v.y += d.y; v.z += d.z; v.w += d.w; }
+      if (!pick) x4[i] = v;
+      r4[i] = v;
+      ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+    }
+  } else {
+    for (int i = tid; i < n; i += 256) {
+      float v;
+      if (tokens) v = ok ? to_f32(embed[(int64_t)tok * n + i]) : 0.f;
+      else v = x[t * n + i] + (delta ? delta[t * n + i] : 0.f);
+      if (!pick) x[t * n + i] = v;
+      if (cap >= 0) capture[(int64_t)cap * n + i] = v;
+      row[i] = v;
+      ss += v * v;
+    }
   }
 #pragma unroll
   for (int off = 16; off > 0; off >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, off);
@@ -355,8 +377,17 @@ __global__ void __launch_bounds__(256) rows_norm_kernel(float* __restrict__ x, c
 #pragma unroll
   for (int i = 0; i < 8; ++i) tot += red[i];
   const float inv = 1.0f / sqrtf(tot / (float)n + eps);
-  if (xn)
-    for (int i = tid; i < n; i += 256) xn[(int64_t)i0 * ldn + i] = from_f32<WT>(row[i] * inv * w[i]);
+  if (!xn) return;
+  if ((n & 3) == 0 && (ldn & 3) == 0) {
+    const float4* r4 = reinterpret_cast<const float4*>(row);
+    const float4* w4 = reinterpret_cast<const float4*>(w);
+    for (int i = tid; i < (n >> 2); i += 256) {
+      const float4 v = r4[i], g = w4[i];
+      store4(xn + (int64_t)i0 * ldn + 4 * i, v.x * inv * g.x, v.y * inv * g.y, v.z * inv * g.z, v.w * inv * g.w);
+    }
+    return;
+  }
+  for (int i = tid; i < n; i += 256) xn[(int64_t)i0 * ldn + i] = from_f32<WT>(row[i] * inv * w[i]);
 }
 
 // float32 GEMM over many tokens on the CUDA cores: 64 rows x 64 tokens per CTA, W in the 16 x 32 tiles of the float32 layout
