@@ -95,3 +95,28 @@ def test_ragged_whisper_positions(lib_built, device):
     assert np.abs(lg[1] - hist[1][1][1]).max() <= 1e-4
     assert nxt[1] == hist[1][0][1]
     sess.close(); model.close()
+
+
+def test_extend_mixes_portions_and_single_tokens(lib_built, device):
+    """lmb200_extend on a Llama: portions, single tokens and sequences that stand still in one call, logits at any place."""
+    L = lib_built
+    cfg = O.CONFIGS["tiny_gqa128"]
+    w = O.synth_llama_weights(cfg, seed=23)
+    toks = [O.synth_tokens(23, 700 + b, (n,), cfg["vocab"]) for b, n in enumerate((14, 6, 10))]
+    refs = [np.concatenate([lg.reshape(1, -1, cfg["vocab"])[:, -1] for lg in _step_logits(w, cfg, t)]) for t in toks]
+    model = make_model(L, device, cfg, w, "f32")
+    sess = L.Session(model, 3, 32)
+    at = [0, 0, 0]
+    for plan in ((4, 1, 3), (1, 0, 1), (6, 2, 1), (1, 1, 1), (2, 2, 4)):
+        part = [t[a:a + n] for t, a, n in zip(toks, at, plan)]
+        got = sess.extend(part, [list(range(n)) for n in plan])
+        want = np.concatenate([r[a:a + n] for r, a, n in zip(refs, at, plan)])
+        assert np.abs(got - want).max() <= 1e-3, plan
+        at = [a + n for a, n in zip(at, plan)]
+        assert list(sess.positions()) == at
+    sess.close(); model.close()
+
+
+def _step_logits(w, cfg, toks):
+    m = O.CachedLlama(w, cfg, 1, 64)
+    return [m.forward(np.asarray([[t]])) for t in toks]
