@@ -520,7 +520,9 @@ __device__ __forceinline__ void tmem_load_row<16>(float (&v)[16], uint32_t taddr
 // block -- the pairs the fused epilogues combine -- are 8 lanes apart in the same warp.
 // The thread holds batch columns b0 .. b0+NV-1 of the row (the whole row when NV == BP); BP is the
 // batch padding of the activation buffers.
-template <int NV, int BP>
+// X: the epilogues of decoders described layer by layer (softcap, EPI_STORE_RELU2) are compiled in.  They have instantiations of their
+// own: the other models' kernels carry no code of them.
+template <int NV, int BP, bool X>
 __device__ __forceinline__ void row_epilogue(const GemvParams& p, float (&v)[NV], int row, int b0, const float* s_inv) {
   typedef Layout<__nv_bfloat16> LY;
   constexpr int N = NV;
@@ -541,7 +543,7 @@ __device__ __forceinline__ void row_epilogue(const GemvParams& p, float (&v)[NV]
   }
   if (p.epi == EPI_STORE_F32) {
     if (row < p.rows) {
-      if (p.softcap > 0.f) {
+      if (X && p.softcap > 0.f) {
 #pragma unroll
         for (int b = 0; b < N; ++b) v[b] = p.softcap * tanhf(v[b] / p.softcap);
       }
@@ -551,7 +553,7 @@ __device__ __forceinline__ void row_epilogue(const GemvParams& p, float (&v)[NV]
     }
     return;
   }
-  if (p.epi == EPI_STORE_RELU2) {
+  if (X && p.epi == EPI_STORE_RELU2) {
     if (row < p.act_row0) {
 #pragma unroll
       for (int b = 0; b < N; ++b)
@@ -898,7 +900,7 @@ __device__ __forceinline__ void resid_norm_tile(const GemvParams& p, const unsig
   }
 }
 
-template <int N>
+template <int N, bool X>
 __global__ void __launch_bounds__(kTcThreads, 1) gemv_tc_kernel(const GemvParams p, int* err) {
   constexpr int kXStage = N * 256;
   constexpr int kStage = kWStage + kXStage;
@@ -1004,7 +1006,7 @@ __global__ void __launch_bounds__(kTcThreads, 1) gemv_tc_kernel(const GemvParams
       int c_first, n;
       contributors(ur, r, &c_first, &n);
       if (n == 1) {
-        row_epilogue<N, N>(p, v, r * 128 + row_in_group, 0, s_inv);
+        row_epilogue<N, N, X>(p, v, r * 128 + row_in_group, 0, s_inv);
         continue;
       }
       float4* part = reinterpret_cast<float4*>(p.partials) + (int64_t)r * p.ksplit * (128 * N / 4);
@@ -1073,7 +1075,7 @@ __global__ void __launch_bounds__(kTcThreads, 1) gemv_tc_kernel(const GemvParams
             const float4 t = lds4(slot);
             v4[0] += t.x; v4[1] += t.y; v4[2] += t.z; v4[3] += t.w;
           }
-          row_epilogue<4, N>(p, v4, pend_r[ip] * 128 + 16 * (ci_[ip] + jj * n_[ip]) + row16, 4 * cg, s_inv);
+          row_epilogue<4, N, X>(p, v4, pend_r[ip] * 128 + 16 * (ci_[ip] + jj * n_[ip]) + row16, 4 * cg, s_inv);
         }
         return slot;
       };
@@ -1105,7 +1107,7 @@ __global__ void __launch_bounds__(kTcThreads, 1) gemv_tc_kernel(const GemvParams
               v4[0] += t.x; v4[1] += t.y; v4[2] += t.z; v4[3] += t.w;
             }
           }
-          row_epilogue<4, N>(p, v4, pend_r[ip] * 128 + 16 * ci_[ip] + row16, 4 * cg, s_inv);
+          row_epilogue<4, N, X>(p, v4, pend_r[ip] * 128 + 16 * ci_[ip] + row16, 4 * cg, s_inv);
         }
       }
       if (tid == 64) LMB_TRACE(13);
@@ -1163,7 +1165,7 @@ __device__ __forceinline__ void cluster_sync_all() {
   asm volatile("barrier.cluster.wait.acquire.aligned;\n" ::: "memory");
 }
 
-template <int N>
+template <int N, bool X>
 __global__ void __launch_bounds__(kTcThreads, 1) gemv_cl_kernel(const GemvParams p, int* err) {
   constexpr int kXStage = N * 256;
   constexpr int kStage = kWStage + kXStage;
@@ -1305,7 +1307,7 @@ __global__ void __launch_bounds__(kTcThreads, 1) gemv_cl_kernel(const GemvParams
           const float4 t = recv[((src * rows_per + 16 * j + row16) * N) / 4 + cg];
           v4[0] += t.x; v4[1] += t.y; v4[2] += t.z; v4[3] += t.w;
         }
-        row_epilogue<4, N>(p, v4, r * 128 + c * rows_per + 16 * j + row16, 4 * cg, s_inv);
+        row_epilogue<4, N, X>(p, v4, r * 128 + c * rows_per + 16 * j + row16, 4 * cg, s_inv);
       }
     }
   }
@@ -1318,6 +1320,8 @@ __global__ void __launch_bounds__(kTcThreads, 1) gemv_cl_kernel(const GemvParams
   }
   if (tid == 0) { LMB_TRACE(9); LMB_TRACE_NS(11); }
 }
+
+bool layered_epilogue(const GemvParams& p) { return p.epi == EPI_STORE_RELU2 || p.softcap > 0.f; }
 
 template <int Bp>
 constexpr size_t cluster_smem() {
@@ -1340,7 +1344,7 @@ int32_t launch_cluster(Ctx* ctx, const GemvParams& p, cudaStream_t stream) {
   attr[1].val.programmaticStreamSerializationAllowed = 1;
   cfg.attrs = attr;
   cfg.numAttrs = pdl_enabled() ? 2 : 1;
-  LMB_CUDA(cudaLaunchKernelEx(&cfg, gemv_cl_kernel<Bp>, p, ctx->dev_err));
+  LMB_CUDA(cudaLaunchKernelEx(&cfg, layered_epilogue(p) ? gemv_cl_kernel<Bp, true> : gemv_cl_kernel<Bp, false>, p, ctx->dev_err));
   ctx->launches++;
   return LMB200_OK;
 }
@@ -1364,7 +1368,7 @@ int cluster_choice(const Ctx* ctx, int rows, int K) {
     cfg.attrs = attr;
     cfg.numAttrs = 1;
     int n_clusters = 0;
-    if (cudaOccupancyMaxActiveClusters(&n_clusters, gemv_cl_kernel<Bp>, &cfg) != cudaSuccess) {
+    if (cudaOccupancyMaxActiveClusters(&n_clusters, gemv_cl_kernel<Bp, false>, &cfg) != cudaSuccess) {
       cudaGetLastError();
       continue;
     }
@@ -1394,7 +1398,7 @@ constexpr size_t stream_smem() {
 template <int Bp>
 int32_t launch_bf16(Ctx* ctx, const GemvParams& p, cudaStream_t stream) {
   if (p.cluster >= 1) return launch_cluster<Bp>(ctx, p, stream);
-  LMB_CUDA(launch_k(gemv_tc_kernel<Bp>, dim3(p.grid), dim3(kTcThreads), stream_smem<Bp>(), stream, p, ctx->dev_err));
+  LMB_CUDA(launch_k(layered_epilogue(p) ? gemv_tc_kernel<Bp, true> : gemv_tc_kernel<Bp, false>, dim3(p.grid), dim3(kTcThreads), stream_smem<Bp>(), stream, p, ctx->dev_err));
   ctx->launches++;
   return LMB200_OK;
 }
@@ -1498,10 +1502,14 @@ int32_t gemv_configure() {
   LMB_CFG((gemv_ring_kernel<float, 1, kMtF32, 3>), kMaxSmem);
   LMB_CFG((gemv_ring_kernel<float, 2, kMtF32, 3>), kMaxSmem);
   LMB_CFG((gemv_ring_kernel<float, 4, kMtF32, 2>), kMaxSmem);
-  LMB_CFG(gemv_tc_kernel<16>, stream_smem<16>());
-  LMB_CFG(gemv_tc_kernel<32>, stream_smem<32>());
-  LMB_CFG(gemv_cl_kernel<16>, cluster_smem<16>());
-  LMB_CFG(gemv_cl_kernel<32>, cluster_smem<32>());
+  LMB_CFG((gemv_tc_kernel<16, false>), stream_smem<16>());
+  LMB_CFG((gemv_tc_kernel<16, true>), stream_smem<16>());
+  LMB_CFG((gemv_tc_kernel<32, false>), stream_smem<32>());
+  LMB_CFG((gemv_tc_kernel<32, true>), stream_smem<32>());
+  LMB_CFG((gemv_cl_kernel<16, false>), cluster_smem<16>());
+  LMB_CFG((gemv_cl_kernel<16, true>), cluster_smem<16>());
+  LMB_CFG((gemv_cl_kernel<32, false>), cluster_smem<32>());
+  LMB_CFG((gemv_cl_kernel<32, true>), cluster_smem<32>());
 #undef LMB_CFG
   return LMB200_OK;
 }
