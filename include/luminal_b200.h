@@ -270,18 +270,34 @@ enum { LMB200_ARCH_LLAMA = 0, LMB200_ARCH_WHISPER_DECODER = 1, LMB200_ARCH_LAYER
 int32_t lmb200_model_create(lmb200_ctx ctx, const lmb200_model_config* cfg, lmb200_model* model);
 
 /* A decoder whose layers are described one by one (LMB200_ARCH_LAYERED): every layer has its own mixer, sizes and
- * constants.  Layer i is x <- x + (mixer(h) + ff(h)) with h the RMSNorm of x; the head follows a final RMSNorm and may be
- * bounded by softcap * tanh(. / softcap).  Not in the reference, whose models repeat one kind of layer (src/NN.jl:417-507).
+ * constants.  Not in the reference, whose models repeat one kind of layer (src/NN.jl:417-507).  Two ways to arrange a layer
+ * (lmb200_layered_config.block):
+ *  - LMB200_BLOCK_PARALLEL: x <- x + (mixer(h) + ff(h)) with h the RMSNorm of x.
+ *  - LMB200_BLOCK_POSTNORM: x <- x + norm1(mixer(x)); x <- x + norm2(ff(x)); and, with side_dim > 0, x <- x + side.norm(side.proj
+ *    (gelu(side.gate x) * e)) with e the layer's side_dim columns of the token's row of "side.embed".
+ * The head follows a final RMSNorm and may be bounded by softcap * tanh(. / softcap).
  *  - LMB200_MIXER_LATENT_ATTENTION: causal attention whose keys and values are linear in one cached latent per token
  *    (kv_rank wide) plus one rotated key part shared by the heads (rot_dim wide); queries come from a latent of q_rank;
  *    every head's output is multiplied by a sigmoid gate.  kv_from >= 0: the layer has no latent of its own and reads the
  *    cache of that earlier layer.
  *  - LMB200_MIXER_RETENTION: linear attention with a fixed decay per head over a float32 state [dim, vdim] per head; the
  *    output of a head is divided by its root mean square and gated with silu.
- * Tensor names: "embed", "final.norm", "head"; per layer i "l<i>.norm1", "l<i>.mlp.up", "l<i>.mlp.down", and under
- * "l<i>.mix.": latent attention dq, dq.norm, uq, dkv, dkv.norm, uk, uv, g, o; retention q, k, v, g, o. */
-enum { LMB200_MIXER_LATENT_ATTENTION = 0, LMB200_MIXER_RETENTION = 1 };
+ *  - LMB200_MIXER_ATTENTION: grouped-query attention over a window of the last `window` positions (0: all); queries and keys are
+ *    rotated and divided by their root mean square per head; scores pass score_cap * tanh(. / score_cap) (0: not bounded).
+ *    kv_from >= 0: the layer has no keys and values of its own and reads the cache of that earlier layer.
+ *  - LMB200_MIXER_CHANNEL_DELTA: delta rule over a float32 state [dim, vdim] per head with one decay per key channel; q, k, v pass a
+ *    causal convolution of `conv` taps and silu, q and k are unit vectors; the head outputs are normed and gated.
+ *  - LMB200_MIXER_LIGHTNING: linear attention with a fixed decay per head, silu on q, k and v; the heads' outputs are normed
+ *    together and gated with a sigmoid.
+ * Tensor names: "embed", "final.norm", "head" (not with tied_head), "side.embed"; per layer i "l<i>.norm1", "l<i>.norm2",
+ * "l<i>.mlp.gate", "l<i>.mlp.up", "l<i>.mlp.down", "l<i>.side.gate", "l<i>.side.proj", "l<i>.side.norm", and under "l<i>.mix.":
+ * latent attention dq, dq.norm, uq, dkv, dkv.norm, uk, uv, g, o; retention q, k, v, g, o; attention q, k, v, o; channel delta q, k, v
+ * (and q.conv, k.conv, v.conv), b, A_log, dt_bias, a1, a2, g1, g2, norm, o; lightning q, k, v, g, norm, o. */
+enum { LMB200_MIXER_LATENT_ATTENTION = 0, LMB200_MIXER_RETENTION = 1, LMB200_MIXER_ATTENTION = 2, LMB200_MIXER_CHANNEL_DELTA = 3,
+       LMB200_MIXER_LIGHTNING = 4 };
 enum { LMB200_ROT_HALF = 0, LMB200_ROT_INTERLEAVED = 1 };   /* pairs (i, i + rot_dims/2), or (2i, 2i + 1) */
+enum { LMB200_BLOCK_PARALLEL = 0, LMB200_BLOCK_POSTNORM = 1 };
+enum { LMB200_FF_RELU2 = 0, LMB200_FF_SILU_GATE = 1 };      /* down(relu(up h)^2), or down(silu(gate h) * up h) */
 typedef struct {
   int32_t mixer;
   int32_t heads;
@@ -290,22 +306,37 @@ typedef struct {
   int32_t q_rank;          /* latent attention */
   int32_t kv_rank;         /* latent attention */
   int32_t rot_dim;         /* latent attention: width of the part with positions */
-  int32_t kv_from;         /* latent attention: -1, or the layer whose latent cache is read */
+  int32_t kv_from;         /* attention of either kind: -1, or the layer whose cache is read */
   int32_t rot_dims;        /* features that are rotated, from the first on (0: none; latent attention: rot_dim) */
   int32_t rot_layout;      /* LMB200_ROT_* */
-  int32_t ff;              /* width of the feed-forward down(relu(up h)^2); 0: none */
-  float scale;             /* latent attention: factor of the scores */
+  int32_t ff;              /* width of the feed-forward; 0: none */
+  float scale;             /* attention of either kind: factor of the scores */
   double rot_base;         /* frequency i is rot_base^(-2 i / rot_dims) */
-  const double* decay;     /* retention: [heads], each in (0, 1]; copied */
+  const double* decay;     /* retention, lightning: [heads], each in (0, 1]; copied */
+  int32_t ff_kind;         /* LMB200_FF_*: RELU2 with LMB200_BLOCK_PARALLEL, SILU_GATE with LMB200_BLOCK_POSTNORM */
+  int32_t kv_heads;        /* attention: key / value heads; channel delta: query / key heads; divides heads (0: heads) */
+  int32_t window;          /* attention */
+  float score_cap;         /* attention */
+  int32_t conv;            /* channel delta: taps */
+  int32_t decay_rank;      /* channel delta: rows of a1 */
+  int32_t gate_rank;       /* channel delta: rows of g1 */
+  /* attention: frequencies stretched by rot_factor (0: not) where a feature turns less than rot_slow times over rot_original
+   * positions, kept where it turns more than rot_fast times, blended linearly in between; cosine and sine times
+   * 0.1 ln(rot_factor) + 1 (YaRN) */
+  double rot_factor, rot_original, rot_fast, rot_slow;
 } lmb200_layer_config;
 typedef struct {
   int32_t n_layers;
   int32_t width;
   int32_t vocab;
-  int32_t dtype;           /* LMB200_F32, or LMB200_BF16: weights, latent cache and GEMM inputs bf16; residual, norms, scores,
+  int32_t dtype;           /* LMB200_F32, or LMB200_BF16: weights, caches and GEMM inputs bf16; residual, norms, scores,
                               states and accumulation float32 */
   float eps;               /* of every RMSNorm */
   float softcap;           /* 0: the logits are not bounded */
+  int32_t block;           /* LMB200_BLOCK_* */
+  int32_t side_dim;        /* LMB200_BLOCK_POSTNORM: width of the per-layer token input (0: none) */
+  int32_t tied_head;       /* the head is the embedding table */
+  float embed_scale;       /* factor of the embedding rows (0: 1) */
 } lmb200_layered_config;
 int32_t lmb200_model_create_layered(lmb200_ctx ctx, const lmb200_layered_config* cfg, const lmb200_layer_config* layers,
                                     lmb200_model* model);

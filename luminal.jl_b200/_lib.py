@@ -36,12 +36,14 @@ class ModelConfig(C.Structure):
 class LayerConfig(C.Structure):
     _fields_ = [(n, C.c_int32) for n in ("mixer", "heads", "dim", "vdim", "q_rank", "kv_rank", "rot_dim", "kv_from", "rot_dims",
                                          "rot_layout", "ff")] + \
-               [("scale", C.c_float), ("rot_base", C.c_double), ("decay", C.POINTER(C.c_double))]
+               [("scale", C.c_float), ("rot_base", C.c_double), ("decay", C.POINTER(C.c_double)), ("ff_kind", C.c_int32),
+                ("kv_heads", C.c_int32), ("window", C.c_int32), ("score_cap", C.c_float), ("conv", C.c_int32), ("decay_rank", C.c_int32),
+                ("gate_rank", C.c_int32)] + [(n, C.c_double) for n in ("rot_factor", "rot_original", "rot_fast", "rot_slow")]
 
 
 class LayeredConfig(C.Structure):
     _fields_ = [("n_layers", C.c_int32), ("width", C.c_int32), ("vocab", C.c_int32), ("dtype", C.c_int32), ("eps", C.c_float),
-                ("softcap", C.c_float)]
+                ("softcap", C.c_float), ("block", C.c_int32), ("side_dim", C.c_int32), ("tied_head", C.c_int32), ("embed_scale", C.c_float)]
 
 
 _i32, _i64, _u64, _f32, _vp = C.c_int32, C.c_int64, C.c_uint64, C.c_float, C.c_void_p

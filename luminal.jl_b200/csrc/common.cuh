@@ -187,6 +187,15 @@ struct FlashSplitView {
   int gate_pitch = 0;
 };
 
+// Grouped-query attention over the last `window` positions (0: all) with scores bounded by cap tanh(. / cap) (0: not): G query heads
+// per key head, widths dn and dv; the S queries are the last of Sk positions.
+struct FlashWindowView {
+  int H = 1, G = 1, dn = 0, dv = 0, window = 0;
+  float cap = 0.f;
+  int64_t q_b = 0, q_h = 0, q_s = 0, o_b = 0, o_h = 0, o_s = 0;
+  int64_t k_b = 0, k_h = 0, k_s = 0, v_b = 0, v_h = 0, v_s = 0;
+};
+
 static inline int64_t ceil_div(int64_t a, int64_t b) { return (a + b - 1) / b; }
 static inline int64_t round_up(int64_t a, int64_t b) { return ceil_div(a, b) * b; }
 

@@ -48,6 +48,12 @@ __device__ __forceinline__ float ex2_approx(float x) {
   return y;
 }
 
+__device__ __forceinline__ float rcp_approx(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
+  return y;
+}
+
 // chunk (row, d8) of a [rows x D] row-major tile -> canonical offset [d8][row/8][row%8][16 B]
 __device__ __forceinline__ uint32_t canon(int row, int c8, int rows) {
   return (uint32_t)(c8 * (rows * 16) + (row >> 3) * 128 + (row & 7) * 16);
@@ -117,6 +123,8 @@ struct FlashExtra {
   int64_t o_b = 0, o_h = 0, o_s = 0;
   const float* gate = nullptr;
   int gate_pitch = 0;
+  int window = 0;                   // a query sees the last `window` positions (0: all)
+  float cap = 0.f;                  // scores pass cap tanh(. / cap) (0: not)
 };
 
 __device__ __forceinline__ void mma_f16_ts(uint32_t tmem_d, uint32_t tmem_a, uint64_t bdesc, uint32_t idesc, uint32_t accumulate) {
@@ -125,7 +133,8 @@ __device__ __forceinline__ void mma_f16_ts(uint32_t tmem_d, uint32_t tmem_a, uin
       "r"(tmem_a), "l"(bdesc), "r"(idesc), "r"(accumulate)
       : "memory");
 }
-template <int DN, int DR, int DV>
+// WIN: windows, bounded scores and padded head widths are compiled in; the other models' kernels carry no code of them
+template <int DN, int DR, int DV, bool WIN>
 __global__ void __launch_bounds__(kThreads, 1)
 flash_tc_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict__ q, const __grid_constant__ CUtensorMap kmap,
                    const __grid_constant__ CUtensorMap vmap, const __grid_constant__ CUtensorMap rmap, const FlashView fv, const FlashExtra ex, int S,
@@ -155,14 +164,16 @@ flash_tc_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict
   __nv_bfloat16* ob_base = out + bi * ex.o_b + hi * ex.o_h;
   const int64_t q_s = fv.q_s;
   const int Sk = ex.Sk, q_off = ex.q_off;
-  int n_tiles[2];
+  int n_tiles[2], first[2];                           // key tiles first[t] .. n_tiles[t] - 1
 #pragma unroll
   for (int t = 0; t < 2; ++t) {
     const int qt0 = q0 + t * kBM;
     const int k_stop = qt0 >= S ? 0 : (causal ? min(Sk, q_off + qt0 + kBM) : Sk);
     n_tiles[t] = (k_stop + kBN - 1) / kBN;
+    first[t] = WIN && ex.window > 0 ? min(n_tiles[t], max(0, q_off + qt0 - ex.window + 1) / kBN) : 0;
   }
   const int n_max = max(n_tiles[0], n_tiles[1]);
+  const int jb = WIN ? first[0] : 0;                  // the first query tile is never empty and starts no later than the second
 
   if (tid == 0) {
     mbar_init(&q_full, kLoaders / 32);
@@ -186,7 +197,7 @@ flash_tc_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict
       const int row = i / (D / 8), c8 = i - row * (D / 8);
       const int qi = q0 + row;
       const int d = c8 * 8;                                  // the padding behind either part of a query is zero
-      const bool valid = qi < S && (DR == 0 || (d < DN ? d < ex.dn : d - DN < ex.dr));
+      const bool valid = qi < S && ((DR == 0 && !WIN) || (d < DN ? d < ex.dn : d - DN < ex.dr));
       const int src = DR == 0 || d < DN ? d : ex.dn + d - DN;
       cp_async16(sQ + (row >> 7) * SM::kQ + canon(row & 127, c8, kBM), qb + (int64_t)min(qi, S - 1) * q_s + (valid ? src : 0), valid ? 16u : 0u);
     }
@@ -200,9 +211,9 @@ flash_tc_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict
     const CUtensorMap* map = lw == 0 ? &kmap : &vmap;
     const int off = lw == 0 ? SM::offK : SM::offV;
     const int stages = lw == 0 ? kStages : vStages, stage_bytes = lw == 0 ? SM::kK : SM::kV, subs = (lw == 0 ? DN : DV) / W;
-    for (int j = 0; j < n_max; ++j) {
-      const int s = j % stages;
-      mbar_wait(&empty[s], ((j / stages) & 1) ^ 1, dead, err);
+    for (int j = jb; j < n_max; ++j) {
+      const int s = (j - jb) % stages;
+      mbar_wait(&empty[s], (((j - jb) / stages) & 1) ^ 1, dead, err);
       if (lane == 0) {
         mbar_expect_tx(&full[s], (uint32_t)stage_bytes);
         unsigned char* at = smem + off + s * stage_bytes;
@@ -220,7 +231,7 @@ flash_tc_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict
     auto issue_s = [&](int j, int t) {                // S[t] = Q[t] K(j)^T
       if (lane == 0) {
         const uint64_t adesc = smem_desc(smem_u32(smem + SM::offQ + t * SM::kQ), kBM * 16, 128);
-        const uint32_t sK = smem_u32(smem + SM::offK + (j % kStages) * SM::kK);
+        const uint32_t sK = smem_u32(smem + SM::offK + ((j - jb) % kStages) * SM::kK);
 #pragma unroll
         for (int ks = 0; ks < D / 16; ++ks) {
           const uint64_t bdesc = smem_desc_swz(sK + ((16 * ks) / W) * kSub + ((16 * ks) % W) * 2, 16, 16 * W, kSwz);
@@ -232,32 +243,37 @@ flash_tc_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict
     };
     auto issue_pv = [&](int j, int t) {               // O[t] += P[t] V(j), P read from tensor memory
       if (lane == 0) {
-        const uint64_t bdesc = smem_desc_swz(smem_u32(smem + SM::offV + (j % vStages) * SM::kV), kSub, 16 * W, kSwz);
+        const uint64_t bdesc = smem_desc_swz(smem_u32(smem + SM::offV + ((j - jb) % vStages) * SM::kV), kSub, 16 * W, kSwz);
 #pragma unroll
         for (int ks = 0; ks < kBN / 16; ++ks)
           mma_f16_ts(tmem + kColO + t * DV, tmem + kColS + t * kBN + ks * 8, bdesc + (uint64_t)(ks * ((32 * W) >> 4)), kIdescPV,
-                     (j > 0 || ks > 0) ? 1u : 0u);
+                     (j > first[t] || ks > 0) ? 1u : 0u);
         if (j == n_tiles[t] - 1) commit(&o_done[t]);
       }
       __syncwarp();
     };
-    if (n_max >= 1) {
+    if (n_max > jb) {
       mbar_wait(&k_full[0], 0, dead, err);
       fence_after();
 #pragma unroll
       for (int t = 0; t < 2; ++t)
-        if (n_tiles[t] >= 1) issue_s(0, t);
+        if (first[t] == jb && n_tiles[t] > jb) issue_s(jb, t);
       if (lane == 0) commit(&k_empty[0]);
       __syncwarp();
     }
-    for (int j = 0; j < n_max; ++j) {
-      const int s = j % vStages, s1 = (j + 1) % kStages;
-      mbar_wait(&v_full[s], (j / vStages) & 1, dead, err);
-      if (j + 1 < n_max) mbar_wait(&k_full[s1], ((j + 1) / kStages) & 1, dead, err);
+    for (int j = jb; j < n_max; ++j) {
+      const int i = j - jb, s = i % vStages, s1 = (i + 1) % kStages;
+      mbar_wait(&v_full[s], (i / vStages) & 1, dead, err);
+      if (j + 1 < n_max) mbar_wait(&k_full[s1], ((i + 1) / kStages) & 1, dead, err);
 #pragma unroll
       for (int t = 0; t < 2; ++t) {
         if (j >= n_tiles[t]) continue;
-        mbar_wait(&p_full[t], j & 1, dead, err);
+        if (WIN && j < first[t]) {                       // the second query tile's window starts one key tile later
+          fence_after();
+          if (j + 1 == first[t] && j + 1 < n_tiles[t]) issue_s(j + 1, t);
+          continue;
+        }
+        mbar_wait(&p_full[t], (j - first[t]) & 1, dead, err);
         fence_after();
         issue_pv(j, t);
         if (j + 1 < n_tiles[t]) issue_s(j + 1, t);       // runs after P V(j) in the tensor pipe: S overwrites P's columns
@@ -282,12 +298,18 @@ flash_tc_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict
     const int pair_bar = 1 + t * 4 + wq;              // named barrier of the two warps that share these rows
     const float c = scale * kLog2e;
     const int nt = n_tiles[t];
+    const int j0 = first[t];
+    // a score in log2 units: s c, or cap tanh(s scale / cap) log2(e) as cap' - 2 cap' / (1 + 2^(s k2)) with cap' = cap log2(e)
+    const float capl = WIN ? ex.cap * kLog2e : 0.f, k2 = WIN && ex.cap > 0.f ? 2.0f * c / ex.cap : 0.f;
+    auto bounded = [&](float x) { return fmaf(-2.0f * capl, rcp_approx(1.0f + ex2_approx(x * k2)), capl); };
+    auto hidden = [&](int key) { return key >= Sk || (causal && key > q_off + qi) || (WIN && ex.window > 0 && key <= q_off + qi - ex.window); };
     float m = -CUDART_INF_F, l = 0.f;
-    for (int j = 0; j < nt; ++j) {
-      mbar_wait(&s_full[t], j & 1, dead, err);          // S(j) is complete, and with it (pipe order) P V(j - 1): O is at rest
+    for (int j = j0; j < nt; ++j) {
+      mbar_wait(&s_full[t], (j - j0) & 1, dead, err);          // S(j) is complete, and with it (pipe order) P V(j - 1): O is at rest
       fence_after();
       const int key0 = j * kBN + h * 64;
-      const bool inside = (j + 1) * kBN <= Sk && (!causal || (j + 1) * kBN - 1 <= q_off + q0 + t * kBM);   // no key of the tile is masked
+      const bool inside = (j + 1) * kBN <= Sk && (!causal || (j + 1) * kBN - 1 <= q_off + q0 + t * kBM) &&
+                          (!WIN || ex.window == 0 || j * kBN > q_off + q0 + t * kBM + kBM - 1 - ex.window);   // no key of the tile is masked
       // pass 1: the maximum of this thread's 64 scores
       float mx4[4] = {-CUDART_INF_F, -CUDART_INF_F, -CUDART_INF_F, -CUDART_INF_F};
 #pragma unroll
@@ -301,7 +323,7 @@ flash_tc_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict
 #pragma unroll
           for (int i = 0; i < 32; ++i) {
             const int key = key0 + qd * 32 + i;
-            if (!(key >= Sk || (causal && key > q_off + qi))) mx4[i & 3] = fmaxf(mx4[i & 3], sv[i]);
+            if (!hidden(key)) mx4[i & 3] = fmaxf(mx4[i & 3], sv[i]);
           }
         }
       }
@@ -309,10 +331,11 @@ flash_tc_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict
       xch[t][h][r] = mx;
       asm volatile("bar.sync %0, 64;\n" ::"r"(pair_bar) : "memory");
       mx = fmaxf(mx, xch[t][h ^ 1][r]);
-      mx *= c;
-      const bool first = m == -CUDART_INF_F && mx > -CUDART_INF_F;
+      if (WIN && capl > 0.f) mx = mx > -CUDART_INF_F ? bounded(mx) : mx;
+      else mx *= c;
+      const bool starts = m == -CUDART_INF_F && mx > -CUDART_INF_F;
       const bool raise = m > -CUDART_INF_F && mx > m + kRescaleStep;
-      if (__any_sync(0xffffffffu, raise) && j > 0) {      // both halves decide alike; each rescales its half of O's columns
+      if (__any_sync(0xffffffffu, raise) && j > j0) {      // both halves decide alike; each rescales its half of O's columns
         const float alpha = raise ? exp2f(m - mx) : 1.0f;
 #pragma unroll
         for (int ch = 0; ch < DV / 32; ++ch) {
@@ -327,7 +350,7 @@ flash_tc_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict
         }
       }
       if (raise) { l *= exp2f(m - mx); m = mx; }
-      if (first) m = mx;
+      if (starts) m = mx;
       const float neg_m = m == -CUDART_INF_F ? 0.f : -m;
       // pass 2: p = exp2(s c - m) as bf16 pairs, kept in registers until the other half has read its scores too
       uint64_t sum2[4] = {0ull, 0ull, 0ull, 0ull};           // four chains of (even, odd) partial sums
@@ -340,13 +363,22 @@ flash_tc_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict
 #pragma unroll
         for (int i = 0; i < 16; i += 2) {
           float a0 = sv[i], a1 = sv[i + 1];
-          if (!inside) {
-            const int key = key0 + qd * 16 + i;
-            if (key >= Sk || (causal && key > q_off + qi)) a0 = -CUDART_INF_F;
-            if (key + 1 >= Sk || (causal && key + 1 > q_off + qi)) a1 = -CUDART_INF_F;
-          }
+          const int key = key0 + qd * 16 + i;
           float x0, x1;
-          unpack2(fma2(pack2(a0, a1), c2, negm2), x0, x1);
+          if (WIN && capl > 0.f) {
+            x0 = bounded(a0) + neg_m;
+            x1 = bounded(a1) + neg_m;
+            if (!inside) {
+              if (hidden(key)) x0 = -CUDART_INF_F;
+              if (hidden(key + 1)) x1 = -CUDART_INF_F;
+            }
+          } else {
+            if (!inside) {
+              if (hidden(key)) a0 = -CUDART_INF_F;
+              if (hidden(key + 1)) a1 = -CUDART_INF_F;
+            }
+            unpack2(fma2(pack2(a0, a1), c2, negm2), x0, x1);
+          }
           const float p0 = ex2_approx(x0), p1 = ex2_approx(x1);
           sum2[(i >> 1) & 3] = add2(sum2[(i >> 1) & 3], pack2(p0, p1));
           const __nv_bfloat162 pb2 = __floats2bfloat162_rn(p0, p1);
@@ -371,7 +403,7 @@ flash_tc_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict
       __syncwarp();
       if (lane == 0) mbar_arrive(&p_full[t]);
     }
-    if (nt >= 1) {
+    if (nt > j0) {
       xch[t][h][r] = l;
       asm volatile("bar.sync %0, 64;\n" ::"r"(pair_bar) : "memory");
       l += xch[t][h ^ 1][r];
@@ -387,7 +419,7 @@ flash_tc_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict
         if (qi < S) {
 #pragma unroll
           for (int i = 0; i < 16; i += 8) {
-            if (DR > 0 && h * (DV / 2) + ch * 16 + i >= ex.dv) continue;      // padding behind the value's width
+            if ((DR > 0 || WIN) && h * (DV / 2) + ch * 16 + i >= ex.dv) continue;      // padding behind the value's width
             uint4 w;
             __nv_bfloat162 a0 = __floats2bfloat162_rn(o[i] * inv, o[i + 1] * inv), a1 = __floats2bfloat162_rn(o[i + 2] * inv, o[i + 3] * inv);
             __nv_bfloat162 a2 = __floats2bfloat162_rn(o[i + 4] * inv, o[i + 5] * inv), a3 = __floats2bfloat162_rn(o[i + 6] * inv, o[i + 7] * inv);
@@ -411,15 +443,19 @@ flash_tc_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict
 }  // namespace
 
 int32_t flash_tc_configure() {
-#define LMB_CFG(...) \
-  LMB_CUDA(cudaFuncSetAttribute(flash_tc_kernel<__VA_ARGS__>, cudaFuncAttributeMaxDynamicSharedMemorySize, Smem<__VA_ARGS__>::total + 1024))
-  LMB_CFG(128, 0, 128);
-  LMB_CFG(96, 0, 96);
-  LMB_CFG(64, 0, 64);
-  LMB_CFG(64, 64, 64);
-  LMB_CFG(64, 64, 128);
-  LMB_CFG(128, 64, 64);
-  LMB_CFG(128, 64, 128);
+#define LMB_CFG(DN, DR, DV, WIN) \
+  LMB_CUDA(cudaFuncSetAttribute(flash_tc_kernel<DN, DR, DV, WIN>, cudaFuncAttributeMaxDynamicSharedMemorySize, Smem<DN, DR, DV>::total + 1024))
+  LMB_CFG(128, 0, 128, false);
+  LMB_CFG(96, 0, 96, false);
+  LMB_CFG(64, 0, 64, false);
+  LMB_CFG(64, 64, 64, false);
+  LMB_CFG(64, 64, 128, false);
+  LMB_CFG(128, 64, 64, false);
+  LMB_CFG(128, 64, 128, false);
+  LMB_CFG(64, 0, 64, true);
+  LMB_CFG(64, 0, 128, true);
+  LMB_CFG(128, 0, 64, true);
+  LMB_CFG(128, 0, 128, true);
 #undef LMB_CFG
   return LMB200_OK;
 }
@@ -477,7 +513,7 @@ int32_t flash_tc_launch_view(Ctx* ctx, void* out, const void* q, const void* k, 
   ex.Sk = (int)S; ex.dn = ex.dv = (int)D;
   ex.o_b = fv.q_b; ex.o_h = fv.q_h; ex.o_s = fv.q_s;
 #define LMB_FLASH(DD)                                                                                                   \
-  flash_tc_kernel<DD, 0, DD><<<grid, kThreads, Smem<DD, 0, DD>::total + 1024, stream>>>(                          \
+  flash_tc_kernel<DD, 0, DD, false><<<grid, kThreads, Smem<DD, 0, DD>::total + 1024, stream>>>(                          \
       (__nv_bfloat16*)out, (const __nv_bfloat16*)q, kmap, vmap, kmap, fv, ex, (int)S, scale, causal, ctx->dev_err)
   if (D == 128) LMB_FLASH(128);
   else if (D == 96) LMB_FLASH(96);
@@ -515,8 +551,42 @@ int32_t flash_tc_launch_split(Ctx* ctx, void* out, const void* q, const void* k,
   ex.gate = f.gate; ex.gate_pitch = f.gate_pitch;
   const dim3 grid((unsigned)ceil_div(Sq, 2 * kBM), (unsigned)(B * f.H));
 #define LMB_FLASH(DN, DV)                                                                                              \
-  flash_tc_kernel<DN, 64, DV><<<grid, kThreads, Smem<DN, 64, DV>::total + 1024, stream>>>(                       \
+  flash_tc_kernel<DN, 64, DV, false><<<grid, kThreads, Smem<DN, 64, DV>::total + 1024, stream>>>(                       \
       (__nv_bfloat16*)out, (const __nv_bfloat16*)q, kmap, vmap, rmap, fv, ex, (int)Sq, scale, 1, ctx->dev_err)
+  if (f.dn <= 64 && f.dv <= 64) LMB_FLASH(64, 64);
+  else if (f.dn <= 64) LMB_FLASH(64, 128);
+  else if (f.dv <= 64) LMB_FLASH(128, 64);
+  else LMB_FLASH(128, 128);
+#undef LMB_FLASH
+  ctx->launches++;
+  LMB_CUDA(cudaGetLastError());
+  return LMB200_OK;
+}
+
+bool flash_tc_window_supported(int dn, int dv) { return dn >= 8 && dn <= 128 && dn % 8 == 0 && dv >= 8 && dv <= 128 && dv % 8 == 0; }
+
+// causal attention of the last Sq of Sk positions over the last f.window positions, scores bounded by f.cap
+int32_t flash_tc_launch_window(Ctx* ctx, void* out, const void* q, const void* k, const void* v, const FlashWindowView& f, int64_t B, int64_t Sq,
+                               int64_t Sk, float scale, cudaStream_t stream) {
+  LMB_REQUIRE(flash_tc_window_supported(f.dn, f.dv), "flash attention: head widths %d, %d", f.dn, f.dv);
+  LMB_REQUIRE(Sq >= 1 && Sk >= Sq && B * f.H <= 65535, "flash attention: %lld queries, %lld keys", (long long)Sq, (long long)Sk);
+  LMB_REQUIRE((reinterpret_cast<uintptr_t>(q) & 15) == 0 && (reinterpret_cast<uintptr_t>(out) & 15) == 0 && f.q_s % 8 == 0 && f.q_h % 8 == 0 &&
+                  f.q_b % 8 == 0 && f.o_s % 8 == 0 && f.o_h % 8 == 0 && f.o_b % 8 == 0,
+              "flash attention: query and output rows must start on 16 bytes");
+  CUtensorMap kmap, vmap;
+  LMB_TRY(kv_tensor_map(&kmap, k, f.H / f.G, B, Sk, f.dn, f.k_s, f.k_h, f.k_b, 64));
+  LMB_TRY(kv_tensor_map(&vmap, v, f.H / f.G, B, Sk, f.dv, f.v_s, f.v_h, f.v_b, 64));
+  FlashView fv;
+  fv.H = f.H; fv.G = f.G;
+  fv.q_b = f.q_b; fv.q_h = f.q_h; fv.q_s = f.q_s;
+  FlashExtra ex;
+  ex.Sk = (int)Sk; ex.q_off = (int)(Sk - Sq); ex.dn = f.dn; ex.dv = f.dv;
+  ex.o_b = f.o_b; ex.o_h = f.o_h; ex.o_s = f.o_s;
+  ex.window = f.window; ex.cap = f.cap;
+  const dim3 grid((unsigned)ceil_div(Sq, 2 * kBM), (unsigned)(B * f.H));
+#define LMB_FLASH(DN, DV)                                                                                              \
+  flash_tc_kernel<DN, 0, DV, true><<<grid, kThreads, Smem<DN, 0, DV>::total + 1024, stream>>>(                         \
+      (__nv_bfloat16*)out, (const __nv_bfloat16*)q, kmap, vmap, kmap, fv, ex, (int)Sq, scale, 1, ctx->dev_err)
   if (f.dn <= 64 && f.dv <= 64) LMB_FLASH(64, 64);
   else if (f.dn <= 64) LMB_FLASH(64, 128);
   else if (f.dv <= 64) LMB_FLASH(128, 64);

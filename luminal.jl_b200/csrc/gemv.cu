@@ -553,7 +553,7 @@ __device__ __forceinline__ void row_epilogue(const GemvParams& p, float (&v)[NV]
     }
     return;
   }
-  if (X && p.epi == EPI_STORE_RELU2) {
+  if (X && (p.epi == EPI_STORE_RELU2 || p.epi == EPI_STORE_ACT)) {
     if (row < p.act_row0) {
 #pragma unroll
       for (int b = 0; b < N; ++b)
@@ -563,7 +563,21 @@ __device__ __forceinline__ void row_epilogue(const GemvParams& p, float (&v)[NV]
 #pragma unroll
       for (int b = 0; b < N; ++b) {
         const float u = fmaxf(v[b], 0.f);
-        if (b0 + b < p.B) act[LY::x_offset(b0 + b, p.act_col0 + row - p.act_row0, BP)] = __float2bfloat16_rn(u * u);
+        if (b0 + b < p.B) act[LY::x_offset(b0 + b, p.act_col0 + row - p.act_row0, BP)] = __float2bfloat16_rn(p.epi == EPI_STORE_ACT ? v[b] : u * u);
+      }
+    }
+    return;
+  }
+  if (X && p.epi == EPI_GELU_TOKEN) {
+    if (row < p.rows) {
+      __nv_bfloat16* act = reinterpret_cast<__nv_bfloat16*>(p.act);
+      const __nv_bfloat16* table = reinterpret_cast<const __nv_bfloat16*>(p.token_table);
+#pragma unroll
+      for (int b = 0; b < N; ++b) {
+        if (b0 + b >= p.B) continue;
+        const int tok = p.tokens[b0 + b];
+        const float e = tok >= 0 && tok < p.token_rows ? __bfloat162float(table[(int64_t)tok * p.token_pitch + row]) : 0.f;
+        act[LY::x_offset(b0 + b, row, BP)] = __float2bfloat16_rn(gelu_ref(v[b]) * e);
       }
     }
     return;
@@ -900,6 +914,109 @@ __device__ __forceinline__ void resid_norm_tile(const GemvParams& p, const unsig
   }
 }
 
+// EPI_POST_NORM on the tile a cluster CTA finalises; threads and rows as in resid_norm_tile.
+template <int N>
+__device__ __forceinline__ void post_norm_tile(const GemvParams& p, const unsigned char* recv_raw, int C, int c, int r, int e, float* s_red,
+                                               float* s_scale, const float* s_inv, int* err) {
+  constexpr int BG = N / 8;
+  const int lane = e & 31, we = e >> 5;
+  const int rows_per = 128 / C;
+  const int bg = e & 3, rl0 = e >> 2;
+  const int row0 = r * 128 + c * rows_per;
+  const int iters = (rows_per + 31) >> 5;
+  const float4* recv = reinterpret_cast<const float4*>(recv_raw);
+  float acc[4][8], xv[4][8], ss[8];
+  bool valid[4];
+#pragma unroll
+  for (int i = 0; i < 8; ++i) ss[i] = 0.f;
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    const int rl = rl0 + 32 * j;
+    valid[j] = j < iters && bg < BG && rl < rows_per && row0 + rl < p.rows;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) acc[j][i] = xv[j][i] = 0.f;
+    if (!valid[j]) continue;
+    for (int src = 0; src < C; ++src) {
+      const float4 t0 = recv[((src * rows_per + rl) * N + 8 * bg) / 4], t1 = recv[((src * rows_per + rl) * N + 8 * bg) / 4 + 1];
+      acc[j][0] += t0.x; acc[j][1] += t0.y; acc[j][2] += t0.z; acc[j][3] += t0.w;
+      acc[j][4] += t1.x; acc[j][5] += t1.y; acc[j][6] += t1.z; acc[j][7] += t1.w;
+    }
+    const float4* xr = reinterpret_cast<const float4*>(p.pn.x + (size_t)(row0 + rl) * N + 8 * bg);
+    const float4 x0 = xr[0], x1 = xr[1];
+    xv[j][0] = x0.x; xv[j][1] = x0.y; xv[j][2] = x0.z; xv[j][3] = x0.w;
+    xv[j][4] = x1.x; xv[j][5] = x1.y; xv[j][6] = x1.z; xv[j][7] = x1.w;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      if (s_inv) acc[j][i] *= s_inv[8 * bg + i];
+      ss[i] += acc[j][i] * acc[j][i];
+    }
+  }
+  auto publish = [&](float* slots) {                           // per-CTA sums of ss over the rows
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      ss[i] += __shfl_xor_sync(0xffffffffu, ss[i], 4);
+      ss[i] += __shfl_xor_sync(0xffffffffu, ss[i], 8);
+      ss[i] += __shfl_xor_sync(0xffffffffu, ss[i], 16);
+    }
+    if (lane < 4) {
+#pragma unroll
+      for (int i = 0; i < 8; ++i) s_red[we * 32 + 8 * lane + i] = ss[i];
+    }
+    asm volatile("bar.sync 1, 128;\n" ::: "memory");
+    if (e < 32) slots[(size_t)blockIdx.x * 32 + e] = ((s_red[e] + s_red[32 + e]) + s_red[64 + e]) + s_red[96 + e];
+  };
+  publish(p.pn.slots);
+  __threadfence();
+  asm volatile("bar.sync 1, 128;\n" ::: "memory");
+  if (e == 0) {
+    atomicAdd(p.pn.counter, 1u);
+    const long long t0 = clock64();
+    for (;;) {
+      unsigned seen;
+      asm volatile("ld.acquire.gpu.global.u32 %0, [%1];\n" : "=r"(seen) : "l"(p.pn.counter) : "memory");
+      if (seen >= gridDim.x) break;
+      if (clock64() - t0 > kWaitLimit) { if (err) atomicExch(err, 1); break; }
+    }
+  }
+  asm volatile("bar.sync 1, 128;\n" ::: "memory");
+  {                                                            // four lanes per sequence, the same sums in every CTA
+    const int b = e >> 2, part = e & 3;
+    float s = 0.f;
+#pragma unroll 8
+    for (int t = part; t < (int)gridDim.x; t += 4) s += __ldcg(p.pn.slots + t * 32 + b);
+    s += __shfl_xor_sync(0xffffffffu, s, 1);
+    s += __shfl_xor_sync(0xffffffffu, s, 2);
+    if (part == 0) s_scale[b] = 1.0f / sqrtf(s / (float)p.rows + p.pn.eps);
+  }
+  asm volatile("bar.sync 1, 128;\n" ::: "memory");
+  if (e == 0 && atomicAdd(p.pn.counter + 1, 1u) == gridDim.x - 1) { p.pn.counter[0] = 0u; p.pn.counter[1] = 0u; }
+  __nv_bfloat16* xg = reinterpret_cast<__nv_bfloat16*>(p.pn.xg);
+#pragma unroll
+  for (int i = 0; i < 8; ++i) ss[i] = 0.f;
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    if (!valid[j]) continue;
+    const int grow = row0 + rl0 + 32 * j;
+    const float w = p.pn.w[grow], g = p.pn.gain ? p.pn.gain[grow] : 1.0f;
+    __nv_bfloat16* o = xg + (size_t)(grow >> 3) * (N * 8) + bg * 64 + (grow & 7);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      xv[j][i] += acc[j][i] * s_scale[8 * bg + i] * w;
+      o[8 * i] = __float2bfloat16_rn(xv[j][i] * g);
+      ss[i] += xv[j][i] * xv[j][i];
+    }
+    float4* xr = reinterpret_cast<float4*>(p.pn.x + (size_t)grow * N + 8 * bg);
+    xr[0] = make_float4(xv[j][0], xv[j][1], xv[j][2], xv[j][3]);
+    xr[1] = make_float4(xv[j][4], xv[j][5], xv[j][6], xv[j][7]);
+    if (p.pn.capture) {
+#pragma unroll
+      for (int i = 0; i < 8; ++i)
+        if (8 * bg + i < p.B) p.pn.capture[(size_t)(8 * bg + i) * p.rows + grow] = xv[j][i];
+    }
+  }
+  if (p.pn.ssq) publish(p.pn.ssq);
+}
+
 template <int N, bool X>
 __global__ void __launch_bounds__(kTcThreads, 1) gemv_tc_kernel(const GemvParams p, int* err) {
   constexpr int kXStage = N * 256;
@@ -1178,6 +1295,7 @@ __global__ void __launch_bounds__(kTcThreads, 1) gemv_cl_kernel(const GemvParams
   __shared__ uint32_t tmem_base_slot;
   __shared__ float s_inv_buf[64];        // [0, 32): inv per sequence, [32, 64): mean * inv (LayerNorm)
   __shared__ float s_red[128];
+  __shared__ float s_scale[X ? 32 : 1];
   const float* s_inv = p.inv.ssq ? s_inv_buf : nullptr;
 
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
@@ -1295,6 +1413,8 @@ __global__ void __launch_bounds__(kTcThreads, 1) gemv_cl_kernel(const GemvParams
   if (tid == 64) LMB_TRACE(7);
   if (warp >= 2 && p.epi == EPI_RESID_NORM) {
     resid_norm_tile<N>(p, smem + kStages * kStage, C, c, r, tid - 64, s_red);
+  } else if (X && warp >= 2 && p.epi == EPI_POST_NORM) {
+    post_norm_tile<N>(p, smem + kStages * kStage, C, c, r, tid - 64, s_red, s_scale, s_inv, err);
   } else if (warp >= 2) {
     const int e = tid - 64;
     const int rows_per = 128 / C;
@@ -1321,7 +1441,9 @@ __global__ void __launch_bounds__(kTcThreads, 1) gemv_cl_kernel(const GemvParams
   if (tid == 0) { LMB_TRACE(9); LMB_TRACE_NS(11); }
 }
 
-bool layered_epilogue(const GemvParams& p) { return p.epi == EPI_STORE_RELU2 || p.softcap > 0.f; }
+bool layered_epilogue(const GemvParams& p) {
+  return p.epi == EPI_STORE_RELU2 || p.epi == EPI_STORE_ACT || p.epi == EPI_GELU_TOKEN || p.epi == EPI_POST_NORM || p.softcap > 0.f;
+}
 
 template <int Bp>
 constexpr size_t cluster_smem() {
@@ -1398,6 +1520,7 @@ constexpr size_t stream_smem() {
 template <int Bp>
 int32_t launch_bf16(Ctx* ctx, const GemvParams& p, cudaStream_t stream) {
   if (p.cluster >= 1) return launch_cluster<Bp>(ctx, p, stream);
+  LMB_REQUIRE(p.epi != EPI_RESID_NORM && p.epi != EPI_POST_NORM, "gemv: this epilogue needs a plan of gemv_plan_resid");
   LMB_CUDA(launch_k(layered_epilogue(p) ? gemv_tc_kernel<Bp, true> : gemv_tc_kernel<Bp, false>, dim3(p.grid), dim3(kTcThreads), stream_smem<Bp>(), stream, p, ctx->dev_err));
   ctx->launches++;
   return LMB200_OK;

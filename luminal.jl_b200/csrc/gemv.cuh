@@ -12,7 +12,10 @@ enum GemvEpilogue {
   EPI_QKV_ROPE = 2,    // RoPE on q and k (if `rope`), q -> q_out, k/v appended to the cache at *pos
   EPI_GELU_ACT = 3,    // act[b, row] = gelu(acc)                  (Whisper fc1)
   EPI_STORE_RELU2 = 5, // rows < act_row0: out[b, row] = acc; rows from act_row0: act[b, act_col0 + row - act_row0] = relu(acc)^2
-  EPI_RESID_NORM = 4   // row-parallel projection + all-reduce + residual add + RMSNorm preparation (ResidNorm below)
+  EPI_RESID_NORM = 4,  // row-parallel projection + all-reduce + residual add + RMSNorm preparation (ResidNorm below)
+  EPI_STORE_ACT = 6,   // like EPI_STORE_RELU2 with act = acc
+  EPI_GELU_TOKEN = 7,  // act[b, row] = gelu(acc) * token_table[tokens[b] * token_pitch + row]
+  EPI_POST_NORM = 8    // residual add of the projection's own RMSNorm (PostNorm below)
 };
 
 // Exchange of a row-parallel projection's partial results between the tensor-parallel ranks, done by
@@ -57,6 +60,24 @@ struct ResidNorm {
   float* capture = nullptr;                // [B][rows] float32 copy of the new residual rows (parity tests) or NULL
 };
 
+// EPI_POST_NORM: a sublayer that is normed on its output.  With y = acc (times the input's scale, InvScale),
+//   x[row][b] += y / sqrt(mean over the rows of y^2 + eps) * w[row]
+//   xg[b, row] = bf16(x * gain[row])                            (gain NULL: 1)
+//   ssq[cta][b] = sum over this CTA's rows of the new x^2       (NULL: not wanted)
+// The mean needs every row: the CTAs (all resident, one wave) leave their sums in slots[cta][32], count themselves in at counter[0],
+// wait (bounded) for the others and add the slots in CTA order.  counter[0..1] are zero between launches.
+struct PostNorm {
+  float* x = nullptr;
+  const float* w = nullptr;
+  void* xg = nullptr;
+  const float* gain = nullptr;
+  float* ssq = nullptr;
+  float* capture = nullptr;                // [B][rows] float32 copy of the new residual rows, or NULL
+  float* slots = nullptr;
+  unsigned* counter = nullptr;
+  float eps = 0.f;
+};
+
 // Consumer side: inv[b] = 1 / sqrt(sum_t ssq[t][b] * (1/n) + eps) multiplies every accumulator of batch
 // column b before the rest of the epilogue.  ssq == NULL: no scaling.
 // LayerNorm (sum != NULL; src/NN.jl:138-173, src/HighLevelOps.jl:292-304): with mu = mean(x) and inv = 1 / sqrt(mean(x*x)
@@ -93,7 +114,10 @@ struct GemvParams {
   float* out = nullptr;
   int out_pitch = 0;
   float softcap = 0.f;       // > 0: out = softcap * tanh(acc / softcap)
-  int act_row0 = 0, act_col0 = 0;   // EPI_STORE_RELU2
+  int act_row0 = 0, act_col0 = 0;   // EPI_STORE_RELU2, EPI_STORE_ACT
+  const void* token_table = nullptr;   // EPI_GELU_TOKEN: bf16
+  int token_pitch = 0, token_rows = 0;
+  const int* tokens = nullptr;
   // EPI_SILU_GATE: act is a GEMV activation buffer of the same batch padding as x
   void* act = nullptr;
   int n_act = 0;
@@ -114,6 +138,7 @@ struct GemvParams {
   InvScale inv;              // per-sequence RMSNorm scale applied to the accumulators (before the bias)
   const float* ln_wg = nullptr;  // LayerNorm input: W g per internal row (see InvScale)
   ResidNorm rn;              // EPI_RESID_NORM
+  PostNorm pn;               // EPI_POST_NORM (a plan of gemv_plan_resid)
   PeerPush push;             // EPI_RESID_NORM under tensor parallelism (n > 1)
   // L2 prefetch for the GEMV that runs next (bf16 tensor-core kernels): once a CTA's producer has issued
   // its last copy, HBM would idle through this kernel's fold, epilogue and drain; instead it pulls the

@@ -576,7 +576,7 @@ __global__ void __launch_bounds__(256) argmax_tp_select_kernel(const PeerReduce 
 // (e >> 2) + 32 j of the CTA's rows and batch columns 8 (e & 3) .. + 7.
 template <int N>
 __global__ void __launch_bounds__(128) embed_prep_kernel(const int* __restrict__ tokens, const __nv_bfloat16* __restrict__ embed,
-                                                         int vocab, int hidden, int B, const float* __restrict__ gain,
+                                                         int vocab, int hidden, int B, const float* __restrict__ gain, float scale,
                                                          float* __restrict__ x, __nv_bfloat16* __restrict__ xg,
                                                          float* __restrict__ ssq_out, int rows_per_cta) {
   __shared__ float s_red[128];
@@ -599,11 +599,11 @@ __global__ void __launch_bounds__(128) embed_prep_kernel(const int* __restrict__
     if (k >= hidden || bg >= N / 8) continue;
     float xv[8];
 #pragma unroll
-    for (int i = 0; i < 8; ++i) xv[i] = tok[i] >= 0 ? __bfloat162float(embed[(int64_t)tok[i] * hidden + k]) : 0.f;
+    for (int i = 0; i < 8; ++i) xv[i] = tok[i] >= 0 ? __bfloat162float(embed[(int64_t)tok[i] * hidden + k]) * scale : 0.f;
     float4* xr = reinterpret_cast<float4*>(x + (size_t)k * N + 8 * bg);
     xr[0] = make_float4(xv[0], xv[1], xv[2], xv[3]);
     xr[1] = make_float4(xv[4], xv[5], xv[6], xv[7]);
-    const float g = gain[k];
+    const float g = gain ? gain[k] : 1.0f;
     __nv_bfloat16* o = xg + (size_t)(k >> 3) * (N * 8) + bg * 64 + (k & 7);
 #pragma unroll
     for (int i = 0; i < 8; ++i) {
@@ -1440,12 +1440,12 @@ PeerPush peer_push(Session* S, int index) {
 }  // namespace
 
 // first launch of a fused step: residual stream, first norm's input and its sums of squares from the embedding rows
-int32_t embed_prep_launch(Session* S, const float* gain, cudaStream_t st) {
+int32_t embed_prep_launch(Session* S, const float* gain, cudaStream_t st, float scale) {
   const Model* M = S->m;
   const int rows_per = S->embed_rows_per_cta, hid = M->cfg.hidden;
   const dim3 grid((unsigned)ceil_div(hid, rows_per));
   LMB_CUDA(launch_k(S->Bp == 16 ? embed_prep_kernel<16> : embed_prep_kernel<32>, grid, dim3(128), 0, st, (const int*)S->tokens,
-                    reinterpret_cast<const __nv_bfloat16*>(M->embed), M->cfg.vocab, hid, S->B, gain, S->xT,
+                    reinterpret_cast<const __nv_bfloat16*>(M->embed), M->cfg.vocab, hid, S->B, gain, scale, S->xT,
                     reinterpret_cast<__nv_bfloat16*>(S->xn), S->ssq, rows_per));
   M->ctx->launches++;
   return LMB200_OK;

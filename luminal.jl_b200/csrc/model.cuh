@@ -12,7 +12,7 @@
 namespace lmb {
 
 enum MapKind { MAP_PLAIN = 0, MAP_QKV = 1, MAP_O = 2, MAP_GATEUP = 3, MAP_DOWN = 4, MAP_STACK = 5 };
-constexpr int kMaxSrc = 5;             // logical tensors one internal matrix can hold
+constexpr int kMaxSrc = 6;             // logical tensors one internal matrix can hold
 
 // How one internal (tiled) matrix maps onto up to kMaxSrc logical [out,in] tensors of the
 // reference (src/NN.jl:330-341, 238-244) -- including the head split f = h + H*d that the
@@ -25,16 +25,16 @@ struct WMap {
   int RB = 0, KC = 0;        // padded extent in 16-row blocks / 32-k chunks
   int H = 0, KV = 0, D = 0, G = 0, Hl = 0, KVl = 0, kv_off = 0;
   int inter_l = 0, inter_off = 0;
-  int src_rows[kMaxSrc] = {0, 0, 0, 0, 0};
-  int src_cols[kMaxSrc] = {0, 0, 0, 0, 0};
+  int src_rows[kMaxSrc] = {0, 0, 0, 0, 0, 0};
+  int src_cols[kMaxSrc] = {0, 0, 0, 0, 0, 0};
   // MAP_STACK: tensor s occupies rows row_off[s] .. + src_rows[s] and columns col_off[s] .. + src_cols[s], the rest is zero
   int n_src = 0;
-  int row_off[kMaxSrc] = {0, 0, 0, 0, 0};
-  int col_off[kMaxSrc] = {0, 0, 0, 0, 0};
+  int row_off[kMaxSrc] = {0, 0, 0, 0, 0, 0};
+  int col_off[kMaxSrc] = {0, 0, 0, 0, 0, 0};
   // rows of heads pair_head[s] wide whose first pair_dims[s] features rotate in half-split pairs (i, i + dims / 2): internal rows 2i and
   // 2i + 1 hold pair i.  Applied to queries and keys alike it changes no product, and a pair always sits in neighbouring rows.
-  int pair_head[kMaxSrc] = {0, 0, 0, 0, 0};
-  int pair_dims[kMaxSrc] = {0, 0, 0, 0, 0};
+  int pair_head[kMaxSrc] = {0, 0, 0, 0, 0, 0};
+  int pair_dims[kMaxSrc] = {0, 0, 0, 0, 0, 0};
 };
 
 struct LayerWeights {
@@ -67,20 +67,30 @@ struct LayerWeights {
 struct LayerSpec {
   lmb200_layer_config c{};
   std::vector<double> decay;
-  // input projections, all reading the layer's norm: latent attention [dq | dkv | g | up], retention [q | k | v | g | up].
+  // input projections, all reading the same vector: latent attention [dq | dkv | g | up], retention [q | k | v | g | up], attention
+  // [q | k | v], channel delta [q | k | v | b | a1 | g1], lightning [q | k | v | g].
   // Every part starts on a multiple of 32 rows.  The first n_store rows are mixer inputs, the rest the feed-forward's.
   WMap m_in;
-  int row0[kMaxSrc] = {0, 0, 0, 0, 0};
+  int row0[kMaxSrc] = {0, 0, 0, 0, 0, 0};
   int n_store = 0;
   WMap m_uq, m_ukv;          // latent attention: queries from their latent; [uk | uv], per-head keys and values from the latent
   WMap m_out;                // [o | down] side by side: mixer output columns from 0, feed-forward columns from cat0
   int cat0 = 0;
+  // LMB200_BLOCK_POSTNORM: feed-forward, token input
+  WMap m_gu, m_down, m_sg, m_sp;
+  WMap m_lr;                 // channel delta: [a2 over the a1 columns; g2 over the g1 columns]
+  int lr_g1 = 0;             // column of g1's output in m_lr's input
+  int k_ld = 0, v_ld = 0;    // attention: cached key and value rows (widths rounded up to 8, the gap zero)
   int lat_rot = 0, lat_ld = 0;   // latent cache row: latent from 0, rotated key part from lat_rot, lat_ld elements in all
 };
 struct LayeredWeights {
   void *w_in = nullptr, *w_out = nullptr, *w_uq = nullptr, *w_ukv = nullptr;
   void *w_ukt = nullptr, *w_uv = nullptr;     // row-major [heads, kv_rank, dim] and [heads * vdim, kv_rank] (absorbed attention)
   float *norm = nullptr, *q_norm = nullptr, *kv_norm = nullptr;
+  void *w_gu = nullptr, *w_down = nullptr, *w_sg = nullptr, *w_sp = nullptr, *w_lr = nullptr;
+  float *norm2 = nullptr, *side_norm = nullptr, *mix_norm = nullptr;
+  float *conv = nullptr;                      // channel delta: [taps][channels of q | k | v], tap 0 meets the current token
+  float *a_log = nullptr, *dt_bias = nullptr;
   float *inv_freq = nullptr;                  // [rot_dims / 2]
   int rot_id = -1;                            // layers with the same frequencies share an angle table (Model::rot_freqs)
   float *decay = nullptr;                     // retention: [heads][kDecayPow]: decay^0 .. decay^(kDecayPow - 1)
@@ -110,7 +120,10 @@ struct Model {
   // LMB200_ARCH_LAYERED
   std::vector<LayerSpec> specs;
   std::vector<LayeredWeights> lw;
-  float softcap = 0.f;
+  float softcap = 0.f, embed_scale = 1.f;
+  int block = 0, side_dim = 0;
+  bool tied_head = false;
+  void* side_embed = nullptr;   // [vocab, n_layers * side_dim], model dtype
   std::vector<std::vector<float>> rot_freqs;   // the distinct frequency lists of the layers
   std::set<std::string> weights_set;   // registry names given through lmb200_model_set_weight
   bool all_weights_set = false;        // lmb200_model_init_random filled everything
@@ -184,8 +197,10 @@ struct Session {
   int graph_nodes_full = 0, graph_nodes_body = 0, graph_nodes_tok = 0;
   // LMB200_ARCH_LAYERED (csrc/layered.cu): per layer a latent cache [B][cap][lat_ld], a recurrent state
   // [B][heads][dim][round_up(vdim, 4)] float32, or NULL (a layer that reads another layer's latent cache)
-  std::vector<void*> latent;
-  std::vector<float*> state;
+  // attention: keys [B][kv_heads][cap][k_ld] and values [B][kv_heads][cap][v_ld]; channel delta also the last raw inputs of its
+  // convolutions, position p in slot p % taps of [B][taps][channels] float32
+  std::vector<void*> latent, keys, values;
+  std::vector<float*> state, conv;
   struct LayeredScratch* lay = nullptr;
   // a batch above 32: this session owns nothing on the device, it is a row of sub-sessions of at most 32 sequences
   std::vector<uint64_t> parts;
@@ -251,7 +266,7 @@ int64_t tiled_elems(const WMap& m, int dtype);
 void finish_map(WMap& m);
 int32_t dmalloc(void** p, int64_t bytes, bool zero, cudaStream_t st);
 int32_t push_positions(Session* S);
-int32_t embed_prep_launch(Session* S, const float* gain, cudaStream_t st);
+int32_t embed_prep_launch(Session* S, const float* gain, cudaStream_t st, float scale = 1.0f);
 GemvParams gemv_params(Session* S, const void* W, const WMap& m, const GemvPlan& pl, const void* x);
 int32_t argmax_launch(Session* S, cudaStream_t st);       // greedy tokens of S->logits into S->tokens
 int32_t advance_launch(Session* S, cudaStream_t st);      // end of a step on one GPU
@@ -265,7 +280,10 @@ enum RowSegKind {
   SEG_RELU2 = 2,      // relu(v)^2, model dtype
   SEG_SILU = 3,       // silu(v), model dtype
   SEG_SOFTCAP = 4,    // softcap * tanh(v / softcap), float32 (softcap 0: v)
-  SEG_ROT = 5         // bf16: neighbouring rows (2i, 2i + 1) of every head are rotated by angle i of the token's table row
+  SEG_ROT = 5,        // bf16: neighbouring rows (2i, 2i + 1) of every head are rotated by angle i of the token's table row
+  SEG_SIGMOID = 6,    // sigmoid(v), model dtype
+  SEG_DECAY = 7,      // -exp(rate[r / head]) softplus(v + bias[r]), float32
+  SEG_GELU_TOKEN = 8  // gelu(v) * table[tokens[t] * table_pitch + r], model dtype
 };
 struct RowSeg {
   int row0 = 0, rows = 0, kind = SEG_F32, pitch = 0;
@@ -273,8 +291,13 @@ struct RowSeg {
   // SEG_ROT: heads of rot_head rows, features rot_off .. rot_off + rot_dims - 1 rotate (all even); rot[token * rot_dims / 2 + i] = (cos, sin)
   const float2* rot = nullptr;
   int rot_head = 0, rot_off = 0, rot_dims = 0;
+  const float *rate = nullptr, *bias = nullptr;        // SEG_DECAY
+  int head = 1;
+  const void* table = nullptr;                         // SEG_GELU_TOKEN: model dtype, table_rows tokens
+  const int* tokens = nullptr;
+  int table_pitch = 0, table_rows = 0;
 };
-constexpr int kMaxSegs = 5;
+constexpr int kMaxSegs = 6;
 struct RowSegs {
   RowSeg s[kMaxSegs];
   int n = 0;
@@ -283,6 +306,8 @@ struct RowSegs {
 };
 // rows of W (bf16 weight layout) times X [T, ldx] row-major bf16 (columns past K are not read), each row to its segment
 int32_t gemm_segments_bf16(Ctx* ctx, const void* W, const void* X, int ldx, int T, int rows, int K, const RowSegs& segs, cudaStream_t st);
+// act[t * ld_act + i] = silu(gate_i) up_i over MAP_GATEUP rows (bf16), i < n_act
+int32_t gemm_silu_gate_bf16(Ctx* ctx, const void* W, const void* X, int ldx, int T, int rows, int K, void* act, int ld_act, int n_act, cudaStream_t st);
 // prompt phase as GEMMs + flash attention (csrc/prefill.cu)
 int32_t prefill_configure();
 bool prefill_gemm_ok(const Session* S, int n);

@@ -21,6 +21,7 @@
 
 #include <algorithm>
 
+#include "activations.cuh"
 #include "model.cuh"
 #include "tc.cuh"
 
@@ -101,6 +102,24 @@ __device__ __forceinline__ void segment_epilogue(const GemmParams& p, float (&v)
       if (t0 + i < t_end) out[(int64_t)(t0 + i) * sg.pitch + r] = cap > 0.f ? cap * tanhf(v[i] / cap) : v[i];
     return;
   }
+  if (sg.kind == SEG_DECAY) {
+    if (r >= sg.rows) return;
+    float* out = reinterpret_cast<float*>(sg.dst);
+    const float rate = -expf(sg.rate[r / sg.head]), bias = sg.bias[r];
+#pragma unroll
+    for (int i = 0; i < 32; ++i)
+      if (t0 + i < t_end) out[(int64_t)(t0 + i) * sg.pitch + r] = rate * softplus_f32(v[i] + bias);
+    return;
+  }
+  if (sg.kind == SEG_GELU_TOKEN) {
+    const __nv_bfloat16* table = reinterpret_cast<const __nv_bfloat16*>(sg.table);
+    const int tok = t0 + lane < t_end ? sg.tokens[t0 + lane] : -1;
+#pragma unroll
+    for (int i = 0; i < 32; ++i) {
+      const int tk = __shfl_sync(0xffffffffu, tok, i);
+      v[i] = tk >= 0 && tk < sg.table_rows && r < sg.rows ? gelu_ref(v[i]) * __bfloat162float(table[(int64_t)tk * sg.table_pitch + r]) : 0.f;
+    }
+  }
   if (sg.kind == SEG_ROT) {
     const int f = r % sg.rot_head - sg.rot_off;         // partner rows are neighbouring lanes
     const bool turn = f >= 0 && f < sg.rot_dims;
@@ -123,6 +142,7 @@ __device__ __forceinline__ void segment_epilogue(const GemmParams& p, float (&v)
     float y = v[i];
     if (sg.kind == SEG_RELU2) { y = fmaxf(y, 0.f); y = y * y; }
     else if (sg.kind == SEG_SILU) y = y / (1.0f + expf(-y));
+    else if (sg.kind == SEG_SIGMOID) y = sigmoid_f32(y);
     st[i * kPitch + lane] = __float2bfloat16_rn(y);
   }
   __syncwarp();
@@ -854,6 +874,13 @@ int32_t gemm_segments_bf16(Ctx* ctx, const void* W, const void* X, int ldx, int 
   p.W = reinterpret_cast<const __nv_bfloat16*>(W); p.X = reinterpret_cast<const __nv_bfloat16*>(X); p.ldx = ldx; p.T = T; p.rows = rows; p.K = K;
   p.epi = GEMM_SEGMENTS; p.segs = segs;
   for (int i = 0; i < segs.n; ++i) LMB_REQUIRE(segs.s[i].row0 % 32 == 0, "gemm: a segment starts at row %d", segs.s[i].row0);
+  return gemm_launch(ctx, p, st);
+}
+
+int32_t gemm_silu_gate_bf16(Ctx* ctx, const void* W, const void* X, int ldx, int T, int rows, int K, void* act, int ld_act, int n_act, cudaStream_t st) {
+  GemmParams p;
+  p.W = reinterpret_cast<const __nv_bfloat16*>(W); p.X = reinterpret_cast<const __nv_bfloat16*>(X); p.ldx = ldx; p.T = T; p.rows = rows; p.K = K;
+  p.epi = GEMM_SILU_GATE; p.act = reinterpret_cast<__nv_bfloat16*>(act); p.ld_act = ld_act; p.n_act = n_act;
   return gemm_launch(ctx, p, st);
 }
 

@@ -1,4 +1,5 @@
 // Kernels of retention (see retention.cuh).
+#include "activations.cuh"
 #include "pdl.cuh"
 #include "retention.cuh"
 
@@ -26,7 +27,7 @@ __global__ void __launch_bounds__(kStepMax) retention_step_kernel(const Retentio
   const int n = v.len[b], t0 = v.start[b], p0 = v.pos0[b];
   if (n <= 0) return;
   const float decay = v.decay[h * v.decay_pitch + 1];
-  const float kscale = 1.0f / sqrtf((float)D);
+  const float kscale = v.k_scale;
   float4* S = reinterpret_cast<float4*>(v.state) + ((int64_t)b * v.H + h) * D * V4;
   const int c0 = tid % cols, w = tid / cols;
   for (int i = 0; i < n; ++i) {
@@ -36,6 +37,7 @@ __global__ void __launch_bounds__(kStepMax) retention_step_kernel(const Retentio
     const IT* vv = reinterpret_cast<const IT*>(v.v) + t * v.v_pitch + h * V;
     for (int d = tid; d < D; d += kStepThreads) {
       float qv = to_f32(q[d]), kv = to_f32(k[d]);
+      if (v.raw_act) { qv = silu_f32(qv); kv = silu_f32(kv); }
       if (d < v.rot_dims) {
         float s, c;
         sincosf((float)(p0 + i) * v.inv_freq[d >> 1], &s, &c);
@@ -46,7 +48,7 @@ __global__ void __launch_bounds__(kStepMax) retention_step_kernel(const Retentio
       qs[d] = qv;
       ks[d] = kv * kscale;
     }
-    for (int d = tid; d < 4 * V4; d += kStepThreads) vs[d] = d < V ? to_f32(vv[d]) : 0.f;
+    for (int d = tid; d < 4 * V4; d += kStepThreads) vs[d] = d >= V ? 0.f : v.raw_act ? silu_f32(to_f32(vv[d])) : to_f32(vv[d]);
     __syncthreads();
     if (w < W) {
       for (int c = c0; c < V4; c += cols) {
@@ -78,13 +80,15 @@ __global__ void __launch_bounds__(kStepMax) retention_step_kernel(const Retentio
     __syncthreads();
     float tot = 0.f;
     for (int j = 0; j < kStepThreads / 32; ++j) tot += red[j];
-    const float inv = 1.0f / sqrtf(tot / (float)V + v.eps);
+    const float inv = v.ssq ? 1.0f : 1.0f / sqrtf(tot / (float)V + v.eps);
+    if (v.ssq && tid == 0) v.ssq[t * v.ssq_t + h * v.ssq_h] = tot;
     const IT* g = reinterpret_cast<const IT*>(v.g) + t * v.g_pitch + h * V;
     OT* out = reinterpret_cast<OT*>(v.out);
     for (int d = tid; d < V; d += kStepThreads) {
       float gv = to_f32(g[d]);
-      if (v.raw_gate) gv = gv / (1.0f + expf(-gv));
+      if (v.raw_gate) gv = v.raw_gate == 1 ? silu_f32(gv) : sigmoid_f32(gv);
       const int col = h * V + d;
+      if (v.out_w) gv *= v.out_w[col];
       out[v.bp > 0 ? Layout<OT>::x_offset((int)t, col, v.bp) : t * v.ldo + col] = from_f32<OT>(vs[d] * inv * gv);
     }
     __syncthreads();                   // vs, red and os are rewritten by the next token
@@ -162,7 +166,7 @@ __global__ void __launch_bounds__(128 * NG, 1) retention_chunk_kernel(const Rete
   if (n_all <= 0) return;
   const int D = v.dim, V = v.vdim, ld = (V + 3) & ~3;
   const int c0 = slice * DVC;                                       // first value column of this CTA
-  const float scale = 1.0f / sqrtf((float)D);
+  const float scale = v.k_scale;
   for (int i = tid; i <= kC; i += kThreads) s_pw[i] = v.decay[h * v.decay_pitch + i];
 
   auto load = [&](int c) {
@@ -370,7 +374,12 @@ __global__ void __launch_bounds__(128 * NG, 1) retention_chunk_kernel(const Rete
     }
     q0 = q1 = 0.f;
     for (int k = 0; k < n_sums; ++k) { q0 += sums[k * kC + r0 + g]; q1 += sums[k * kC + r0 + g + 8]; }
-    const float i0 = 1.0f / sqrtf(q0 / (float)V + v.eps), i1 = 1.0f / sqrtf(q1 / (float)V + v.eps);
+    const float i0 = v.ssq ? 1.0f : 1.0f / sqrtf(q0 / (float)V + v.eps), i1 = v.ssq ? 1.0f : 1.0f / sqrtf(q1 / (float)V + v.eps);
+    if (v.ssq && slice == 0 && cg == 0 && tq == 0) {
+      const int64_t t = t_first + (int64_t)c * kC + r0 + g;
+      if (r0 + g < n) v.ssq[t * v.ssq_t + h * v.ssq_h] = q0;
+      if (r0 + g + 8 < n) v.ssq[(t + 8) * v.ssq_t + h * v.ssq_h] = q1;
+    }
 #pragma unroll
     for (int e2 = 0; e2 < 2; ++e2) {
       const int row = r0 + g + e2 * 8;
@@ -389,7 +398,8 @@ __global__ void __launch_bounds__(128 * NG, 1) retention_chunk_kernel(const Rete
       for (int nt = 0; nt < NT; ++nt) {
         const int col = c0 + cg * CG + nt * 8 + 2 * tq;
         if (col >= V) continue;
-        const float2 gv = unpack_bf16(gu[nt]);
+        float2 gv = unpack_bf16(gu[nt]);
+        if (v.out_w) { gv.x *= v.out_w[h * V + col]; gv.y *= v.out_w[h * V + col + 1]; }
         *reinterpret_cast<__nv_bfloat162*>(out + col) = __floats2bfloat162_rn(O[nt][2 * e2] * inv * gv.x, O[nt][2 * e2 + 1] * inv * gv.y);
       }
     }

@@ -2,6 +2,9 @@
 //   S_t = decay S_{t-1} + (R_t k_t / sqrt(dim)) v_t^T,   o_t = S_t^T R_t q_t,   y_t = o_t / rms(o_t) * silu(g_t)
 // over a float32 state S [dim, vdim] that a sequence carries from token to token.  Not in the reference (all of its attention
 // is softmax attention, src/NN.jl:343-387).
+// Lightning attention is the same recurrence without rotation and key scale, silu on q, k and v, and one norm over all heads' outputs
+// together: with `ssq` set the kernels leave y_t = o_t w gate and the heads' sums of o_t^2; whoever multiplies y by the output
+// projection applies the norm's scale, one number per token.
 #pragma once
 #include "common.cuh"
 
@@ -20,11 +23,16 @@ struct RetentionView {
   const float* decay = nullptr;       // [H][decay_pitch]: powers 0 .. decay_pitch - 1
   int decay_pitch = 0;
   float eps = 0.f;
+  float k_scale = 1.f;
   float* state = nullptr;             // [B][H][dim][round_up(vdim, 4)]
-  // rows [T, pitch] of the projections: head a of q at column a * dim and so on; g with silu still to be applied if raw_gate
+  // rows [T, pitch] of the projections: head a of q at column a * dim and so on;
+  // raw_gate: what is still to be applied to g (1: silu, 2: sigmoid); raw_act: q, k and v still lack their silu (token by token only)
   const void *q = nullptr, *k = nullptr, *v = nullptr, *g = nullptr;
   int q_pitch = 0, k_pitch = 0, v_pitch = 0, g_pitch = 0;
-  int in_f32 = 1, raw_gate = 1;
+  int in_f32 = 1, raw_gate = 1, raw_act = 0;
+  const float* out_w = nullptr;       // [H * vdim] (with ssq)
+  float* ssq = nullptr;               // token t, head a: ssq[t * ssq_t + a * ssq_h]
+  int ssq_t = 0, ssq_h = 0;
   void* out = nullptr;                // model dtype: [T, ldo] row-major, or GEMV activations of padding bp
   int ldo = 0, bp = 0;
 };

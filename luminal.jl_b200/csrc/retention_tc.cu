@@ -113,7 +113,7 @@ __global__ void __launch_bounds__(kThreads, 1) retention_tc_kernel(const Retenti
   const int chunks = (n_all + kT - 1) / kT;              // 0: nothing to do (uniform over the pair)
   const int D = v.dim, V = v.vdim, ld = (V + 3) & ~3, c0 = slice * 128;
   const float* pw = tl.pw;
-  const float scale = 1.0f / sqrtf((float)D);
+  const float scale = v.k_scale;
   const uint32_t lane_base = (uint32_t)(32 * (warp & 3)) << 16;
 
   if (warp == 17) {
@@ -340,8 +340,9 @@ __global__ void __launch_bounds__(kThreads, 1) retention_tc_kernel(const Retenti
         mbar_wait_cluster(&tl.x_full, c & 1, dead, err);
         ss += tl.peer[c & 1][row];
       }
-      const float inv = 1.0f / sqrtf(ss / (float)V + v.eps);
+      const float inv = v.ssq ? 1.0f : 1.0f / sqrtf(ss / (float)V + v.eps);
       if (row < n) {
+        if (v.ssq && half == 0 && slice == 0) v.ssq[t * v.ssq_t + h * v.ssq_h] = ss;
         __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(v.out) + t * v.ldo + col;
 #pragma unroll
         for (int q0 = 0; q0 < 8; q0 += 4) {                                    // four gate vectors in flight
@@ -354,8 +355,9 @@ __global__ void __launch_bounds__(kThreads, 1) retention_tc_kernel(const Retenti
             uint32_t* gi = reinterpret_cast<uint32_t*>(&gu[q]);
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
-              const float2 g = unpack2bf(gi[e]);
+              float2 g = unpack2bf(gi[e]);
               const int i = (q0 + q) * 8 + 2 * e;
+              if (v.out_w && i < left) { const float2 w = __ldg(reinterpret_cast<const float2*>(v.out_w + col + i)); g.x *= w.x; g.y *= w.y; }
               const __nv_bfloat162 r = __floats2bfloat162_rn(o[i] * inv * g.x, o[i + 1] * inv * g.y);
               gi[e] = *reinterpret_cast<const uint32_t*>(&r);
             }

@@ -7,13 +7,14 @@ import json
 import os
 
 from .session import LayeredModel, Model
-from .weights import load_safetensors
+from .weights import load_safetensors, safetensors_shapes
 
 REGISTRY = {}
 
 
 def register(*names):
-    """Registers a builder (device, config, dtype) -> model for the architecture names of a config.json."""
+    """Registers a builder (device, config, dtype, shapes) -> model for the architecture names of a config.json.  `shapes` (name ->
+    shape of the weight file's tensors) is for sizes that no key of the configuration gives."""
     def add(fn):
         for n in names:
             REGISTRY[n] = fn
@@ -33,13 +34,13 @@ def architecture(config):
     return name
 
 
-def build_model(device, config, dtype="bf16"):
-    return REGISTRY[architecture(config)](device, config, dtype)
+def build_model(device, config, dtype="bf16", shapes=None):
+    return REGISTRY[architecture(config)](device, config, dtype, shapes or {})
 
 
 def load_model(device, path, dtype="bf16"):
     """The model of a folder (config.json + *.safetensors).  A tensor the configuration needs and no file has is an error."""
-    model = build_model(device, read_config(path), dtype)
+    model = build_model(device, read_config(path), dtype, safetensors_shapes(path))
     load_safetensors(model, path, warn_missing=False)
     missing = model.missing_weights()
     if missing:
@@ -49,7 +50,7 @@ def load_model(device, path, dtype="bf16"):
 
 
 @register("LlamaForCausalLM")
-def llama(device, config, dtype):
+def llama(device, config, dtype, shapes):
     return Model(device, n_layers=config["num_hidden_layers"], hidden=config["hidden_size"], n_heads=config["num_attention_heads"],
                  n_kv_heads=config.get("num_key_value_heads") or config["num_attention_heads"], intermediate=config["intermediate_size"],
                  vocab=config["vocab_size"], eps=config["rms_norm_eps"], rope_base=config.get("rope_theta", 10000.0), dtype=dtype)
@@ -78,6 +79,40 @@ def gibutar_layers(config):
 
 
 @register("Gibutar")
-def gibutar(device, config, dtype):
+def gibutar(device, config, dtype, shapes):
     return LayeredModel(device, width=config["width"], vocab=config["vocab"], layers=gibutar_layers(config), eps=config["norm"]["eps"],
                         softcap=config.get("logit_softcap") or 0.0, dtype=dtype)
+
+
+def kevatar_layers(config, shapes):
+    """Layer descriptions (LayeredModel) of a Kevatar configuration.  Fixed by the design: rotations of interleaved pairs, unit key
+    heads, the feed-forward down(silu(gate h) * up h).  The ranks of a channel-delta layer's decay and gate come from its tensors."""
+    layers = []
+    for i, layer in enumerate(config["layers"]):
+        mx, mlp, kind = layer["mixer"], layer.get("mlp"), layer["type"]
+        if mlp and mlp.get("kind", "dense") != "dense":
+            raise ValueError(f"layer {i}: feed-forward of kind {mlp['kind']!r}")
+        d = dict(mixer=kind, heads=mx["heads"], dim=mx["dim"], vdim=mx["vdim"], ff=mlp["ff"] if mlp else 0, ff_kind="silu_gate",
+                 rot_layout="interleaved")
+        if kind == "attention":
+            rot = mx.get("rot") or {}
+            d.update(kv_heads=mx["kv_heads"], scale=mx["scale"], score_cap=mx.get("softcap"), window=(mx.get("mask") or {}).get("size"),
+                     kv_from=mx.get("kv_from"), rot_dims=rot.get("dims", 0), rot_base=rot.get("base"), rot_scaling=rot.get("scaling"))
+        elif kind == "channel_delta":
+            ranks = [shapes.get(f"l{i}.mix.{n}") for n in ("a1", "g1")]
+            if None in ranks:
+                raise ValueError(f"layer {i}: the shapes of l{i}.mix.a1 and l{i}.mix.g1 are needed for its ranks")
+            d.update(kv_heads=mx["kv_heads"], conv=mx["conv"], decay_rank=ranks[0][0], gate_rank=ranks[1][0])
+        elif kind == "lightning":
+            d.update(decay=mx["decay"])
+        else:
+            raise ValueError(f"layer {i}: mixer {kind!r}")
+        layers.append(d)
+    return layers
+
+
+@register("Kevatar")
+def kevatar(device, config, dtype, shapes):
+    return LayeredModel(device, width=config["width"], vocab=config["vocab"], layers=kevatar_layers(config, shapes), eps=config["norm"]["eps"],
+                        block="postnorm", side_dim=(config.get("token_side") or {}).get("dim", 0), tied_head=True,
+                        embed_scale=config["embedding"]["scale"], dtype=dtype)

@@ -88,17 +88,21 @@ def WhisperDecoderModel(device, *, d_model, heads, layers, ffn, vocab, max_posit
                  cross_len=cross_len)
 
 
-MIXERS = {"latent_attention": 0, "retention": 1}
+MIXERS = {"latent_attention": 0, "retention": 1, "attention": 2, "channel_delta": 3, "lightning": 4}
 ROTATIONS = {"half": 0, "interleaved": 1}
+BLOCKS = {"parallel": 0, "postnorm": 1}
+FEED_FORWARDS = {"relu2": 0, "silu_gate": 1}
 
 
 class LayeredModel(Model):
-    """A decoder described layer by layer (lmb200_model_create_layered).  `layers`: one dict per layer with `mixer`
-    ('latent_attention' or 'retention'), heads, dim, vdim, ff (0: no feed-forward), rot_dims, rot_base, rot_layout ('half' or
-    'interleaved'); latent attention also q_rank, kv_rank, rot_dim, scale, kv_from (None, or the layer whose latent cache it
-    reads); retention also decay (one value per head)."""
+    """A decoder described layer by layer (lmb200_model_create_layered).  `layers`: one dict per layer with `mixer` (a key of
+    MIXERS), heads, dim, vdim, ff (0: no feed-forward), ff_kind, rot_dims, rot_base, rot_layout ('half' or 'interleaved'); latent
+    attention also q_rank, kv_rank, rot_dim, scale, kv_from (None, or the layer whose cache it reads); attention kv_heads, window,
+    scale, score_cap, kv_from and rot_scaling (None, or factor, original, fast, slow); channel delta kv_heads, conv, decay_rank,
+    gate_rank; retention and lightning decay (one value per head).  block: 'parallel' or 'postnorm'."""
 
-    def __init__(self, device, *, width, vocab, layers, eps, softcap=0.0, dtype="bf16"):
+    def __init__(self, device, *, width, vocab, layers, eps, softcap=0.0, block="parallel", side_dim=0, tied_head=False, embed_scale=1.0,
+                 dtype="bf16"):
         self.device = device
         code = _dtype_code(dtype)
         arr = (_lib.LayerConfig * len(layers))()
@@ -107,19 +111,24 @@ class LayeredModel(Model):
             c.mixer = MIXERS[layer["mixer"]]
             for k in ("heads", "dim", "vdim"):
                 setattr(c, k, int(layer[k]))
-            for k in ("q_rank", "kv_rank", "rot_dim", "rot_dims", "ff"):
+            for k in ("q_rank", "kv_rank", "rot_dim", "rot_dims", "ff", "kv_heads", "window", "conv", "decay_rank", "gate_rank"):
                 setattr(c, k, int(layer.get(k) or 0))
             c.kv_from = -1 if layer.get("kv_from") is None else int(layer["kv_from"])
             c.rot_layout = ROTATIONS[layer.get("rot_layout", "half")]
+            c.ff_kind = FEED_FORWARDS[layer.get("ff_kind", "relu2")]
             c.rot_base = float(layer.get("rot_base") or 1.0)
             c.scale = float(layer.get("scale", 1.0))
+            c.score_cap = float(layer.get("score_cap") or 0.0)
+            for k, v in (layer.get("rot_scaling") or {}).items():
+                setattr(c, "rot_" + k, float(v))
             if "decay" in layer:
                 if len(layer["decay"]) != c.heads:
                     raise ValueError(f"{len(layer['decay'])} decays for {c.heads} heads")
                 keep.append((C.c_double * c.heads)(*[float(d) for d in layer["decay"]]))
                 c.decay = C.cast(keep[-1], C.POINTER(C.c_double))
         cfg = _lib.LayeredConfig(n_layers=len(layers), width=int(width), vocab=int(vocab), dtype=code, eps=float(eps),
-                                 softcap=float(softcap or 0.0))
+                                 softcap=float(softcap or 0.0), block=BLOCKS[block], side_dim=int(side_dim or 0),
+                                 tied_head=int(bool(tied_head)), embed_scale=float(embed_scale))
         h = C.c_uint64(0)
         _lib.call("lmb200_model_create_layered", device.handle, C.byref(cfg), arr, C.byref(h))
         self.handle = h

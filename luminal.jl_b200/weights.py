@@ -25,16 +25,29 @@ def _to_f32(raw, dtype):
     return raw.astype(np.float32)
 
 
+def _header(f):
+    """(tensor name -> entry, where the data starts) of an open safetensors file."""
+    (hlen,) = struct.unpack("<Q", f.read(8))
+    header = json.loads(f.read(hlen).decode("utf-8"))
+    header.pop("__metadata__", None)
+    return header, 8 + hlen
+
+
+def safetensors_shapes(path):
+    """name -> shape of every tensor of a file or of a directory's shards, without reading the data."""
+    out = {}
+    for file in _files(path):
+        with open(file, "rb") as f:
+            out.update({name: tuple(int(s) for s in info["shape"]) for name, info in _header(f)[0].items()})
+    return out
+
+
 def read_safetensors(path):
     """name -> float32 array of every tensor in one file (F32, F16, BF16 or F64 on disk)."""
     with open(path, "rb") as f:
-        (hlen,) = struct.unpack("<Q", f.read(8))
-        header = json.loads(f.read(hlen).decode("utf-8"))
-        base = 8 + hlen
+        header, base = _header(f)
         out = {}
         for name, info in header.items():
-            if name == "__metadata__":
-                continue
             if info["dtype"] not in _DTYPES:
                 raise ValueError(f"{path}: tensor {name} has unsupported dtype {info['dtype']}")
             np_dt, esz = _DTYPES[info["dtype"]]
