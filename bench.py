@@ -1,7 +1,7 @@
 #!/usr/bin/env python
 """Throughput of the B200 backend on the reference's benchmark configurations.
 
-    python bench.py [--config llama3_8b|phi3_mini|whisper_base|small_llama|flash|gibutar]
+    python bench.py [--config llama3_8b|phi3_mini|whisper_base|small_llama|flash|gibutar|kevatar]
                     [--gpus N] [--steps K] [--warmup W] [--repeats R] [--impl ours|reference]
 
 Default: the Llama-3-8B-shape decode (32 layers, hidden 4096, 32 q / 8 kv heads x 128, MLP 14336,
@@ -295,7 +295,7 @@ def run_reference(args):
         return
     if args.config == "small_llama":
         return run_reference_small_llama(args)
-    if args.config == "gibutar":
+    if args.config in LAYERED:
         print(json.dumps({"impl": "reference", "unavailable": "the reference has no such model"}))
         return
     name = args.config if args.config in DECODE else "llama3_8b"
@@ -755,7 +755,7 @@ def run_whisper(args):
 
 
 # -------------------------------------------------------------------------------------------------
-# gibutar: latent attention + retention layers at the sizes of real models' layers, beside Llama at equal width
+# gibutar, kevatar: decoders described layer by layer at the sizes of real models' layers, beside Llama at equal width
 # -------------------------------------------------------------------------------------------------
 def gibutar_size(width, heads, ff, kv_rank, q_rank, layers, vocab=32064):
     """One latent-attention layer to three retention layers, the second latent layer of a pair reading the first one's cache."""
@@ -797,10 +797,65 @@ def gibutar_flops(cfg, n):
     return total
 
 
-def run_gibutar(args):
+def kevatar_size(width, heads, kv_heads, ff, side, window, layers, vocab=32064):
+    """Of eight layers two windowed attention (the second reading the first one's cache), two channel delta and four lightning."""
+    dim = width // heads
+    out = []
+    for i in range(layers):
+        if i % 4 == 0:
+            mx = dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=dim, scale=dim ** -0.5, softcap=30.0, mask=dict(size=window),
+                      rot=dict(base=500000.0, dims=dim // 2, scaling=dict(factor=4.0, original=8192, fast=32.0, slow=1.0)))
+            if i % 8 == 4:
+                mx["kv_from"] = i - 4
+            kind = "attention"
+        elif i % 4 == 2:
+            mx, kind = dict(heads=heads, kv_heads=heads // 2, dim=dim, vdim=dim, conv=4), "channel_delta"
+        else:
+            mx, kind = dict(heads=heads, dim=dim, vdim=dim, decay=[1.0 - 2.0 ** -(5 + 4 * h / heads) for h in range(heads)]), "lightning"
+        out.append(dict(type=kind, mixer=mx, mlp=dict(kind="dense", ff=ff)))
+    return dict(architecture="Kevatar", width=width, vocab=vocab, norm=dict(eps=1e-5), embedding=dict(scale=1.0), token_side=dict(dim=side), layers=out)
+
+
+KEVATAR_SIZES = {
+    "w4096": dict(width=4096, heads=32, kv_heads=8, ff=14336, side=256, window=1024, layers=8),
+    "w2048": dict(width=2048, heads=16, kv_heads=4, ff=8192, side=128, window=1024, layers=8),
+}
+
+
+def kevatar_shapes(cfg):
+    """the low-rank matrices' shapes, which a configuration does not give: ranks as wide as a head"""
+    return {f"l{i}.mix.{t}": (x["mixer"]["dim"], cfg["width"]) for i, x in enumerate(cfg["layers"]) if x["type"] == "channel_delta" for t in ("a1", "g1")}
+
+
+def kevatar_flops(cfg, n):
+    total = 0
+    for layer in cfg["layers"]:
+        mx, W = layer["mixer"], cfg["width"]
+        H, d, v = mx["heads"], mx["dim"], mx["vdim"]
+        total += 6 * W * layer["mlp"]["ff"] + 2 * W * H * v + 4 * W * cfg["token_side"]["dim"]
+        if layer["type"] == "attention":
+            w = min(n, mx["mask"]["size"])
+            total += 2 * W * H * d + (0 if "kv_from" in mx else 2 * W * mx["kv_heads"] * (d + v)) + 2 * H * (d + v) * (w - w * w / (2.0 * n))
+        elif layer["type"] == "channel_delta":
+            total += 2 * W * (2 * mx["kv_heads"] * d + H * v + 2 * d + H) + 2 * d * H * (d + v) + 6 * H * d * v
+        else:
+            total += 4 * W * H * (d + v) + 4 * H * d * v
+    return total
+
+
+LAYERED = {
+    "gibutar": dict(sizes=GIBUTAR_SIZES, build=gibutar_size, flops=gibutar_flops, shapes=lambda cfg: {}, title="Gibutar",
+                    layers="1 latent attention : 3 retention, feed-forward on every layer"),
+    "kevatar": dict(sizes=KEVATAR_SIZES, build=kevatar_size, flops=kevatar_flops, shapes=kevatar_shapes, title="Kevatar",
+                    layers="1 windowed attention : 1 channel delta : 2 lightning, feed-forward and token input on every layer"),
+}
+
+
+def run_layered(args):
     import numpy as np
     import torch
     import luminal_jl_b200 as L
+    spec = LAYERED[args.config]
     D = Dist(1)
     stream = torch.cuda.Stream()
     dev = L.B200Device(0, stream=stream.cuda_stream)
@@ -859,11 +914,11 @@ def run_gibutar(args):
         return out, launches[batch]
 
     variants, total_launches = {}, 0
-    for name, sz in GIBUTAR_SIZES.items():
-        cfg = gibutar_size(**sz)
-        model = L.models.build_model(dev, cfg, "bf16")
+    for name, sz in spec["sizes"].items():
+        cfg = spec["build"](**sz)
+        model = L.models.build_model(dev, cfg, "bf16", shapes=spec["shapes"](cfg))
         model.init_random(1234, 0.02)
-        ours, n_launch = measure(model, lambda n: gibutar_flops(cfg, n))
+        ours, n_launch = measure(model, lambda n: spec["flops"](cfg, n))
         total_launches = total_launches or n_launch
         model.close()
         kv = max(1, sz["heads"] // 4)
@@ -873,15 +928,15 @@ def run_gibutar(args):
         per_tok = 2 * (model_params(lc) - 2 * lc["vocab"] * lc["hidden"])
         llama, _ = measure(model, lambda n: per_tok + 4 * lc["n_layers"] * lc["hidden"] * (n / 2.0))
         model.close()
-        variants[name] = {"sizes": sz, "gibutar": ours, "llama_same_width": llama}
-    head = variants["w4096"]["gibutar"]
+        variants[name] = {"sizes": sz, args.config: ours, "llama_same_width": llama}
+    head = variants["w4096"][args.config]
     print(json.dumps({
         "metric": METRIC, "value": head[f"decode_b{batch}"]["tokens_per_s"], "unit": "tokens/s", "n_gpus": 1, "steps": steps, "warmup": warm,
         "ms_per_step": head[f"decode_b{batch}"]["ms_per_step"], "higher_is_better": True, "scaling": "weak", "vs_baseline": None, "dtype": "bf16",
         "data": "synthetic",
-        "config": {"workload": f"Gibutar layers (1 latent attention : 3 retention, feed-forward on every layer), 8 layers, bf16, random weights; decode "
+        "config": {"workload": f"{spec['title']} layers ({spec['layers']}), 8 layers, bf16, random weights; decode "
                                f"batch {batch} and 1 with the context ending at {ctx}, prompts {p_batch} x {p_len} and 1 x 8192; Llama (8 layers, GQA 4:1) at equal width",
-                   "name": "gibutar", "batch": batch,
+                   "name": args.config, "batch": batch,
                    "l2": "a step streams several GB of weights, latents and states: inputs larger than L2"},
         "e2e": {"value": batch / head["e2e_ms_per_step"] * 1e3, "unit": "tokens/s", "h2d_bytes_per_step": batch * 4, "d2h_bytes_per_step": batch * 4},
         "gpu_launches": int(total_launches), "clocks": sampler.stop(), "variants": variants, "roofline": None, "cpu_baseline": None,
@@ -890,7 +945,7 @@ def run_gibutar(args):
 
 def main():
     ap = argparse.ArgumentParser()
-    ap.add_argument("--config", default="llama3_8b", choices=["llama3_8b", "phi3_mini", "whisper_base", "small_llama", "flash", "gibutar"])
+    ap.add_argument("--config", default="llama3_8b", choices=["llama3_8b", "phi3_mini", "whisper_base", "small_llama", "flash", "gibutar", "kevatar"])
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=256)
     ap.add_argument("--warmup", type=int, default=3)
@@ -912,8 +967,8 @@ def main():
         run_small_llama(args)
     elif args.config == "flash":
         run_flash(args)
-    elif args.config == "gibutar":
-        run_gibutar(args)
+    elif args.config in LAYERED:
+        run_layered(args)
     else:
         run_whisper(args)
 

@@ -291,7 +291,7 @@ int32_t conv_launch(const DeltaView& v, T* out, float* rq, float* rk, cudaStream
 
 }  // namespace
 
-int32_t delta_configure() { return LMB200_OK; }
+int32_t delta_configure() { return delta_chunk_configure(); }
 
 int32_t delta_conv(Ctx* ctx, int dtype, const DeltaView& v, void* out, float* rq, float* rk, cudaStream_t st) {
   LMB_TRY(check(v));

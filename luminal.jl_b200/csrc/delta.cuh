@@ -43,5 +43,9 @@ int32_t delta_configure();
 int32_t delta_conv(Ctx* ctx, int dtype, const DeltaView& v, void* out, float* rq, float* rk, cudaStream_t st);
 // token after token: decoding, short portions, float32
 int32_t delta_steps(Ctx* ctx, int dtype, const DeltaView& v, cudaStream_t st);
+// chunks of 64 tokens on the tensor cores (csrc/delta_chunk.cu): bf16 prepared rows, heads up to 128 wide
+bool delta_chunks_ok(const DeltaView& v);
+int32_t delta_chunks(Ctx* ctx, const DeltaView& v, cudaStream_t st);
+int32_t delta_chunk_configure();
 
 }  // namespace lmb

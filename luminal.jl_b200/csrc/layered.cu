@@ -74,7 +74,7 @@ struct LayeredScratch {
 
 namespace {
 
-constexpr int kChunkMin = 8, kTcMin = 80;   // longest portion from which retention runs in chunks of 64, of 128 tokens
+constexpr int kChunkMin = 8, kTcMin = 80;   // longest portion from which retention (and the delta rule) runs in chunks of 64, of 128 tokens
 constexpr int kFlashMin = 32;           // shortest portion whose context is expanded to keys and values
 constexpr int kBlockTokens = 2048;      // tokens per round of the absorbed attention in a rows step (bounds its scratch)
 constexpr uint64_t kIdLayered = 0x200000, kIdLayeredState = 0x300000;
@@ -268,6 +268,7 @@ struct Target {
   int slot = 0;
   void* plain = nullptr;         // row-major copy in the model dtype (float32 for vectors)
   bool vec = false;
+  float offset = 1.f;            // what generated values of a vector lie around
   int head = 0;                  // the copy holds heads of this many rows transposed
   float* conv = nullptr;         // taps of a convolution: [cols][conv_C] from channel conv_at on, last column first
   int conv_C = 0, conv_at = 0;
@@ -320,8 +321,8 @@ bool find_target(Model* M, const std::string& n, Target* t) {
     if (tail == "mix.a2") return mat(w.w_lr, s.m_lr, 0);
     if (tail == "mix.g2") return mat(w.w_lr, s.m_lr, 1);
     if (tail == "mix.norm") return vec(w.mix_norm, s.c.vdim);
-    if (tail == "mix.A_log") return vec(w.a_log, s.c.heads);
-    if (tail == "mix.dt_bias") return vec(w.dt_bias, (int64_t)s.c.heads * s.c.dim);
+    if (tail == "mix.A_log") { t->offset = 0.f; return vec(w.a_log, s.c.heads); }
+    if (tail == "mix.dt_bias") { t->offset = -2.f; return vec(w.dt_bias, (int64_t)s.c.heads * s.c.dim); }      // decays of about 0.9
     const int kd = s.c.kv_heads * s.c.dim;
     auto conv = [&](int at, int rows) { t->conv = w.conv; t->conv_C = delta_channels(s); t->conv_at = at; t->rows = rows; t->cols = s.c.conv; return true; };
     if (tail == "mix.q.conv") return conv(0, kd);
@@ -366,7 +367,7 @@ int32_t fill_target(Model* M, const Target& t, uint64_t key, const float* src, i
     LMB_CUDA(cudaGetLastError());
     return LMB200_OK;
   }
-  if (t.vec) return fill_plain_dt(M, LMB200_F32, t.plain, t.rows, t.cols, key, src, 0, scale, src ? 0.f : 1.f);
+  if (t.vec) return fill_plain_dt(M, LMB200_F32, t.plain, t.rows, t.cols, key, src, 0, scale, src ? 0.f : t.offset);
   if (t.plain) LMB_TRY(fill_plain_dt(M, M->cfg.dtype, t.plain, t.rows, t.cols, key, src, layout, scale, 0.f, t.head));
   if (!t.tiled) return LMB200_OK;
   FillSrc f{};
@@ -1057,6 +1058,7 @@ int32_t delta_rows(Session* S, RowsBuf& r, const RowsRun& run, int l, cudaStream
   v.decay = r.log_g; v.decay_pitch = hd;
   v.gate = r.gate; v.gate_pitch = ld_g;
   v.out = r.cat; v.ldo = row_ld(s.m_out.K); v.bp = 0;
+  if (dt == LMB200_BF16 && run.max_len >= kChunkMin && delta_chunks_ok(v)) return delta_chunks(ctx, v, st);
   return delta_steps(ctx, dt, v, st);
 }
 
@@ -1652,7 +1654,7 @@ int64_t layered_step_bytes(const Session* S, int32_t T) {
   int64_t n = (int64_t)M->cfg.vocab * W * e + W * 4 + B * W * e;
   for (int l = 0; l < M->cfg.n_layers; ++l) {
     const LayerSpec& s = M->specs[l];
-    auto mat = [&](const WMap& m) { int64_t k = 0; for (int i = 0; i < m.n_src; ++i) k += (int64_t)m.src_rows[i] * m.src_cols[i]; return k * e; };
+    auto mat = [&](const WMap& m) { int64_t k = 0; for (int i = 0; i < kMaxSrc; ++i) k += (int64_t)m.src_rows[i] * m.src_cols[i]; return k * e; };
     n += mat(s.m_in) + mat(s.m_out) + W * 4;
     if (post_norm(M)) n += mat(s.m_gu) + mat(s.m_down) + mat(s.m_sg) + mat(s.m_sp) + mat(s.m_lr) + 2 * W * 4 + B * M->side_dim * e;
     if (is_attention(s)) n += B * (int64_t)((s.c.window > 0 ? std::min(T, s.c.window) : T) + (s.c.kv_from < 0 ? 1 : 0)) * s.c.kv_heads * (s.c.dim + s.c.vdim) * e;

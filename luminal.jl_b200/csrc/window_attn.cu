@@ -3,6 +3,7 @@
 
 #include <algorithm>
 
+#include "mma_sync.cuh"
 #include "pdl.cuh"
 #include "tc.cuh"
 #include "window_attn.cuh"
@@ -24,7 +25,12 @@ __device__ __forceinline__ float2 turn(const WindowView& v, int t, int pos, int 
     const float2 cs = __ldg(v.angles + (int64_t)t * (v.rot_dims >> 1) + p);
     c = cs.x; s = cs.y;
   } else {
-    sincosf((float)pos * v.inv_freq[p], &s, &c);
+    // the product's rounding error is turned back to first order: at position 1000 it is 1000 times a float's resolution
+    const float f = v.inv_freq[p], x = (float)pos * f, err = fmaf((float)pos, f, -x);
+    sincosf(x, &s, &c);
+    const float s0 = s;
+    s = fmaf(err, c, s);
+    c = fmaf(-err, s0, c);
   }
   c *= v.rot_scale; s *= v.rot_scale;
   return make_float2(a * c - b * s, b * c + a * s);
@@ -174,18 +180,6 @@ __global__ void __launch_bounds__(kSimple) window_simple_kernel(const WindowView
 // ---------------------------------------------------------------------------------------------
 constexpr int kThreads = 128, kRing = 3;
 
-__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t addr) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];\n" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void ldsm4_trans(uint32_t (&r)[4], uint32_t addr) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];\n" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void mma16816(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile(
-      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
-      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
 __device__ __forceinline__ uint32_t movmatrix_trans(uint32_t a) {
   uint32_t d;
   asm volatile("movmatrix.sync.aligned.m8n8.trans.b16 %0, %1;\n" : "=r"(d) : "r"(a));

@@ -155,8 +155,9 @@ def token_side(x, e, w, p, eps):
     return rms(g @ w[p + "proj"].T, eps, w[p + "norm"])
 
 
-def forward(cfg, w, tokens, dtype=np.float64, return_layers=False):
-    """Logits [T, vocab] of one sequence (and the residual stream after every layer)."""
+def forward(cfg, w, tokens, dtype=np.float64, return_layers=False, rounded=lambda x: x):
+    """Logits [T, vocab] of one sequence (and the residual stream after every layer).  `rounded` is applied to what every sublayer and
+    the head read: with a rounding it shows how far rounding alone moves the logits."""
     w = {k: np.asarray(v, dtype=dtype) for k, v in w.items()}
     eps = cfg["norm"]["eps"]
     tokens = np.asarray(tokens)
@@ -168,20 +169,20 @@ def forward(cfg, w, tokens, dtype=np.float64, return_layers=False):
         if layer["type"] == "attention":
             src = mx.get("kv_from")
             if src is None:
-                kvs[i] = cached_keys_values(x, w, p + "mix.", mx, eps, pos)
-            y = attention(x, w, p + "mix.", mx, eps, pos, kvs[i if src is None else src])
+                kvs[i] = cached_keys_values(rounded(x), w, p + "mix.", mx, eps, pos)
+            y = attention(rounded(x), w, p + "mix.", mx, eps, pos, kvs[i if src is None else src])
         elif layer["type"] == "channel_delta":
-            y = channel_delta(x, w, p + "mix.", mx, eps)
+            y = channel_delta(rounded(x), w, p + "mix.", mx, eps)
         else:
-            y = lightning(x, w, p + "mix.", mx, eps)
+            y = lightning(rounded(x), w, p + "mix.", mx, eps)
         x = x + rms(y, eps, w[p + "norm1"])
         if layer.get("mlp"):
-            x = x + rms(feed_forward(x, w, p + "mlp."), eps, w[p + "norm2"])
+            x = x + rms(feed_forward(rounded(x), w, p + "mlp."), eps, w[p + "norm2"])
         if cfg.get("token_side"):
             n = cfg["token_side"]["dim"]
-            x = x + token_side(x, w["side.embed"][tokens, i * n:(i + 1) * n], w, p + "side.", eps)
+            x = x + token_side(rounded(x), w["side.embed"][tokens, i * n:(i + 1) * n], w, p + "side.", eps)
         outs.append(x)
-    logits = rms(x, eps, w["final.norm"]) @ w["embed"].T
+    logits = rounded(rms(x, eps, w["final.norm"])) @ w["embed"].T
     return (logits, outs) if return_layers else logits
 
 
