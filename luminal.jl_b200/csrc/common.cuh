@@ -192,6 +192,7 @@ struct FlashSplitView {
 struct FlashWindowView {
   int H = 1, G = 1, dn = 0, dv = 0, window = 0;
   float cap = 0.f;
+  float max_dot = 0.f;                // a bound on |q . k|, or 0: not known
   int64_t q_b = 0, q_h = 0, q_s = 0, o_b = 0, o_h = 0, o_s = 0;
   int64_t k_b = 0, k_h = 0, k_s = 0, v_b = 0, v_h = 0, v_s = 0;
 };

@@ -19,6 +19,8 @@ template <> struct Pair<float> { typedef float2 V; };
 template <> struct Pair<__nv_bfloat16> { typedef __nv_bfloat162 V; };
 __device__ __forceinline__ float2 pair_f32(float2 v) { return v; }
 __device__ __forceinline__ float2 pair_f32(__nv_bfloat162 v) { return __bfloat1622float2(v); }
+__device__ __forceinline__ float conv_silu(float x, float) { return silu_f32(x); }
+__device__ __forceinline__ float conv_silu(float x, __nv_bfloat16) { return __fdividef(x, 1.0f + __expf(-x)); }      // rounded to bf16 next
 __device__ __forceinline__ void put_pair(float* p, float2 v) { *reinterpret_cast<float2*>(p) = v; }
 __device__ __forceinline__ void put_pair(__nv_bfloat16* p, float2 v) { *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(v.x, v.y); }
 
@@ -53,9 +55,25 @@ __global__ void __launch_bounds__(256) delta_conv_kernel(const DeltaView v, T* _
       const float* p = v.conv + (int64_t)j * C + c0 + c;
       w[j][i] = j < v.taps && c < width ? make_float2(p[0], c + 1 < width ? p[1] : 0.f) : make_float2(0.f, 0.f);
     }
+  // few taps: all rows of the run are in flight at once
+  constexpr bool kAhead = MAXT <= 4;
+  constexpr int kRows = kAhead ? kRun : 1;
+  const int n = (int)min((int64_t)kRun, v.total - first);
+  const int my_seq = lane < n ? v.seq[first + lane] : 0, my_pos = lane < n ? v.pos[first + lane] : 0;
+  typename Pair<T>::V ahead[kRows][NP];
+  if (kAhead && even) {
+#pragma unroll
+    for (int r = 0; r < kRows; ++r)
+#pragma unroll
+      for (int i = 0; i < NP; ++i) {
+        const int c = 2 * (lane + 32 * i);
+        if (r < n && c < width) ahead[r][i] = *reinterpret_cast<const typename Pair<T>::V*>(src + (first + r) * pitch + c);
+      }
+  }
   int last = -1;
-  for (int64_t t = first; t < min((int64_t)v.total, first + kRun); ++t) {
-    const int s = v.seq[t], p = v.pos[t];
+  auto token = [&](int r, auto x_of) {
+    const int64_t t = first + r;
+    const int s = __shfl_sync(0xffffffffu, my_seq, r), p = __shfl_sync(0xffffffffu, my_pos, r);
     if (s != last) {                       // a run starts, or another sequence: the rows before this one
       last = s;
 #pragma unroll
@@ -67,8 +85,8 @@ __global__ void __launch_bounds__(256) delta_conv_kernel(const DeltaView v, T* _
           if (j < v.taps && p - j >= 0 && c < width) {
             if (t - j >= v.start[s]) x = raw(t - j, c);
             else {
-              const float* r = v.ring + ((int64_t)s * v.taps + (p - j) % v.taps) * C + c0 + c;
-              x = make_float2(r[0], c + 1 < width ? r[1] : 0.f);
+              const float* q = v.ring + ((int64_t)s * v.taps + (p - j) % v.taps) * C + c0 + c;
+              x = make_float2(q[0], c + 1 < width ? q[1] : 0.f);
             }
           }
           h[j - 1][i] = x;
@@ -80,14 +98,14 @@ __global__ void __launch_bounds__(256) delta_conv_kernel(const DeltaView v, T* _
     for (int i = 0; i < NP; ++i) {
       const int c = 2 * (lane + 32 * i);
       if (c >= width) continue;
-      const float2 x = raw(t, c);
+      const float2 x = x_of(i, c);
       float2 y = make_float2(w[0][i].x * x.x, w[0][i].y * x.y);
 #pragma unroll
       for (int j = 1; j < MAXT; ++j) { y.x = fmaf(w[j][i].x, h[j - 1][i].x, y.x); y.y = fmaf(w[j][i].y, h[j - 1][i].y, y.y); }
 #pragma unroll
       for (int j = MAXT - 2; j > 0; --j) h[j][i] = h[j - 1][i];
       h[0][i] = x;
-      T r0 = from_f32<T>(silu_f32(y.x)), r1 = from_f32<T>(c + 1 < width ? silu_f32(y.y) : 0.f);
+      const T r0 = from_f32<T>(conv_silu(y.x, T())), r1 = from_f32<T>(c + 1 < width ? conv_silu(y.y, T()) : 0.f);
       const float z0 = to_f32(r0), z1 = to_f32(r1);              // the length is that of the stored vector
       ss += z0 * z0 + z1 * z1;
       if (even) put_pair(o + c, make_float2(z0, z1));
@@ -96,13 +114,20 @@ __global__ void __launch_bounds__(256) delta_conv_kernel(const DeltaView v, T* _
         if (c + 1 < width) o[c + 1] = r1;
       }
     }
-    if (kind == 2) continue;
+    if (kind == 2) return;
     ss = warp_sum(ss);
     if (lane == 0) {
-      const float r = 1.0f / sqrtf(ss + kUnitEps);
-      if (kind == 0) rq[t * v.G + a] = r / sqrtf((float)v.dim);
-      else rk[t * v.G + a] = r;
+      const float f = 1.0f / sqrtf(ss + kUnitEps);
+      if (kind == 0) rq[t * v.G + a] = f / sqrtf((float)v.dim);
+      else rk[t * v.G + a] = f;
     }
+  };
+  if (kAhead && even) {
+#pragma unroll
+    for (int r = 0; r < kRows; ++r)
+      if (r < n) token(r, [&](int i, int) { return pair_f32(ahead[r][i]); });
+  } else {
+    for (int r = 0; r < n; ++r) token(r, [&](int, int c) { return raw(first + r, c); });
   }
 }
 
@@ -127,7 +152,7 @@ __global__ void __launch_bounds__(256) delta_ring_kernel(const DeltaView v) {
 // One CTA per (value head, sequence).  Thread (c, w): value columns 4 c .., rows w, w + W, ... of the state.  One pass over the state per
 // token gives both S^T k and S^T q after the decay; with u the written value, o = S^T q + (k . q) u and S <- S + k u^T.  KEEP: the
 // thread's part of the state stays in registers over all tokens.
-constexpr int kStep = 256, kKeep = 16;
+constexpr int kStep = 512, kKeep = 8;
 
 template <typename IT, typename OT, bool RAW, bool KEEP>
 __global__ void __launch_bounds__(kStep, 2) delta_step_kernel(const DeltaView v) {
@@ -162,23 +187,32 @@ __global__ void __launch_bounds__(kStep, 2) delta_step_kernel(const DeltaView v)
     const int64_t t = t0 + it;
     float beta = 0.f;
     if (RAW) {
-      const int C = 2 * v.G * D + v.H * V, p = p0 + it;
+      const int C = 2 * v.G * D + v.H * V, p = p0 + it, now = p % v.taps;
       float* ring = v.ring + (int64_t)b * v.taps * C;
-      auto conv = [&](const void* src, int pitch, int col, int ch, bool keep) {
-        const float x = reinterpret_cast<const float*>(src)[t * pitch + col];
-        float y = v.conv[ch] * x;
-        for (int j = 1; j < v.taps; ++j)
-          if (p - j >= 0) y = fmaf(v.conv[(int64_t)j * C + ch], ring[((p - j) % v.taps) * C + ch], y);
-        if (keep) ring[(p % v.taps) * C + ch] = x;              // a slot no tap of this token reads
-        return to_f32(from_f32<IT>(silu_f32(y)));
-      };
       const bool owner = h == a * gq;
-      for (int d = tid; d < D; d += kStep) {
-        qs[d] = conv(v.q, v.q_pitch, a * D + d, a * D + d, owner);
-        ks[d] = conv(v.k, v.k_pitch, a * D + d, v.G * D + a * D + d, owner);
-        gs[d] = expf(log_decay_f32(v.decay[t * v.decay_pitch + h * D + d], v.a_log[h], v.dt_bias[h * D + d]));
+      for (int i = tid; i < 3 * D + 4 * V4; i += kStep) {       // q, k, log g, v: the taps' loads are independent
+        const int kind = i < 3 * D ? i / D : 3, d = i - kind * D;
+        if (kind == 2) {
+          gs[d] = expf(log_decay_f32(v.decay[t * v.decay_pitch + h * D + d], v.a_log[h], v.dt_bias[h * D + d]));
+          continue;
+        }
+        if (kind == 3 && d >= V) { vs[d] = 0.f; continue; }
+        const int col = kind == 3 ? h * V + d : a * D + d, ch = kind == 0 ? col : kind == 1 ? v.G * D + col : 2 * v.G * D + col;
+        const float x = kind == 0 ? reinterpret_cast<const float*>(v.q)[t * v.q_pitch + col]
+                                  : kind == 1 ? reinterpret_cast<const float*>(v.k)[t * v.k_pitch + col] : reinterpret_cast<const float*>(v.v)[t * v.v_pitch + col];
+        float y = v.conv[ch] * x;
+        int slot = now;
+#pragma unroll 4
+        for (int j = 1; j < v.taps; ++j) {
+          slot = slot == 0 ? v.taps - 1 : slot - 1;
+          if (p - j >= 0) y = fmaf(v.conv[(int64_t)j * C + ch], ring[slot * C + ch], y);
+        }
+        if (kind == 3 || owner) ring[now * C + ch] = x;         // a slot no tap of this token reads
+        const float r = to_f32(from_f32<IT>(silu_f32(y)));
+        if (kind == 0) qs[d] = r;
+        else if (kind == 1) ks[d] = r;
+        else vs[d] = r;
       }
-      for (int d = tid; d < 4 * V4; d += kStep) vs[d] = d < V ? conv(v.v, v.v_pitch, h * V + d, 2 * v.G * D + h * V + d, true) : 0.f;
     } else {
       const IT* q = reinterpret_cast<const IT*>(v.q) + t * v.q_pitch + a * D;
       const IT* k = reinterpret_cast<const IT*>(v.k) + t * v.k_pitch + a * D;

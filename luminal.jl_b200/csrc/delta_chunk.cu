@@ -5,9 +5,9 @@
 //   A_ts = beta_t sum_d k_t k_s e^{G_t - G_s} (s < t),   B_ts = sum_d q_t k_s e^{G_t - G_s} (s <= t)
 // the recurrence is
 //   (I + A) U = beta (V - kt S),   O = qt S + B U,   S <- diag(e^{G_end}) S + kb^T U
-// No exponent is ever positive, whatever the decays: the rows t of a 16-token block are taken relative to the block's start R,
-// e^{G_t - R} e^{R - G_s}; inside the block, where the second factor grows, only as far as float32 reaches (kDiagMax), else the block's
-// 16 x 16 sums are taken term by term.  (I + A) is solved block by block with the inverses of its 16 x 16 diagonal blocks.
+// A and B for any decays: where a whole chunk decays by no more than 2^-kDiagMax, they are products of kt, qt and k_s e^{-G_s}.  Else the
+// rows t of a 16-token block are taken relative to the block's start R, e^{G_t - R} e^{R - G_s}, and no exponent is positive for s in an
+// earlier block; inside the block the second factor grows, again no further than 2^kDiagMax, or its 16 x 16 sums are taken term by term.  (I + A) is solved block by block with the inverses of its 16 x 16 diagonal blocks.
 // Everything the decays or the state touch enters the products as bf16 pairs hi + lo (x to about 2^-17) in three products.
 // All products are taken transposed (M = 16 value columns): a warp owns 16 value columns, its part of the state stays in its
 // accumulator registers over the whole portion and is an A operand without a move, and so is U; warps meet only to share
@@ -145,6 +145,7 @@ __global__ void __launch_bounds__(Smem<DK, DV>::kThreads, 1) delta_chunk_kernel(
     __syncthreads();
     // ---- running sums of the log decays (log2 units): in sG from the block's start on (a large decay costs only its own block
     // precision), R[b] = the sum before block b, R[4] = G_end
+    int mild = 1;
     for (int d = tid; d < DK; d += NT) {
       float R = 0.f;
 #pragma unroll
@@ -159,34 +160,46 @@ __global__ void __launch_bounds__(Smem<DK, DV>::kThreads, 1) delta_chunk_kernel(
         R += s;
       }
       sR[kB * DK + d] = R;
+      mild = mild && R >= -kDiagMax;
     }
-    __syncthreads();
-    // ---- kt, qt, kb
-    for (int i = tid; i < kC * (DK / 2); i += NT) {
-      const int r = i / (DK / 2), d = (i - r * (DK / 2)) * 2;
-      const float2 G = *reinterpret_cast<const float2*>(sG + r * pg + d), E = *reinterpret_cast<const float2*>(sR + kB * DK + d);
-      const float2 Rv = *reinterpret_cast<const float2*>(sR + (r >> 4) * DK + d);
-      const float2 k = unpack_bf16(*reinterpret_cast<const uint32_t*>(sK + r * pk + d)), q = unpack_bf16(*reinterpret_cast<const uint32_t*>(sQ + r * pk + d));
-      const float e0 = ex2(Rv.x + G.x), e1 = ex2(Rv.y + G.y), kr = rk[r], qr = rq[r];
-      uint32_t hi, lo;
-      split2(k.x * kr * e0, k.y * kr * e1, hi, lo);
-      *reinterpret_cast<uint32_t*>(sKt + r * pk + d) = hi;
-      *reinterpret_cast<uint32_t*>(sKt + kLoT + r * pk + d) = lo;
-      split2(q.x * qr * e0, q.y * qr * e1, hi, lo);
-      *reinterpret_cast<uint32_t*>(sQt + r * pk + d) = hi;
-      *reinterpret_cast<uint32_t*>(sQt + kLoT + r * pk + d) = lo;
-      split2(k.x * kr * ex2(E.x - Rv.x - G.x), k.y * kr * ex2(E.y - Rv.y - G.y), hi, lo);
-      *reinterpret_cast<uint32_t*>(sKb + r * pk + d) = hi;
-      *reinterpret_cast<uint32_t*>(sKb + kLoT + r * pk + d) = lo;
+    mild = __syncthreads_and(mild);
+    // ---- kt, qt, kb; mild chunks: k e^{-G} over the raw rows (hi over K, lo over Q)
+#pragma unroll 2
+    for (int i = tid; i < kC * (DK / 4); i += NT) {
+      const int r = i / (DK / 4), d = (i - r * (DK / 4)) * 4, at = r * pk + d;
+      const float4 L = *reinterpret_cast<const float4*>(sG + r * pg + d), E = *reinterpret_cast<const float4*>(sR + kB * DK + d);
+      const float4 Rv = *reinterpret_cast<const float4*>(sR + (r >> 4) * DK + d);
+      const uint2 ku = *reinterpret_cast<const uint2*>(sK + at), qu = *reinterpret_cast<const uint2*>(sQ + at);
+      const float2 k0 = unpack_bf16(ku.x), k1 = unpack_bf16(ku.y), q0 = unpack_bf16(qu.x), q1 = unpack_bf16(qu.y);
+      const float kr = rk[r], qr = rq[r];
+      const float G[4] = {Rv.x + L.x, Rv.y + L.y, Rv.z + L.z, Rv.w + L.w};
+      const float Eb[4] = {E.x - Rv.x - L.x, E.y - Rv.y - L.y, E.z - Rv.z - L.z, E.w - Rv.w - L.w};
+      const float k[4] = {k0.x * kr, k0.y * kr, k1.x * kr, k1.y * kr}, q[4] = {q0.x * qr, q0.y * qr, q1.x * qr, q1.y * qr};
+      float e[4];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) e[j] = ex2(G[j]);
+      auto put = [&](bf* m, float x0, float x1, float x2, float x3) {
+        uint2 hi, lo;
+        split2(x0, x1, hi.x, lo.x);
+        split2(x2, x3, hi.y, lo.y);
+        *reinterpret_cast<uint2*>(m + at) = hi;
+        return lo;
+      };
+      *reinterpret_cast<uint2*>(sKt + kLoT + at) = put(sKt, k[0] * e[0], k[1] * e[1], k[2] * e[2], k[3] * e[3]);
+      *reinterpret_cast<uint2*>(sQt + kLoT + at) = put(sQt, q[0] * e[0], q[1] * e[1], q[2] * e[2], q[3] * e[3]);
+      *reinterpret_cast<uint2*>(sKb + kLoT + at) = put(sKb, k[0] * ex2(Eb[0]), k[1] * ex2(Eb[1]), k[2] * ex2(Eb[2]), k[3] * ex2(Eb[3]));
+      if (mild) *reinterpret_cast<uint2*>(sQ + at) = put(sK, k[0] * ex2(-G[0]), k[1] * ex2(-G[1]), k[2] * ex2(-G[2]), k[3] * ex2(-G[3]));
     }
+    if (mild) __syncthreads();
     // ---- blocks (rt, st), st <= rt, of A and B: M = 16 rows t, N = 16 rows s
+    // the diagonal ones, which also are inverted, first
     for (int task = warp; task < 10; task += NW) {
-      const int rt = task < 4 ? 3 : task < 7 ? 2 : task < 9 ? 1 : 0, st = task < 4 ? task : task < 7 ? task - 4 : task < 9 ? task - 7 : 0;
+      const int off = task - 4, rt = task < 4 ? task : off == 0 ? 1 : off < 3 ? 2 : 3, st = task < 4 ? task : off == 0 ? 0 : off < 3 ? off - 1 : off - 3;
       if (16 * rt >= n) continue;                               // rows behind the portion's end
       const float* R = sR + rt * DK;
       const bool diag = rt == st;
       bool direct = false;
-      if (diag) {
+      if (diag && !mild) {
         float m = 0.f;
         for (int d = lane; d < DK; d += 32) m = fmaxf(m, -sG[(rt * 16 + 15) * pg + d]);
         direct = __any_sync(0xffffffffu, !(m <= kDiagMax));
@@ -196,7 +209,23 @@ __global__ void __launch_bounds__(Smem<DK, DV>::kThreads, 1) delta_chunk_kernel(
       for (int j = 0; j < 2; ++j)
 #pragma unroll
         for (int e = 0; e < 4; ++e) ca[j][e] = cb[j][e] = 0.f;
-      if (!direct) {
+      if (mild) {
+        const uint32_t ao = (uint32_t)((rt * 16 + (lane & 15)) * pk + (lane >> 4) * 8) * 2;
+        const uint32_t bo = (uint32_t)((st * 16 + (lane & 7) + ((lane >> 4) << 3)) * pk + ((lane >> 3) & 1) * 8) * 2;
+        const uint32_t kt = smem_addr(sKt) + ao, qt = smem_addr(sQt) + ao, k2h = smem_addr(sK) + bo, k2l = smem_addr(sQ) + bo;
+#pragma unroll 2
+        for (int kk = 0; kk < ND; ++kk) {
+          uint32_t ah[4], al[4], bh[4], bl[4];
+          ldsm4(bh, k2h + kk * 32);
+          ldsm4(bl, k2l + kk * 32);
+          ldsm4(ah, kt + kk * 32);
+          ldsm4(al, kt + kLoT * 2 + kk * 32);
+          mma3(ca[0], ca[1], ah, al, bh, bl);
+          ldsm4(ah, qt + kk * 32);
+          ldsm4(al, qt + kLoT * 2 + kk * 32);
+          mma3(cb[0], cb[1], ah, al, bh, bl);
+        }
+      } else if (!direct) {
 #pragma unroll 2
         for (int kk = 0; kk < ND; ++kk) {
           uint32_t kh[4], kl[4], qh[4], ql[4], bh[4], bl[4];
@@ -243,7 +272,7 @@ __global__ void __launch_bounds__(Smem<DK, DV>::kThreads, 1) delta_chunk_kernel(
 #pragma unroll
         for (int e2 = 0; e2 < 2; ++e2) {
           const int tl = g + 8 * e2, sl = 8 * j + 2 * tq, t = rt * 16 + tl, s = st * 16 + sl;
-          const float bt = beta[t] * rk[t], qt = rq[t], k0 = rk[s], k1 = rk[s + 1];
+          const float bt = mild ? beta[t] : beta[t] * rk[t], qt = mild ? 1.f : rq[t], k0 = mild ? 1.f : rk[s], k1 = mild ? 1.f : rk[s + 1];
           float a0 = ca[j][2 * e2] * bt * k0, a1 = ca[j][2 * e2 + 1] * bt * k1;
           float b0 = cb[j][2 * e2] * qt * k0, b1 = cb[j][2 * e2 + 1] * qt * k1;
           if (diag) {
@@ -388,6 +417,14 @@ __global__ void __launch_bounds__(Smem<DK, DV>::kThreads, 1) delta_chunk_kernel(
       }
     }
     // ---- outputs: sums of squares over the value columns, then whole token rows
+    constexpr int kVec = kC * (DV / 8) / NT;                    // 16-byte pieces of the gate and of the output per thread
+    uint4 gates[kVec];
+#pragma unroll
+    for (int j = 0; j < kVec; ++j) {
+      const int i = tid + j * NT, r = i / (DV / 8), d = (i - r * (DV / 8)) * 8;
+      gates[j] = r < n && d < V ? __ldg(reinterpret_cast<const uint4*>(reinterpret_cast<const bf*>(v.gate) + (t_first + (int64_t)c * kC + r) * v.gate_pitch + h * V + d))
+                                : make_uint4(0, 0, 0, 0);
+    }
 #pragma unroll
     for (int i = 0; i < 2 * kB; ++i) {
       float s0 = O[i][0] * O[i][0] + O[i][2] * O[i][2], s1 = O[i][1] * O[i][1] + O[i][3] * O[i][3];
@@ -409,15 +446,16 @@ __global__ void __launch_bounds__(Smem<DK, DV>::kThreads, 1) delta_chunk_kernel(
 #pragma unroll
       for (int e = 0; e < 4; ++e) sO[(8 * i + 2 * tq + (e & 1)) * SM::po + vc + 8 * (e >> 1)] = O[i][e];
     __syncthreads();
-    for (int i = tid; i < n * (DV / 8); i += NT) {
-      const int r = i / (DV / 8), d = (i - r * (DV / 8)) * 8;
-      if (d >= V) continue;
+#pragma unroll
+    for (int j = 0; j < kVec; ++j) {
+      const int i = tid + j * NT, r = i / (DV / 8), d = (i - r * (DV / 8)) * 8;
+      if (r >= n || d >= V) continue;
       float ss = 0.f;
 #pragma unroll
       for (int w = 0; w < NW; ++w) ss += sSum[w * kC + r];
       const float inv = 1.0f / sqrtf(ss / (float)V + v.eps);
       const int64_t t = t_first + (int64_t)c * kC + r;
-      uint4 gu = *reinterpret_cast<const uint4*>(reinterpret_cast<const bf*>(v.gate) + t * v.gate_pitch + h * V + d);
+      uint4 gu = gates[j];
       uint32_t* gi = reinterpret_cast<uint32_t*>(&gu);
 #pragma unroll
       for (int e = 0; e < 4; ++e) {

@@ -29,6 +29,7 @@
 // Causal: key tiles beyond a query tile's diagonal are never computed; inside the diagonal tile
 // keys j > i are masked -- the reference's `if causal && j > i continue`.
 #include <cuda.h>
+#include <math.h>
 #include <math_constants.h>
 
 #include "common.cuh"
@@ -92,6 +93,11 @@ __device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
   asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
   return d;
 }
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
+  uint64_t d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
 __device__ __forceinline__ uint64_t add2(uint64_t a, uint64_t b) {
   uint64_t d;
   asm("add.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
@@ -125,6 +131,8 @@ struct FlashExtra {
   int gate_pitch = 0;
   int window = 0;                   // a query sees the last `window` positions (0: all)
   float cap = 0.f;                  // scores pass cap tanh(. / cap) (0: not)
+  int n_poly = 0;                   // 4 or 7: cap tanh(z) log2(e) = z (poly[0] + poly[1] z^2 + ...) for every z that occurs
+  float poly[7] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
 };
 
 __device__ __forceinline__ void mma_f16_ts(uint32_t tmem_d, uint32_t tmem_a, uint64_t bdesc, uint32_t idesc, uint32_t accumulate) {
@@ -302,6 +310,22 @@ flash_tc_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict
     // a score in log2 units: s c, or cap tanh(s scale / cap) log2(e) as cap' - 2 cap' / (1 + 2^(s k2)) with cap' = cap log2(e)
     const float capl = WIN ? ex.cap * kLog2e : 0.f, k2 = WIN && ex.cap > 0.f ? 2.0f * c / ex.cap : 0.f;
     auto bounded = [&](float x) { return fmaf(-2.0f * capl, rcp_approx(1.0f + ex2_approx(x * k2)), capl); };
+    // with a bound on the scores: a polynomial on the FMA pipe, which leaves the exp2 unit to the softmax
+    const float kz = WIN && ex.cap > 0.f ? scale / ex.cap : 0.f;
+    auto poly2 = [&](uint64_t s2) {
+      const uint64_t z = mul2(s2, pack2(kz, kz)), u = mul2(z, z);
+      uint64_t p = pack2(ex.poly[3], ex.poly[3]);
+      if (ex.n_poly > 4) {
+        p = pack2(ex.poly[6], ex.poly[6]);
+        p = fma2(p, u, pack2(ex.poly[5], ex.poly[5]));
+        p = fma2(p, u, pack2(ex.poly[4], ex.poly[4]));
+        p = fma2(p, u, pack2(ex.poly[3], ex.poly[3]));
+      }
+      p = fma2(p, u, pack2(ex.poly[2], ex.poly[2]));
+      p = fma2(p, u, pack2(ex.poly[1], ex.poly[1]));
+      p = fma2(p, u, pack2(ex.poly[0], ex.poly[0]));
+      return mul2(z, p);
+    };
     auto hidden = [&](int key) { return key >= Sk || (causal && key > q_off + qi) || (WIN && ex.window > 0 && key <= q_off + qi - ex.window); };
     float m = -CUDART_INF_F, l = 0.f;
     for (int j = j0; j < nt; ++j) {
@@ -331,7 +355,13 @@ flash_tc_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict
       xch[t][h][r] = mx;
       asm volatile("bar.sync %0, 64;\n" ::"r"(pair_bar) : "memory");
       mx = fmaxf(mx, xch[t][h ^ 1][r]);
-      if (WIN && capl > 0.f) mx = mx > -CUDART_INF_F ? bounded(mx) : mx;
+      if (WIN && capl > 0.f) {
+        if (mx > -CUDART_INF_F) {
+          float z0, z1;
+          if (ex.n_poly) { unpack2(poly2(pack2(mx, mx)), z0, z1); mx = z0; }
+          else mx = bounded(mx);
+        }
+      }
       else mx *= c;
       const bool starts = m == -CUDART_INF_F && mx > -CUDART_INF_F;
       const bool raise = m > -CUDART_INF_F && mx > m + kRescaleStep;
@@ -366,8 +396,12 @@ flash_tc_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict
           const int key = key0 + qd * 16 + i;
           float x0, x1;
           if (WIN && capl > 0.f) {
-            x0 = bounded(a0) + neg_m;
-            x1 = bounded(a1) + neg_m;
+            if (ex.n_poly) {
+              unpack2(add2(poly2(pack2(a0, a1)), negm2), x0, x1);
+            } else {
+              x0 = bounded(a0) + neg_m;
+              x1 = bounded(a1) + neg_m;
+            }
             if (!inside) {
               if (hidden(key)) x0 = -CUDART_INF_F;
               if (hidden(key + 1)) x1 = -CUDART_INF_F;
@@ -563,6 +597,25 @@ int32_t flash_tc_launch_split(Ctx* ctx, void* out, const void* q, const void* k,
   return LMB200_OK;
 }
 
+// g(u) = tanh(sqrt u) / sqrt u on [0, z_max^2] through n Chebyshev points, times `factor`, as a polynomial in u
+static void tanh_poly(double z_max, int n, double factor, float* poly) {
+  double x[8], y[8], c[8] = {0}, basis[9] = {1.0};
+  const double len = z_max * z_max;
+  for (int i = 0; i < n; ++i) {
+    x[i] = 0.5 * len * (1.0 - cos((i + 0.5) * 3.14159265358979323846 / n));
+    const double r = sqrt(x[i]);
+    y[i] = tanh(r) / r;
+  }
+  for (int j = 1; j < n; ++j)                                   // divided differences, then Newton's form multiplied out
+    for (int i = n - 1; i >= j; --i) y[i] = (y[i] - y[i - 1]) / (x[i] - x[i - j]);
+  for (int j = 0; j < n; ++j) {
+    for (int i = 0; i <= j; ++i) c[i] += y[j] * basis[i];
+    for (int i = j + 1; i > 0; --i) basis[i] = basis[i - 1] - x[j] * basis[i];
+    basis[0] *= -x[j];
+  }
+  for (int i = 0; i < n; ++i) poly[i] = (float)(c[i] * factor);
+}
+
 bool flash_tc_window_supported(int dn, int dv) { return dn >= 8 && dn <= 128 && dn % 8 == 0 && dv >= 8 && dv <= 128 && dv % 8 == 0; }
 
 // causal attention of the last Sq of Sk positions over the last f.window positions, scores bounded by f.cap
@@ -583,6 +636,11 @@ int32_t flash_tc_launch_window(Ctx* ctx, void* out, const void* q, const void* k
   ex.Sk = (int)Sk; ex.q_off = (int)(Sk - Sq); ex.dn = f.dn; ex.dv = f.dv;
   ex.o_b = f.o_b; ex.o_h = f.o_h; ex.o_s = f.o_s;
   ex.window = f.window; ex.cap = f.cap;
+  const double z_max = f.cap > 0.f && f.max_dot > 0.f ? (double)scale * f.max_dot / f.cap : 2.0;
+  if (z_max <= 1.0) {                                           // relative errors about 1e-7 and 3e-8
+    ex.n_poly = z_max <= 0.45 ? 4 : 7;
+    tanh_poly(z_max, ex.n_poly, (double)f.cap * kLog2e, ex.poly);
+  }
   const dim3 grid((unsigned)ceil_div(Sq, 2 * kBM), (unsigned)(B * f.H));
 #define LMB_FLASH(DN, DV)                                                                                              \
   flash_tc_kernel<DN, 0, DV, true><<<grid, kThreads, Smem<DN, 0, DV>::total + 1024, stream>>>(                         \

@@ -237,7 +237,8 @@ void derive_layer(LayerSpec& s, int width, int block, int side_dim) {
     s.n_store = at;
     if (c.ff && block == LMB200_BLOCK_PARALLEL) part(R_UP, c.ff);
   }
-  s.m_in.rows = at; s.m_in.K = width;
+  s.m_in.rows = at > 1024 ? (int)round_up(at, 256) : at;        // whole row pairs for the prompt GEMM
+  s.m_in.K = width;
   s.cat0 = (int)round_up(out_width(s), 32);
   stack(s.m_out, 0, 0, width, 0, out_width(s));
   s.m_out.rows = width; s.m_out.K = out_width(s);
@@ -1004,6 +1005,7 @@ int32_t attention_rows(Session* S, RowsBuf& r, const RowsRun& run, int l, bool g
   auto flash = [&](int b, int n_batch, int t0, int n, int ctx_rows) -> int32_t {
     FlashWindowView f;
     f.H = v.H; f.G = v.H / v.G; f.dn = v.dim; f.dv = v.vdim; f.window = v.window; f.cap = v.score_cap;
+    f.max_dot = 1.01f * v.dim;                                 // unit root mean squares, rounded to bf16
     f.q_s = qw; f.q_h = v.dim; f.q_b = (int64_t)n * qw;
     f.o_s = ldc; f.o_h = v.vdim; f.o_b = (int64_t)n * ldc;
     f.k_s = v.k_ld; f.k_h = (int64_t)v.cap * v.k_ld; f.k_b = v.G * f.k_h;

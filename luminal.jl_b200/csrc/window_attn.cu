@@ -13,6 +13,11 @@ namespace {
 
 constexpr float kLog2e = 1.4426950408889634f;
 
+__device__ __forceinline__ float2 load_pair(const float* p) { return *reinterpret_cast<const float2*>(p); }
+__device__ __forceinline__ float2 load_pair(const __nv_bfloat16* p) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p)); }
+__device__ __forceinline__ void store_pair(float* p, float a, float b) { *reinterpret_cast<float2*>(p) = make_float2(a, b); }
+__device__ __forceinline__ void store_pair(__nv_bfloat16* p, float a, float b) { *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(a, b); }
+
 // pair p of a head: features lo and hi; the first rot_dims / 2 pairs rotate
 __device__ __forceinline__ void pair_of(const WindowView& v, int p, int* lo, int* hi) {
   const int half = v.rot_dims >> 1;
@@ -102,6 +107,75 @@ __global__ void __launch_bounds__(256) window_prep_kernel(const WindowView v, co
     WT* o = reinterpret_cast<WT*>(v.values) + row * v.v_ld;
     const IT* s = reinterpret_cast<const IT*>(in.v) + (int64_t)t * in.v_pitch + a * v.vdim;
     for (int d = lane; d < v.vdim; d += 32) o[d] = from_f32<WT>(to_f32(s[d]));
+  }
+}
+
+// The same for neighbouring pairs and even widths up to 64 NP: a warp takes kHeads heads of one token, their loads in flight together; the
+// token's angles are read once
+constexpr int kHeads = 4;
+template <typename IT, typename WT, int NP>
+__global__ void __launch_bounds__(256) window_prep_rows_kernel(const WindowView v, const WindowRows in, WT* q_out) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int lane = threadIdx.x & 31;
+  const int units = v.H + (in.k ? v.G : 0), groups = (units + kHeads - 1) / kHeads, vgroups = in.k ? (v.G + kHeads - 1) / kHeads : 0;
+  const int64_t id = (int64_t)blockIdx.x * 8 + (threadIdx.x >> 5);
+  if (id >= (int64_t)v.T * (groups + vgroups)) return;
+  const int t = (int)(id / (groups + vgroups)), gr = (int)(id - (int64_t)t * (groups + vgroups));
+  const int pos = v.pos[t];
+  const bool cached = pos >= 0 && pos < v.cap;
+  const int64_t row0 = (int64_t)v.seq[t] * v.G * v.cap + pos;          // key head a: + a * cap
+  if (gr >= groups) {
+    if (!cached) return;
+    for (int a = (gr - groups) * kHeads; a < min(v.G, (gr - groups + 1) * kHeads); ++a) {
+      WT* o = reinterpret_cast<WT*>(v.values) + (row0 + (int64_t)a * v.cap) * v.v_ld;
+      const IT* s = reinterpret_cast<const IT*>(in.v) + (int64_t)t * in.v_pitch + a * v.vdim;
+      for (int d = lane; d < v.vdim; d += 32) o[d] = from_f32<WT>(to_f32(s[d]));
+    }
+    return;
+  }
+  float2 x[kHeads][NP];
+#pragma unroll
+  for (int e = 0; e < kHeads; ++e) {
+    const int u = gr * kHeads + e;
+    const IT* s = u < v.H ? reinterpret_cast<const IT*>(in.q) + (int64_t)t * in.q_pitch + u * v.dim
+                          : reinterpret_cast<const IT*>(in.k) + (int64_t)t * in.k_pitch + (u - v.H) * v.dim;
+#pragma unroll
+    for (int i = 0; i < NP; ++i) {
+      const int d = 2 * (lane + 32 * i);
+      x[e][i] = u < units && d < v.dim ? load_pair(s + d) : make_float2(0.f, 0.f);
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < NP; ++i) {
+    const int p = lane + 32 * i;
+    if (p >= (v.rot_dims >> 1)) continue;
+    const float2 cs = turn(v, t, pos, p, 1.f, 0.f);                  // (cosine, sine), scaled
+#pragma unroll
+    for (int e = 0; e < kHeads; ++e) x[e][i] = make_float2(x[e][i].x * cs.x - x[e][i].y * cs.y, x[e][i].y * cs.x + x[e][i].x * cs.y);
+  }
+  float ss[kHeads];
+#pragma unroll
+  for (int e = 0; e < kHeads; ++e) {
+    ss[e] = 0.f;
+#pragma unroll
+    for (int i = 0; i < NP; ++i) ss[e] += x[e][i].x * x[e][i].x + x[e][i].y * x[e][i].y;
+  }
+#pragma unroll
+  for (int off = 16; off > 0; off >>= 1)
+#pragma unroll
+    for (int e = 0; e < kHeads; ++e) ss[e] += __shfl_xor_sync(0xffffffffu, ss[e], off);
+#pragma unroll
+  for (int e = 0; e < kHeads; ++e) {
+    const int u = gr * kHeads + e;
+    if (u >= units || (u >= v.H && !cached)) continue;
+    const float inv = 1.0f / sqrtf(ss[e] / (float)v.dim + v.eps);
+    WT* o = u < v.H ? q_out + ((int64_t)t * v.H + u) * v.dim : reinterpret_cast<WT*>(v.keys) + (row0 + (int64_t)(u - v.H) * v.cap) * v.k_ld;
+#pragma unroll
+    for (int i = 0; i < NP; ++i) {
+      const int d = 2 * (lane + 32 * i);
+      if (d < v.dim) store_pair(o + d, x[e][i].x * inv, x[e][i].y * inv);
+    }
   }
 }
 
@@ -229,6 +303,32 @@ __global__ void __launch_bounds__(kThreads) window_split_kernel(const WindowView
   __nv_bfloat16* K = reinterpret_cast<__nv_bfloat16*>(v.keys) + ((int64_t)v.seq[t] * v.G + a) * v.cap * v.k_ld;
   __nv_bfloat16* V = reinterpret_cast<__nv_bfloat16*>(v.values) + ((int64_t)v.seq[t] * v.G + a) * v.cap * v.v_ld;
   __syncthreads();
+  const int kpw = kpc >> 2, wb = k_begin + warp * kpw, we = min(k_end, wb + kpw);
+  const int blocks = we > wb ? (we - wb + 15) >> 4 : 0;
+  const int kc = v.k_ld >> 3, vc = v.v_ld >> 3;
+  auto load = [&](int i) {
+    __nv_bfloat16* sk = stage + (i % kRing) * 16 * (PK + PV);
+    __nv_bfloat16* sv = sk + 16 * PK;
+    const int key0 = wb + i * 16;
+#pragma unroll
+    for (int rr = 0; rr < 2; ++rr) {
+      const int r = (lane >> 2) + 8 * rr;
+      const __nv_bfloat16* kr = K + (int64_t)(key0 + r) * v.k_ld;
+      const __nv_bfloat16* vr = V + (int64_t)(key0 + r) * v.v_ld;
+#pragma unroll
+      for (int c0 = 0; c0 < DK / 8; c0 += 4)
+        if (c0 + tq < kc) tc::cp_async16(tc::smem_u32(sk + r * PK + (c0 + tq) * 8), kr + (c0 + tq) * 8, 16u);
+#pragma unroll
+      for (int c0 = 0; c0 < DV / 8; c0 += 4)
+        if (c0 + tq < vc) tc::cp_async16(tc::smem_u32(sv + r * PV + (c0 + tq) * 8), vr + (c0 + tq) * 8, 16u);
+    }
+  };
+  // the first blocks are on their way while the queries are prepared (not the one that gets the newest key)
+  int early = 0;
+#pragma unroll
+  for (int i = 0; i < kRing - 1; ++i) {
+    if (i < blocks && (!PREP || wb + i * 16 + 16 <= pos)) { load(i); early = i + 1; }
+  }
   if (PREP) {
     const bool newest = in.k && k_end == pos + 1;
     for (int u = warp; u < nh + (newest ? 2 : 0); u += 4) {
@@ -257,26 +357,6 @@ __global__ void __launch_bounds__(kThreads) window_split_kernel(const WindowView
     qf[dk][0] = *reinterpret_cast<const uint32_t*>(sQ + g * PK + 16 * dk + 2 * tq);
     qf[dk][1] = *reinterpret_cast<const uint32_t*>(sQ + g * PK + 16 * dk + 2 * tq + 8);
   }
-  const int kpw = kpc >> 2, wb = k_begin + warp * kpw, we = min(k_end, wb + kpw);
-  const int blocks = we > wb ? (we - wb + 15) >> 4 : 0;
-  const int kc = v.k_ld >> 3, vc = v.v_ld >> 3;
-  auto load = [&](int i) {
-    __nv_bfloat16* sk = stage + (i % kRing) * 16 * (PK + PV);
-    __nv_bfloat16* sv = sk + 16 * PK;
-    const int key0 = wb + i * 16;
-#pragma unroll
-    for (int rr = 0; rr < 2; ++rr) {
-      const int r = (lane >> 2) + 8 * rr;
-      const __nv_bfloat16* kr = K + (int64_t)(key0 + r) * v.k_ld;
-      const __nv_bfloat16* vr = V + (int64_t)(key0 + r) * v.v_ld;
-#pragma unroll
-      for (int c0 = 0; c0 < DK / 8; c0 += 4)
-        if (c0 + tq < kc) tc::cp_async16(tc::smem_u32(sk + r * PK + (c0 + tq) * 8), kr + (c0 + tq) * 8, 16u);
-#pragma unroll
-      for (int c0 = 0; c0 < DV / 8; c0 += 4)
-        if (c0 + tq < vc) tc::cp_async16(tc::smem_u32(sv + r * PV + (c0 + tq) * 8), vr + (c0 + tq) * 8, 16u);
-    }
-  };
   float m0 = -CUDART_INF_F, m1 = -CUDART_INF_F, l0 = 0.f, l1 = 0.f;
   float o[NV][4];
 #pragma unroll
@@ -284,7 +364,7 @@ __global__ void __launch_bounds__(kThreads) window_split_kernel(const WindowView
   const float two_over_cap = v.score_cap > 0.f ? 2.0f / v.score_cap : 0.f;
 #pragma unroll
   for (int i = 0; i < kRing - 1; ++i) {
-    if (i < blocks) load(i);
+    if (i < blocks && i >= early) load(i);
     tc::cp_async_commit();
   }
   for (int i = 0; i < blocks; ++i) {
@@ -434,7 +514,22 @@ int32_t window_configure() {
   return LMB200_OK;
 }
 
+template <typename IT, typename WT>
+int32_t prep_rows(const WindowView& v, const WindowRows& in, void* q_out, cudaStream_t st) {
+  const int64_t warps = (int64_t)v.T * (ceil_div(v.H + (in.k ? v.G : 0), kHeads) + (in.k ? ceil_div(v.G, kHeads) : 0));
+  const dim3 grid((unsigned)ceil_div(warps, 8));
+  if (v.dim <= 64) LMB_CUDA(launch_k(window_prep_rows_kernel<IT, WT, 1>, grid, dim3(256), 0, st, v, in, (WT*)q_out));
+  else if (v.dim <= 128) LMB_CUDA(launch_k(window_prep_rows_kernel<IT, WT, 2>, grid, dim3(256), 0, st, v, in, (WT*)q_out));
+  else LMB_CUDA(launch_k(window_prep_rows_kernel<IT, WT, 4>, grid, dim3(256), 0, st, v, in, (WT*)q_out));
+  return LMB200_OK;
+}
+
 int32_t window_prep(Ctx* ctx, int dtype, const WindowView& v, const WindowRows& in, void* q_out, cudaStream_t st) {
+  if (v.rot_interleaved && v.dim % 2 == 0 && v.dim <= 256 && in.q_pitch % 2 == 0 && in.k_pitch % 2 == 0 && v.k_ld % 2 == 0) {
+    ctx->launches++;
+    if (dtype != LMB200_BF16) return prep_rows<float, float>(v, in, q_out, st);
+    return in.in_f32 ? prep_rows<float, __nv_bfloat16>(v, in, q_out, st) : prep_rows<__nv_bfloat16, __nv_bfloat16>(v, in, q_out, st);
+  }
   const int units = v.H + (in.k ? 2 * v.G : 0);
   const dim3 grid((unsigned)ceil_div((int64_t)v.T * units, 8));
   if (dtype != LMB200_BF16)
