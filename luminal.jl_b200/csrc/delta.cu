@@ -7,7 +7,7 @@ namespace lmb {
 namespace {
 
 constexpr float kUnitEps = 1e-6f;
-constexpr int kRun = 16;                 // tokens a warp of the convolution walks over
+constexpr int kRun = 8;                  // tokens a warp of the convolution walks over
 
 __device__ __forceinline__ float warp_sum(float x) {
 #pragma unroll
@@ -55,35 +55,40 @@ __global__ void __launch_bounds__(256) delta_conv_kernel(const DeltaView v, T* _
       const float* p = v.conv + (int64_t)j * C + c0 + c;
       w[j][i] = j < v.taps && c < width ? make_float2(p[0], c + 1 < width ? p[1] : 0.f) : make_float2(0.f, 0.f);
     }
-  // few taps: all rows of the run are in flight at once
+  // few taps: all rows of the run, and the ones before it, are in flight at once
   constexpr bool kAhead = MAXT <= 4;
-  constexpr int kRows = kAhead ? kRun : 1;
+  constexpr int kBack = kAhead ? MAXT - 1 : 0, kRows = kAhead ? kRun : 1;
   const int n = (int)min((int64_t)kRun, v.total - first);
-  const int my_seq = lane < n ? v.seq[first + lane] : 0, my_pos = lane < n ? v.pos[first + lane] : 0;
-  typename Pair<T>::V ahead[kRows][NP];
+  // lane r: row first - (MAXT - 1) + r
+  const int64_t mine = first - (MAXT - 1) + lane;
+  const bool have = lane < n + MAXT - 1 && mine >= 0;
+  const int my_seq = have ? v.seq[mine] : -1, my_pos = have ? v.pos[mine] : 0;
+  typename Pair<T>::V ahead[kBack + kRows][NP];
   if (kAhead && even) {
 #pragma unroll
-    for (int r = 0; r < kRows; ++r)
+    for (int r = 0; r < kBack + kRows; ++r)
 #pragma unroll
       for (int i = 0; i < NP; ++i) {
         const int c = 2 * (lane + 32 * i);
-        if (r < n && c < width) ahead[r][i] = *reinterpret_cast<const typename Pair<T>::V*>(src + (first + r) * pitch + c);
+        const int64_t t = first - kBack + r;
+        if (t >= 0 && r < kBack + n && c < width) ahead[r][i] = *reinterpret_cast<const typename Pair<T>::V*>(src + t * pitch + c);
       }
   }
   int last = -1;
   auto token = [&](int r, auto x_of) {
     const int64_t t = first + r;
-    const int s = __shfl_sync(0xffffffffu, my_seq, r), p = __shfl_sync(0xffffffffu, my_pos, r);
+    const int s = __shfl_sync(0xffffffffu, my_seq, r + MAXT - 1), p = __shfl_sync(0xffffffffu, my_pos, r + MAXT - 1);
     if (s != last) {                       // a run starts, or another sequence: the rows before this one
       last = s;
 #pragma unroll
-      for (int j = 1; j < MAXT; ++j)
+      for (int j = 1; j < MAXT; ++j) {
+        const bool packed = __shfl_sync(0xffffffffu, my_seq, r + MAXT - 1 - j) == s;      // the row before is in this call too
 #pragma unroll
         for (int i = 0; i < NP; ++i) {
           const int c = 2 * (lane + 32 * i);
           float2 x = make_float2(0.f, 0.f);
           if (j < v.taps && p - j >= 0 && c < width) {
-            if (t - j >= v.start[s]) x = raw(t - j, c);
+            if (packed) x = x_of(r - j, i, c);
             else {
               const float* q = v.ring + ((int64_t)s * v.taps + (p - j) % v.taps) * C + c0 + c;
               x = make_float2(q[0], c + 1 < width ? q[1] : 0.f);
@@ -91,6 +96,7 @@ __global__ void __launch_bounds__(256) delta_conv_kernel(const DeltaView v, T* _
           }
           h[j - 1][i] = x;
         }
+      }
     }
     float ss = 0.f;
     T* o = out + t * C + c0;
@@ -98,7 +104,7 @@ __global__ void __launch_bounds__(256) delta_conv_kernel(const DeltaView v, T* _
     for (int i = 0; i < NP; ++i) {
       const int c = 2 * (lane + 32 * i);
       if (c >= width) continue;
-      const float2 x = x_of(i, c);
+      const float2 x = x_of(r, i, c);
       float2 y = make_float2(w[0][i].x * x.x, w[0][i].y * x.y);
 #pragma unroll
       for (int j = 1; j < MAXT; ++j) { y.x = fmaf(w[j][i].x, h[j - 1][i].x, y.x); y.y = fmaf(w[j][i].y, h[j - 1][i].y, y.y); }
@@ -114,20 +120,30 @@ __global__ void __launch_bounds__(256) delta_conv_kernel(const DeltaView v, T* _
         if (c + 1 < width) o[c + 1] = r1;
       }
     }
-    if (kind == 2) return;
-    ss = warp_sum(ss);
-    if (lane == 0) {
-      const float f = 1.0f / sqrtf(ss + kUnitEps);
-      if (kind == 0) rq[t * v.G + a] = f / sqrtf((float)v.dim);
-      else rk[t * v.G + a] = f;
-    }
+    return ss;
   };
+  float my_ss = 0.f;                       // lane r: token r's sum
   if (kAhead && even) {
+    float ss[kRows];
 #pragma unroll
-    for (int r = 0; r < kRows; ++r)
-      if (r < n) token(r, [&](int i, int) { return pair_f32(ahead[r][i]); });
+    for (int r = 0; r < kRows; ++r) ss[r] = r < n ? token(r, [&](int q, int i, int) { return pair_f32(ahead[kBack + q][i]); }) : 0.f;
+    if (kind < 2) {
+#pragma unroll
+      for (int r = 0; r < kRows; ++r) {
+        const float s = warp_sum(ss[r]);
+        if (lane == r) my_ss = s;
+      }
+    }
   } else {
-    for (int r = 0; r < n; ++r) token(r, [&](int, int c) { return raw(first + r, c); });
+    for (int r = 0; r < n; ++r) {
+      const float s = warp_sum(token(r, [&](int q, int, int c) { return raw(first + q, c); }));
+      if (lane == r) my_ss = s;
+    }
+  }
+  if (kind < 2 && lane < n) {
+    const float f = 1.0f / sqrtf(my_ss + kUnitEps);
+    if (kind == 0) rq[(first + lane) * v.G + a] = f / sqrtf((float)v.dim);
+    else rk[(first + lane) * v.G + a] = f;
   }
 }
 
@@ -160,24 +176,50 @@ __global__ void __launch_bounds__(kStep, 2) delta_step_kernel(const DeltaView v)
   __shared__ float red[kStep / 32], s_dot[3];
   pdl_launch_dependents();
   const int h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const int D = v.dim, V = v.vdim, V4 = (V + 3) >> 2, W = kStep / V4;
+  const int D = v.dim, V = v.vdim, V4 = (V + 3) >> 2;
   const int gq = v.H / v.G, a = h / gq;
   float* qs = sm;
   float* ks = qs + ((D + 3) & ~3);
   float* gs = ks + ((D + 3) & ~3);
   float* vs = gs + ((D + 3) & ~3);         // [4 V4] v, then o
   float* us = vs + 4 * V4;                 // [4 V4]
-  float* os = us + 4 * V4;                 // [W][2][4 V4]
+  float* os = us + 4 * V4;                 // [parts][2][4 V4]
   float4* S = reinterpret_cast<float4*>(v.state) + ((int64_t)b * v.H + h) * D * V4;
-  const int c = tid % V4, w = tid / V4;
-  if (KEEP && w < W) {                     // the state into L2 while the projection finishes
-#pragma unroll
-    for (int i = 0; i < kKeep; ++i)
-      if (w + i * W < D && (c & 7) == 0) asm volatile("prefetch.global.L2 [%0];\n" ::"l"(S + (int64_t)(w + i * W) * V4 + c));
-  }
+  // quad: a warp covers 8 column groups x 4 rows, so that shuffles add four rows and few partial sums meet in shared memory
+  const int blocks = V4 >> 3;
+  const bool quad = (V4 & 7) == 0 && (kStep / 32) % blocks == 0;
+  const int W = quad ? kStep / 32 / blocks * 4 : kStep / V4, parts = quad ? W / 4 : W;
+  const int c = quad ? (warp % blocks) * 8 + (lane & 7) : tid % V4, w = quad ? warp / blocks * 4 + (lane >> 3) : tid / V4;
   pdl_wait();
   const int n = v.len[b], t0 = v.start[b], p0 = v.pos0[b];
   if (n <= 0) return;
+  // The single raw token of a decoding step: its inputs' loads go out before the state's.  Item tid: one element of q, k, log g or v
+  constexpr int kTaps = 4;
+  const int C = 2 * v.G * D + v.H * V, items = 3 * D + V;
+  const bool early = RAW && v.taps <= kTaps && items <= kStep;
+  const int kind = tid < 3 * D ? tid / D : 3, di = tid - kind * D;
+  const bool owner = h == a * gq;
+  int ch = 0;
+  float raw_x = 0.f, raw_t[kTaps], raw_w[kTaps];
+  float* ring = v.ring + (int64_t)b * v.taps * C;
+  if (early && tid < items) {
+    const int64_t t = t0;
+    if (kind == 2) {
+      raw_x = v.decay[t * v.decay_pitch + h * D + di];
+      raw_t[0] = v.a_log[h];
+      raw_t[1] = v.dt_bias[h * D + di];
+    } else {
+      const int col = kind == 3 ? h * V + di : a * D + di;
+      ch = kind == 0 ? col : kind == 1 ? v.G * D + col : 2 * v.G * D + col;
+      raw_x = kind == 0 ? reinterpret_cast<const float*>(v.q)[t * v.q_pitch + col]
+                        : kind == 1 ? reinterpret_cast<const float*>(v.k)[t * v.k_pitch + col] : reinterpret_cast<const float*>(v.v)[t * v.v_pitch + col];
+#pragma unroll
+      for (int j = 0; j < kTaps; ++j) {
+        raw_w[j] = j < v.taps ? v.conv[(int64_t)j * C + ch] : 0.f;
+        raw_t[j] = j > 0 && j < v.taps && p0 - j >= 0 ? ring[(p0 - j) % v.taps * C + ch] : 0.f;
+      }
+    }
+  }
   float4 s[kKeep];
   if (KEEP && w < W) {
 #pragma unroll
@@ -186,10 +228,20 @@ __global__ void __launch_bounds__(kStep, 2) delta_step_kernel(const DeltaView v)
   for (int it = 0; it < n; ++it) {
     const int64_t t = t0 + it;
     float beta = 0.f;
-    if (RAW) {
-      const int C = 2 * v.G * D + v.H * V, p = p0 + it, now = p % v.taps;
-      float* ring = v.ring + (int64_t)b * v.taps * C;
-      const bool owner = h == a * gq;
+    if (early) {
+      if (tid < items) {
+        if (kind == 2) gs[di] = expf(log_decay_f32(raw_x, raw_t[0], raw_t[1]));
+        else {
+          float y = raw_w[0] * raw_x;
+#pragma unroll
+          for (int j = 1; j < kTaps; ++j) y = fmaf(raw_w[j], raw_t[j], y);
+          if (kind == 3 || owner) ring[p0 % v.taps * C + ch] = raw_x;     // a slot no tap of this token reads
+          (kind == 0 ? qs : kind == 1 ? ks : vs)[di] = to_f32(from_f32<IT>(silu_f32(y)));
+        }
+      }
+      for (int d = V + tid; d < 4 * V4; d += kStep) vs[d] = 0.f;
+    } else if (RAW) {
+      const int p = p0 + it, now = p % v.taps;
       for (int i = tid; i < 3 * D + 4 * V4; i += kStep) {       // q, k, log g, v: the taps' loads are independent
         const int kind = i < 3 * D ? i / D : 3, d = i - kind * D;
         if (kind == 2) {
@@ -251,8 +303,20 @@ __global__ void __launch_bounds__(kStep, 2) delta_step_kernel(const DeltaView v)
           row(d, x);
         }
       }
-      *reinterpret_cast<float4*>(os + (w * 2) * 4 * V4 + 4 * c) = ak;
-      *reinterpret_cast<float4*>(os + (w * 2 + 1) * 4 * V4 + 4 * c) = aq;
+      if (quad) {
+#pragma unroll
+        for (int off = 8; off < 32; off <<= 1) {
+          ak.x += __shfl_xor_sync(0xffffffffu, ak.x, off); ak.y += __shfl_xor_sync(0xffffffffu, ak.y, off);
+          ak.z += __shfl_xor_sync(0xffffffffu, ak.z, off); ak.w += __shfl_xor_sync(0xffffffffu, ak.w, off);
+          aq.x += __shfl_xor_sync(0xffffffffu, aq.x, off); aq.y += __shfl_xor_sync(0xffffffffu, aq.y, off);
+          aq.z += __shfl_xor_sync(0xffffffffu, aq.z, off); aq.w += __shfl_xor_sync(0xffffffffu, aq.w, off);
+        }
+      }
+      if (!quad || lane < 8) {
+        const int part = quad ? w >> 2 : w;
+        *reinterpret_cast<float4*>(os + (part * 2) * 4 * V4 + 4 * c) = ak;
+        *reinterpret_cast<float4*>(os + (part * 2 + 1) * 4 * V4 + 4 * c) = aq;
+      }
     }
     __syncthreads();
     float rq, rk;
@@ -262,7 +326,7 @@ __global__ void __launch_bounds__(kStep, 2) delta_step_kernel(const DeltaView v)
     float ss = 0.f;
     for (int d = tid; d < 4 * V4; d += kStep) {
       float x = 0.f, y = 0.f;
-      for (int j = 0; j < W; ++j) { x += os[(j * 2) * 4 * V4 + d]; y += os[(j * 2 + 1) * 4 * V4 + d]; }
+      for (int j = 0; j < parts; ++j) { x += os[(j * 2) * 4 * V4 + d]; y += os[(j * 2 + 1) * 4 * V4 + d]; }
       const float u = d < V ? beta * (vs[d] - x * rk) : 0.f, o = y * rq + kq * u;
       us[d] = u * rk;                      // the key's scale on the way into the state
       vs[d] = o;
@@ -336,7 +400,7 @@ int32_t delta_conv(Ctx* ctx, int dtype, const DeltaView& v, void* out, float* rq
 
 int32_t delta_steps(Ctx* ctx, int dtype, const DeltaView& v, cudaStream_t st) {
   LMB_TRY(check(v));
-  const int V4 = (v.vdim + 3) >> 2, W = kStep / V4;
+  const int V4 = (v.vdim + 3) >> 2, blocks = V4 >> 3, W = (V4 & 7) == 0 && (kStep / 32) % blocks == 0 ? kStep / 32 / blocks * 4 : kStep / V4;
   const size_t smem = (size_t)(3 * ((v.dim + 3) & ~3) + 8 * V4 + W * 8 * V4) * 4;
   const bool keep = v.dim <= W * kKeep, bf = dtype == LMB200_BF16;
   const dim3 grid((unsigned)v.H, (unsigned)v.B);

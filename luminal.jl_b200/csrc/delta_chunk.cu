@@ -38,10 +38,9 @@ struct Smem {
   static constexpr int oK = oT + 2 * 4 * kBlk * 2, oQ = oK + kRow, oG = oQ + kRow;   // raw rows; G float32
   static constexpr int oV = oG + kC * pg * 4;
   static constexpr int oD = oV + kC * pv * 2;                                        // 4 diagonal blocks float32 [16][17]
-  static constexpr int oR = oD + 4 * 16 * 17 * 4;                                    // [5][DK]: G before each block, and G_end
+  static constexpr int oR = oD + 4 * 16 * 17 * 4;                                    // [5][DK]: e^{G_end}, G before blocks 1 .. 3, G_end
   static constexpr int oRow = oR + 5 * DK * 4;                                       // beta, rk, rq: 2 x [3][64]
-  static constexpr int oSum = oRow + 2 * 3 * kC * 4;                                 // [kWarps][64]
-  static constexpr int total = oSum + kWarps * kC * 4;
+  static constexpr int total = oRow + 2 * 3 * kC * 4;
   static_assert(kC * po * 4 <= 4 * kRow, "the staged outputs fit over kt and qt");
   static_assert(total <= 227 * 1024, "shared memory");
 };
@@ -79,7 +78,7 @@ __global__ void __launch_bounds__(Smem<DK, DV>::kThreads, 1) delta_chunk_kernel(
   bf *sKt = (bf*)(sm + SM::oKt), *sQt = (bf*)(sm + SM::oQt), *sKb = (bf*)(sm + SM::oKb);
   bf *sA = (bf*)(sm + SM::oA), *sB = (bf*)(sm + SM::oB), *sT = (bf*)(sm + SM::oT);
   bf *sK = (bf*)(sm + SM::oK), *sQ = (bf*)(sm + SM::oQ), *sV = (bf*)(sm + SM::oV);
-  float *sG = (float*)(sm + SM::oG), *sD = (float*)(sm + SM::oD), *sR = (float*)(sm + SM::oR), *sRow = (float*)(sm + SM::oRow), *sSum = (float*)(sm + SM::oSum);
+  float *sG = (float*)(sm + SM::oG), *sD = (float*)(sm + SM::oD), *sR = (float*)(sm + SM::oR), *sRow = (float*)(sm + SM::oRow);
   float* sO = (float*)(sm + SM::oKt);
   constexpr int kLoT = kC * pk, kLoA = 6 * kBlk, kLoB = 10 * kBlk, kLoI = 4 * kBlk;          // distance of the low parts (elements)
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, tq = lane & 3;
@@ -90,39 +89,64 @@ __global__ void __launch_bounds__(Smem<DK, DV>::kThreads, 1) delta_chunk_kernel(
   if (n_all <= 0) return;
   const int chunks = (n_all + kC - 1) / kC;
 
+  // a thread copies 16-byte pieces of one column range, rows r0, r0 + step, ...
+  float row_b = 0.f, row_k = 0.f, row_q = 0.f;                 // of token tid, on their way to sRow
   auto load_kqg = [&](int c) {
     const int64_t t0 = t_first + (int64_t)c * kC;
     const int n = min(kC, n_all - c * kC);
-    for (int i = tid; i < kC * (DK / 8); i += NT) {
-      const int r = i / (DK / 8), d = (i - r * (DK / 8)) * 8;
-      const bool ok = r < n && d < D;
-      const int64_t t = t0 + (ok ? r : 0);
-      tc::cp_async16(smem_addr(sK + r * pk + d), reinterpret_cast<const bf*>(v.k) + t * v.k_pitch + a * D + (ok ? d : 0), ok ? 16u : 0u);
-      tc::cp_async16(smem_addr(sQ + r * pk + d), reinterpret_cast<const bf*>(v.q) + t * v.q_pitch + a * D + (ok ? d : 0), ok ? 16u : 0u);
+    {
+      constexpr int step = NT / (DK / 8);
+      const int r0 = tid / (DK / 8), d = (tid - r0 * (DK / 8)) * 8;
+      const bool in = d < D;
+      const bf* k = reinterpret_cast<const bf*>(v.k) + t0 * v.k_pitch + a * D + (in ? d : 0);
+      const bf* q = reinterpret_cast<const bf*>(v.q) + t0 * v.q_pitch + a * D + (in ? d : 0);
+#pragma unroll
+      for (int r = r0; r < kC; r += step) {
+        const bool ok = in && r < n;
+        tc::cp_async16(smem_addr(sK + r * pk + d), k + (ok ? r * v.k_pitch : 0), ok ? 16u : 0u);
+        tc::cp_async16(smem_addr(sQ + r * pk + d), q + (ok ? r * v.q_pitch : 0), ok ? 16u : 0u);
+      }
     }
-    for (int i = tid; i < kC * (DK / 4); i += NT) {
-      const int r = i / (DK / 4), d = (i - r * (DK / 4)) * 4;
-      const bool ok = r < n && d < D;
-      tc::cp_async16(smem_addr(sG + r * pg + d), v.decay + (t0 + (ok ? r : 0)) * v.decay_pitch + h * D + (ok ? d : 0), ok ? 16u : 0u);
+    {
+      constexpr int step = NT / (DK / 4);
+      const int r0 = tid / (DK / 4), d = (tid - r0 * (DK / 4)) * 4;
+      const bool in = d < D;
+      const float* x = v.decay + t0 * v.decay_pitch + h * D + (in ? d : 0);
+#pragma unroll
+      for (int r = r0; r < kC; r += step) {
+        const bool ok = in && r < n;
+        tc::cp_async16(smem_addr(sG + r * pg + d), x + (ok ? r * v.decay_pitch : 0), ok ? 16u : 0u);
+      }
     }
-    float* row = sRow + (c & 1) * 3 * kC;
     if (tid < kC) {
       const bool ok = tid < n;
-      row[tid] = ok ? 1.0f / (1.0f + expf(-v.b[(t0 + tid) * v.b_pitch + h])) : 0.f;
-      row[kC + tid] = ok ? v.rk[(t0 + tid) * v.G + a] : 0.f;
-      row[2 * kC + tid] = ok ? v.rq[(t0 + tid) * v.G + a] : 0.f;
+      row_b = ok ? v.b[(t0 + tid) * v.b_pitch + h] : 0.f;
+      row_k = ok ? v.rk[(t0 + tid) * v.G + a] : 0.f;
+      row_q = ok ? v.rq[(t0 + tid) * v.G + a] : 0.f;
     }
+  };
+  auto store_rows = [&](int c) {
+    if (tid >= kC) return;
+    float* row = sRow + (c & 1) * 3 * kC;
+    row[tid] = c * kC + tid < n_all ? 1.0f / (1.0f + expf(-row_b)) : 0.f;
+    row[kC + tid] = row_k;
+    row[2 * kC + tid] = row_q;
   };
   auto load_v = [&](int c) {
     const int64_t t0 = t_first + (int64_t)c * kC;
     const int n = min(kC, n_all - c * kC);
-    for (int i = tid; i < kC * (DV / 8); i += NT) {
-      const int r = i / (DV / 8), d = (i - r * (DV / 8)) * 8;
-      const bool ok = r < n && d < V;
-      tc::cp_async16(smem_addr(sV + r * pv + d), reinterpret_cast<const bf*>(v.v) + (t0 + (ok ? r : 0)) * v.v_pitch + h * V + (ok ? d : 0), ok ? 16u : 0u);
+    constexpr int step = NT / (DV / 8);
+    const int r0 = tid / (DV / 8), d = (tid - r0 * (DV / 8)) * 8;
+    const bool in = d < V;
+    const bf* x = reinterpret_cast<const bf*>(v.v) + t0 * v.v_pitch + h * V + (in ? d : 0);
+#pragma unroll
+    for (int r = r0; r < kC; r += step) {
+      const bool ok = in && r < n;
+      tc::cp_async16(smem_addr(sV + r * pv + d), x + (ok ? r * v.v_pitch : 0), ok ? 16u : 0u);
     }
   };
   load_kqg(0);
+  store_rows(0);
   load_v(0);
   tc::cp_async_commit();
 
@@ -144,13 +168,13 @@ __global__ void __launch_bounds__(Smem<DK, DV>::kThreads, 1) delta_chunk_kernel(
     tc::cp_async_wait<0>();
     __syncthreads();
     // ---- running sums of the log decays (log2 units): in sG from the block's start on (a large decay costs only its own block
-    // precision), R[b] = the sum before block b, R[4] = G_end
+    // precision), R[b] = the sum before block b > 0, R[4] = G_end, R[0] = e^{G_end}
     int mild = 1;
     for (int d = tid; d < DK; d += NT) {
       float R = 0.f;
 #pragma unroll
       for (int blk = 0; blk < kB; ++blk) {
-        sR[blk * DK + d] = R;
+        if (blk) sR[blk * DK + d] = R;
         float s = 0.f;
 #pragma unroll
         for (int r = 0; r < 16; ++r) {
@@ -160,6 +184,7 @@ __global__ void __launch_bounds__(Smem<DK, DV>::kThreads, 1) delta_chunk_kernel(
         R += s;
       }
       sR[kB * DK + d] = R;
+      sR[d] = ex2(R);
       mild = mild && R >= -kDiagMax;
     }
     mild = __syncthreads_and(mild);
@@ -168,7 +193,7 @@ __global__ void __launch_bounds__(Smem<DK, DV>::kThreads, 1) delta_chunk_kernel(
     for (int i = tid; i < kC * (DK / 4); i += NT) {
       const int r = i / (DK / 4), d = (i - r * (DK / 4)) * 4, at = r * pk + d;
       const float4 L = *reinterpret_cast<const float4*>(sG + r * pg + d), E = *reinterpret_cast<const float4*>(sR + kB * DK + d);
-      const float4 Rv = *reinterpret_cast<const float4*>(sR + (r >> 4) * DK + d);
+      const float4 Rv = r < 16 ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4*>(sR + (r >> 4) * DK + d);
       const uint2 ku = *reinterpret_cast<const uint2*>(sK + at), qu = *reinterpret_cast<const uint2*>(sQ + at);
       const float2 k0 = unpack_bf16(ku.x), k1 = unpack_bf16(ku.y), q0 = unpack_bf16(qu.x), q1 = unpack_bf16(qu.y);
       const float kr = rk[r], qr = rq[r];
@@ -187,14 +212,21 @@ __global__ void __launch_bounds__(Smem<DK, DV>::kThreads, 1) delta_chunk_kernel(
       };
       *reinterpret_cast<uint2*>(sKt + kLoT + at) = put(sKt, k[0] * e[0], k[1] * e[1], k[2] * e[2], k[3] * e[3]);
       *reinterpret_cast<uint2*>(sQt + kLoT + at) = put(sQt, q[0] * e[0], q[1] * e[1], q[2] * e[2], q[3] * e[3]);
-      *reinterpret_cast<uint2*>(sKb + kLoT + at) = put(sKb, k[0] * ex2(Eb[0]), k[1] * ex2(Eb[1]), k[2] * ex2(Eb[2]), k[3] * ex2(Eb[3]));
-      if (mild) *reinterpret_cast<uint2*>(sQ + at) = put(sK, k[0] * ex2(-G[0]), k[1] * ex2(-G[1]), k[2] * ex2(-G[2]), k[3] * ex2(-G[3]));
+      if (mild) {
+        const float4 X = *reinterpret_cast<const float4*>(sR + d);                              // e^{G_end}
+        const float m[4] = {k[0] * ex2(-G[0]), k[1] * ex2(-G[1]), k[2] * ex2(-G[2]), k[3] * ex2(-G[3])};
+        *reinterpret_cast<uint2*>(sKb + kLoT + at) = put(sKb, m[0] * X.x, m[1] * X.y, m[2] * X.z, m[3] * X.w);
+        *reinterpret_cast<uint2*>(sQ + at) = put(sK, m[0], m[1], m[2], m[3]);
+      } else {
+        *reinterpret_cast<uint2*>(sKb + kLoT + at) = put(sKb, k[0] * ex2(Eb[0]), k[1] * ex2(Eb[1]), k[2] * ex2(Eb[2]), k[3] * ex2(Eb[3]));
+      }
     }
     if (mild) __syncthreads();
     // ---- blocks (rt, st), st <= rt, of A and B: M = 16 rows t, N = 16 rows s
-    // the diagonal ones, which also are inverted, first
-    for (int task = warp; task < 10; task += NW) {
-      const int off = task - 4, rt = task < 4 ? task : off == 0 ? 1 : off < 3 ? 2 : 3, st = task < 4 ? task : off == 0 ? 0 : off < 3 ? off - 1 : off - 3;
+    // tasks 0 - 3: the diagonal ones, which also are inverted; then the A and the B part of the six others
+    for (int task = warp; task < 16; task += NW) {
+      const int off = (task - 4) >> 1, rt = task < 4 ? task : off == 0 ? 1 : off < 3 ? 2 : 3, st = task < 4 ? task : off == 0 ? 0 : off < 3 ? off - 1 : off - 3;
+      const bool do_a = task < 4 || (task & 1) == 0, do_b = task < 4 || (task & 1);
       if (16 * rt >= n) continue;                               // rows behind the portion's end
       const float* R = sR + rt * DK;
       const bool diag = rt == st;
@@ -213,18 +245,37 @@ __global__ void __launch_bounds__(Smem<DK, DV>::kThreads, 1) delta_chunk_kernel(
         const uint32_t ao = (uint32_t)((rt * 16 + (lane & 15)) * pk + (lane >> 4) * 8) * 2;
         const uint32_t bo = (uint32_t)((st * 16 + (lane & 7) + ((lane >> 4) << 3)) * pk + ((lane >> 3) & 1) * 8) * 2;
         const uint32_t kt = smem_addr(sKt) + ao, qt = smem_addr(sQt) + ao, k2h = smem_addr(sK) + bo, k2l = smem_addr(sQ) + bo;
+        float cx[2][2][4], cy[2][2][4];                         // the three products on accumulators of their own: short chains
+#pragma unroll
+        for (int j = 0; j < 2; ++j)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) cx[0][j][e] = cx[1][j][e] = cy[0][j][e] = cy[1][j][e] = 0.f;
+        auto three = [&](float (&c0)[2][4], float (&c1)[2][4], float (&c2)[2][4], const uint32_t (&ah)[4], const uint32_t (&al)[4], const uint32_t (&bh)[4],
+                         const uint32_t (&bl)[4]) {
+          mma16816(c0[0], ah, bh[0], bh[1]); mma16816(c0[1], ah, bh[2], bh[3]);
+          mma16816(c1[0], al, bh[0], bh[1]); mma16816(c1[1], al, bh[2], bh[3]);
+          mma16816(c2[0], ah, bl[0], bl[1]); mma16816(c2[1], ah, bl[2], bl[3]);
+        };
 #pragma unroll 2
         for (int kk = 0; kk < ND; ++kk) {
           uint32_t ah[4], al[4], bh[4], bl[4];
           ldsm4(bh, k2h + kk * 32);
           ldsm4(bl, k2l + kk * 32);
-          ldsm4(ah, kt + kk * 32);
-          ldsm4(al, kt + kLoT * 2 + kk * 32);
-          mma3(ca[0], ca[1], ah, al, bh, bl);
-          ldsm4(ah, qt + kk * 32);
-          ldsm4(al, qt + kLoT * 2 + kk * 32);
-          mma3(cb[0], cb[1], ah, al, bh, bl);
+          if (do_a) {
+            ldsm4(ah, kt + kk * 32);
+            ldsm4(al, kt + kLoT * 2 + kk * 32);
+            three(ca, cx[0], cx[1], ah, al, bh, bl);
+          }
+          if (do_b) {
+            ldsm4(ah, qt + kk * 32);
+            ldsm4(al, qt + kLoT * 2 + kk * 32);
+            three(cb, cy[0], cy[1], ah, al, bh, bl);
+          }
         }
+#pragma unroll
+        for (int j = 0; j < 2; ++j)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) { ca[j][e] += cx[0][j][e] + cx[1][j][e]; cb[j][e] += cy[0][j][e] + cy[1][j][e]; }
       } else if (!direct) {
 #pragma unroll 2
         for (int kk = 0; kk < ND; ++kk) {
@@ -235,18 +286,19 @@ __global__ void __launch_bounds__(Smem<DK, DV>::kThreads, 1) delta_chunk_kernel(
             const float2 G = *reinterpret_cast<const float2*>(sG + r * pg + d);
             const float e0 = ex2(G.x), e1 = ex2(G.y);
             const float2 k = unpack_bf16(*reinterpret_cast<const uint32_t*>(sK + r * pk + d)), q = unpack_bf16(*reinterpret_cast<const uint32_t*>(sQ + r * pk + d));
-            split2(k.x * e0, k.y * e1, kh[e], kl[e]);
-            split2(q.x * e0, q.y * e1, qh[e], ql[e]);
+            if (do_a) split2(k.x * e0, k.y * e1, kh[e], kl[e]);
+            if (do_b) split2(q.x * e0, q.y * e1, qh[e], ql[e]);
           }
 #pragma unroll
           for (int e = 0; e < 4; ++e) {                         // B operand: column tile e >> 1, channels 2 tq + 8 (e & 1)
             const int r = st * 16 + g + 8 * (e >> 1), d = kk * 16 + 2 * tq + 8 * (e & 1);
-            const float2 G = *reinterpret_cast<const float2*>(sG + r * pg + d), Rt = *reinterpret_cast<const float2*>(R + d), Rs = *reinterpret_cast<const float2*>(sR + st * DK + d);
+            const float2 G = *reinterpret_cast<const float2*>(sG + r * pg + d), Rt = rt ? *reinterpret_cast<const float2*>(R + d) : make_float2(0.f, 0.f);
+            const float2 Rs = st ? *reinterpret_cast<const float2*>(sR + st * DK + d) : make_float2(0.f, 0.f);
             const float2 k = unpack_bf16(*reinterpret_cast<const uint32_t*>(sK + r * pk + d));
             split2(k.x * ex2(Rt.x - Rs.x - G.x), k.y * ex2(Rt.y - Rs.y - G.y), bh[e], bl[e]);
           }
-          mma3(ca[0], ca[1], kh, kl, bh, bl);
-          mma3(cb[0], cb[1], qh, ql, bh, bl);
+          if (do_a) mma3(ca[0], ca[1], kh, kl, bh, bl);
+          if (do_b) mma3(cb[0], cb[1], qh, ql, bh, bl);
         }
       } else {
 #pragma unroll
@@ -284,10 +336,12 @@ __global__ void __launch_bounds__(Smem<DK, DV>::kThreads, 1) delta_chunk_kernel(
             sD[(rt * 16 + tl) * 17 + sl + 1] = a1;
           }
           uint32_t hi, lo;
-          split2(b0, b1, hi, lo);
-          *reinterpret_cast<uint32_t*>(sB + blk * kBlk + tl * 24 + sl) = hi;
-          *reinterpret_cast<uint32_t*>(sB + kLoB + blk * kBlk + tl * 24 + sl) = lo;
-          if (!diag) {                                          // subtracted where it is used
+          if (do_b) {
+            split2(b0, b1, hi, lo);
+            *reinterpret_cast<uint32_t*>(sB + blk * kBlk + tl * 24 + sl) = hi;
+            *reinterpret_cast<uint32_t*>(sB + kLoB + blk * kBlk + tl * 24 + sl) = lo;
+          }
+          if (!diag && do_a) {                                          // subtracted where it is used
             split2(-a0, -a1, hi, lo);
             *reinterpret_cast<uint32_t*>(sA + blk_a * kBlk + tl * 24 + sl) = hi;
             *reinterpret_cast<uint32_t*>(sA + kLoA + blk_a * kBlk + tl * 24 + sl) = lo;
@@ -398,9 +452,8 @@ __global__ void __launch_bounds__(Smem<DK, DV>::kThreads, 1) delta_chunk_kernel(
     // ---- S <- e^{G_end} S + kb^T U
 #pragma unroll
     for (int j = 0; j < DK / 8; ++j) {
-      const float2 E = *reinterpret_cast<const float2*>(sR + kB * DK + 8 * j + 2 * tq);
-      const float e0 = ex2(E.x), e1 = ex2(E.y);
-      S[j][0] *= e0; S[j][1] *= e1; S[j][2] *= e0; S[j][3] *= e1;
+      const float2 E = *reinterpret_cast<const float2*>(sR + 8 * j + 2 * tq);
+      S[j][0] *= E.x; S[j][1] *= E.y; S[j][2] *= E.x; S[j][3] *= E.y;
     }
     {
       const uint32_t kb = smem_addr(sKb) + (uint32_t)((lane & 15) * pk + (lane >> 4) * 8) * 2;
@@ -416,7 +469,7 @@ __global__ void __launch_bounds__(Smem<DK, DV>::kThreads, 1) delta_chunk_kernel(
         }
       }
     }
-    // ---- outputs: sums of squares over the value columns, then whole token rows
+    // ---- outputs: through shared memory to whole token rows
     constexpr int kVec = kC * (DV / 8) / NT;                    // 16-byte pieces of the gate and of the output per thread
     uint4 gates[kVec];
 #pragma unroll
@@ -424,19 +477,6 @@ __global__ void __launch_bounds__(Smem<DK, DV>::kThreads, 1) delta_chunk_kernel(
       const int i = tid + j * NT, r = i / (DV / 8), d = (i - r * (DV / 8)) * 8;
       gates[j] = r < n && d < V ? __ldg(reinterpret_cast<const uint4*>(reinterpret_cast<const bf*>(v.gate) + (t_first + (int64_t)c * kC + r) * v.gate_pitch + h * V + d))
                                 : make_uint4(0, 0, 0, 0);
-    }
-#pragma unroll
-    for (int i = 0; i < 2 * kB; ++i) {
-      float s0 = O[i][0] * O[i][0] + O[i][2] * O[i][2], s1 = O[i][1] * O[i][1] + O[i][3] * O[i][3];
-#pragma unroll
-      for (int off = 4; off < 32; off <<= 1) {
-        s0 += __shfl_xor_sync(0xffffffffu, s0, off);
-        s1 += __shfl_xor_sync(0xffffffffu, s1, off);
-      }
-      if (g == 0) {
-        sSum[warp * kC + 8 * i + 2 * tq] = s0;
-        sSum[warp * kC + 8 * i + 2 * tq + 1] = s1;
-      }
     }
     __syncthreads();                                            // kt and qt have been read by everyone
     if (c + 1 < chunks) load_v(c + 1);
@@ -446,25 +486,42 @@ __global__ void __launch_bounds__(Smem<DK, DV>::kThreads, 1) delta_chunk_kernel(
 #pragma unroll
       for (int e = 0; e < 4; ++e) sO[(8 * i + 2 * tq + (e & 1)) * SM::po + vc + 8 * (e >> 1)] = O[i][e];
     __syncthreads();
+    {
+      constexpr int L = DV / 8;                                 // lanes that share a token row
+      const int d = (tid % L) * 8;
+      float w[8];
 #pragma unroll
-    for (int j = 0; j < kVec; ++j) {
-      const int i = tid + j * NT, r = i / (DV / 8), d = (i - r * (DV / 8)) * 8;
-      if (r >= n || d >= V) continue;
-      float ss = 0.f;
+      for (int e = 0; e < 8; ++e) w[e] = d < V ? __ldg(v.norm + d + e) : 0.f;
+      float o[kVec][8], ss[kVec];
 #pragma unroll
-      for (int w = 0; w < NW; ++w) ss += sSum[w * kC + r];
-      const float inv = 1.0f / sqrtf(ss / (float)V + v.eps);
-      const int64_t t = t_first + (int64_t)c * kC + r;
-      uint4 gu = gates[j];
-      uint32_t* gi = reinterpret_cast<uint32_t*>(&gu);
+      for (int j = 0; j < kVec; ++j) {
+        const float* row = sO + (tid / L + j * (NT / L)) * SM::po + d;
+        const float4 x = *reinterpret_cast<const float4*>(row), y = *reinterpret_cast<const float4*>(row + 4);
+        o[j][0] = x.x; o[j][1] = x.y; o[j][2] = x.z; o[j][3] = x.w; o[j][4] = y.x; o[j][5] = y.y; o[j][6] = y.z; o[j][7] = y.w;
+        ss[j] = 0.f;
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const float2 gt = unpack_bf16(gi[e]), o = *reinterpret_cast<const float2*>(sO + r * SM::po + d + 2 * e), w = __ldg(reinterpret_cast<const float2*>(v.norm + d + 2 * e));
-        const __nv_bfloat162 y = __floats2bfloat162_rn(o.x * inv * w.x * gt.x, o.y * inv * w.y * gt.y);
-        gi[e] = *reinterpret_cast<const uint32_t*>(&y);
+        for (int e = 0; e < 8; ++e) ss[j] = fmaf(o[j][e], o[j][e], ss[j]);      // zero behind the width
       }
-      *reinterpret_cast<uint4*>(reinterpret_cast<bf*>(v.out) + t * v.ldo + h * V + d) = gu;
+#pragma unroll
+      for (int off = L / 2; off > 0; off >>= 1)
+#pragma unroll
+        for (int j = 0; j < kVec; ++j) ss[j] += __shfl_xor_sync(0xffffffffu, ss[j], off);
+#pragma unroll
+      for (int j = 0; j < kVec; ++j) {
+        const int r = tid / L + j * (NT / L);
+        if (r >= n || d >= V) continue;
+        const float inv = 1.0f / sqrtf(ss[j] / (float)V + v.eps);
+        uint32_t* gi = reinterpret_cast<uint32_t*>(&gates[j]);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const float2 gt = unpack_bf16(gi[e]);
+          const __nv_bfloat162 y = __floats2bfloat162_rn(o[j][2 * e] * inv * w[2 * e] * gt.x, o[j][2 * e + 1] * inv * w[2 * e + 1] * gt.y);
+          gi[e] = *reinterpret_cast<const uint32_t*>(&y);
+        }
+        *reinterpret_cast<uint4*>(reinterpret_cast<bf*>(v.out) + (t_first + (int64_t)c * kC + r) * v.ldo + h * V + d) = gates[j];
+      }
     }
+    if (c + 1 < chunks) store_rows(c + 1);
   }
 #pragma unroll
   for (int j = 0; j < DK / 8; ++j)

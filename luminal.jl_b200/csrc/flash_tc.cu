@@ -93,6 +93,12 @@ __device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
   asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
   return d;
 }
+// the pair (a, a) as a value the compiler keeps instead of rebuilding it from the kernel's parameters
+__device__ __forceinline__ uint64_t keep2(float a) {
+  uint64_t r;
+  asm volatile("mov.b64 %0, {%1, %1};" : "=l"(r) : "f"(a));
+  return r;
+}
 __device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
   uint64_t d;
   asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
@@ -131,8 +137,7 @@ struct FlashExtra {
   int gate_pitch = 0;
   int window = 0;                   // a query sees the last `window` positions (0: all)
   float cap = 0.f;                  // scores pass cap tanh(. / cap) (0: not)
-  int n_poly = 0;                   // 4 or 7: cap tanh(z) log2(e) = z (poly[0] + poly[1] z^2 + ...) for every z that occurs
-  float poly[7] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+  float poly[4] = {0.f, 0.f, 0.f, 0.f};      // WIN 2: cap tanh(z) log2(e) = z (poly[0] + poly[1] z^2 + ...) for every z that occurs
 };
 
 __device__ __forceinline__ void mma_f16_ts(uint32_t tmem_d, uint32_t tmem_a, uint64_t bdesc, uint32_t idesc, uint32_t accumulate) {
@@ -141,8 +146,9 @@ __device__ __forceinline__ void mma_f16_ts(uint32_t tmem_d, uint32_t tmem_a, uin
       "r"(tmem_a), "l"(bdesc), "r"(idesc), "r"(accumulate)
       : "memory");
 }
-// WIN: windows, bounded scores and padded head widths are compiled in; the other models' kernels carry no code of them
-template <int DN, int DR, int DV, bool WIN>
+// WIN: windows, bounded scores and padded head widths are compiled in (2: the bound as a polynomial); the other models' kernels carry no
+// code of them
+template <int DN, int DR, int DV, int WIN>
 __global__ void __launch_bounds__(kThreads, 1)
 flash_tc_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict__ q, const __grid_constant__ CUtensorMap kmap,
                    const __grid_constant__ CUtensorMap vmap, const __grid_constant__ CUtensorMap rmap, const FlashView fv, const FlashExtra ex, int S,
@@ -310,23 +316,26 @@ flash_tc_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict
     // a score in log2 units: s c, or cap tanh(s scale / cap) log2(e) as cap' - 2 cap' / (1 + 2^(s k2)) with cap' = cap log2(e)
     const float capl = WIN ? ex.cap * kLog2e : 0.f, k2 = WIN && ex.cap > 0.f ? 2.0f * c / ex.cap : 0.f;
     auto bounded = [&](float x) { return fmaf(-2.0f * capl, rcp_approx(1.0f + ex2_approx(x * k2)), capl); };
-    // with a bound on the scores: a polynomial on the FMA pipe, which leaves the exp2 unit to the softmax
+    // small scores: a polynomial on the FMA pipe, which leaves the exp2 unit to the softmax.  The coefficients stay in register pairs
     const float kz = WIN && ex.cap > 0.f ? scale / ex.cap : 0.f;
-    auto poly2 = [&](uint64_t s2) {
-      const uint64_t z = mul2(s2, pack2(kz, kz)), u = mul2(z, z);
-      uint64_t p = pack2(ex.poly[3], ex.poly[3]);
-      if (ex.n_poly > 4) {
-        p = pack2(ex.poly[6], ex.poly[6]);
-        p = fma2(p, u, pack2(ex.poly[5], ex.poly[5]));
-        p = fma2(p, u, pack2(ex.poly[4], ex.poly[4]));
-        p = fma2(p, u, pack2(ex.poly[3], ex.poly[3]));
-      }
-      p = fma2(p, u, pack2(ex.poly[2], ex.poly[2]));
-      p = fma2(p, u, pack2(ex.poly[1], ex.poly[1]));
-      p = fma2(p, u, pack2(ex.poly[0], ex.poly[0]));
-      return mul2(z, p);
+    uint64_t pc[4], kz2 = 0ull;
+    if (WIN == 2) {
+      kz2 = keep2(kz);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) pc[i] = keep2(ex.poly[i]);
+    }
+    auto poly2 = [&](uint64_t s2, uint64_t plus) {
+      const uint64_t z = mul2(s2, kz2), u = mul2(z, z);
+      uint64_t p = fma2(pc[3], u, pc[2]);
+      p = fma2(p, u, pc[1]);
+      p = fma2(p, u, pc[0]);
+      return fma2(z, p, plus);
     };
     auto hidden = [&](int key) { return key >= Sk || (causal && key > q_off + qi) || (WIN && ex.window > 0 && key <= q_off + qi - ex.window); };
+    // keys key_lo .. key_lo + key_span are visible to this row
+    const int key_hi = min(Sk - 1, causal ? q_off + qi : Sk - 1), key_lo = WIN && ex.window > 0 ? q_off + qi - ex.window + 1 : 0;
+    const unsigned key_span = (unsigned)max(key_hi - key_lo, 0);      // (rows behind the last query are never stored)
+    const uint64_t k22 = WIN ? pack2(k2, k2) : 0ull, one2 = WIN ? pack2(1.f, 1.f) : 0ull, m2capl2 = WIN ? pack2(-2.f * capl, -2.f * capl) : 0ull;
     float m = -CUDART_INF_F, l = 0.f;
     for (int j = j0; j < nt; ++j) {
       mbar_wait(&s_full[t], (j - j0) & 1, dead, err);          // S(j) is complete, and with it (pipe order) P V(j - 1): O is at rest
@@ -347,7 +356,7 @@ flash_tc_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict
 #pragma unroll
           for (int i = 0; i < 32; ++i) {
             const int key = key0 + qd * 32 + i;
-            if (!hidden(key)) mx4[i & 3] = fmaxf(mx4[i & 3], sv[i]);
+            if (WIN ? (unsigned)(key - key_lo) <= key_span : !hidden(key)) mx4[i & 3] = fmaxf(mx4[i & 3], sv[i]);
           }
         }
       }
@@ -357,8 +366,8 @@ flash_tc_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict
       mx = fmaxf(mx, xch[t][h ^ 1][r]);
       if (WIN && capl > 0.f) {
         if (mx > -CUDART_INF_F) {
-          float z0, z1;
-          if (ex.n_poly) { unpack2(poly2(pack2(mx, mx)), z0, z1); mx = z0; }
+          float z1;
+          if (WIN == 2) unpack2(poly2(pack2(mx, mx), 0ull), mx, z1);
           else mx = bounded(mx);
         }
       }
@@ -396,15 +405,16 @@ flash_tc_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict
           const int key = key0 + qd * 16 + i;
           float x0, x1;
           if (WIN && capl > 0.f) {
-            if (ex.n_poly) {
-              unpack2(add2(poly2(pack2(a0, a1)), negm2), x0, x1);
+            if (WIN == 2 && (i & 2)) {                     // every other pair on the FMA pipe, the others on the exp2 unit
+              unpack2(poly2(pack2(a0, a1), negm2), x0, x1);
             } else {
-              x0 = bounded(a0) + neg_m;
-              x1 = bounded(a1) + neg_m;
+              unpack2(mul2(pack2(a0, a1), k22), x0, x1);
+              unpack2(add2(pack2(ex2_approx(x0), ex2_approx(x1)), one2), x0, x1);
+              unpack2(fma2(pack2(rcp_approx(x0), rcp_approx(x1)), m2capl2, pack2(capl + neg_m, capl + neg_m)), x0, x1);
             }
             if (!inside) {
-              if (hidden(key)) x0 = -CUDART_INF_F;
-              if (hidden(key + 1)) x1 = -CUDART_INF_F;
+              if ((unsigned)(key - key_lo) > key_span) x0 = -CUDART_INF_F;
+              if ((unsigned)(key + 1 - key_lo) > key_span) x1 = -CUDART_INF_F;
             }
           } else {
             if (!inside) {
@@ -479,17 +489,21 @@ flash_tc_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict
 int32_t flash_tc_configure() {
 #define LMB_CFG(DN, DR, DV, WIN) \
   LMB_CUDA(cudaFuncSetAttribute(flash_tc_kernel<DN, DR, DV, WIN>, cudaFuncAttributeMaxDynamicSharedMemorySize, Smem<DN, DR, DV>::total + 1024))
-  LMB_CFG(128, 0, 128, false);
-  LMB_CFG(96, 0, 96, false);
-  LMB_CFG(64, 0, 64, false);
-  LMB_CFG(64, 64, 64, false);
-  LMB_CFG(64, 64, 128, false);
-  LMB_CFG(128, 64, 64, false);
-  LMB_CFG(128, 64, 128, false);
-  LMB_CFG(64, 0, 64, true);
-  LMB_CFG(64, 0, 128, true);
-  LMB_CFG(128, 0, 64, true);
-  LMB_CFG(128, 0, 128, true);
+  LMB_CFG(128, 0, 128, 0);
+  LMB_CFG(96, 0, 96, 0);
+  LMB_CFG(64, 0, 64, 0);
+  LMB_CFG(64, 64, 64, 0);
+  LMB_CFG(64, 64, 128, 0);
+  LMB_CFG(128, 64, 64, 0);
+  LMB_CFG(128, 64, 128, 0);
+  LMB_CFG(64, 0, 64, 1);
+  LMB_CFG(64, 0, 64, 2);
+  LMB_CFG(64, 0, 128, 1);
+  LMB_CFG(64, 0, 128, 2);
+  LMB_CFG(128, 0, 64, 1);
+  LMB_CFG(128, 0, 64, 2);
+  LMB_CFG(128, 0, 128, 1);
+  LMB_CFG(128, 0, 128, 2);
 #undef LMB_CFG
   return LMB200_OK;
 }
@@ -547,7 +561,7 @@ int32_t flash_tc_launch_view(Ctx* ctx, void* out, const void* q, const void* k, 
   ex.Sk = (int)S; ex.dn = ex.dv = (int)D;
   ex.o_b = fv.q_b; ex.o_h = fv.q_h; ex.o_s = fv.q_s;
 #define LMB_FLASH(DD)                                                                                                   \
-  flash_tc_kernel<DD, 0, DD, false><<<grid, kThreads, Smem<DD, 0, DD>::total + 1024, stream>>>(                          \
+  flash_tc_kernel<DD, 0, DD, 0><<<grid, kThreads, Smem<DD, 0, DD>::total + 1024, stream>>>(                          \
       (__nv_bfloat16*)out, (const __nv_bfloat16*)q, kmap, vmap, kmap, fv, ex, (int)S, scale, causal, ctx->dev_err)
   if (D == 128) LMB_FLASH(128);
   else if (D == 96) LMB_FLASH(96);
@@ -585,7 +599,7 @@ int32_t flash_tc_launch_split(Ctx* ctx, void* out, const void* q, const void* k,
   ex.gate = f.gate; ex.gate_pitch = f.gate_pitch;
   const dim3 grid((unsigned)ceil_div(Sq, 2 * kBM), (unsigned)(B * f.H));
 #define LMB_FLASH(DN, DV)                                                                                              \
-  flash_tc_kernel<DN, 64, DV, false><<<grid, kThreads, Smem<DN, 64, DV>::total + 1024, stream>>>(                       \
+  flash_tc_kernel<DN, 64, DV, 0><<<grid, kThreads, Smem<DN, 64, DV>::total + 1024, stream>>>(                       \
       (__nv_bfloat16*)out, (const __nv_bfloat16*)q, kmap, vmap, rmap, fv, ex, (int)Sq, scale, 1, ctx->dev_err)
   if (f.dn <= 64 && f.dv <= 64) LMB_FLASH(64, 64);
   else if (f.dn <= 64) LMB_FLASH(64, 128);
@@ -637,18 +651,18 @@ int32_t flash_tc_launch_window(Ctx* ctx, void* out, const void* q, const void* k
   ex.o_b = f.o_b; ex.o_h = f.o_h; ex.o_s = f.o_s;
   ex.window = f.window; ex.cap = f.cap;
   const double z_max = f.cap > 0.f && f.max_dot > 0.f ? (double)scale * f.max_dot / f.cap : 2.0;
-  if (z_max <= 1.0) {                                           // relative errors about 1e-7 and 3e-8
-    ex.n_poly = z_max <= 0.45 ? 4 : 7;
-    tanh_poly(z_max, ex.n_poly, (double)f.cap * kLog2e, ex.poly);
-  }
+  const bool poly = z_max <= 0.45;                              // four coefficients: an error of 1e-7 of the bound at most
+  if (poly) tanh_poly(z_max, 4, (double)f.cap * kLog2e, ex.poly);
   const dim3 grid((unsigned)ceil_div(Sq, 2 * kBM), (unsigned)(B * f.H));
-#define LMB_FLASH(DN, DV)                                                                                              \
-  flash_tc_kernel<DN, 0, DV, true><<<grid, kThreads, Smem<DN, 0, DV>::total + 1024, stream>>>(                         \
+#define LMB_FLASH(DN, DV, W)                                                                                           \
+  flash_tc_kernel<DN, 0, DV, W><<<grid, kThreads, Smem<DN, 0, DV>::total + 1024, stream>>>(                            \
       (__nv_bfloat16*)out, (const __nv_bfloat16*)q, kmap, vmap, kmap, fv, ex, (int)Sq, scale, 1, ctx->dev_err)
-  if (f.dn <= 64 && f.dv <= 64) LMB_FLASH(64, 64);
-  else if (f.dn <= 64) LMB_FLASH(64, 128);
-  else if (f.dv <= 64) LMB_FLASH(128, 64);
-  else LMB_FLASH(128, 128);
+#define LMB_PICK(DN, DV) do { if (poly) LMB_FLASH(DN, DV, 2); else LMB_FLASH(DN, DV, 1); } while (0)
+  if (f.dn <= 64 && f.dv <= 64) LMB_PICK(64, 64);
+  else if (f.dn <= 64) LMB_PICK(64, 128);
+  else if (f.dv <= 64) LMB_PICK(128, 64);
+  else LMB_PICK(128, 128);
+#undef LMB_PICK
 #undef LMB_FLASH
   ctx->launches++;
   LMB_CUDA(cudaGetLastError());

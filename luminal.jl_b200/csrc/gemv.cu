@@ -951,7 +951,7 @@ __device__ __forceinline__ void post_norm_tile(const GemvParams& p, const unsign
       ss[i] += acc[j][i] * acc[j][i];
     }
   }
-  auto publish = [&](float* slots) {                           // per-CTA sums of ss over the rows
+  auto publish = [&](float* slots, bool flagged) {             // per-CTA sums of ss over the rows
 #pragma unroll
     for (int i = 0; i < 8; ++i) {
       ss[i] += __shfl_xor_sync(0xffffffffu, ss[i], 4);
@@ -963,33 +963,48 @@ __device__ __forceinline__ void post_norm_tile(const GemvParams& p, const unsign
       for (int i = 0; i < 8; ++i) s_red[we * 32 + 8 * lane + i] = ss[i];
     }
     asm volatile("bar.sync 1, 128;\n" ::: "memory");
-    if (e < 32) slots[(size_t)blockIdx.x * 32 + e] = ((s_red[e] + s_red[32 + e]) + s_red[64 + e]) + s_red[96 + e];
-  };
-  publish(p.pn.slots);
-  __threadfence();
-  asm volatile("bar.sync 1, 128;\n" ::: "memory");
-  if (e == 0) {
-    atomicAdd(p.pn.counter, 1u);
-    const long long t0 = clock64();
-    for (;;) {
-      unsigned seen;
-      asm volatile("ld.acquire.gpu.global.u32 %0, [%1];\n" : "=r"(seen) : "l"(p.pn.counter) : "memory");
-      if (seen >= gridDim.x) break;
-      if (clock64() - t0 > kWaitLimit) { if (err) atomicExch(err, 1); break; }
+    if (e < 32) {
+      const float t = ((s_red[e] + s_red[32 + e]) + s_red[64 + e]) + s_red[96 + e];
+      unsigned u = __float_as_uint(t);
+      if (flagged && u == kSlotEmpty) u = 0x7FC00000u;
+      asm volatile("st.relaxed.gpu.global.u32 [%0], %1;\n" ::"l"(slots + (size_t)blockIdx.x * 32 + e), "r"(u) : "memory");
     }
-  }
-  asm volatile("bar.sync 1, 128;\n" ::: "memory");
+  };
+  publish(p.pn.slots, true);
+  if (p.pn.clear)
+    for (int i = blockIdx.x * 32 + (e & 31); i < kPushMaxCtas * 32; i += gridDim.x * 32)
+      if (e < 32) p.pn.clear[i] = __uint_as_float(kSlotEmpty);
   {                                                            // four lanes per sequence, the same sums in every CTA
-    const int b = e >> 2, part = e & 3;
+    const int b = e >> 2, part = e & 3, n = (int)gridDim.x;
     float s = 0.f;
-#pragma unroll 8
-    for (int t = part; t < (int)gridDim.x; t += 4) s += __ldcg(p.pn.slots + t * 32 + b);
+    const long long t0 = clock64();
+    bool late = false;
+    for (int first = part; first < n; first += 32) {           // eight slots in flight
+      unsigned u[8];
+      bool wait = true;
+      while (wait) {
+        wait = false;
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+          u[i] = 0u;
+          if (first + 4 * i < n) asm volatile("ld.relaxed.gpu.global.u32 %0, [%1];\n" : "=r"(u[i]) : "l"(p.pn.slots + (first + 4 * i) * 32 + b) : "memory");
+        }
+#pragma unroll
+        for (int i = 0; i < 8; ++i) wait = wait || u[i] == kSlotEmpty;
+        if (wait && (late || clock64() - t0 > kWaitLimit)) {
+          if (!late && err) atomicExch(err, 1);
+          late = true;
+          wait = false;
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < 8; ++i) s += __uint_as_float(u[i]);
+    }
     s += __shfl_xor_sync(0xffffffffu, s, 1);
     s += __shfl_xor_sync(0xffffffffu, s, 2);
     if (part == 0) s_scale[b] = 1.0f / sqrtf(s / (float)p.rows + p.pn.eps);
   }
   asm volatile("bar.sync 1, 128;\n" ::: "memory");
-  if (e == 0 && atomicAdd(p.pn.counter + 1, 1u) == gridDim.x - 1) { p.pn.counter[0] = 0u; p.pn.counter[1] = 0u; }
   __nv_bfloat16* xg = reinterpret_cast<__nv_bfloat16*>(p.pn.xg);
 #pragma unroll
   for (int i = 0; i < 8; ++i) ss[i] = 0.f;
@@ -1014,7 +1029,7 @@ __device__ __forceinline__ void post_norm_tile(const GemvParams& p, const unsign
         if (8 * bg + i < p.B) p.pn.capture[(size_t)(8 * bg + i) * p.rows + grow] = xv[j][i];
     }
   }
-  if (p.pn.ssq) publish(p.pn.ssq);
+  if (p.pn.ssq) publish(p.pn.ssq, false);
 }
 
 template <int N, bool X>

@@ -64,8 +64,11 @@ struct ResidNorm {
 //   x[row][b] += y / sqrt(mean over the rows of y^2 + eps) * w[row]
 //   xg[b, row] = bf16(x * gain[row])                            (gain NULL: 1)
 //   ssq[cta][b] = sum over this CTA's rows of the new x^2       (NULL: not wanted)
-// The mean needs every row: the CTAs (all resident, one wave) leave their sums in slots[cta][32], count themselves in at counter[0],
-// wait (bounded) for the others and add the slots in CTA order.  counter[0..1] are zero between launches.
+// The mean needs every row: the CTAs (all resident, one wave) leave their sums in slots[cta][32], where every word starts as
+// kSlotEmpty ("not written yet"), read the others' words until none is (bounded) and add them in CTA order: no flag and no fence sit
+// between a sum and its use.  The launch also empties `clear`, the slots of the launch that uses them next: never its own, and the
+// last launch that read them has completed.
+constexpr unsigned kSlotEmpty = 0xFFFFFFFFu;        // a NaN no sum is stored as
 struct PostNorm {
   float* x = nullptr;
   const float* w = nullptr;
@@ -73,8 +76,8 @@ struct PostNorm {
   const float* gain = nullptr;
   float* ssq = nullptr;
   float* capture = nullptr;                // [B][rows] float32 copy of the new residual rows, or NULL
-  float* slots = nullptr;
-  unsigned* counter = nullptr;
+  float* slots = nullptr;                  // [kPushMaxCtas][32]
+  float* clear = nullptr;                  // the same, or NULL
   float eps = 0.f;
 };
 

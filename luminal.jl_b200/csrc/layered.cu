@@ -60,8 +60,7 @@ struct LayeredScratch {
   int64_t prompt_cnt_n = 0;
   std::vector<GemvPlan> p_gu, p_down, p_sg, p_sp, p_lr;
   void *act_ff = nullptr, *act_side = nullptr, *lr_in = nullptr, *qw = nullptr;   // GEMV inputs; prepared queries (CUDA-core attention)
-  float *lr = nullptr, *mix_ssq = nullptr, *post_slots = nullptr;
-  unsigned* post_cnt = nullptr;
+  float *lr = nullptr, *mix_ssq = nullptr, *post_slots = nullptr;                 // post_slots: [3][kPushMaxCtas][32]
   RowsBuf step, prompt;                          // float32 decode step; everything longer
   float* want_logits = nullptr;
   void* want_xn = nullptr;
@@ -1201,6 +1200,11 @@ int32_t fused_post_step(Session* S, cudaStream_t st, bool with_head) {
   LayeredScratch& Z = *S->lay;
   const int B = S->B, hid = M->cfg.hidden, L = M->cfg.n_layers, dt = LMB200_BF16;
   int tiles = 1;                                             // CTAs of the last output projection
+  // Slots of the step's n_post output norms: two sets in turn, and a third for the last of an odd number, so that a launch and the
+  // one after it (the step is replayed) never share a set
+  int n_post = 0, at_post = 0;
+  for (const LayerSpec& s : M->specs) n_post += 1 + (s.c.ff > 0) + (M->side_dim > 0);
+  auto slots = [&](int i) { return Z.post_slots + (int64_t)(n_post % 2 && i == n_post - 1 ? 2 : i & 1) * kPushMaxCtas * 32; };
   // the matrix that follows: its weights are drawn into L2 while this one drains
   struct Next { const void* W = nullptr; const WMap* m = nullptr; const GemvPlan* pl = nullptr; };
   auto launch = [&](GemvParams& p, const Next& nx) -> int32_t {
@@ -1213,7 +1217,10 @@ int32_t fused_post_step(Session* S, cudaStream_t st, bool with_head) {
   auto post = [&](int l, const void* W, const WMap& m, const GemvPlan& pl, const void* x, const float* w, InvScale iv, bool layer_end, const Next& nx) -> int32_t {
     GemvParams p = gemv_params(S, W, m, pl, x);
     p.epi = EPI_POST_NORM; p.inv = iv;
-    p.pn.x = S->xT; p.pn.w = w; p.pn.xg = S->xn; p.pn.slots = Z.post_slots; p.pn.counter = Z.post_cnt; p.pn.eps = M->cfg.rms_eps;
+    p.pn.x = S->xT; p.pn.w = w; p.pn.xg = S->xn; p.pn.eps = M->cfg.rms_eps;
+    p.pn.slots = slots(at_post); p.pn.clear = n_post > 1 ? slots((at_post + 1) % n_post) : nullptr;
+    if (n_post == 1) LMB_CUDA(cudaMemsetAsync(p.pn.slots, 0xFF, (size_t)kPushMaxCtas * 32 * 4, st));
+    ++at_post;
     if (layer_end && S->capture_on) p.pn.capture = S->capture + (int64_t)l * B * hid;
     if (layer_end && l + 1 == L) { p.pn.gain = M->final_norm; p.pn.ssq = S->ssq; }
     tiles = gemv_plan_ctas(pl, m.rows);
@@ -1474,8 +1481,9 @@ int32_t layered_session_create(Model* M, int batch, int max_ctx, lmb200_session*
       alloc(&Z.lr_in, x_bytes(std::max<int64_t>(1, max_over(M, [](const LayerSpec& s) { return s.m_lr.K; }))));
       alloc((void**)&Z.lr, batch * max_over(M, [](const LayerSpec& s) { return s.m_lr.rows; }) * 4);
       alloc((void**)&Z.mix_ssq, max_over(M, [](const LayerSpec& s) { return is_lightning(s) ? s.c.heads : 0; }) * 32 * 4);
-      alloc((void**)&Z.post_slots, (int64_t)kPushMaxCtas * 32 * 4);
-      alloc((void**)&Z.post_cnt, 8);
+      alloc((void**)&Z.post_slots, (int64_t)3 * kPushMaxCtas * 32 * 4);
+      if (rc == LMB200_OK && cudaMemsetAsync(Z.post_slots, 0xFF, (size_t)3 * kPushMaxCtas * 32 * 4, ctx->stream) != cudaSuccess)
+        rc = fail(LMB200_ECUDA, "session_create: memset failed");
       alloc(&Z.qw, batch * qw * 2);
     }
     S->fused = true;
@@ -1525,7 +1533,7 @@ void layered_session_free(Session* S) {
   LayeredScratch& Z = *S->lay;
   cudaFree(Z.proj); cudaFree(Z.qf); cudaFree(Z.xq); cudaFree(Z.qa); cudaFree(Z.iota); cudaFree(Z.ones);
   cudaFree(Z.attn_part); cudaFree(Z.prompt_part); cudaFree(Z.win_cnt); cudaFree(Z.prompt_cnt);
-  cudaFree(Z.act_ff); cudaFree(Z.act_side); cudaFree(Z.lr_in); cudaFree(Z.qw); cudaFree(Z.lr); cudaFree(Z.mix_ssq); cudaFree(Z.post_slots); cudaFree(Z.post_cnt);
+  cudaFree(Z.act_ff); cudaFree(Z.act_side); cudaFree(Z.lr_in); cudaFree(Z.qw); cudaFree(Z.lr); cudaFree(Z.mix_ssq); cudaFree(Z.post_slots);
   cudaFree(Z.want_logits); cudaFree(Z.want_xn); cudaFree(Z.expanded);
   free_rows(Z.step);
   free_rows(Z.prompt);

@@ -279,6 +279,7 @@ __global__ void __launch_bounds__(kThreads) window_split_kernel(const WindowView
   extern __shared__ __align__(16) unsigned char sm_raw[];
   __shared__ float sm_m[4][8], sm_l[4][8];
   __shared__ int is_last;
+  __shared__ float2 s_cs[PREP ? DK / 2 : 1];
   __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(sm_raw);            // [8][PK]
   __nv_bfloat16* ring = sQ + 8 * PK;                                       // [4 warps][kRing][16][PK | PV]
   pdl_launch_dependents();
@@ -331,18 +332,40 @@ __global__ void __launch_bounds__(kThreads) window_split_kernel(const WindowView
   }
   if (PREP) {
     const bool newest = in.k && k_end == pos + 1;
-    for (int u = warp; u < nh + (newest ? 2 : 0); u += 4) {
-      if (u < nh) {
-        norm_head(v, reinterpret_cast<const float*>(in.q) + (int64_t)t * in.q_pitch + (h0 + u) * v.dim, t, pos, lane,
-                  [&](int d, float x) { sQ[u * PK + d] = __float2bfloat16_rn(x); });
-      } else if (u == nh) {
-        __nv_bfloat16* o = K + (int64_t)pos * v.k_ld;
-        norm_head(v, reinterpret_cast<const float*>(in.k) + (int64_t)t * in.k_pitch + a * v.dim, t, pos, lane,
-                  [&](int d, float x) { o[d] = __float2bfloat16_rn(x); });
-      } else {
-        __nv_bfloat16* o = V + (int64_t)pos * v.v_ld;
-        const float* s = reinterpret_cast<const float*>(in.v) + (int64_t)t * in.v_pitch + a * v.vdim;
-        for (int d = lane; d < v.vdim; d += 32) o[d] = __float2bfloat16_rn(s[d]);
+    for (int p = tid; p < (v.rot_dims >> 1); p += kThreads) s_cs[p] = turn(v, t, pos, p, 1.f, 0.f);
+    if (newest) {
+      __nv_bfloat16* o = V + (int64_t)pos * v.v_ld;
+      const float* x = reinterpret_cast<const float*>(in.v) + (int64_t)t * in.v_pitch + a * v.vdim;
+      for (int d = tid; d < v.vdim; d += kThreads) o[d] = __float2bfloat16_rn(x[d]);
+    }
+    __syncthreads();
+    for (int u = warp; u < nh + (newest ? 1 : 0); u += 4) {
+      const float* x = u < nh ? reinterpret_cast<const float*>(in.q) + (int64_t)t * in.q_pitch + (h0 + u) * v.dim
+                              : reinterpret_cast<const float*>(in.k) + (int64_t)t * in.k_pitch + a * v.dim;
+      __nv_bfloat16* o = u < nh ? sQ + u * PK : K + (int64_t)pos * v.k_ld;
+      float2 y[DK / 64];
+      float ss = 0.f;
+#pragma unroll
+      for (int i = 0; i < DK / 64; ++i) {
+        const int p = lane + 32 * i;
+        int lo, hi;
+        pair_of(v, p, &lo, &hi);
+        y[i] = make_float2(lo < v.dim ? x[lo] : 0.f, hi < v.dim ? x[hi] : 0.f);
+        if (p < (v.rot_dims >> 1)) {
+          const float2 cs = s_cs[p];
+          y[i] = make_float2(y[i].x * cs.x - y[i].y * cs.y, y[i].y * cs.x + y[i].x * cs.y);
+        }
+        ss += y[i].x * y[i].x + y[i].y * y[i].y;
+      }
+#pragma unroll
+      for (int off = 16; off > 0; off >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, off);
+      const float inv = 1.0f / sqrtf(ss / (float)v.dim + v.eps);
+#pragma unroll
+      for (int i = 0; i < DK / 64; ++i) {
+        int lo, hi;
+        pair_of(v, lane + 32 * i, &lo, &hi);
+        if (lo < v.dim) o[lo] = __float2bfloat16_rn(y[i].x * inv);
+        if (hi < v.dim) o[hi] = __float2bfloat16_rn(y[i].y * inv);
       }
     }
     __threadfence_block();
