@@ -2,6 +2,7 @@
 #include "activations.cuh"
 #include "delta.cuh"
 #include "pdl.cuh"
+#include "tc.cuh"
 
 namespace lmb {
 namespace {
@@ -74,30 +75,28 @@ __global__ void __launch_bounds__(256) delta_conv_kernel(const DeltaView v, T* _
         if (t >= 0 && r < kBack + n && c < width) ahead[r][i] = *reinterpret_cast<const typename Pair<T>::V*>(src + t * pitch + c);
       }
   }
-  int last = -1;
-  auto token = [&](int r, auto x_of) {
-    const int64_t t = first + r;
-    const int s = __shfl_sync(0xffffffffu, my_seq, r + MAXT - 1), p = __shfl_sync(0xffffffffu, my_pos, r + MAXT - 1);
-    if (s != last) {                       // a run starts, or another sequence: the rows before this one
-      last = s;
+  // the rows before packed row first + r, of sequence s at position p
+  auto history = [&](int r, int s, int p, auto x_of) {
 #pragma unroll
-      for (int j = 1; j < MAXT; ++j) {
-        const bool packed = __shfl_sync(0xffffffffu, my_seq, r + MAXT - 1 - j) == s;      // the row before is in this call too
+    for (int j = 1; j < MAXT; ++j) {
+      const bool packed = __shfl_sync(0xffffffffu, my_seq, r + MAXT - 1 - j) == s;        // the row before is in this call too
 #pragma unroll
-        for (int i = 0; i < NP; ++i) {
-          const int c = 2 * (lane + 32 * i);
-          float2 x = make_float2(0.f, 0.f);
-          if (j < v.taps && p - j >= 0 && c < width) {
-            if (packed) x = x_of(r - j, i, c);
-            else {
-              const float* q = v.ring + ((int64_t)s * v.taps + (p - j) % v.taps) * C + c0 + c;
-              x = make_float2(q[0], c + 1 < width ? q[1] : 0.f);
-            }
+      for (int i = 0; i < NP; ++i) {
+        const int c = 2 * (lane + 32 * i);
+        float2 x = make_float2(0.f, 0.f);
+        if (j < v.taps && p - j >= 0 && c < width) {
+          if (packed) x = x_of(r - j, i, c);
+          else {
+            const float* q = v.ring + ((int64_t)s * v.taps + (p - j) % v.taps) * C + c0 + c;
+            x = make_float2(q[0], c + 1 < width ? q[1] : 0.f);
           }
-          h[j - 1][i] = x;
         }
+        h[j - 1][i] = x;
       }
     }
+  };
+  auto token = [&](int r, auto x_of) {
+    const int64_t t = first + r;
     float ss = 0.f;
     T* o = out + t * C + c0;
 #pragma unroll
@@ -123,10 +122,14 @@ __global__ void __launch_bounds__(256) delta_conv_kernel(const DeltaView v, T* _
     return ss;
   };
   float my_ss = 0.f;                       // lane r: token r's sum
-  if (kAhead && even) {
+  const int s0 = __shfl_sync(0xffffffffu, my_seq, MAXT - 1), p0 = __shfl_sync(0xffffffffu, my_pos, MAXT - 1);
+  const bool one = __all_sync(0xffffffffu, lane < MAXT - 1 || lane >= n + MAXT - 1 || my_seq == s0);
+  if (kAhead && even && one) {
+    auto x_of = [&](int r, int i, int) { return pair_f32(ahead[kBack + r][i]); };
+    history(0, s0, p0, x_of);
     float ss[kRows];
 #pragma unroll
-    for (int r = 0; r < kRows; ++r) ss[r] = r < n ? token(r, [&](int q, int i, int) { return pair_f32(ahead[kBack + q][i]); }) : 0.f;
+    for (int r = 0; r < kRows; ++r) ss[r] = r < n ? token(r, x_of) : 0.f;
     if (kind < 2) {
 #pragma unroll
       for (int r = 0; r < kRows; ++r) {
@@ -135,9 +138,15 @@ __global__ void __launch_bounds__(256) delta_conv_kernel(const DeltaView v, T* _
       }
     }
   } else {
+    auto x_of = [&](int r, int, int c) { return raw(first + r, c); };
+    int last = -1;
+#pragma unroll 1
     for (int r = 0; r < n; ++r) {
-      const float s = warp_sum(token(r, [&](int q, int, int c) { return raw(first + q, c); }));
-      if (lane == r) my_ss = s;
+      const int s = __shfl_sync(0xffffffffu, my_seq, r + MAXT - 1), p = __shfl_sync(0xffffffffu, my_pos, r + MAXT - 1);
+      if (s != last) history(r, s, p, x_of);
+      last = s;
+      const float y = warp_sum(token(r, x_of));
+      if (lane == r) my_ss = y;
     }
   }
   if (kind < 2 && lane < n) {
@@ -166,17 +175,37 @@ __global__ void __launch_bounds__(256) delta_ring_kernel(const DeltaView v) {
 }
 
 // One CTA per (value head, sequence).  Thread (c, w): value columns 4 c .., rows w, w + W, ... of the state.  One pass over the state per
-// token gives both S^T k and S^T q after the decay; with u the written value, o = S^T q + (k . q) u and S <- S + k u^T.  KEEP: the
-// thread's part of the state stays in registers over all tokens.
-constexpr int kStep = 512, kKeep = 8;
+// token gives both S^T k and S^T q after the decay; with u the written value, o = S^T q + (k . q) u and S <- S + k u^T.  KEEP: the state
+// lies in shared memory over all tokens (one bulk copy brings it while the inputs are prepared); else it is read twice per token.
+constexpr int kStep = 256;
+constexpr size_t kKeepMax = 100 * 1024;
+
+struct StepShape {
+  int V4, blocks, W, parts;
+  bool quad;                             // a warp covers 8 column groups x 4 rows: shuffles add four rows, few partial sums meet in shared memory
+};
+__host__ __device__ inline StepShape step_shape(int vdim) {
+  StepShape p;
+  p.V4 = (vdim + 3) >> 2;
+  p.blocks = p.V4 >> 3;
+  p.quad = (p.V4 & 7) == 0 && (kStep / 32) % p.blocks == 0;
+  p.W = p.quad ? kStep / 32 / p.blocks * 4 : kStep / p.V4;
+  p.parts = p.quad ? p.W / 4 : p.W;
+  return p;
+}
+__host__ __device__ inline size_t step_vectors(int dim, const StepShape& p) {        // floats
+  return (size_t)(3 * ((dim + 3) & ~3) + 8 * p.V4 + p.parts * 8 * p.V4);
+}
 
 template <typename IT, typename OT, bool RAW, bool KEEP>
-__global__ void __launch_bounds__(kStep, 2) delta_step_kernel(const DeltaView v) {
-  extern __shared__ float sm[];
+__global__ void __launch_bounds__(kStep, 3) delta_step_kernel(const DeltaView v, int* err) {
+  extern __shared__ __align__(16) float sm[];
   __shared__ float red[kStep / 32], s_dot[3];
-  pdl_launch_dependents();
+  __shared__ __align__(8) uint64_t full;
   const int h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const int D = v.dim, V = v.vdim, V4 = (V + 3) >> 2;
+  const int D = v.dim, V = v.vdim;
+  const StepShape sh = step_shape(V);
+  const int V4 = sh.V4, W = sh.W, parts = sh.parts;
   const int gq = v.H / v.G, a = h / gq;
   float* qs = sm;
   float* ks = qs + ((D + 3) & ~3);
@@ -184,86 +213,68 @@ __global__ void __launch_bounds__(kStep, 2) delta_step_kernel(const DeltaView v)
   float* vs = gs + ((D + 3) & ~3);         // [4 V4] v, then o
   float* us = vs + 4 * V4;                 // [4 V4]
   float* os = us + 4 * V4;                 // [parts][2][4 V4]
-  float4* S = reinterpret_cast<float4*>(v.state) + ((int64_t)b * v.H + h) * D * V4;
-  // quad: a warp covers 8 column groups x 4 rows, so that shuffles add four rows and few partial sums meet in shared memory
-  const int blocks = V4 >> 3;
-  const bool quad = (V4 & 7) == 0 && (kStep / 32) % blocks == 0;
-  const int W = quad ? kStep / 32 / blocks * 4 : kStep / V4, parts = quad ? W / 4 : W;
-  const int c = quad ? (warp % blocks) * 8 + (lane & 7) : tid % V4, w = quad ? warp / blocks * 4 + (lane >> 3) : tid / V4;
+  float4* const state = reinterpret_cast<float4*>(v.state) + ((int64_t)b * v.H + h) * D * V4;
+  float4* const S = KEEP ? reinterpret_cast<float4*>(sm + step_vectors(D, sh)) : state;
+  const int c = sh.quad ? (warp % sh.blocks) * 8 + (lane & 7) : tid % V4, w = sh.quad ? warp / sh.blocks * 4 + (lane >> 3) : tid / V4;
+  if (KEEP && tid == 0) {
+    tc::mbar_init(&full, 1);
+    tc::mbar_init_fence();
+  }
+  pdl_launch_dependents();
   pdl_wait();
   const int n = v.len[b], t0 = v.start[b], p0 = v.pos0[b];
   if (n <= 0) return;
-  // The single raw token of a decoding step: its inputs' loads go out before the state's.  Item tid: one element of q, k, log g or v
-  constexpr int kTaps = 4;
-  const int C = 2 * v.G * D + v.H * V, items = 3 * D + V;
-  const bool early = RAW && v.taps <= kTaps && items <= kStep;
-  const int kind = tid < 3 * D ? tid / D : 3, di = tid - kind * D;
-  const bool owner = h == a * gq;
-  int ch = 0;
-  float raw_x = 0.f, raw_t[kTaps], raw_w[kTaps];
-  float* ring = v.ring + (int64_t)b * v.taps * C;
-  if (early && tid < items) {
-    const int64_t t = t0;
-    if (kind == 2) {
-      raw_x = v.decay[t * v.decay_pitch + h * D + di];
-      raw_t[0] = v.a_log[h];
-      raw_t[1] = v.dt_bias[h * D + di];
-    } else {
-      const int col = kind == 3 ? h * V + di : a * D + di;
-      ch = kind == 0 ? col : kind == 1 ? v.G * D + col : 2 * v.G * D + col;
-      raw_x = kind == 0 ? reinterpret_cast<const float*>(v.q)[t * v.q_pitch + col]
-                        : kind == 1 ? reinterpret_cast<const float*>(v.k)[t * v.k_pitch + col] : reinterpret_cast<const float*>(v.v)[t * v.v_pitch + col];
-#pragma unroll
-      for (int j = 0; j < kTaps; ++j) {
-        raw_w[j] = j < v.taps ? v.conv[(int64_t)j * C + ch] : 0.f;
-        raw_t[j] = j > 0 && j < v.taps && p0 - j >= 0 ? ring[(p0 - j) % v.taps * C + ch] : 0.f;
-      }
-    }
+  if (KEEP && tid == 0) {
+    tc::mbar_expect_tx(&full, (uint32_t)(D * V4 * 16));
+    tc::bulk_g2s(S, state, (uint32_t)(D * V4 * 16), &full);
   }
-  float4 s[kKeep];
-  if (KEEP && w < W) {
-#pragma unroll
-    for (int i = 0; i < kKeep; ++i) s[i] = w + i * W < D ? S[(int64_t)(w + i * W) * V4 + c] : make_float4(0.f, 0.f, 0.f, 0.f);
-  }
+  bool dead = false;
   for (int it = 0; it < n; ++it) {
     const int64_t t = t0 + it;
-    float beta = 0.f;
-    if (early) {
-      if (tid < items) {
-        if (kind == 2) gs[di] = expf(log_decay_f32(raw_x, raw_t[0], raw_t[1]));
-        else {
-          float y = raw_w[0] * raw_x;
+    if (RAW) {
+      const int C = 2 * v.G * D + v.H * V, now = p0 % v.taps, items = 3 * D + 4 * V4;
+      float* ring = v.ring + (int64_t)b * v.taps * C;
+      const bool owner = h == a * gq;
+      // two elements of q, k, log g or v per round; all of their loads go out before any is used
+      for (int i0 = tid; i0 < items; i0 += 2 * kStep) {
+        float x[2], tap[2][4], wgt[2][4];
+        int kind[2], di[2], ch[2];
 #pragma unroll
-          for (int j = 1; j < kTaps; ++j) y = fmaf(raw_w[j], raw_t[j], y);
-          if (kind == 3 || owner) ring[p0 % v.taps * C + ch] = raw_x;     // a slot no tap of this token reads
-          (kind == 0 ? qs : kind == 1 ? ks : vs)[di] = to_f32(from_f32<IT>(silu_f32(y)));
+        for (int e = 0; e < 2; ++e) {
+          const int i = i0 + e * kStep;
+          kind[e] = i >= items ? 4 : i < 3 * D ? i / D : 3;
+          di[e] = i - min(kind[e], 3) * D;
+          ch[e] = 0;
+          x[e] = 0.f;
+          if (kind[e] == 4 || (kind[e] == 3 && di[e] >= V)) continue;
+          if (kind[e] == 2) {
+            x[e] = v.decay[t * v.decay_pitch + h * D + di[e]];
+            tap[e][0] = v.a_log[h];
+            tap[e][1] = v.dt_bias[h * D + di[e]];
+            continue;
+          }
+          const int col = kind[e] == 3 ? h * V + di[e] : a * D + di[e];
+          ch[e] = kind[e] == 0 ? col : kind[e] == 1 ? v.G * D + col : 2 * v.G * D + col;
+          x[e] = reinterpret_cast<const float*>(kind[e] == 0 ? v.q : kind[e] == 1 ? v.k : v.v)[t * (kind[e] == 0 ? v.q_pitch : kind[e] == 1 ? v.k_pitch : v.v_pitch) + col];
+#pragma unroll
+          for (int j = 0; j < 4; ++j) {
+            wgt[e][j] = j < v.taps ? v.conv[(int64_t)j * C + ch[e]] : 0.f;
+            tap[e][j] = j > 0 && j < v.taps && p0 - j >= 0 ? ring[(now - j < 0 ? now - j + v.taps : now - j) * C + ch[e]] : 0.f;
+          }
         }
-      }
-      for (int d = V + tid; d < 4 * V4; d += kStep) vs[d] = 0.f;
-    } else if (RAW) {
-      const int p = p0 + it, now = p % v.taps;
-      for (int i = tid; i < 3 * D + 4 * V4; i += kStep) {       // q, k, log g, v: the taps' loads are independent
-        const int kind = i < 3 * D ? i / D : 3, d = i - kind * D;
-        if (kind == 2) {
-          gs[d] = expf(log_decay_f32(v.decay[t * v.decay_pitch + h * D + d], v.a_log[h], v.dt_bias[h * D + d]));
-          continue;
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          if (kind[e] == 4) continue;
+          if (kind[e] == 2) { gs[di[e]] = expf(log_decay_f32(x[e], tap[e][0], tap[e][1])); continue; }
+          if (kind[e] == 3 && di[e] >= V) { vs[di[e]] = 0.f; continue; }
+          float y = wgt[e][0] * x[e];
+#pragma unroll
+          for (int j = 1; j < 4; ++j) y = fmaf(wgt[e][j], tap[e][j], y);
+          for (int j = 4; j < v.taps; ++j)
+            if (p0 - j >= 0) y = fmaf(v.conv[(int64_t)j * C + ch[e]], ring[(p0 - j) % v.taps * C + ch[e]], y);
+          if (kind[e] == 3 || owner) ring[now * C + ch[e]] = x[e];          // a slot no tap of this token reads
+          (kind[e] == 0 ? qs : kind[e] == 1 ? ks : vs)[di[e]] = to_f32(from_f32<IT>(silu_f32(y)));
         }
-        if (kind == 3 && d >= V) { vs[d] = 0.f; continue; }
-        const int col = kind == 3 ? h * V + d : a * D + d, ch = kind == 0 ? col : kind == 1 ? v.G * D + col : 2 * v.G * D + col;
-        const float x = kind == 0 ? reinterpret_cast<const float*>(v.q)[t * v.q_pitch + col]
-                                  : kind == 1 ? reinterpret_cast<const float*>(v.k)[t * v.k_pitch + col] : reinterpret_cast<const float*>(v.v)[t * v.v_pitch + col];
-        float y = v.conv[ch] * x;
-        int slot = now;
-#pragma unroll 4
-        for (int j = 1; j < v.taps; ++j) {
-          slot = slot == 0 ? v.taps - 1 : slot - 1;
-          if (p - j >= 0) y = fmaf(v.conv[(int64_t)j * C + ch], ring[slot * C + ch], y);
-        }
-        if (kind == 3 || owner) ring[now * C + ch] = x;         // a slot no tap of this token reads
-        const float r = to_f32(from_f32<IT>(silu_f32(y)));
-        if (kind == 0) qs[d] = r;
-        else if (kind == 1) ks[d] = r;
-        else vs[d] = r;
       }
     } else {
       const IT* q = reinterpret_cast<const IT*>(v.q) + t * v.q_pitch + a * D;
@@ -276,8 +287,9 @@ __global__ void __launch_bounds__(kStep, 2) delta_step_kernel(const DeltaView v)
       }
       for (int d = tid; d < 4 * V4; d += kStep) vs[d] = d < V ? to_f32(x[d]) : 0.f;
     }
-    beta = sigmoid_f32(v.b[t * v.b_pitch + h]);
+    const float beta = sigmoid_f32(v.b[t * v.b_pitch + h]);
     __syncthreads();
+    if (KEEP && it == 0) tc::mbar_wait(&full, 0, dead, err);
     // the vectors stay unscaled in shared memory; their scales multiply the sums
     if (warp < 3) {
       float x = 0.f;
@@ -287,23 +299,15 @@ __global__ void __launch_bounds__(kStep, 2) delta_step_kernel(const DeltaView v)
     }
     float4 ak = make_float4(0.f, 0.f, 0.f, 0.f), aq = ak;
     if (w < W) {
-      auto row = [&](int d, float4& x) {
+#pragma unroll 4
+      for (int d = w; d < D; d += W) {
+        float4 x = S[(int64_t)d * V4 + c];
         const float g = gs[d], kd = ks[d], qd = qs[d];
         x.x *= g; x.y *= g; x.z *= g; x.w *= g;
         ak.x = fmaf(kd, x.x, ak.x); ak.y = fmaf(kd, x.y, ak.y); ak.z = fmaf(kd, x.z, ak.z); ak.w = fmaf(kd, x.w, ak.w);
         aq.x = fmaf(qd, x.x, aq.x); aq.y = fmaf(qd, x.y, aq.y); aq.z = fmaf(qd, x.z, aq.z); aq.w = fmaf(qd, x.w, aq.w);
-      };
-      if (KEEP) {
-#pragma unroll
-        for (int i = 0; i < kKeep; ++i)
-          if (w + i * W < D) row(w + i * W, s[i]);
-      } else {
-        for (int d = w; d < D; d += W) {
-          float4 x = S[(int64_t)d * V4 + c];
-          row(d, x);
-        }
       }
-      if (quad) {
+      if (sh.quad) {
 #pragma unroll
         for (int off = 8; off < 32; off <<= 1) {
           ak.x += __shfl_xor_sync(0xffffffffu, ak.x, off); ak.y += __shfl_xor_sync(0xffffffffu, ak.y, off);
@@ -312,8 +316,8 @@ __global__ void __launch_bounds__(kStep, 2) delta_step_kernel(const DeltaView v)
           aq.z += __shfl_xor_sync(0xffffffffu, aq.z, off); aq.w += __shfl_xor_sync(0xffffffffu, aq.w, off);
         }
       }
-      if (!quad || lane < 8) {
-        const int part = quad ? w >> 2 : w;
+      if (!sh.quad || lane < 8) {
+        const int part = sh.quad ? w >> 2 : w;
         *reinterpret_cast<float4*>(os + (part * 2) * 4 * V4 + 4 * c) = ak;
         *reinterpret_cast<float4*>(os + (part * 2 + 1) * 4 * V4 + 4 * c) = aq;
       }
@@ -341,22 +345,14 @@ __global__ void __launch_bounds__(kStep, 2) delta_step_kernel(const DeltaView v)
     const float inv = 1.0f / sqrtf(tot / (float)V + v.eps);
     if (w < W) {
       const float4 u = *reinterpret_cast<const float4*>(us + 4 * c);
-      if (KEEP) {
-#pragma unroll
-        for (int i = 0; i < kKeep; ++i) {
-          const int d = w + i * W;
-          if (d >= D) continue;
-          const float kd = ks[d];
-          s[i].x = fmaf(kd, u.x, s[i].x); s[i].y = fmaf(kd, u.y, s[i].y); s[i].z = fmaf(kd, u.z, s[i].z); s[i].w = fmaf(kd, u.w, s[i].w);
-          if (it == n - 1) S[(int64_t)d * V4 + c] = s[i];
-        }
-      } else {
-        for (int d = w; d < D; d += W) {
-          float4 x = S[(int64_t)d * V4 + c];
-          const float g = gs[d], kd = ks[d];
-          x.x = fmaf(kd, u.x, g * x.x); x.y = fmaf(kd, u.y, g * x.y); x.z = fmaf(kd, u.z, g * x.z); x.w = fmaf(kd, u.w, g * x.w);
-          S[(int64_t)d * V4 + c] = x;
-        }
+      const bool leave = it == n - 1;
+#pragma unroll 4
+      for (int d = w; d < D; d += W) {
+        float4 x = S[(int64_t)d * V4 + c];
+        const float g = gs[d], kd = ks[d];
+        x.x = fmaf(kd, u.x, g * x.x); x.y = fmaf(kd, u.y, g * x.y); x.z = fmaf(kd, u.z, g * x.z); x.w = fmaf(kd, u.w, g * x.w);
+        if (KEEP && leave) state[(int64_t)d * V4 + c] = x;
+        else S[(int64_t)d * V4 + c] = x;
       }
     }
     OT* out = reinterpret_cast<OT*>(v.out);
@@ -389,7 +385,13 @@ int32_t conv_launch(const DeltaView& v, T* out, float* rq, float* rk, cudaStream
 
 }  // namespace
 
-int32_t delta_configure() { return delta_chunk_configure(); }
+int32_t delta_configure() {
+  typedef __nv_bfloat16 bf16;
+  LMB_CUDA(cudaFuncSetAttribute(delta_step_kernel<bf16, bf16, true, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kKeepMax));
+  LMB_CUDA(cudaFuncSetAttribute(delta_step_kernel<bf16, bf16, false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kKeepMax));
+  LMB_CUDA(cudaFuncSetAttribute(delta_step_kernel<float, float, false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kKeepMax));
+  return delta_chunk_configure();
+}
 
 int32_t delta_conv(Ctx* ctx, int dtype, const DeltaView& v, void* out, float* rq, float* rk, cudaStream_t st) {
   LMB_TRY(check(v));
@@ -400,16 +402,17 @@ int32_t delta_conv(Ctx* ctx, int dtype, const DeltaView& v, void* out, float* rq
 
 int32_t delta_steps(Ctx* ctx, int dtype, const DeltaView& v, cudaStream_t st) {
   LMB_TRY(check(v));
-  const int V4 = (v.vdim + 3) >> 2, blocks = V4 >> 3, W = (V4 & 7) == 0 && (kStep / 32) % blocks == 0 ? kStep / 32 / blocks * 4 : kStep / V4;
-  const size_t smem = (size_t)(3 * ((v.dim + 3) & ~3) + 8 * V4 + W * 8 * V4) * 4;
-  const bool keep = v.dim <= W * kKeep, bf = dtype == LMB200_BF16;
+  const StepShape sh = step_shape(v.vdim);
+  const size_t vectors = step_vectors(v.dim, sh) * 4, whole = vectors + (size_t)v.dim * sh.V4 * 16;
+  const bool keep = whole <= kKeepMax, bf = dtype == LMB200_BF16;
+  const size_t smem = keep ? whole : vectors;
   const dim3 grid((unsigned)v.H, (unsigned)v.B);
   typedef __nv_bfloat16 bf16;
-  if (bf && v.raw) LMB_CUDA(launch_k(keep ? delta_step_kernel<bf16, bf16, true, true> : delta_step_kernel<bf16, bf16, true, false>, grid, dim3(kStep), smem, st, v));
-  else if (bf) LMB_CUDA(launch_k(keep ? delta_step_kernel<bf16, bf16, false, true> : delta_step_kernel<bf16, bf16, false, false>, grid, dim3(kStep), smem, st, v));
+  if (bf && v.raw) LMB_CUDA(launch_k(keep ? delta_step_kernel<bf16, bf16, true, true> : delta_step_kernel<bf16, bf16, true, false>, grid, dim3(kStep), smem, st, v, ctx->dev_err));
+  else if (bf) LMB_CUDA(launch_k(keep ? delta_step_kernel<bf16, bf16, false, true> : delta_step_kernel<bf16, bf16, false, false>, grid, dim3(kStep), smem, st, v, ctx->dev_err));
   else {
     LMB_REQUIRE(!v.raw, "delta rule: float32 models prepare their rows");
-    LMB_CUDA(launch_k(keep ? delta_step_kernel<float, float, false, true> : delta_step_kernel<float, float, false, false>, grid, dim3(kStep), smem, st, v));
+    LMB_CUDA(launch_k(keep ? delta_step_kernel<float, float, false, true> : delta_step_kernel<float, float, false, false>, grid, dim3(kStep), smem, st, v, ctx->dev_err));
   }
   ctx->launches++;
   return LMB200_OK;

@@ -497,18 +497,30 @@ __global__ void __launch_bounds__(kThreads) window_split_kernel(const WindowView
   __syncthreads();
   if (!is_last) return;
   __threadfence();
+  // weights of the parts, then their weighted sum
+  float* wt = reinterpret_cast<float*>(ring);           // [nvalid][8]
+  for (int h = warp; h < nh; h += 4) {
+    float M = -CUDART_INF_F;
+    for (int sp = lane; sp < nvalid; sp += 32) M = fmaxf(M, __ldcg(part_ml + ((slot0 + sp) * 8 + h) * 2));
+#pragma unroll
+    for (int off = 16; off > 0; off >>= 1) M = fmaxf(M, __shfl_xor_sync(0xffffffffu, M, off));
+    float den = 0.f;
+    for (int sp = lane; sp < nvalid; sp += 32) {
+      const float w = exp2f((__ldcg(part_ml + ((slot0 + sp) * 8 + h) * 2) - M) * kLog2e);
+      wt[sp * 8 + h] = w;
+      den += w * __ldcg(part_ml + ((slot0 + sp) * 8 + h) * 2 + 1);
+    }
+#pragma unroll
+    for (int off = 16; off > 0; off >>= 1) den += __shfl_xor_sync(0xffffffffu, den, off);
+    if (lane == 0) sm_l[0][h] = 1.0f / den;
+  }
+  __syncthreads();
   for (int i = tid; i < nh * v.vdim; i += kThreads) {
     const int h = i / v.vdim, d = i - h * v.vdim;
-    float M = -CUDART_INF_F;
-    for (int sp = 0; sp < nvalid; ++sp) M = fmaxf(M, __ldcg(part_ml + ((slot0 + sp) * 8 + h) * 2));
-    float acc = 0.f, den = 0.f;
-#pragma unroll 4
-    for (int sp = 0; sp < nvalid; ++sp) {
-      const float wgt = exp2f((__ldcg(part_ml + ((slot0 + sp) * 8 + h) * 2) - M) * kLog2e);
-      den += wgt * __ldcg(part_ml + ((slot0 + sp) * 8 + h) * 2 + 1);
-      acc += wgt * __ldcg(part_o + ((slot0 + sp) * 8 + h) * v.vdim + d);
-    }
-    put(h, d, acc / den);
+    float acc = 0.f;
+#pragma unroll 8
+    for (int sp = 0; sp < nvalid; ++sp) acc += wt[sp * 8 + h] * __ldcg(part_o + ((slot0 + sp) * 8 + h) * v.vdim + d);
+    put(h, d, acc * sm_l[0][h]);
   }
 }
 
