@@ -390,7 +390,8 @@ int32_t delta_configure() {
   LMB_CUDA(cudaFuncSetAttribute(delta_step_kernel<bf16, bf16, true, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kKeepMax));
   LMB_CUDA(cudaFuncSetAttribute(delta_step_kernel<bf16, bf16, false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kKeepMax));
   LMB_CUDA(cudaFuncSetAttribute(delta_step_kernel<float, float, false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kKeepMax));
-  return delta_chunk_configure();
+  LMB_TRY(delta_chunk_configure());
+  return delta_tc_configure();
 }
 
 int32_t delta_conv(Ctx* ctx, int dtype, const DeltaView& v, void* out, float* rq, float* rk, cudaStream_t st) {

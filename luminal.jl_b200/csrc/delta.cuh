@@ -47,5 +47,9 @@ int32_t delta_steps(Ctx* ctx, int dtype, const DeltaView& v, cudaStream_t st);
 bool delta_chunks_ok(const DeltaView& v);
 int32_t delta_chunks(Ctx* ctx, const DeltaView& v, cudaStream_t st);
 int32_t delta_chunk_configure();
+// the same with tcgen05 (csrc/delta_tc.cu), for heads wider than 64
+bool delta_tc_ok(const DeltaView& v);
+int32_t delta_tc(Ctx* ctx, const DeltaView& v, cudaStream_t st);
+int32_t delta_tc_configure();
 
 }  // namespace lmb

@@ -1,0 +1,650 @@
+// Channel-wise gated delta rule over long portions on the fifth-generation tensor cores: the algorithm of csrc/delta_chunk.cu (chunks of
+// 64 tokens; kt, qt, kb, A, B as defined there) with its products on tcgen05.mma and the state in tensor memory.
+//
+// One CTA per (value head, sequence).  Everything is transposed: the 128 lanes of tensor memory are value columns.  Per chunk
+//   [Y | O]^T = S^T [kt | qt]^T        S^T from tensor memory as bf16 pairs hi | lo, kt and qt hi and lo in shared memory
+//   X = beta (V - Y),  U^T = X^T T^T   T = (I + A)^-1, 64 x 64
+//   O^T += U^T B^T,   S^T = S^T diag(e^{G_end}) + U^T kb
+// every product as hi hi + lo hi + hi lo (x = hi + lo to about 2^-17), accumulated in float32.
+// Tensor memory columns: [Y then U | O] 128, S 128, [S hi | S lo, later X hi | X lo] 128, [U hi | U lo] 64.
+// Warps: 0-7 own the value columns (two threads per column): they turn S, X and U into operands and write the outputs; 8-15 prepare the
+// next chunk (decay sums, kt, qt, kb; A and B with mma.sync; T in float32) while the others work on this one; 16 issues the
+// MMAs, 17 the row copies.  All waits are bounded.
+#include "delta.cuh"
+#include "mma_sync.cuh"
+#include "pdl.cuh"
+#include "tc.cuh"
+
+namespace lmb {
+namespace {
+
+constexpr int kC = 64, kW = 128;                        // tokens per chunk; head width, padded with zeros
+constexpr float kLog2e = 1.4426950408889634f;
+constexpr float kDiagMax = 80.0f, kDecayMin = -150.0f;  // as in csrc/delta_chunk.cu
+constexpr int kThreads = 18 * 32;
+constexpr uint32_t cYO = 0, cS = 128, cSh = 256, cSl = 320, cXh = 256, cXl = 288, cUh = 384, cUl = 416;
+constexpr int kPk = kW + 8, kPg = kW + 4, kPt = 66;     // row pitches: raw rows, decay sums, float32 A and T
+// shared memory; tiles in the 128-byte swizzle
+constexpr int kSub = 128 * 128, kSubKb = 64 * 128;      // sub-tiles [128 rows][64 columns], [64 rows][64 columns]
+constexpr int oKQh = 0, oKQl = oKQh + 2 * kSub;         // rows 0-63 kt, 64-127 qt
+constexpr int oKbh = oKQl + 2 * kSub, oKbl = oKbh + 2 * kSubKb;
+constexpr int oTh = oKbl + 2 * kSubKb, oTl = oTh + kSubKb, oBh = oTl + kSubKb, oBl = oBh + kSubKb;
+constexpr int oK = oBl + kSubKb, oQ = oK + kC * kPk * 2, oV = oQ + kC * kPk * 2;          // raw rows; mild chunks: k e^{-G} hi over K, lo over Q
+constexpr int oG = oV + kC * kPk * 2;                   // decay sums; later A and T in float32
+constexpr int oEnd = oG + kC * kPg * 4;
+static_assert(2 * kC * kPt * 4 <= kC * kPg * 4, "A and T fit over the decay sums");
+struct Tail {
+  uint64_t raw_full, raw_empty, v_full, v_empty, kq_ready, tb_ready, s_ready, x_ready, u_ready, yo_done, u_done, o_done, s_done;
+  uint32_t tmem;
+  alignas(16) float R[5][kW];                                       // decay sums before blocks 1 .. 3 of 16 tokens, and of the whole chunk
+  alignas(16) float E[2][kW];                                       // e^{G_end}, by chunk parity
+  float row[2][3][kC];                                  // beta, 1 / |k|, 1 / |q| / sqrt(dim), by chunk parity
+  float sum[4][kC];                                     // sums of squares of the outputs per 32 value columns
+};
+constexpr size_t kSmem = (size_t)oEnd + sizeof(Tail);
+static_assert(kSmem <= 227 * 1024 && oEnd % 16 == 0, "shared memory");
+
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ uint64_t desc(uint32_t saddr, uint32_t lbo, uint32_t sbo) {       // 128-byte swizzle
+  return (uint64_t)((saddr & 0x3FFFF) >> 4) | ((uint64_t)(lbo >> 4) << 16) | ((uint64_t)(sbo >> 4) << 32) | (1ull << 46) | (2ull << 61);
+}
+__device__ __forceinline__ void mma_ts(uint32_t d, uint32_t a, uint64_t b, uint32_t idesc, uint32_t acc) {        // A from tensor memory
+  asm volatile(
+      "{\n.reg .pred p;\nsetp.ne.b32 p, %4, 0;\ntcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n}\n" ::"r"(d), "r"(a), "l"(b), "r"(idesc), "r"(acc)
+      : "memory");
+}
+// byte of (row, column) in a swizzled tile of sub-tiles `sub` bytes apart
+__device__ __forceinline__ int swz(int row, int col, int sub) { return (col >> 6) * sub + row * 128 + ((((col & 63) >> 3) ^ (row & 7)) << 4) + (col & 7) * 2; }
+__device__ __forceinline__ void prep_sync() { asm volatile("bar.sync 3, 256;\n" ::: "memory"); }
+
+__global__ void __launch_bounds__(kThreads, 1) delta_tc_kernel(const DeltaView v, int* err) {
+  using namespace tc;
+  typedef __nv_bfloat16 bf;
+  extern __shared__ __align__(1024) unsigned char smem[];
+  Tail& tl = *reinterpret_cast<Tail*>(smem + oEnd);
+  bf *sK = (bf*)(smem + oK), *sQ = (bf*)(smem + oQ), *sV = (bf*)(smem + oV);
+  float* sG = (float*)(smem + oG);
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int h = blockIdx.x, b = blockIdx.y, D = v.dim, V = v.vdim, ld = (V + 3) & ~3, a = h / (v.H / v.G);
+  if (tid == 0) {
+    if (smem_u32(smem) & 1023) atomicExch(err, 1);       // the swizzle needs 1024-byte tiles
+    mbar_init(&tl.raw_full, 1); mbar_init(&tl.v_full, 1); mbar_init(&tl.yo_done, 1); mbar_init(&tl.u_done, 1); mbar_init(&tl.o_done, 1); mbar_init(&tl.s_done, 1);
+    mbar_init(&tl.raw_empty, 8); mbar_init(&tl.v_empty, 8); mbar_init(&tl.kq_ready, 8); mbar_init(&tl.tb_ready, 8);
+    mbar_init(&tl.s_ready, 8); mbar_init(&tl.x_ready, 8); mbar_init(&tl.u_ready, 8);
+    mbar_init_fence();
+  }
+  // what lies behind the widths and above the triangles stays zero
+  for (int i = tid; i < (oG - oTh) / 16; i += kThreads) reinterpret_cast<uint4*>(smem + oTh)[i] = make_uint4(0, 0, 0, 0);
+  fence_async_smem();
+  if (warp == 16) tmem_alloc(&tl.tmem, 512);
+  fence_before();
+  __syncthreads();
+  fence_after();
+  const uint32_t tmem = tl.tmem;
+  pdl_launch_dependents();
+  pdl_wait();
+  bool dead = false;
+  const int n_all = v.len[b], t_first = v.start[b];
+  const int chunks = (n_all + kC - 1) / kC;              // 0: nothing to do
+
+  if (warp == 17) {
+    // ------------------------------ rows of k, q and v ------------------------------
+    for (int c = 0; c < chunks; ++c) {
+      const int64_t t0 = t_first + (int64_t)c * kC;
+      const int n = min(kC, n_all - c * kC);             // behind the portion's end the last row again: its beta and decay are zero
+      mbar_wait(&tl.raw_empty, (c & 1) ^ 1, dead, err);
+      if (lane == 0) mbar_expect_tx(&tl.raw_full, (uint32_t)(2 * kC * D * 2));
+      __syncwarp();
+      for (int r = lane; r < kC; r += 32) {
+        const int64_t t = t0 + min(r, n - 1);
+        bulk_g2s(sK + r * kPk, reinterpret_cast<const bf*>(v.k) + t * v.k_pitch + a * D, (uint32_t)D * 2, &tl.raw_full);
+        bulk_g2s(sQ + r * kPk, reinterpret_cast<const bf*>(v.q) + t * v.q_pitch + a * D, (uint32_t)D * 2, &tl.raw_full);
+      }
+      mbar_wait(&tl.v_empty, (c & 1) ^ 1, dead, err);
+      if (lane == 0) mbar_expect_tx(&tl.v_full, (uint32_t)(kC * V * 2));
+      __syncwarp();
+      for (int r = lane; r < kC; r += 32)
+        bulk_g2s(sV + r * kPk, reinterpret_cast<const bf*>(v.v) + (t0 + min(r, n - 1)) * v.v_pitch + h * V, (uint32_t)V * 2, &tl.v_full);
+    }
+  } else if (warp == 16) {
+    // ------------------------------ MMA issue ------------------------------
+    constexpr uint32_t kN128 = idesc_bf16(128, 128, false, false), kN64 = idesc_bf16(128, 64, false, false), kN128m = idesc_bf16(128, 128, false, true);
+    const uint32_t base = smem_u32(smem);
+    for (int c = 0; c < chunks; ++c) {
+      mbar_wait(&tl.kq_ready, c & 1, dead, err);
+      mbar_wait(&tl.s_ready, c & 1, dead, err);
+      fence_after();
+      if (lane == 0) {
+#pragma unroll
+        for (int p = 0; p < 3; ++p)                      // hi hi, lo hi, hi lo
+          for (int ks = 0; ks < 8; ++ks)
+            mma_ts(tmem + cYO, tmem + (p == 1 ? cSl : cSh) + ks * 8, desc(base + (p == 2 ? oKQl : oKQh) + (ks >> 2) * kSub + (ks & 3) * 32, 16, 1024), kN128, p | ks ? 1u : 0u);
+        commit(&tl.yo_done);
+      }
+      __syncwarp();
+      mbar_wait(&tl.tb_ready, c & 1, dead, err);
+      mbar_wait(&tl.x_ready, c & 1, dead, err);
+      fence_after();
+      if (lane == 0) {
+#pragma unroll
+        for (int p = 0; p < 3; ++p)
+          for (int ks = 0; ks < 4; ++ks)
+            mma_ts(tmem + cYO, tmem + (p == 1 ? cXl : cXh) + ks * 8, desc(base + (p == 2 ? oTl : oTh) + ks * 32, 16, 1024), kN64, p | ks ? 1u : 0u);
+        commit(&tl.u_done);
+      }
+      __syncwarp();
+      mbar_wait(&tl.u_ready, c & 1, dead, err);
+      fence_after();
+      if (lane == 0) {
+#pragma unroll
+        for (int p = 0; p < 3; ++p)
+          for (int ks = 0; ks < 4; ++ks)
+            mma_ts(tmem + cYO + 64, tmem + (p == 1 ? cUl : cUh) + ks * 8, desc(base + (p == 2 ? oBl : oBh) + ks * 32, 16, 1024), kN64, 1u);
+        commit(&tl.o_done);
+#pragma unroll
+        for (int p = 0; p < 3; ++p)
+          for (int ks = 0; ks < 4; ++ks)
+            mma_ts(tmem + cS, tmem + (p == 1 ? cUl : cUh) + ks * 8, desc(base + (p == 2 ? oKbl : oKbh) + ks * 2048, kSubKb, 1024), kN128m, 1u);
+        commit(&tl.s_done);
+      }
+      __syncwarp();
+    }
+  } else if (warp >= 8) {
+    // ------------------------------ preparation of a chunk ------------------------------
+    const int pt = tid - 256, pw = warp - 8, g = lane >> 2, tq = lane & 3;
+    const int ch = pt >> 1, hf = pt & 1;                 // decay sums: channel, half of the chunk
+    float gl[32];                                        // its log decays
+    float rb = 0.f, rk_ = 0.f, rq_ = 0.f;
+    auto fetch = [&](int c) {
+      const int64_t t0 = t_first + (int64_t)c * kC;
+      const int n = min(kC, n_all - c * kC);
+#pragma unroll
+      for (int r = 0; r < 32; ++r) gl[r] = ch < D && hf * 32 + r < n ? __ldg(v.decay + (t0 + hf * 32 + r) * v.decay_pitch + h * D + ch) : 0.f;
+      if (pt < kC) {
+        const bool ok = pt < n;
+        rb = ok ? v.b[(t0 + pt) * v.b_pitch + h] : 0.f;
+        rk_ = ok ? v.rk[(t0 + pt) * v.G + a] : 0.f;
+        rq_ = ok ? v.rq[(t0 + pt) * v.G + a] : 0.f;
+      }
+    };
+    if (chunks > 0) fetch(0);
+    for (int c = 0; c < chunks; ++c) {
+      const int n = min(kC, n_all - c * kC);
+      float *beta = tl.row[c & 1][0], *rk = tl.row[c & 1][1], *rq = tl.row[c & 1][2], *E = tl.E[c & 1];
+      // ---- decay sums (log2 units): in sG from the start of each block of 16 tokens, in R before the block
+      if (pt < kC) {
+        beta[pt] = pt < n ? 1.0f / (1.0f + expf(-rb)) : 0.f;
+        rk[pt] = rk_;
+        rq[pt] = rq_;
+      }
+      float tot[2];
+#pragma unroll
+      for (int q = 0; q < 2; ++q) {
+        float s = 0.f;
+#pragma unroll
+        for (int r = 0; r < 16; ++r) {
+          s += fmaxf(gl[q * 16 + r] * kLog2e, kDecayMin);
+          sG[(hf * 32 + q * 16 + r) * kPg + ch] = s;
+        }
+        tot[q] = s;
+      }
+      const float mine = tot[0] + tot[1], other = __shfl_xor_sync(0xffffffffu, mine, 1), before = hf ? other : 0.f;
+      if (hf) tl.R[2][ch] = before;
+      tl.R[hf ? 3 : 1][ch] = before + tot[0];
+      const float all = hf ? other + mine : mine + other;
+      if (!hf) {
+        tl.R[4][ch] = all;
+        E[ch] = ex2(all);
+      }
+      mbar_wait(&tl.raw_full, c & 1, dead, err);
+      int mild;
+      {                                                  // bar.red over the preparing warps
+        int p = all >= -kDiagMax;
+        asm volatile("{\n.reg .pred p, q;\nsetp.ne.s32 p, %1, 0;\nbarrier.red.and.pred q, 3, 256, p;\nselp.s32 %0, 1, 0, q;\n}\n" : "=r"(mild) : "r"(p) : "memory");
+      }
+      // ---- kt, qt (and k e^{-G} over the raw rows)
+      if (c) mbar_wait(&tl.yo_done, (c - 1) & 1, dead, err);
+#pragma unroll 2
+      for (int i = pt; i < kC * (kW / 4); i += 256) {
+        const int r = i >> 5, d = (i & 31) * 4, at = r * kPk + d;
+        const float4 L = *reinterpret_cast<const float4*>(sG + r * kPg + d);
+        const float4 Rv = r < 16 ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4*>(&tl.R[r >> 4][d]);
+        const uint2 ku = *reinterpret_cast<const uint2*>(sK + at), qu = *reinterpret_cast<const uint2*>(sQ + at);
+        const float2 k0 = unpack_bf16(ku.x), k1 = unpack_bf16(ku.y), q0 = unpack_bf16(qu.x), q1 = unpack_bf16(qu.y);
+        const float kr = rk[r], qr = rq[r];
+        const float G[4] = {Rv.x + L.x, Rv.y + L.y, Rv.z + L.z, Rv.w + L.w};
+        const float k[4] = {k0.x * kr, k0.y * kr, k1.x * kr, k1.y * kr}, q[4] = {q0.x * qr, q0.y * qr, q1.x * qr, q1.y * qr};
+        float e[4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) e[j] = ex2(G[j]);
+        const int to = swz(r, d, kSub);
+        uint2 hi, lo;
+        split2(k[0] * e[0], k[1] * e[1], hi.x, lo.x);
+        split2(k[2] * e[2], k[3] * e[3], hi.y, lo.y);
+        *reinterpret_cast<uint2*>(smem + oKQh + to) = hi;
+        *reinterpret_cast<uint2*>(smem + oKQl + to) = lo;
+        split2(q[0] * e[0], q[1] * e[1], hi.x, lo.x);
+        split2(q[2] * e[2], q[3] * e[3], hi.y, lo.y);
+        *reinterpret_cast<uint2*>(smem + oKQh + to + 64 * 128) = hi;
+        *reinterpret_cast<uint2*>(smem + oKQl + to + 64 * 128) = lo;
+        if (mild) {
+          split2(k[0] * ex2(-G[0]), k[1] * ex2(-G[1]), hi.x, lo.x);
+          split2(k[2] * ex2(-G[2]), k[3] * ex2(-G[3]), hi.y, lo.y);
+          *reinterpret_cast<uint2*>(sK + at) = hi;
+          *reinterpret_cast<uint2*>(sQ + at) = lo;
+        }
+      }
+      fence_async_smem();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&tl.kq_ready);
+      prep_sync();
+      // ---- blocks of A and B, kept in registers: first one block per warp (0-3 on the diagonal), then the A or the B part of two more
+      auto block_of = [](int task, int* rt, int* st) {
+        const int off = task - 4;
+        *rt = task < 4 ? task : off == 0 ? 1 : off < 3 ? 2 : 3;
+        *st = task < 4 ? task : off == 0 ? 0 : off < 3 ? off - 1 : off - 3;
+      };
+      auto block = [&](int rt, int st, bool do_a, bool do_b, float (&ca)[2][4], float (&cb)[2][4]) {
+#pragma unroll
+        for (int j = 0; j < 2; ++j)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) ca[j][e] = cb[j][e] = 0.f;
+        if (16 * rt >= n) return;
+        const bool diag = rt == st;
+        if (mild) {
+          const int ra = rt * 16 + (lane & 15);
+          const uint32_t k2h = smem_addr(sK + (st * 16 + (lane & 7) + ((lane >> 4) << 3)) * kPk + ((lane >> 3) & 1) * 8), k2l = k2h + (uint32_t)(oQ - oK);
+          const uint32_t kq = smem_addr(smem + oKQh) + ra * 128;
+          float c1[2][4], c2[2][4];                      // the three products on accumulators of their own: short chains
+#pragma unroll
+          for (int part = 0; part < 2; ++part) {
+            if (part == 0 ? !do_a : !do_b) continue;
+            float (&cc)[2][4] = part == 0 ? ca : cb;
+#pragma unroll
+            for (int j = 0; j < 2; ++j)
+#pragma unroll
+              for (int e = 0; e < 4; ++e) c1[j][e] = c2[j][e] = 0.f;
+#pragma unroll 4
+            for (int kk = 0; kk < 8; ++kk) {
+              uint32_t ah[4], al[4], bh[4], bl[4];
+              const uint32_t at = kq + part * 64 * 128 + (kk >> 2) * kSub + (((((kk & 3) * 2) + (lane >> 4)) ^ (ra & 7)) << 4);
+              ldsm4(bh, k2h + kk * 32);
+              ldsm4(bl, k2l + kk * 32);
+              ldsm4(ah, at);
+              ldsm4(al, at + (oKQl - oKQh));
+              mma16816(cc[0], ah, bh[0], bh[1]); mma16816(cc[1], ah, bh[2], bh[3]);
+              mma16816(c1[0], al, bh[0], bh[1]); mma16816(c1[1], al, bh[2], bh[3]);
+              mma16816(c2[0], ah, bl[0], bl[1]); mma16816(c2[1], ah, bl[2], bl[3]);
+            }
+#pragma unroll
+            for (int j = 0; j < 2; ++j)
+#pragma unroll
+              for (int e = 0; e < 4; ++e) cc[j][e] += c1[j][e] + c2[j][e];
+          }
+        } else {
+          bool direct = false;
+          if (diag) {
+            float m = 0.f;
+            for (int d = lane; d < kW; d += 32) m = fmaxf(m, -sG[(rt * 16 + 15) * kPg + d]);
+            direct = __any_sync(0xffffffffu, !(m <= kDiagMax));
+          }
+          if (!direct) {
+#pragma unroll 1
+            for (int kk = 0; kk < 8; ++kk) {
+              uint32_t xh[4], xl[4], bh[4], bl[4];
+#pragma unroll
+              for (int e = 0; e < 4; ++e) {              // B operand: column tile e >> 1, channels 2 tq + 8 (e & 1)
+                const int r = st * 16 + g + 8 * (e >> 1), d = kk * 16 + 2 * tq + 8 * (e & 1);
+                const float2 G = *reinterpret_cast<const float2*>(sG + r * kPg + d), Rt = rt ? *reinterpret_cast<const float2*>(&tl.R[rt][d]) : make_float2(0.f, 0.f);
+                const float2 Rs = st ? *reinterpret_cast<const float2*>(&tl.R[st][d]) : make_float2(0.f, 0.f);
+                const float2 k = unpack_bf16(*reinterpret_cast<const uint32_t*>(sK + r * kPk + d));
+                split2(k.x * ex2(Rt.x - Rs.x - G.x), k.y * ex2(Rt.y - Rs.y - G.y), bh[e], bl[e]);
+              }
+#pragma unroll
+              for (int part = 0; part < 2; ++part) {
+                if (part == 0 ? !do_a : !do_b) continue;
+                const bf* src = part == 0 ? sK : sQ;
+                float (&cc)[2][4] = part == 0 ? ca : cb;
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {            // A operand: rows g + 8 (e & 1), channels 2 tq + 8 (e >> 1)
+                  const int r = rt * 16 + g + 8 * (e & 1), d = kk * 16 + 2 * tq + 8 * (e >> 1);
+                  const float2 G = *reinterpret_cast<const float2*>(sG + r * kPg + d), x = unpack_bf16(*reinterpret_cast<const uint32_t*>(src + r * kPk + d));
+                  split2(x.x * ex2(G.x), x.y * ex2(G.y), xh[e], xl[e]);
+                }
+                mma16816(cc[0], xh, bh[0], bh[1]); mma16816(cc[1], xh, bh[2], bh[3]);
+                mma16816(cc[0], xl, bh[0], bh[1]); mma16816(cc[1], xl, bh[2], bh[3]);
+                mma16816(cc[0], xh, bl[0], bl[1]); mma16816(cc[1], xh, bl[2], bl[3]);
+              }
+            }
+          } else {
+#pragma unroll
+            for (int j = 0; j < 2; ++j)
+#pragma unroll
+              for (int e = 0; e < 4; ++e) {
+                const int r = rt * 16 + g + 8 * (e >> 1), s = rt * 16 + 8 * j + 2 * tq + (e & 1);
+                if (s > r) continue;
+                float x = 0.f, y = 0.f;
+                for (int d = 0; d < D; ++d) {
+                  const float w = __bfloat162float(sK[s * kPk + d]) * ex2(sG[r * kPg + d] - sG[s * kPg + d]);
+                  x = fmaf(__bfloat162float(sK[r * kPk + d]), w, x);
+                  y = fmaf(__bfloat162float(sQ[r * kPk + d]), w, y);
+                }
+                ca[j][e] = x;
+                cb[j][e] = y;
+              }
+          }
+        }
+        // scales and the triangle
+#pragma unroll
+        for (int j = 0; j < 2; ++j)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const int tl_ = g + 8 * (e >> 1), sl = 8 * j + 2 * tq + (e & 1), t = rt * 16 + tl_, s = st * 16 + sl;
+            const float ks = mild ? 1.f : rk[s];
+            ca[j][e] *= (mild ? beta[t] : beta[t] * rk[t]) * ks;
+            cb[j][e] *= (mild ? 1.f : rq[t]) * ks;
+            if (diag && sl >= tl_) ca[j][e] = 0.f;
+            if (diag && sl > tl_) cb[j][e] = 0.f;
+          }
+      };
+      float a1[2][4], b1[2][4], a2[2][4], b2[2][4];
+      int rt1, st1, rt2 = 0, st2 = 0;
+      block_of(pw, &rt1, &st1);
+      block(rt1, st1, true, true, a1, b1);
+      if (pw < 4) {
+        block_of(8 + (pw >> 1), &rt2, &st2);
+        block(rt2, st2, (pw & 1) == 0, pw & 1, a2, b2);
+      }
+      if (c) mbar_wait(&tl.s_done, (c - 1) & 1, dead, err);      // kb, B and T of the chunk before have been multiplied
+      // ---- kb
+#pragma unroll 2
+      for (int i = pt; i < kC * (kW / 4); i += 256) {
+        const int r = i >> 5, d = (i & 31) * 4, at = r * kPk + d, to = swz(r, d, kSubKb);
+        const uint2 ku = *reinterpret_cast<const uint2*>(sK + at);
+        float2 k0 = unpack_bf16(ku.x), k1 = unpack_bf16(ku.y);
+        float f[4];
+        if (mild) {
+          const float4 X = *reinterpret_cast<const float4*>(E + d);
+          const uint2 lu = *reinterpret_cast<const uint2*>(sQ + at);
+          const float2 l0 = unpack_bf16(lu.x), l1 = unpack_bf16(lu.y);
+          k0.x += l0.x; k0.y += l0.y; k1.x += l1.x; k1.y += l1.y;
+          f[0] = X.x; f[1] = X.y; f[2] = X.z; f[3] = X.w;
+        } else {
+          const float4 L = *reinterpret_cast<const float4*>(sG + r * kPg + d), all4 = *reinterpret_cast<const float4*>(&tl.R[4][d]);
+          const float4 Rv = r < 16 ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4*>(&tl.R[r >> 4][d]);
+          const float kr = rk[r];
+          f[0] = kr * ex2(all4.x - Rv.x - L.x); f[1] = kr * ex2(all4.y - Rv.y - L.y); f[2] = kr * ex2(all4.z - Rv.z - L.z); f[3] = kr * ex2(all4.w - Rv.w - L.w);
+        }
+        uint2 hi, lo;
+        split2(k0.x * f[0], k0.y * f[1], hi.x, lo.x);
+        split2(k1.x * f[2], k1.y * f[3], hi.y, lo.y);
+        *reinterpret_cast<uint2*>(smem + oKbh + to) = hi;
+        *reinterpret_cast<uint2*>(smem + oKbl + to) = lo;
+      }
+      // ---- B
+      auto put_b = [&](int rt, int st, const float (&cb)[2][4]) {
+#pragma unroll
+        for (int j = 0; j < 2; ++j)
+#pragma unroll
+          for (int e2 = 0; e2 < 2; ++e2) {
+            uint32_t hi, lo;
+            split2(cb[j][2 * e2], cb[j][2 * e2 + 1], hi, lo);
+            const int to = swz(rt * 16 + g + 8 * e2, st * 16 + 8 * j + 2 * tq, 0);
+            *reinterpret_cast<uint32_t*>(smem + oBh + to) = hi;
+            *reinterpret_cast<uint32_t*>(smem + oBl + to) = lo;
+          }
+      };
+      put_b(rt1, st1, b1);
+      if (pw < 4 && (pw & 1)) put_b(rt2, st2, b2);
+      fence_async_smem();
+      prep_sync();
+      // ---- raw rows are free; the next chunk's decays are on their way; A in float32 over the decay sums
+      if (lane == 0) mbar_arrive(&tl.raw_empty);
+      if (c + 1 < chunks) fetch(c + 1);
+      float *sA = sG, *sT = sG + kC * kPt;
+      auto put_a = [&](int rt, int st, const float (&ca)[2][4]) {
+#pragma unroll
+        for (int j = 0; j < 2; ++j)
+#pragma unroll
+          for (int e2 = 0; e2 < 2; ++e2)
+            *reinterpret_cast<float2*>(sA + (rt * 16 + g + 8 * e2) * kPt + st * 16 + 8 * j + 2 * tq) = make_float2(ca[j][2 * e2], ca[j][2 * e2 + 1]);
+      };
+      put_a(rt1, st1, a1);
+      if (pw < 4 && (pw & 1) == 0) put_a(rt2, st2, a2);
+      // ---- T = (I + A)^-1: 16 x 16 diagonal blocks, then twice [[P, 0], [R, Q]]^-1 = [[P', 0], [-Q' R P', Q']]
+      if (pw < 4) {
+        __syncwarp();
+        const float* M = sA + (pw * 16) * kPt + pw * 16;
+        float x[16];
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+          float y = i == (lane & 15) ? 1.f : 0.f;
+#pragma unroll
+          for (int k = 0; k < i; ++k) y = fmaf(-M[i * kPt + k], x[k], y);
+          x[i] = y;
+        }
+        if (lane < 16) {
+#pragma unroll
+          for (int i = 0; i < 16; ++i) sT[(pw * 16 + i) * kPt + pw * 16 + lane] = x[i];
+        }
+      }
+      prep_sync();
+      {                                                  // R P' of the two 32-blocks, into the empty blocks above the diagonal
+        const int blk = pt >> 7, i = (pt & 127) >> 3, j = (pt & 7) * 2;
+        const float *Rm = sA + (blk * 32 + 16 + i) * kPt + blk * 32, *P = sT + (blk * 32) * kPt + blk * 32 + j;
+        float x = 0.f, y = 0.f;
+#pragma unroll
+        for (int k = 0; k < 16; ++k) {
+          const float m = Rm[k];
+          const float2 p = *reinterpret_cast<const float2*>(P + k * kPt);
+          x = fmaf(m, p.x, x); y = fmaf(m, p.y, y);
+        }
+        *reinterpret_cast<float2*>(sT + (blk * 32 + i) * kPt + blk * 32 + 16 + j) = make_float2(x, y);
+        prep_sync();
+        const float *Q = sT + (blk * 32 + 16 + i) * kPt + blk * 32 + 16, *Y = sT + (blk * 32) * kPt + blk * 32 + 16 + j;
+        x = y = 0.f;
+#pragma unroll
+        for (int k = 0; k < 16; ++k) {
+          const float m = Q[k];
+          const float2 p = *reinterpret_cast<const float2*>(Y + k * kPt);
+          x = fmaf(m, p.x, x); y = fmaf(m, p.y, y);
+        }
+        *reinterpret_cast<float2*>(sT + (blk * 32 + 16 + i) * kPt + blk * 32 + j) = make_float2(-x, -y);
+      }
+      prep_sync();
+      {                                                  // the same for the halves
+        const int i = pt >> 3, j = (pt & 7) * 4;
+        const float *Rm = sA + (32 + i) * kPt, *P = sT + j;
+        float x[4] = {0.f, 0.f, 0.f, 0.f};
+        for (int k = j & 16; k < 32; k += 2) {           // P' is zero above its diagonal blocks (scratch lies there)
+          const float2 m = *reinterpret_cast<const float2*>(Rm + k);
+          const float2 p0 = *reinterpret_cast<const float2*>(P + k * kPt), p1 = *reinterpret_cast<const float2*>(P + k * kPt + 2);
+          const float2 q0 = *reinterpret_cast<const float2*>(P + (k + 1) * kPt), q1 = *reinterpret_cast<const float2*>(P + (k + 1) * kPt + 2);
+          x[0] = fmaf(m.x, p0.x, x[0]); x[1] = fmaf(m.x, p0.y, x[1]); x[2] = fmaf(m.x, p1.x, x[2]); x[3] = fmaf(m.x, p1.y, x[3]);
+          x[0] = fmaf(m.y, q0.x, x[0]); x[1] = fmaf(m.y, q0.y, x[1]); x[2] = fmaf(m.y, q1.x, x[2]); x[3] = fmaf(m.y, q1.y, x[3]);
+        }
+        float* Y = sT + i * kPt + 32 + j;
+        *reinterpret_cast<float2*>(Y) = make_float2(x[0], x[1]);
+        *reinterpret_cast<float2*>(Y + 2) = make_float2(x[2], x[3]);
+        prep_sync();
+        const float *Q = sT + (32 + i) * kPt + 32, *Z = sT + 32 + j;
+        x[0] = x[1] = x[2] = x[3] = 0.f;
+        for (int k = 0; k < (i & 16) + 16; k += 2) {
+          const float2 m = *reinterpret_cast<const float2*>(Q + k);
+          const float2 p0 = *reinterpret_cast<const float2*>(Z + k * kPt), p1 = *reinterpret_cast<const float2*>(Z + k * kPt + 2);
+          const float2 q0 = *reinterpret_cast<const float2*>(Z + (k + 1) * kPt), q1 = *reinterpret_cast<const float2*>(Z + (k + 1) * kPt + 2);
+          x[0] = fmaf(m.x, p0.x, x[0]); x[1] = fmaf(m.x, p0.y, x[1]); x[2] = fmaf(m.x, p1.x, x[2]); x[3] = fmaf(m.x, p1.y, x[3]);
+          x[0] = fmaf(m.y, q0.x, x[0]); x[1] = fmaf(m.y, q0.y, x[1]); x[2] = fmaf(m.y, q1.x, x[2]); x[3] = fmaf(m.y, q1.y, x[3]);
+        }
+        float* W = sT + (32 + i) * kPt + j;
+        *reinterpret_cast<float2*>(W) = make_float2(-x[0], -x[1]);
+        *reinterpret_cast<float2*>(W + 2) = make_float2(-x[2], -x[3]);
+      }
+      prep_sync();
+      for (int i = pt; i < 10 * 64; i += 256) {          // four elements of a row of one of the ten blocks
+        int rt, st;
+        block_of(i >> 6, &rt, &st);
+        const int r = rt * 16 + ((i & 63) >> 2), col = st * 16 + (i & 3) * 4, to = swz(r, col, 0);
+        const float2 x = *reinterpret_cast<const float2*>(sT + r * kPt + col), y = *reinterpret_cast<const float2*>(sT + r * kPt + col + 2);
+        uint2 hi, lo;
+        split2(x.x, x.y, hi.x, lo.x);
+        split2(y.x, y.y, hi.y, lo.y);
+        *reinterpret_cast<uint2*>(smem + oTh + to) = hi;
+        *reinterpret_cast<uint2*>(smem + oTl + to) = lo;
+      }
+      fence_async_smem();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&tl.tb_ready);
+      prep_sync();                                       // T has been read: the next decay sums go over it
+    }
+  } else {
+    // ------------------------------ value columns ------------------------------
+    const int half = warp >> 2, quad = warp & 3, col = 32 * quad + lane;
+    const uint32_t lanes = tmem + ((uint32_t)(32 * quad) << 16);
+    float* state = v.state + ((int64_t)b * v.H + h) * D * ld + col;
+    const float wn = col < V ? __ldg(v.norm + col) : 0.f;
+    for (int c = 0; c < chunks; ++c) {
+      const int n = min(kC, n_all - c * kC);
+      const int64_t t0 = t_first + (int64_t)c * kC + half * 32;
+      const float *beta = tl.row[c & 1][0] + half * 32, *E = tl.E[c & 1];
+      // ---- S as an operand, and decayed
+      mbar_wait(&tl.kq_ready, c & 1, dead, err);
+      if (c) { mbar_wait(&tl.s_done, (c - 1) & 1, dead, err); fence_after(); }
+#pragma unroll
+      for (int q = 0; q < 4; ++q) {
+        float x[16];
+        const int d0 = half * 64 + q * 16;
+        if (c == 0) {
+#pragma unroll
+          for (int i = 0; i < 16; ++i) x[i] = d0 + i < D && col < V ? state[(int64_t)(d0 + i) * ld] : 0.f;
+        } else {
+          tmem_ld16(x, lanes + cS + d0);
+        }
+        uint32_t hi[8], lo[8], u[16];
+#pragma unroll
+        for (int i = 0; i < 16; i += 2) split2(x[i], x[i + 1], hi[i / 2], lo[i / 2]);
+#pragma unroll
+        for (int i = 0; i < 16; ++i) u[i] = __float_as_uint(x[i] * E[d0 + i]);
+        tmem_st16_nowait(lanes + cS + d0, u);
+        asm volatile("tcgen05.st.sync.aligned.32x32b.x8.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8};\n" ::"r"(lanes + cSh + d0 / 2), "r"(hi[0]), "r"(hi[1]), "r"(hi[2]), "r"(hi[3]),
+                     "r"(hi[4]), "r"(hi[5]), "r"(hi[6]), "r"(hi[7]) : "memory");
+        asm volatile("tcgen05.st.sync.aligned.32x32b.x8.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8};\n" ::"r"(lanes + cSl + d0 / 2), "r"(lo[0]), "r"(lo[1]), "r"(lo[2]), "r"(lo[3]),
+                     "r"(lo[4]), "r"(lo[5]), "r"(lo[6]), "r"(lo[7]) : "memory");
+      }
+      tmem_st_wait();
+      fence_before();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&tl.s_ready);
+      // ---- X
+      mbar_wait(&tl.v_full, c & 1, dead, err);
+      float x[32];
+      uint32_t hi[16], lo[16];
+      {
+        bf vv[32];
+#pragma unroll
+        for (int i = 0; i < 32; ++i) vv[i] = sV[(half * 32 + i) * kPk + col];
+        mbar_wait(&tl.yo_done, c & 1, dead, err);
+        fence_after();
+        tmem_ld32(x, lanes + cYO + half * 32);
+#pragma unroll
+        for (int i = 0; i < 32; i += 2)
+          split2(beta[i] * (__bfloat162float(vv[i]) - x[i]), beta[i + 1] * (__bfloat162float(vv[i + 1]) - x[i + 1]), hi[i / 2], lo[i / 2]);
+      }
+      tmem_st16_nowait(lanes + cXh + half * 16, hi);
+      tmem_st16_nowait(lanes + cXl + half * 16, lo);
+      tmem_st_wait();
+      fence_before();
+      __syncwarp();
+      if (lane == 0) { mbar_arrive(&tl.x_ready); mbar_arrive(&tl.v_empty); }
+      const bf* gate = reinterpret_cast<const bf*>(v.gate) + t0 * v.gate_pitch + h * V + col;
+      if (half * 32 + lane < n && 32 * quad < V) asm volatile("prefetch.global.L2 [%0];\n" ::"l"(gate - lane + (int64_t)lane * v.gate_pitch));
+      mbar_wait(&tl.u_done, c & 1, dead, err);
+      fence_after();
+      tmem_ld32(x, lanes + cYO + half * 32);
+#pragma unroll
+      for (int i = 0; i < 32; i += 2) split2(x[i], x[i + 1], hi[i / 2], lo[i / 2]);
+      tmem_st16_nowait(lanes + cUh + half * 16, hi);
+      tmem_st16_nowait(lanes + cUl + half * 16, lo);
+      tmem_st_wait();
+      fence_before();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&tl.u_ready);
+      // ---- outputs: lane i ends with token i's sum of squares over the warp's 32 value columns
+      mbar_wait(&tl.o_done, c & 1, dead, err);
+      fence_after();
+      tmem_ld32(x, lanes + cYO + 64 + half * 32);
+      float ss[32];
+#pragma unroll
+      for (int i = 0; i < 32; ++i) ss[i] = x[i] * x[i];
+#pragma unroll
+      for (int w = 16; w > 0; w >>= 1) {
+        const bool up = (lane & w) != 0;
+#pragma unroll
+        for (int i = 0; i < w; ++i) {
+          const float send = up ? ss[i] : ss[i + w], keep = up ? ss[i + w] : ss[i];
+          ss[i] = keep + __shfl_xor_sync(0xffffffffu, send, w);
+        }
+      }
+      tl.sum[quad][half * 32 + lane] = ss[0];
+      asm volatile("bar.sync %0, 128;\n" ::"r"(1 + half) : "memory");
+      const float all = tl.sum[0][half * 32 + lane] + tl.sum[1][half * 32 + lane] + tl.sum[2][half * 32 + lane] + tl.sum[3][half * 32 + lane];
+      const float inv = 1.0f / sqrtf(all / (float)V + v.eps);
+      asm volatile("bar.sync %0, 128;\n" ::"r"(1 + half) : "memory");             // the sums have been read
+      bf* out = reinterpret_cast<bf*>(v.out) + t0 * v.ldo + h * V + col;
+      const int rows = col < V ? n - half * 32 : 0;
+#pragma unroll
+      for (int i0 = 0; i0 < 32; i0 += 16) {              // sixteen gate values in flight
+        bf gv[16];
+#pragma unroll
+        for (int i = 0; i < 16; ++i) gv[i] = i0 + i < rows ? __ldg(gate + (int64_t)(i0 + i) * v.gate_pitch) : __float2bfloat16_rn(0.f);
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+          const float f = __shfl_sync(0xffffffffu, inv, i0 + i);
+          if (i0 + i < rows) out[(int64_t)(i0 + i) * v.ldo] = __float2bfloat16_rn(x[i0 + i] * f * wn * __bfloat162float(gv[i]));
+        }
+      }
+    }
+    if (chunks > 0) {
+      mbar_wait(&tl.s_done, (chunks - 1) & 1, dead, err);
+      fence_after();
+#pragma unroll
+      for (int q = 0; q < 4; ++q) {
+        float x[16];
+        const int d0 = half * 64 + q * 16;
+        tmem_ld16(x, lanes + cS + d0);
+#pragma unroll
+        for (int i = 0; i < 16; ++i)
+          if (d0 + i < D && col < V) state[(int64_t)(d0 + i) * ld] = x[i];
+      }
+    }
+  }
+  fence_before();
+  __syncthreads();
+  if (warp == 16) {
+    fence_after();
+    tmem_dealloc(tmem, 512);
+  }
+}
+
+}  // namespace
+
+int32_t delta_tc_configure() {
+  LMB_CUDA(cudaFuncSetAttribute(delta_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSmem));
+  return LMB200_OK;
+}
+
+// heads no wider than a tile; narrow ones (64 x 64 and below) are better off in csrc/delta_chunk.cu
+bool delta_tc_ok(const DeltaView& v) { return delta_chunks_ok(v) && (v.dim > 64 || v.vdim > 64); }
+
+int32_t delta_tc(Ctx* ctx, const DeltaView& v, cudaStream_t st) {
+  LMB_REQUIRE(delta_tc_ok(v), "delta rule: heads of %d x %d have no kernel on tcgen05", v.dim, v.vdim);
+  LMB_CUDA(launch_k(delta_tc_kernel, dim3((unsigned)v.H, (unsigned)v.B), dim3(kThreads), kSmem, st, v, ctx->dev_err));
+  ctx->launches++;
+  return LMB200_OK;
+}
+
+}  // namespace lmb

@@ -74,6 +74,7 @@ struct LayeredScratch {
 namespace {
 
 constexpr int kChunkMin = 8, kTcMin = 80;   // longest portion from which retention (and the delta rule) runs in chunks of 64, of 128 tokens
+constexpr int kDeltaTcMin = 48;         // longest portion from which the delta rule runs on tcgen05
 constexpr int kFlashMin = 32;           // shortest portion whose context is expanded to keys and values
 constexpr int kBlockTokens = 2048;      // tokens per round of the absorbed attention in a rows step (bounds its scratch)
 constexpr uint64_t kIdLayered = 0x200000, kIdLayeredState = 0x300000;
@@ -1059,6 +1060,7 @@ int32_t delta_rows(Session* S, RowsBuf& r, const RowsRun& run, int l, cudaStream
   v.decay = r.log_g; v.decay_pitch = hd;
   v.gate = r.gate; v.gate_pitch = ld_g;
   v.out = r.cat; v.ldo = row_ld(s.m_out.K); v.bp = 0;
+  if (dt == LMB200_BF16 && run.max_len >= kDeltaTcMin && delta_tc_ok(v)) return delta_tc(ctx, v, st);
   if (dt == LMB200_BF16 && run.max_len >= kChunkMin && delta_chunks_ok(v)) return delta_chunks(ctx, v, st);
   return delta_steps(ctx, dt, v, st);
 }
