@@ -6,10 +6,11 @@
 //   X = beta (V - Y),  U^T = X^T T^T   T = (I + A)^-1, 64 x 64
 //   O^T += U^T B^T,   S^T = S^T diag(e^{G_end}) + U^T kb
 // every product as hi hi + lo hi + hi lo (x = hi + lo to about 2^-17), accumulated in float32.
-// Tensor memory columns: [Y then U | O] 128, S 128, [S hi | S lo, later X hi | X lo] 128, [U hi | U lo] 64.
+//   [A | B] = [kt | qt] (k e^{-G})^T   mild chunks (see there), from shared memory; other chunks with mma.sync, block by block
+// Tensor memory columns: [Y then U | O] 128, S 128, [S hi | S lo, later X hi | X lo] 128, [U hi | U lo] 64, [A, B] 64 (lanes: tokens).
 // Warps: 0-7 own the value columns (two threads per column): they turn S, X and U into operands and write the outputs; 8-15 prepare the
-// next chunk (decay sums, kt, qt, kb; A and B with mma.sync; T in float32) while the others work on this one; 16 issues the
-// MMAs, 17 the row copies.  All waits are bounded.
+// next chunk (decay sums, kt, qt, kb, A and B, T in float32) while the others work on this one; 16 issues the other MMAs, 17 the row
+// copies.  All waits are bounded.
 #include "delta.cuh"
 #include "mma_sync.cuh"
 #include "pdl.cuh"
@@ -22,22 +23,23 @@ constexpr int kC = 64, kW = 128;                        // tokens per chunk; hea
 constexpr float kLog2e = 1.4426950408889634f;
 constexpr float kDiagMax = 80.0f, kDecayMin = -150.0f;  // as in csrc/delta_chunk.cu
 constexpr int kThreads = 18 * 32;
-constexpr uint32_t cYO = 0, cS = 128, cSh = 256, cSl = 320, cXh = 256, cXl = 288, cUh = 384, cUl = 416;
-constexpr int kPk = kW + 8, kPg = kW + 4, kPt = 66;     // row pitches: raw rows, decay sums, float32 A and T
+constexpr uint32_t cYO = 0, cS = 128, cSh = 256, cSl = 320, cXh = 256, cXl = 288, cUh = 384, cUl = 416, cBlk = 448;
+constexpr int kPv = kW, kPg = kW + 4, kPt = 66;         // row pitches: raw rows, decay sums, float32 A and T
 // shared memory; tiles in the 128-byte swizzle
-constexpr int kSub = 128 * 128, kSubKb = 64 * 128;      // sub-tiles [128 rows][64 columns], [64 rows][64 columns]
+constexpr int kSub = 128 * 128, kSub64 = 64 * 128;      // sub-tiles [128 rows][64 columns], [64 rows][64 columns]
 constexpr int oKQh = 0, oKQl = oKQh + 2 * kSub;         // rows 0-63 kt, 64-127 qt
-constexpr int oKbh = oKQl + 2 * kSub, oKbl = oKbh + 2 * kSubKb;
-constexpr int oTh = oKbl + 2 * kSubKb, oTl = oTh + kSubKb, oBh = oTl + kSubKb, oBl = oBh + kSubKb;
-constexpr int oK = oBl + kSubKb, oQ = oK + kC * kPk * 2, oV = oQ + kC * kPk * 2;          // raw rows; mild chunks: k e^{-G} hi over K, lo over Q
-constexpr int oG = oV + kC * kPk * 2;                   // decay sums; later A and T in float32
+constexpr int oKbh = oKQl + 2 * kSub, oKbl = oKbh + 2 * kSub64;
+constexpr int oTh = oKbl + 2 * kSub64, oTl = oTh + kSub64, oBh = oTl + kSub64, oBl = oBh + kSub64;
+constexpr int oK = oBl + kSub64, oQ = oK + 2 * kSub64;  // raw rows; mild chunks then k e^{-G} as a tile, hi over K, lo over Q
+constexpr int oV = oQ + 2 * kSub64;                     // v, later the outputs on their way out
+constexpr int oG = oV + 2 * kSub64;                     // log decays, their sums; later A and T in float32
 constexpr int oEnd = oG + kC * kPg * 4;
-static_assert(2 * kC * kPt * 4 <= kC * kPg * 4, "A and T fit over the decay sums");
+static_assert(2 * kC * kPt * 4 <= kC * kPg * 4 && kC * kPv * 2 <= 2 * kSub64, "what lies over something else fits");
 struct Tail {
-  uint64_t raw_full, raw_empty, v_full, v_empty, kq_ready, tb_ready, s_ready, x_ready, u_ready, yo_done, u_done, o_done, s_done;
+  uint64_t raw_full, raw_empty, g_full, g_empty, v_full, v_empty, kq_ready, blk_done, tb_ready, kb_ready, s_ready, x_ready, u_ready, yo_done, u_done, o_done, s_done;
   uint32_t tmem;
-  alignas(16) float R[5][kW];                                       // decay sums before blocks 1 .. 3 of 16 tokens, and of the whole chunk
-  alignas(16) float E[2][kW];                                       // e^{G_end}, by chunk parity
+  alignas(16) float R[5][kW];                           // decay sums before blocks 1 .. 3 of 16 tokens, and of the whole chunk
+  alignas(16) float E[2][kW];                           // e^{G_end}, by chunk parity
   float row[2][3][kC];                                  // beta, 1 / |k|, 1 / |q| / sqrt(dim), by chunk parity
   float sum[4][kC];                                     // sums of squares of the outputs per 32 value columns
 };
@@ -72,8 +74,8 @@ __global__ void __launch_bounds__(kThreads, 1) delta_tc_kernel(const DeltaView v
   const int h = blockIdx.x, b = blockIdx.y, D = v.dim, V = v.vdim, ld = (V + 3) & ~3, a = h / (v.H / v.G);
   if (tid == 0) {
     if (smem_u32(smem) & 1023) atomicExch(err, 1);       // the swizzle needs 1024-byte tiles
-    mbar_init(&tl.raw_full, 1); mbar_init(&tl.v_full, 1); mbar_init(&tl.yo_done, 1); mbar_init(&tl.u_done, 1); mbar_init(&tl.o_done, 1); mbar_init(&tl.s_done, 1);
-    mbar_init(&tl.raw_empty, 8); mbar_init(&tl.v_empty, 8); mbar_init(&tl.kq_ready, 8); mbar_init(&tl.tb_ready, 8);
+    mbar_init(&tl.raw_full, 1); mbar_init(&tl.g_full, 1); mbar_init(&tl.v_full, 1); mbar_init(&tl.blk_done, 1); mbar_init(&tl.yo_done, 1); mbar_init(&tl.u_done, 1); mbar_init(&tl.o_done, 1); mbar_init(&tl.s_done, 1);
+    mbar_init(&tl.raw_empty, 8); mbar_init(&tl.g_empty, 8); mbar_init(&tl.v_empty, 8); mbar_init(&tl.kb_ready, 8); mbar_init(&tl.kq_ready, 8); mbar_init(&tl.tb_ready, 8);
     mbar_init(&tl.s_ready, 8); mbar_init(&tl.x_ready, 8); mbar_init(&tl.u_ready, 8);
     mbar_init_fence();
   }
@@ -92,23 +94,27 @@ __global__ void __launch_bounds__(kThreads, 1) delta_tc_kernel(const DeltaView v
   const int chunks = (n_all + kC - 1) / kC;              // 0: nothing to do
 
   if (warp == 17) {
-    // ------------------------------ rows of k, q and v ------------------------------
+    // ------------------------------ rows of k, q, log g and v ------------------------------
     for (int c = 0; c < chunks; ++c) {
       const int64_t t0 = t_first + (int64_t)c * kC;
-      const int n = min(kC, n_all - c * kC);             // behind the portion's end the last row again: its beta and decay are zero
+      const int n = min(kC, n_all - c * kC);             // behind the portion's end the last row again: its beta and decay count as zero
+      mbar_wait(&tl.g_empty, (c & 1) ^ 1, dead, err);
+      if (lane == 0) mbar_expect_tx(&tl.g_full, (uint32_t)(kC * D * 4));
+      __syncwarp();
+      for (int r = lane; r < kC; r += 32) bulk_g2s(sG + r * kPg, v.decay + (t0 + min(r, n - 1)) * v.decay_pitch + h * D, (uint32_t)D * 4, &tl.g_full);
       mbar_wait(&tl.raw_empty, (c & 1) ^ 1, dead, err);
       if (lane == 0) mbar_expect_tx(&tl.raw_full, (uint32_t)(2 * kC * D * 2));
       __syncwarp();
       for (int r = lane; r < kC; r += 32) {
         const int64_t t = t0 + min(r, n - 1);
-        bulk_g2s(sK + r * kPk, reinterpret_cast<const bf*>(v.k) + t * v.k_pitch + a * D, (uint32_t)D * 2, &tl.raw_full);
-        bulk_g2s(sQ + r * kPk, reinterpret_cast<const bf*>(v.q) + t * v.q_pitch + a * D, (uint32_t)D * 2, &tl.raw_full);
+        bulk_g2s(sK + r * kW, reinterpret_cast<const bf*>(v.k) + t * v.k_pitch + a * D, (uint32_t)D * 2, &tl.raw_full);
+        bulk_g2s(sQ + r * kW, reinterpret_cast<const bf*>(v.q) + t * v.q_pitch + a * D, (uint32_t)D * 2, &tl.raw_full);
       }
       mbar_wait(&tl.v_empty, (c & 1) ^ 1, dead, err);
       if (lane == 0) mbar_expect_tx(&tl.v_full, (uint32_t)(kC * V * 2));
       __syncwarp();
       for (int r = lane; r < kC; r += 32)
-        bulk_g2s(sV + r * kPk, reinterpret_cast<const bf*>(v.v) + (t0 + min(r, n - 1)) * v.v_pitch + h * V, (uint32_t)V * 2, &tl.v_full);
+        bulk_g2s(sV + r * kPv, reinterpret_cast<const bf*>(v.v) + (t0 + min(r, n - 1)) * v.v_pitch + h * V, (uint32_t)V * 2, &tl.v_full);
     }
   } else if (warp == 16) {
     // ------------------------------ MMA issue ------------------------------
@@ -145,10 +151,15 @@ __global__ void __launch_bounds__(kThreads, 1) delta_tc_kernel(const DeltaView v
           for (int ks = 0; ks < 4; ++ks)
             mma_ts(tmem + cYO + 64, tmem + (p == 1 ? cUl : cUh) + ks * 8, desc(base + (p == 2 ? oBl : oBh) + ks * 32, 16, 1024), kN64, 1u);
         commit(&tl.o_done);
+      }
+      __syncwarp();
+      mbar_wait(&tl.kb_ready, c & 1, dead, err);
+      fence_after();
+      if (lane == 0) {
 #pragma unroll
         for (int p = 0; p < 3; ++p)
           for (int ks = 0; ks < 4; ++ks)
-            mma_ts(tmem + cS, tmem + (p == 1 ? cUl : cUh) + ks * 8, desc(base + (p == 2 ? oKbl : oKbh) + ks * 2048, kSubKb, 1024), kN128m, 1u);
+            mma_ts(tmem + cS, tmem + (p == 1 ? cUl : cUh) + ks * 8, desc(base + (p == 2 ? oKbl : oKbh) + ks * 2048, kSub64, 1024), kN128m, 1u);
         commit(&tl.s_done);
       }
       __syncwarp();
@@ -157,37 +168,38 @@ __global__ void __launch_bounds__(kThreads, 1) delta_tc_kernel(const DeltaView v
     // ------------------------------ preparation of a chunk ------------------------------
     const int pt = tid - 256, pw = warp - 8, g = lane >> 2, tq = lane & 3;
     const int ch = pt >> 1, hf = pt & 1;                 // decay sums: channel, half of the chunk
-    float gl[32];                                        // its log decays
+    const int quad = warp & 3, side = pw >> 2;           // A and B: 32 rows of [A | B], half of their columns
+    int n_mild = 0;                                      // phases of blk_done
     float rb = 0.f, rk_ = 0.f, rq_ = 0.f;
-    auto fetch = [&](int c) {
-      const int64_t t0 = t_first + (int64_t)c * kC;
-      const int n = min(kC, n_all - c * kC);
-#pragma unroll
-      for (int r = 0; r < 32; ++r) gl[r] = ch < D && hf * 32 + r < n ? __ldg(v.decay + (t0 + hf * 32 + r) * v.decay_pitch + h * D + ch) : 0.f;
-      if (pt < kC) {
-        const bool ok = pt < n;
-        rb = ok ? v.b[(t0 + pt) * v.b_pitch + h] : 0.f;
-        rk_ = ok ? v.rk[(t0 + pt) * v.G + a] : 0.f;
-        rq_ = ok ? v.rq[(t0 + pt) * v.G + a] : 0.f;
-      }
+    auto fetch = [&](int c) {                            // scalars of token pt
+      const int64_t t = t_first + (int64_t)c * kC + pt;
+      if (pt >= kC) return;
+      const bool ok = c * kC + pt < n_all;
+      rb = ok ? v.b[t * v.b_pitch + h] : 0.f;
+      rk_ = ok ? v.rk[t * v.G + a] : 0.f;
+      rq_ = ok ? v.rq[t * v.G + a] : 0.f;
     };
     if (chunks > 0) fetch(0);
     for (int c = 0; c < chunks; ++c) {
       const int n = min(kC, n_all - c * kC);
       float *beta = tl.row[c & 1][0], *rk = tl.row[c & 1][1], *rq = tl.row[c & 1][2], *E = tl.E[c & 1];
-      // ---- decay sums (log2 units): in sG from the start of each block of 16 tokens, in R before the block
       if (pt < kC) {
         beta[pt] = pt < n ? 1.0f / (1.0f + expf(-rb)) : 0.f;
         rk[pt] = rk_;
         rq[pt] = rq_;
       }
+      if (c + 1 < chunks) fetch(c + 1);
+      // ---- decay sums (log2 units): in sG from the start of each block of 16 tokens, in R before the block
+      mbar_wait(&tl.g_full, c & 1, dead, err);
       float tot[2];
 #pragma unroll
       for (int q = 0; q < 2; ++q) {
-        float s = 0.f;
+        float gl[16], s = 0.f;
+#pragma unroll
+        for (int r = 0; r < 16; ++r) gl[r] = ch < D && hf * 32 + q * 16 + r < n ? sG[(hf * 32 + q * 16 + r) * kPg + ch] : 0.f;
 #pragma unroll
         for (int r = 0; r < 16; ++r) {
-          s += fmaxf(gl[q * 16 + r] * kLog2e, kDecayMin);
+          s += fmaxf(gl[r] * kLog2e, kDecayMin);
           sG[(hf * 32 + q * 16 + r) * kPg + ch] = s;
         }
         tot[q] = s;
@@ -200,49 +212,76 @@ __global__ void __launch_bounds__(kThreads, 1) delta_tc_kernel(const DeltaView v
         tl.R[4][ch] = all;
         E[ch] = ex2(all);
       }
-      mbar_wait(&tl.raw_full, c & 1, dead, err);
       int mild;
-      {                                                  // bar.red over the preparing warps
+      {                                                  // over the preparing warps
         int p = all >= -kDiagMax;
         asm volatile("{\n.reg .pred p, q;\nsetp.ne.s32 p, %1, 0;\nbarrier.red.and.pred q, 3, 256, p;\nselp.s32 %0, 1, 0, q;\n}\n" : "=r"(mild) : "r"(p) : "memory");
       }
-      // ---- kt, qt (and k e^{-G} over the raw rows)
+      // ---- kt, qt, and k e^{-G} over the raw rows
+      mbar_wait(&tl.raw_full, c & 1, dead, err);
       if (c) mbar_wait(&tl.yo_done, (c - 1) & 1, dead, err);
-#pragma unroll 2
-      for (int i = pt; i < kC * (kW / 4); i += 256) {
-        const int r = i >> 5, d = (i & 31) * 4, at = r * kPk + d;
-        const float4 L = *reinterpret_cast<const float4*>(sG + r * kPg + d);
-        const float4 Rv = r < 16 ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4*>(&tl.R[r >> 4][d]);
-        const uint2 ku = *reinterpret_cast<const uint2*>(sK + at), qu = *reinterpret_cast<const uint2*>(sQ + at);
-        const float2 k0 = unpack_bf16(ku.x), k1 = unpack_bf16(ku.y), q0 = unpack_bf16(qu.x), q1 = unpack_bf16(qu.y);
-        const float kr = rk[r], qr = rq[r];
-        const float G[4] = {Rv.x + L.x, Rv.y + L.y, Rv.z + L.z, Rv.w + L.w};
-        const float k[4] = {k0.x * kr, k0.y * kr, k1.x * kr, k1.y * kr}, q[4] = {q0.x * qr, q0.y * qr, q1.x * qr, q1.y * qr};
-        float e[4];
+      {
+        uint2 mh[8], ml[8];
 #pragma unroll
-        for (int j = 0; j < 4; ++j) e[j] = ex2(G[j]);
-        const int to = swz(r, d, kSub);
-        uint2 hi, lo;
-        split2(k[0] * e[0], k[1] * e[1], hi.x, lo.x);
-        split2(k[2] * e[2], k[3] * e[3], hi.y, lo.y);
-        *reinterpret_cast<uint2*>(smem + oKQh + to) = hi;
-        *reinterpret_cast<uint2*>(smem + oKQl + to) = lo;
-        split2(q[0] * e[0], q[1] * e[1], hi.x, lo.x);
-        split2(q[2] * e[2], q[3] * e[3], hi.y, lo.y);
-        *reinterpret_cast<uint2*>(smem + oKQh + to + 64 * 128) = hi;
-        *reinterpret_cast<uint2*>(smem + oKQl + to + 64 * 128) = lo;
+        for (int it = 0; it < 8; ++it) {
+          const int r = (pt >> 5) + 8 * it, d = (pt & 31) * 4, at = r * kW + d;
+          const float4 L = *reinterpret_cast<const float4*>(sG + r * kPg + d);
+          const float4 Rv = it < 2 ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4*>(&tl.R[it >> 1][d]);
+          uint2 ku = *reinterpret_cast<const uint2*>(sK + at), qu = *reinterpret_cast<const uint2*>(sQ + at);
+          if (d >= D) {                                  // behind the width: whatever lay over the raw rows before
+            ku = qu = make_uint2(0u, 0u);
+            if (!mild) *reinterpret_cast<uint2*>(sK + at) = *reinterpret_cast<uint2*>(sQ + at) = ku;
+          }
+          const float2 k0 = unpack_bf16(ku.x), k1 = unpack_bf16(ku.y), q0 = unpack_bf16(qu.x), q1 = unpack_bf16(qu.y);
+          const float kr = rk[r], qr = rq[r];
+          const float G[4] = {Rv.x + L.x, Rv.y + L.y, Rv.z + L.z, Rv.w + L.w};
+          const float k[4] = {k0.x * kr, k0.y * kr, k1.x * kr, k1.y * kr}, q[4] = {q0.x * qr, q0.y * qr, q1.x * qr, q1.y * qr};
+          float e[4];
+#pragma unroll
+          for (int j = 0; j < 4; ++j) e[j] = ex2(G[j]);
+          const int to = swz(r, d, kSub);
+          uint2 hi, lo;
+          split2(k[0] * e[0], k[1] * e[1], hi.x, lo.x);
+          split2(k[2] * e[2], k[3] * e[3], hi.y, lo.y);
+          *reinterpret_cast<uint2*>(smem + oKQh + to) = hi;
+          *reinterpret_cast<uint2*>(smem + oKQl + to) = lo;
+          split2(q[0] * e[0], q[1] * e[1], hi.x, lo.x);
+          split2(q[2] * e[2], q[3] * e[3], hi.y, lo.y);
+          *reinterpret_cast<uint2*>(smem + oKQh + to + 64 * 128) = hi;
+          *reinterpret_cast<uint2*>(smem + oKQl + to + 64 * 128) = lo;
+          if (mild) {
+            split2(k[0] * ex2(-G[0]), k[1] * ex2(-G[1]), mh[it].x, ml[it].x);
+            split2(k[2] * ex2(-G[2]), k[3] * ex2(-G[3]), mh[it].y, ml[it].y);
+          }
+        }
         if (mild) {
-          split2(k[0] * ex2(-G[0]), k[1] * ex2(-G[1]), hi.x, lo.x);
-          split2(k[2] * ex2(-G[2]), k[3] * ex2(-G[3]), hi.y, lo.y);
-          *reinterpret_cast<uint2*>(sK + at) = hi;
-          *reinterpret_cast<uint2*>(sQ + at) = lo;
+          prep_sync();                                   // every raw row has been read
+#pragma unroll
+          for (int it = 0; it < 8; ++it) {
+            const int to = swz((pt >> 5) + 8 * it, (pt & 31) * 4, kSub64);
+            *reinterpret_cast<uint2*>(smem + oK + to) = mh[it];
+            *reinterpret_cast<uint2*>(smem + oQ + to) = ml[it];
+          }
         }
       }
       fence_async_smem();
       __syncwarp();
       if (lane == 0) mbar_arrive(&tl.kq_ready);
       prep_sync();
-      // ---- blocks of A and B, kept in registers: first one block per warp (0-3 on the diagonal), then the A or the B part of two more
+      if (mild && pt == 0) {
+        constexpr uint32_t kN64 = idesc_bf16(128, 64, false, false);
+        const uint32_t base = smem_u32(smem);
+        fence_after();
+#pragma unroll
+        for (int p = 0; p < 3; ++p)
+          for (int ks = 0; ks < 8; ++ks)
+            mma_f16(tmem + cBlk, desc(base + (p == 1 ? oKQl : oKQh) + (ks >> 2) * kSub + (ks & 3) * 32, 16, 1024),
+                    desc(base + (p == 2 ? oQ : oK) + (ks >> 2) * kSub64 + (ks & 3) * 32, 16, 1024), kN64, p | ks ? 1u : 0u);
+        commit(&tl.blk_done);
+      }
+      __syncwarp();
+      // ---- A and B of other than mild chunks: 16 x 16 blocks in registers, first one per warp (0-3 on the diagonal), then the A or the B
+      // part of two more
       auto block_of = [](int task, int* rt, int* st) {
         const int off = task - 4;
         *rt = task < 4 ? task : off == 0 ? 1 : off < 3 ? 2 : 3;
@@ -255,37 +294,7 @@ __global__ void __launch_bounds__(kThreads, 1) delta_tc_kernel(const DeltaView v
           for (int e = 0; e < 4; ++e) ca[j][e] = cb[j][e] = 0.f;
         if (16 * rt >= n) return;
         const bool diag = rt == st;
-        if (mild) {
-          const int ra = rt * 16 + (lane & 15);
-          const uint32_t k2h = smem_addr(sK + (st * 16 + (lane & 7) + ((lane >> 4) << 3)) * kPk + ((lane >> 3) & 1) * 8), k2l = k2h + (uint32_t)(oQ - oK);
-          const uint32_t kq = smem_addr(smem + oKQh) + ra * 128;
-          float c1[2][4], c2[2][4];                      // the three products on accumulators of their own: short chains
-#pragma unroll
-          for (int part = 0; part < 2; ++part) {
-            if (part == 0 ? !do_a : !do_b) continue;
-            float (&cc)[2][4] = part == 0 ? ca : cb;
-#pragma unroll
-            for (int j = 0; j < 2; ++j)
-#pragma unroll
-              for (int e = 0; e < 4; ++e) c1[j][e] = c2[j][e] = 0.f;
-#pragma unroll 4
-            for (int kk = 0; kk < 8; ++kk) {
-              uint32_t ah[4], al[4], bh[4], bl[4];
-              const uint32_t at = kq + part * 64 * 128 + (kk >> 2) * kSub + (((((kk & 3) * 2) + (lane >> 4)) ^ (ra & 7)) << 4);
-              ldsm4(bh, k2h + kk * 32);
-              ldsm4(bl, k2l + kk * 32);
-              ldsm4(ah, at);
-              ldsm4(al, at + (oKQl - oKQh));
-              mma16816(cc[0], ah, bh[0], bh[1]); mma16816(cc[1], ah, bh[2], bh[3]);
-              mma16816(c1[0], al, bh[0], bh[1]); mma16816(c1[1], al, bh[2], bh[3]);
-              mma16816(c2[0], ah, bl[0], bl[1]); mma16816(c2[1], ah, bl[2], bl[3]);
-            }
-#pragma unroll
-            for (int j = 0; j < 2; ++j)
-#pragma unroll
-              for (int e = 0; e < 4; ++e) cc[j][e] += c1[j][e] + c2[j][e];
-          }
-        } else {
+        {
           bool direct = false;
           if (diag) {
             float m = 0.f;
@@ -301,7 +310,7 @@ __global__ void __launch_bounds__(kThreads, 1) delta_tc_kernel(const DeltaView v
                 const int r = st * 16 + g + 8 * (e >> 1), d = kk * 16 + 2 * tq + 8 * (e & 1);
                 const float2 G = *reinterpret_cast<const float2*>(sG + r * kPg + d), Rt = rt ? *reinterpret_cast<const float2*>(&tl.R[rt][d]) : make_float2(0.f, 0.f);
                 const float2 Rs = st ? *reinterpret_cast<const float2*>(&tl.R[st][d]) : make_float2(0.f, 0.f);
-                const float2 k = unpack_bf16(*reinterpret_cast<const uint32_t*>(sK + r * kPk + d));
+                const float2 k = unpack_bf16(*reinterpret_cast<const uint32_t*>(sK + r * kW + d));
                 split2(k.x * ex2(Rt.x - Rs.x - G.x), k.y * ex2(Rt.y - Rs.y - G.y), bh[e], bl[e]);
               }
 #pragma unroll
@@ -312,7 +321,7 @@ __global__ void __launch_bounds__(kThreads, 1) delta_tc_kernel(const DeltaView v
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {            // A operand: rows g + 8 (e & 1), channels 2 tq + 8 (e >> 1)
                   const int r = rt * 16 + g + 8 * (e & 1), d = kk * 16 + 2 * tq + 8 * (e >> 1);
-                  const float2 G = *reinterpret_cast<const float2*>(sG + r * kPg + d), x = unpack_bf16(*reinterpret_cast<const uint32_t*>(src + r * kPk + d));
+                  const float2 G = *reinterpret_cast<const float2*>(sG + r * kPg + d), x = unpack_bf16(*reinterpret_cast<const uint32_t*>(src + r * kW + d));
                   split2(x.x * ex2(G.x), x.y * ex2(G.y), xh[e], xl[e]);
                 }
                 mma16816(cc[0], xh, bh[0], bh[1]); mma16816(cc[1], xh, bh[2], bh[3]);
@@ -329,9 +338,9 @@ __global__ void __launch_bounds__(kThreads, 1) delta_tc_kernel(const DeltaView v
                 if (s > r) continue;
                 float x = 0.f, y = 0.f;
                 for (int d = 0; d < D; ++d) {
-                  const float w = __bfloat162float(sK[s * kPk + d]) * ex2(sG[r * kPg + d] - sG[s * kPg + d]);
-                  x = fmaf(__bfloat162float(sK[r * kPk + d]), w, x);
-                  y = fmaf(__bfloat162float(sQ[r * kPk + d]), w, y);
+                  const float w = __bfloat162float(sK[s * kW + d]) * ex2(sG[r * kPg + d] - sG[s * kPg + d]);
+                  x = fmaf(__bfloat162float(sK[r * kW + d]), w, x);
+                  y = fmaf(__bfloat162float(sQ[r * kW + d]), w, y);
                 }
                 ca[j][e] = x;
                 cb[j][e] = y;
@@ -344,80 +353,104 @@ __global__ void __launch_bounds__(kThreads, 1) delta_tc_kernel(const DeltaView v
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
             const int tl_ = g + 8 * (e >> 1), sl = 8 * j + 2 * tq + (e & 1), t = rt * 16 + tl_, s = st * 16 + sl;
-            const float ks = mild ? 1.f : rk[s];
-            ca[j][e] *= (mild ? beta[t] : beta[t] * rk[t]) * ks;
-            cb[j][e] *= (mild ? 1.f : rq[t]) * ks;
+            ca[j][e] *= beta[t] * rk[t] * rk[s];
+            cb[j][e] *= rq[t] * rk[s];
             if (diag && sl >= tl_) ca[j][e] = 0.f;
             if (diag && sl > tl_) cb[j][e] = 0.f;
           }
       };
-      float a1[2][4], b1[2][4], a2[2][4], b2[2][4];
-      int rt1, st1, rt2 = 0, st2 = 0;
-      block_of(pw, &rt1, &st1);
-      block(rt1, st1, true, true, a1, b1);
-      if (pw < 4) {
-        block_of(8 + (pw >> 1), &rt2, &st2);
-        block(rt2, st2, (pw & 1) == 0, pw & 1, a2, b2);
-      }
-      if (c) mbar_wait(&tl.s_done, (c - 1) & 1, dead, err);      // kb, B and T of the chunk before have been multiplied
-      // ---- kb
-#pragma unroll 2
-      for (int i = pt; i < kC * (kW / 4); i += 256) {
-        const int r = i >> 5, d = (i & 31) * 4, at = r * kPk + d, to = swz(r, d, kSubKb);
-        const uint2 ku = *reinterpret_cast<const uint2*>(sK + at);
-        float2 k0 = unpack_bf16(ku.x), k1 = unpack_bf16(ku.y);
-        float f[4];
-        if (mild) {
-          const float4 X = *reinterpret_cast<const float4*>(E + d);
-          const uint2 lu = *reinterpret_cast<const uint2*>(sQ + at);
-          const float2 l0 = unpack_bf16(lu.x), l1 = unpack_bf16(lu.y);
-          k0.x += l0.x; k0.y += l0.y; k1.x += l1.x; k1.y += l1.y;
-          f[0] = X.x; f[1] = X.y; f[2] = X.z; f[3] = X.w;
-        } else {
-          const float4 L = *reinterpret_cast<const float4*>(sG + r * kPg + d), all4 = *reinterpret_cast<const float4*>(&tl.R[4][d]);
-          const float4 Rv = r < 16 ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4*>(&tl.R[r >> 4][d]);
-          const float kr = rk[r];
-          f[0] = kr * ex2(all4.x - Rv.x - L.x); f[1] = kr * ex2(all4.y - Rv.y - L.y); f[2] = kr * ex2(all4.z - Rv.z - L.z); f[3] = kr * ex2(all4.w - Rv.w - L.w);
-        }
-        uint2 hi, lo;
-        split2(k0.x * f[0], k0.y * f[1], hi.x, lo.x);
-        split2(k1.x * f[2], k1.y * f[3], hi.y, lo.y);
-        *reinterpret_cast<uint2*>(smem + oKbh + to) = hi;
-        *reinterpret_cast<uint2*>(smem + oKbl + to) = lo;
-      }
-      // ---- B
-      auto put_b = [&](int rt, int st, const float (&cb)[2][4]) {
-#pragma unroll
-        for (int j = 0; j < 2; ++j)
-#pragma unroll
-          for (int e2 = 0; e2 < 2; ++e2) {
-            uint32_t hi, lo;
-            split2(cb[j][2 * e2], cb[j][2 * e2 + 1], hi, lo);
-            const int to = swz(rt * 16 + g + 8 * e2, st * 16 + 8 * j + 2 * tq, 0);
-            *reinterpret_cast<uint32_t*>(smem + oBh + to) = hi;
-            *reinterpret_cast<uint32_t*>(smem + oBl + to) = lo;
+      auto write_kb = [&]() {
+#pragma unroll 4
+        for (int it = 0; it < 8; ++it) {
+          const int r = (pt >> 5) + 8 * it, d = (pt & 31) * 4, to = swz(r, d, kSub64);
+          float2 k0, k1;
+          float f[4];
+          if (mild) {
+            const float4 X = *reinterpret_cast<const float4*>(E + d);
+            const uint2 ku = *reinterpret_cast<const uint2*>(smem + oK + to), lu = *reinterpret_cast<const uint2*>(smem + oQ + to);
+            const float2 l0 = unpack_bf16(lu.x), l1 = unpack_bf16(lu.y);
+            k0 = unpack_bf16(ku.x); k1 = unpack_bf16(ku.y);
+            k0.x += l0.x; k0.y += l0.y; k1.x += l1.x; k1.y += l1.y;
+            f[0] = X.x; f[1] = X.y; f[2] = X.z; f[3] = X.w;
+          } else {
+            const uint2 ku = *reinterpret_cast<const uint2*>(sK + r * kW + d);
+            const float4 L = *reinterpret_cast<const float4*>(sG + r * kPg + d), all4 = *reinterpret_cast<const float4*>(&tl.R[4][d]);
+            const float4 Rv = it < 2 ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4*>(&tl.R[it >> 1][d]);
+            const float kr = rk[r];
+            k0 = unpack_bf16(ku.x); k1 = unpack_bf16(ku.y);
+            f[0] = kr * ex2(all4.x - Rv.x - L.x); f[1] = kr * ex2(all4.y - Rv.y - L.y); f[2] = kr * ex2(all4.z - Rv.z - L.z); f[3] = kr * ex2(all4.w - Rv.w - L.w);
           }
+          uint2 hi, lo;
+          split2(k0.x * f[0], k0.y * f[1], hi.x, lo.x);
+          split2(k1.x * f[2], k1.y * f[3], hi.y, lo.y);
+          *reinterpret_cast<uint2*>(smem + oKbh + to) = hi;
+          *reinterpret_cast<uint2*>(smem + oKbl + to) = lo;
+        }
       };
-      put_b(rt1, st1, b1);
-      if (pw < 4 && (pw & 1)) put_b(rt2, st2, b2);
-      fence_async_smem();
-      prep_sync();
-      // ---- raw rows are free; the next chunk's decays are on their way; A in float32 over the decay sums
-      if (lane == 0) mbar_arrive(&tl.raw_empty);
-      if (c + 1 < chunks) fetch(c + 1);
+      // ---- A in float32 over the decay sums, B as an operand
       float *sA = sG, *sT = sG + kC * kPt;
-      auto put_a = [&](int rt, int st, const float (&ca)[2][4]) {
+      if (mild) {
+        mbar_wait(&tl.blk_done, n_mild++ & 1, dead, err);
+        fence_after();
+        float x[32];
+        tmem_ld32(x, tmem + ((uint32_t)(32 * quad) << 16) + cBlk + side * 32);
+        fence_before();
+        const int t = 32 * (quad & 1) + lane, s0 = side * 32;
+        if (quad < 2) {
+          const float bt = beta[t];
 #pragma unroll
-        for (int j = 0; j < 2; ++j)
+          for (int i = 0; i < 32; i += 2) *reinterpret_cast<float2*>(sA + t * kPt + s0 + i) = make_float2(s0 + i < t ? x[i] * bt : 0.f, s0 + i + 1 < t ? x[i + 1] * bt : 0.f);
+        } else {
+          if (c) mbar_wait(&tl.o_done, (c - 1) & 1, dead, err);
 #pragma unroll
-          for (int e2 = 0; e2 < 2; ++e2)
-            *reinterpret_cast<float2*>(sA + (rt * 16 + g + 8 * e2) * kPt + st * 16 + 8 * j + 2 * tq) = make_float2(ca[j][2 * e2], ca[j][2 * e2 + 1]);
-      };
-      put_a(rt1, st1, a1);
-      if (pw < 4 && (pw & 1) == 0) put_a(rt2, st2, a2);
+          for (int i = 0; i < 32; i += 8) {
+            uint4 hi, lo;
+            const auto z = [&](int j) { return s0 + i + j <= t ? x[i + j] : 0.f; };
+            split2(z(0), z(1), hi.x, lo.x); split2(z(2), z(3), hi.y, lo.y); split2(z(4), z(5), hi.z, lo.z); split2(z(6), z(7), hi.w, lo.w);
+            const int to = swz(t, s0 + i, 0);
+            *reinterpret_cast<uint4*>(smem + oBh + to) = hi;
+            *reinterpret_cast<uint4*>(smem + oBl + to) = lo;
+          }
+        }
+      } else {
+        float a1[2][4], b1[2][4], a2[2][4], b2[2][4];
+        int rt1, st1, rt2 = 0, st2 = 0;
+        block_of(pw, &rt1, &st1);
+        block(rt1, st1, true, true, a1, b1);
+        if (pw < 4) {
+          block_of(8 + (pw >> 1), &rt2, &st2);
+          block(rt2, st2, (pw & 1) == 0, pw & 1, a2, b2);
+        }
+        if (c) mbar_wait(&tl.s_done, (c - 1) & 1, dead, err);
+        write_kb();
+        auto put_b = [&](int rt, int st, const float (&cb)[2][4]) {
+#pragma unroll
+          for (int j = 0; j < 2; ++j)
+#pragma unroll
+            for (int e2 = 0; e2 < 2; ++e2) {
+              uint32_t hi, lo;
+              split2(cb[j][2 * e2], cb[j][2 * e2 + 1], hi, lo);
+              const int to = swz(rt * 16 + g + 8 * e2, st * 16 + 8 * j + 2 * tq, 0);
+              *reinterpret_cast<uint32_t*>(smem + oBh + to) = hi;
+              *reinterpret_cast<uint32_t*>(smem + oBl + to) = lo;
+            }
+        };
+        put_b(rt1, st1, b1);
+        if (pw < 4 && (pw & 1)) put_b(rt2, st2, b2);
+        prep_sync();                                     // decay sums and raw rows have been read
+        auto put_a = [&](int rt, int st, const float (&ca)[2][4]) {
+#pragma unroll
+          for (int j = 0; j < 2; ++j)
+#pragma unroll
+            for (int e2 = 0; e2 < 2; ++e2)
+              *reinterpret_cast<float2*>(sA + (rt * 16 + g + 8 * e2) * kPt + st * 16 + 8 * j + 2 * tq) = make_float2(ca[j][2 * e2], ca[j][2 * e2 + 1]);
+        };
+        put_a(rt1, st1, a1);
+        if (pw < 4 && (pw & 1) == 0) put_a(rt2, st2, a2);
+      }
+      prep_sync();
       // ---- T = (I + A)^-1: 16 x 16 diagonal blocks, then twice [[P, 0], [R, Q]]^-1 = [[P', 0], [-Q' R P', Q']]
       if (pw < 4) {
-        __syncwarp();
         const float* M = sA + (pw * 16) * kPt + pw * 16;
         float x[16];
 #pragma unroll
@@ -460,6 +493,7 @@ __global__ void __launch_bounds__(kThreads, 1) delta_tc_kernel(const DeltaView v
         const int i = pt >> 3, j = (pt & 7) * 4;
         const float *Rm = sA + (32 + i) * kPt, *P = sT + j;
         float x[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 4
         for (int k = j & 16; k < 32; k += 2) {           // P' is zero above its diagonal blocks (scratch lies there)
           const float2 m = *reinterpret_cast<const float2*>(Rm + k);
           const float2 p0 = *reinterpret_cast<const float2*>(P + k * kPt), p1 = *reinterpret_cast<const float2*>(P + k * kPt + 2);
@@ -473,6 +507,7 @@ __global__ void __launch_bounds__(kThreads, 1) delta_tc_kernel(const DeltaView v
         prep_sync();
         const float *Q = sT + (32 + i) * kPt + 32, *Z = sT + 32 + j;
         x[0] = x[1] = x[2] = x[3] = 0.f;
+#pragma unroll 4
         for (int k = 0; k < (i & 16) + 16; k += 2) {
           const float2 m = *reinterpret_cast<const float2*>(Q + k);
           const float2 p0 = *reinterpret_cast<const float2*>(Z + k * kPt), p1 = *reinterpret_cast<const float2*>(Z + k * kPt + 2);
@@ -485,21 +520,34 @@ __global__ void __launch_bounds__(kThreads, 1) delta_tc_kernel(const DeltaView v
         *reinterpret_cast<float2*>(W + 2) = make_float2(-x[2], -x[3]);
       }
       prep_sync();
-      for (int i = pt; i < 10 * 64; i += 256) {          // four elements of a row of one of the ten blocks
-        int rt, st;
-        block_of(i >> 6, &rt, &st);
-        const int r = rt * 16 + ((i & 63) >> 2), col = st * 16 + (i & 3) * 4, to = swz(r, col, 0);
-        const float2 x = *reinterpret_cast<const float2*>(sT + r * kPt + col), y = *reinterpret_cast<const float2*>(sT + r * kPt + col + 2);
-        uint2 hi, lo;
-        split2(x.x, x.y, hi.x, lo.x);
-        split2(y.x, y.y, hi.y, lo.y);
-        *reinterpret_cast<uint2*>(smem + oTh + to) = hi;
-        *reinterpret_cast<uint2*>(smem + oTl + to) = lo;
+      if (c) mbar_wait(&tl.u_done, (c - 1) & 1, dead, err);
+      {                                                  // sixteen elements of a row, zero above the triangle
+        const int r = pt >> 2, c0 = (pt & 3) * 16;
+        const bool in = c0 <= r;
+#pragma unroll
+        for (int i = 0; i < 16; i += 8) {
+          const float* x = sT + r * kPt + c0 + i;
+          uint4 hi = make_uint4(0, 0, 0, 0), lo = hi;
+          if (in) {
+            const float2 x0 = *reinterpret_cast<const float2*>(x), x1 = *reinterpret_cast<const float2*>(x + 2), x2 = *reinterpret_cast<const float2*>(x + 4), x3 = *reinterpret_cast<const float2*>(x + 6);
+            split2(x0.x, x0.y, hi.x, lo.x); split2(x1.x, x1.y, hi.y, lo.y); split2(x2.x, x2.y, hi.z, lo.z); split2(x3.x, x3.y, hi.w, lo.w);
+          }
+          const int to = swz(r, c0 + i, 0);
+          *reinterpret_cast<uint4*>(smem + oTh + to) = hi;
+          *reinterpret_cast<uint4*>(smem + oTl + to) = lo;
+        }
       }
       fence_async_smem();
       __syncwarp();
-      if (lane == 0) mbar_arrive(&tl.tb_ready);
-      prep_sync();                                       // T has been read: the next decay sums go over it
+      if (lane == 0) { mbar_arrive(&tl.tb_ready); mbar_arrive(&tl.g_empty); }
+      // ---- kb
+      if (mild) {
+        if (c) mbar_wait(&tl.s_done, (c - 1) & 1, dead, err);
+        write_kb();
+        fence_async_smem();
+        __syncwarp();
+      }
+      if (lane == 0) { mbar_arrive(&tl.kb_ready); mbar_arrive(&tl.raw_empty); }
     }
   } else {
     // ------------------------------ value columns ------------------------------
@@ -546,7 +594,7 @@ __global__ void __launch_bounds__(kThreads, 1) delta_tc_kernel(const DeltaView v
       {
         bf vv[32];
 #pragma unroll
-        for (int i = 0; i < 32; ++i) vv[i] = sV[(half * 32 + i) * kPk + col];
+        for (int i = 0; i < 32; ++i) vv[i] = col < V ? sV[(half * 32 + i) * kPv + col] : __float2bfloat16_rn(0.f);
         mbar_wait(&tl.yo_done, c & 1, dead, err);
         fence_after();
         tmem_ld32(x, lanes + cYO + half * 32);
@@ -559,9 +607,16 @@ __global__ void __launch_bounds__(kThreads, 1) delta_tc_kernel(const DeltaView v
       tmem_st_wait();
       fence_before();
       __syncwarp();
-      if (lane == 0) { mbar_arrive(&tl.x_ready); mbar_arrive(&tl.v_empty); }
-      const bf* gate = reinterpret_cast<const bf*>(v.gate) + t0 * v.gate_pitch + h * V + col;
-      if (half * 32 + lane < n && 32 * quad < V) asm volatile("prefetch.global.L2 [%0];\n" ::"l"(gate - lane + (int64_t)lane * v.gate_pitch));
+      if (lane == 0) mbar_arrive(&tl.x_ready);
+      // the gates of the output pieces this thread will store: pass p, rows of half a chunk's quarter, eight value columns
+      const int hr = tid & 127, piece = (hr & 15) * 8;   // 128 threads: 8 rows x 16 pieces at a time
+      uint4 gates[4];
+#pragma unroll
+      for (int p = 0; p < 4; ++p) {
+        const int r = p * 8 + (hr >> 4);
+        gates[p] = half * 32 + r < n && piece < V ? __ldg(reinterpret_cast<const uint4*>(reinterpret_cast<const bf*>(v.gate) + (t0 + r) * v.gate_pitch + h * V + piece))
+                                                  : make_uint4(0, 0, 0, 0);
+      }
       mbar_wait(&tl.u_done, c & 1, dead, err);
       fence_after();
       tmem_ld32(x, lanes + cYO + half * 32);
@@ -593,20 +648,33 @@ __global__ void __launch_bounds__(kThreads, 1) delta_tc_kernel(const DeltaView v
       asm volatile("bar.sync %0, 128;\n" ::"r"(1 + half) : "memory");
       const float all = tl.sum[0][half * 32 + lane] + tl.sum[1][half * 32 + lane] + tl.sum[2][half * 32 + lane] + tl.sum[3][half * 32 + lane];
       const float inv = 1.0f / sqrtf(all / (float)V + v.eps);
-      asm volatile("bar.sync %0, 128;\n" ::"r"(1 + half) : "memory");             // the sums have been read
-      bf* out = reinterpret_cast<bf*>(v.out) + t0 * v.ldo + h * V + col;
-      const int rows = col < V ? n - half * 32 : 0;
+      // turned through the place of v, sixteen tokens at a time: [16][128] float32 per half, then whole pieces of token rows
+      float* stage = reinterpret_cast<float*>(smem + oV) + half * 16 * kW;
 #pragma unroll
-      for (int i0 = 0; i0 < 32; i0 += 16) {              // sixteen gate values in flight
-        bf gv[16];
+      for (int p = 0; p < 2; ++p) {
 #pragma unroll
-        for (int i = 0; i < 16; ++i) gv[i] = i0 + i < rows ? __ldg(gate + (int64_t)(i0 + i) * v.gate_pitch) : __float2bfloat16_rn(0.f);
+        for (int i = 0; i < 16; ++i) stage[i * kW + col] = x[p * 16 + i] * __shfl_sync(0xffffffffu, inv, p * 16 + i) * wn;
+        asm volatile("bar.sync %0, 128;\n" ::"r"(1 + half) : "memory");
 #pragma unroll
-        for (int i = 0; i < 16; ++i) {
-          const float f = __shfl_sync(0xffffffffu, inv, i0 + i);
-          if (i0 + i < rows) out[(int64_t)(i0 + i) * v.ldo] = __float2bfloat16_rn(x[i0 + i] * f * wn * __bfloat162float(gv[i]));
+        for (int q = 0; q < 2; ++q) {
+          const int rl = q * 8 + (hr >> 4), r = p * 16 + rl;
+          const float4 y0 = *reinterpret_cast<const float4*>(stage + rl * kW + piece), y1 = *reinterpret_cast<const float4*>(stage + rl * kW + piece + 4);
+          uint4 gu = gates[p * 2 + q];
+          const float y[8] = {y0.x, y0.y, y0.z, y0.w, y1.x, y1.y, y1.z, y1.w};
+          uint32_t* gi = reinterpret_cast<uint32_t*>(&gu);
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const float2 gt = unpack_bf16(gi[e]);
+            const __nv_bfloat162 o = __floats2bfloat162_rn(y[2 * e] * gt.x, y[2 * e + 1] * gt.y);
+            gi[e] = *reinterpret_cast<const uint32_t*>(&o);
+          }
+          if (half * 32 + r < n && piece < V) *reinterpret_cast<uint4*>(reinterpret_cast<bf*>(v.out) + (t0 + r) * v.ldo + h * V + piece) = gu;
         }
+        asm volatile("bar.sync %0, 128;\n" ::"r"(1 + half) : "memory");
       }
+      fence_async_smem();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&tl.v_empty);
     }
     if (chunks > 0) {
       mbar_wait(&tl.s_done, (chunks - 1) & 1, dead, err);
