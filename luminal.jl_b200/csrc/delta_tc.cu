@@ -9,8 +9,10 @@
 //   [A | B] = [kt | qt] (k e^{-G})^T   mild chunks (see there), from shared memory; other chunks with mma.sync, block by block
 // Tensor memory columns: [Y then U | O] 128, S 128, [S hi | S lo, later X hi | X lo] 128, [U hi | U lo] 64, [A, B] 64 (lanes: tokens).
 // Warps: 0-7 own the value columns (two threads per column): they turn S, X and U into operands and write the outputs; 8-15 prepare the
-// next chunk (decay sums, kt, qt, kb, A and B, T in float32) while the others work on this one; 16 issues the other MMAs, 17 the row
-// copies.  All waits are bounded.
+// next chunk (decay sums, kt, qt, kb, A and B, T in float32) while the others work on this one; 16 issues the other MMAs, 17
+// and 18 the TMA loads.  All waits are bounded.
+#include <cuda.h>
+
 #include "delta.cuh"
 #include "mma_sync.cuh"
 #include "pdl.cuh"
@@ -22,9 +24,9 @@ namespace {
 constexpr int kC = 64, kW = 128;                        // tokens per chunk; head width, padded with zeros
 constexpr float kLog2e = 1.4426950408889634f;
 constexpr float kDiagMax = 80.0f, kDecayMin = -150.0f;  // as in csrc/delta_chunk.cu
-constexpr int kThreads = 18 * 32;
+constexpr int kThreads = 19 * 32;
 constexpr uint32_t cYO = 0, cS = 128, cSh = 256, cSl = 320, cXh = 256, cXl = 288, cUh = 384, cUl = 416, cBlk = 448;
-constexpr int kPv = kW, kPg = kW + 4, kPt = 66;         // row pitches: raw rows, decay sums, float32 A and T
+constexpr int kPv = kW, kPg = kW, kPt = 66;             // row pitches: raw rows, decay sums, float32 A and T
 // shared memory; tiles in the 128-byte swizzle
 constexpr int kSub = 128 * 128, kSub64 = 64 * 128;      // sub-tiles [128 rows][64 columns], [64 rows][64 columns]
 constexpr int oKQh = 0, oKQl = oKQh + 2 * kSub;         // rows 0-63 kt, 64-127 qt
@@ -33,8 +35,8 @@ constexpr int oTh = oKbl + 2 * kSub64, oTl = oTh + kSub64, oBh = oTl + kSub64, o
 constexpr int oK = oBl + kSub64, oQ = oK + 2 * kSub64;  // raw rows; mild chunks then k e^{-G} as a tile, hi over K, lo over Q
 constexpr int oV = oQ + 2 * kSub64;                     // v, later the outputs on their way out
 constexpr int oG = oV + 2 * kSub64;                     // log decays, their sums; later A and T in float32
-constexpr int oEnd = oG + kC * kPg * 4;
-static_assert(2 * kC * kPt * 4 <= kC * kPg * 4 && kC * kPv * 2 <= 2 * kSub64, "what lies over something else fits");
+constexpr int oEnd = oG + 2 * kC * kPt * 4;
+static_assert(kC * kPg * 4 <= 2 * kC * kPt * 4 && kC * kPv * 2 <= 2 * kSub64, "what lies over something else fits");
 struct Tail {
   uint64_t raw_full, raw_empty, g_full, g_empty, v_full, v_empty, kq_ready, blk_done, tb_ready, kb_ready, s_ready, x_ready, u_ready, yo_done, u_done, o_done, s_done;
   uint32_t tmem;
@@ -61,9 +63,36 @@ __device__ __forceinline__ void mma_ts(uint32_t d, uint32_t a, uint64_t b, uint3
 }
 // byte of (row, column) in a swizzled tile of sub-tiles `sub` bytes apart
 __device__ __forceinline__ int swz(int row, int col, int sub) { return (col >> 6) * sub + row * 128 + ((((col & 63) >> 3) ^ (row & 7)) << 4) + (col & 7) * 2; }
+__device__ __forceinline__ void tma_3d(void* dst, const CUtensorMap* map, int c1, int c2, uint64_t* bar) {
+  asm volatile(
+      "cp.async.bulk.tensor.3d.shared::cluster.global.tile.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3, %4}], [%5];\n" ::"r"(tc::smem_u32(dst)),
+      "l"(reinterpret_cast<uint64_t>(map)), "r"(0), "r"(c1), "r"(c2), "r"(tc::smem_u32(bar))
+      : "memory");
+}
+// one 16 x 8 tile of A B over 16 ks .. contraction steps, A and B row-major float32 of pitch kPt, operands as bf16 pairs hi + lo
+__device__ __forceinline__ void mm_tile(float (&c)[4], const float* A, const float* B, int k0, int k1, int g, int tq) {
+  c[0] = c[1] = c[2] = c[3] = 0.f;
+  for (int k = k0; k < k1; k += 16) {
+    uint32_t ah[4], al[4], bh[2], bl[2];
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const float2 x = *reinterpret_cast<const float2*>(A + (g + 8 * (e & 1)) * kPt + k + 2 * tq + 8 * (e >> 1));
+      split2(x.x, x.y, ah[e], al[e]);
+    }
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const float* x = B + (k + 2 * tq + 8 * e) * kPt + g;
+      split2(x[0], x[kPt], bh[e], bl[e]);
+    }
+    mma16816(c, ah, bh[0], bh[1]);
+    mma16816(c, al, bh[0], bh[1]);
+    mma16816(c, ah, bl[0], bl[1]);
+  }
+}
 __device__ __forceinline__ void prep_sync() { asm volatile("bar.sync 3, 256;\n" ::: "memory"); }
 
-__global__ void __launch_bounds__(kThreads, 1) delta_tc_kernel(const DeltaView v, int* err) {
+__global__ void __launch_bounds__(kThreads, 1) delta_tc_kernel(const DeltaView v, const __grid_constant__ CUtensorMap kmap, const __grid_constant__ CUtensorMap qmap,
+                                                                const __grid_constant__ CUtensorMap vmap, const __grid_constant__ CUtensorMap gmap, int* err) {
   using namespace tc;
   typedef __nv_bfloat16 bf;
   extern __shared__ __align__(1024) unsigned char smem[];
@@ -93,29 +122,27 @@ __global__ void __launch_bounds__(kThreads, 1) delta_tc_kernel(const DeltaView v
   const int n_all = v.len[b], t_first = v.start[b];
   const int chunks = (n_all + kC - 1) / kC;              // 0: nothing to do
 
-  if (warp == 17) {
-    // ------------------------------ rows of k, q, log g and v ------------------------------
-    for (int c = 0; c < chunks; ++c) {
-      const int64_t t0 = t_first + (int64_t)c * kC;
-      const int n = min(kC, n_all - c * kC);             // behind the portion's end the last row again: its beta and decay count as zero
-      mbar_wait(&tl.g_empty, (c & 1) ^ 1, dead, err);
-      if (lane == 0) mbar_expect_tx(&tl.g_full, (uint32_t)(kC * D * 4));
-      __syncwarp();
-      for (int r = lane; r < kC; r += 32) bulk_g2s(sG + r * kPg, v.decay + (t0 + min(r, n - 1)) * v.decay_pitch + h * D, (uint32_t)D * 4, &tl.g_full);
-      mbar_wait(&tl.raw_empty, (c & 1) ^ 1, dead, err);
-      if (lane == 0) mbar_expect_tx(&tl.raw_full, (uint32_t)(2 * kC * D * 2));
-      __syncwarp();
-      for (int r = lane; r < kC; r += 32) {
-        const int64_t t = t0 + min(r, n - 1);
-        bulk_g2s(sK + r * kW, reinterpret_cast<const bf*>(v.k) + t * v.k_pitch + a * D, (uint32_t)D * 2, &tl.raw_full);
-        bulk_g2s(sQ + r * kW, reinterpret_cast<const bf*>(v.q) + t * v.q_pitch + a * D, (uint32_t)D * 2, &tl.raw_full);
+  if (warp >= 17) {
+    // ------------------------------ rows of log g, k and q; of v.  What a box takes in behind the portion counts as zero (beta, decay) ------------------------------
+    if (lane == 0) {
+      for (int c = 0; c < chunks; ++c) {
+        const int t0 = t_first + c * kC;
+        if (warp == 17) {
+          mbar_wait(&tl.g_empty, (c & 1) ^ 1, dead, err);
+          mbar_expect_tx(&tl.g_full, kC * kW * 4);
+          tma_3d(sG, &gmap, h, t0, &tl.g_full);
+          mbar_wait(&tl.raw_empty, (c & 1) ^ 1, dead, err);
+          mbar_expect_tx(&tl.raw_full, 2 * kC * kW * 2);
+          tma_3d(sK, &kmap, a, t0, &tl.raw_full);
+          tma_3d(sQ, &qmap, a, t0, &tl.raw_full);
+        } else {
+          mbar_wait(&tl.v_empty, (c & 1) ^ 1, dead, err);
+          mbar_expect_tx(&tl.v_full, kC * kW * 2);
+          tma_3d(sV, &vmap, h, t0, &tl.v_full);
+        }
       }
-      mbar_wait(&tl.v_empty, (c & 1) ^ 1, dead, err);
-      if (lane == 0) mbar_expect_tx(&tl.v_full, (uint32_t)(kC * V * 2));
-      __syncwarp();
-      for (int r = lane; r < kC; r += 32)
-        bulk_g2s(sV + r * kPv, reinterpret_cast<const bf*>(v.v) + (t0 + min(r, n - 1)) * v.v_pitch + h * V, (uint32_t)V * 2, &tl.v_full);
     }
+    __syncwarp();
   } else if (warp == 16) {
     // ------------------------------ MMA issue ------------------------------
     constexpr uint32_t kN128 = idesc_bf16(128, 128, false, false), kN64 = idesc_bf16(128, 64, false, false), kN128m = idesc_bf16(128, 128, false, true);
@@ -466,58 +493,31 @@ __global__ void __launch_bounds__(kThreads, 1) delta_tc_kernel(const DeltaView v
         }
       }
       prep_sync();
-      {                                                  // R P' of the two 32-blocks, into the empty blocks above the diagonal
-        const int blk = pt >> 7, i = (pt & 127) >> 3, j = (pt & 7) * 2;
-        const float *Rm = sA + (blk * 32 + 16 + i) * kPt + blk * 32, *P = sT + (blk * 32) * kPt + blk * 32 + j;
-        float x = 0.f, y = 0.f;
-#pragma unroll
-        for (int k = 0; k < 16; ++k) {
-          const float m = Rm[k];
-          const float2 p = *reinterpret_cast<const float2*>(P + k * kPt);
-          x = fmaf(m, p.x, x); y = fmaf(m, p.y, y);
+      auto put_tile = [&](float* to, const float (&x)[4], float sign) {
+        *reinterpret_cast<float2*>(to + g * kPt + 2 * tq) = make_float2(sign * x[0], sign * x[1]);
+        *reinterpret_cast<float2*>(to + (g + 8) * kPt + 2 * tq) = make_float2(sign * x[2], sign * x[3]);
+      };
+      {                                                  // R P' of the two 32-blocks, into the empty blocks above the diagonal; then -Q' of it
+        float x[4];
+        const int blk = (pw >> 1) & 1, n0 = (pw & 1) * 8;
+        float *D0 = sT + blk * 32 * kPt + blk * 32, *D1 = D0 + 16 * kPt + 16, *up = D0 + 16, *low = D0 + 16 * kPt;
+        if (pw < 4) {
+          mm_tile(x, sA + (blk * 32 + 16) * kPt + blk * 32, D0 + n0, 0, 16, g, tq);
+          put_tile(up + n0, x, 1.f);
+          __syncwarp();                                  // a warp reads only the columns it wrote
+          mm_tile(x, D1, up + n0, 0, 16, g, tq);
+          put_tile(low + n0, x, -1.f);
         }
-        *reinterpret_cast<float2*>(sT + (blk * 32 + i) * kPt + blk * 32 + 16 + j) = make_float2(x, y);
-        prep_sync();
-        const float *Q = sT + (blk * 32 + 16 + i) * kPt + blk * 32 + 16, *Y = sT + (blk * 32) * kPt + blk * 32 + 16 + j;
-        x = y = 0.f;
-#pragma unroll
-        for (int k = 0; k < 16; ++k) {
-          const float m = Q[k];
-          const float2 p = *reinterpret_cast<const float2*>(Y + k * kPt);
-          x = fmaf(m, p.x, x); y = fmaf(m, p.y, y);
-        }
-        *reinterpret_cast<float2*>(sT + (blk * 32 + 16 + i) * kPt + blk * 32 + j) = make_float2(-x, -y);
       }
       prep_sync();
-      {                                                  // the same for the halves
-        const int i = pt >> 3, j = (pt & 7) * 4;
-        const float *Rm = sA + (32 + i) * kPt, *P = sT + j;
-        float x[4] = {0.f, 0.f, 0.f, 0.f};
-#pragma unroll 4
-        for (int k = j & 16; k < 32; k += 2) {           // P' is zero above its diagonal blocks (scratch lies there)
-          const float2 m = *reinterpret_cast<const float2*>(Rm + k);
-          const float2 p0 = *reinterpret_cast<const float2*>(P + k * kPt), p1 = *reinterpret_cast<const float2*>(P + k * kPt + 2);
-          const float2 q0 = *reinterpret_cast<const float2*>(P + (k + 1) * kPt), q1 = *reinterpret_cast<const float2*>(P + (k + 1) * kPt + 2);
-          x[0] = fmaf(m.x, p0.x, x[0]); x[1] = fmaf(m.x, p0.y, x[1]); x[2] = fmaf(m.x, p1.x, x[2]); x[3] = fmaf(m.x, p1.y, x[3]);
-          x[0] = fmaf(m.y, q0.x, x[0]); x[1] = fmaf(m.y, q0.y, x[1]); x[2] = fmaf(m.y, q1.x, x[2]); x[3] = fmaf(m.y, q1.y, x[3]);
-        }
-        float* Y = sT + i * kPt + 32 + j;
-        *reinterpret_cast<float2*>(Y) = make_float2(x[0], x[1]);
-        *reinterpret_cast<float2*>(Y + 2) = make_float2(x[2], x[3]);
+      {                                                  // the same for the halves; P' and Q' are zero above their diagonal blocks (scratch lies there)
+        float x[4];
+        const int m0 = (pw >> 2) * 16, n0 = (pw & 3) * 8;
+        mm_tile(x, sA + (32 + m0) * kPt, sT + n0, n0 & 16, 32, g, tq);
+        put_tile(sT + m0 * kPt + 32 + n0, x, 1.f);
         prep_sync();
-        const float *Q = sT + (32 + i) * kPt + 32, *Z = sT + 32 + j;
-        x[0] = x[1] = x[2] = x[3] = 0.f;
-#pragma unroll 4
-        for (int k = 0; k < (i & 16) + 16; k += 2) {
-          const float2 m = *reinterpret_cast<const float2*>(Q + k);
-          const float2 p0 = *reinterpret_cast<const float2*>(Z + k * kPt), p1 = *reinterpret_cast<const float2*>(Z + k * kPt + 2);
-          const float2 q0 = *reinterpret_cast<const float2*>(Z + (k + 1) * kPt), q1 = *reinterpret_cast<const float2*>(Z + (k + 1) * kPt + 2);
-          x[0] = fmaf(m.x, p0.x, x[0]); x[1] = fmaf(m.x, p0.y, x[1]); x[2] = fmaf(m.x, p1.x, x[2]); x[3] = fmaf(m.x, p1.y, x[3]);
-          x[0] = fmaf(m.y, q0.x, x[0]); x[1] = fmaf(m.y, q0.y, x[1]); x[2] = fmaf(m.y, q1.x, x[2]); x[3] = fmaf(m.y, q1.y, x[3]);
-        }
-        float* W = sT + (32 + i) * kPt + j;
-        *reinterpret_cast<float2*>(W) = make_float2(-x[0], -x[1]);
-        *reinterpret_cast<float2*>(W + 2) = make_float2(-x[2], -x[3]);
+        mm_tile(x, sT + (32 + m0) * kPt + 32, sT + 32 + n0, 0, m0 + 16, g, tq);
+        put_tile(sT + (32 + m0) * kPt + n0, x, -1.f);
       }
       prep_sync();
       if (c) mbar_wait(&tl.u_done, (c - 1) & 1, dead, err);
@@ -698,6 +698,31 @@ __global__ void __launch_bounds__(kThreads, 1) delta_tc_kernel(const DeltaView v
   }
 }
 
+typedef CUresult (*EncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*, const cuuint32_t*,
+                                  const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
+// [T tokens][heads][width] inside rows of `pitch` elements; a box is 64 tokens x 128 features of one head, rows dense, zeros behind the width
+int32_t rows_map(CUtensorMap* map, const void* base, bool f32, int width, int heads, int T, int pitch) {
+  static EncodeTiledFn enc = nullptr;
+  if (!enc) {
+    void* ptr = nullptr;
+    cudaDriverEntryPointQueryResult qres;
+    if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &ptr, cudaEnableDefault, &qres) != cudaSuccess || qres != cudaDriverEntryPointSuccess) {
+      cudaGetLastError();
+      return fail(LMB200_ECUDA, "delta rule: cuTensorMapEncodeTiled is not available");
+    }
+    enc = reinterpret_cast<EncodeTiledFn>(ptr);
+  }
+  const int e = f32 ? 4 : 2;
+  const cuuint64_t dims[3] = {(cuuint64_t)width, (cuuint64_t)heads, (cuuint64_t)T};
+  const cuuint64_t strides[2] = {(cuuint64_t)width * e, (cuuint64_t)pitch * e};
+  const cuuint32_t box[3] = {(cuuint32_t)kW, 1, (cuuint32_t)kC};
+  const cuuint32_t estr[3] = {1, 1, 1};
+  const CUresult r = enc(map, f32 ? CU_TENSOR_MAP_DATA_TYPE_FLOAT32 : CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(base), dims, strides, box, estr,
+                         CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_NONE, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  if (r != CUDA_SUCCESS) return fail(LMB200_ECUDA, "delta rule: cuTensorMapEncodeTiled failed (%d)", (int)r);
+  return LMB200_OK;
+}
+
 }  // namespace
 
 int32_t delta_tc_configure() {
@@ -710,7 +735,12 @@ bool delta_tc_ok(const DeltaView& v) { return delta_chunks_ok(v) && (v.dim > 64 
 
 int32_t delta_tc(Ctx* ctx, const DeltaView& v, cudaStream_t st) {
   LMB_REQUIRE(delta_tc_ok(v), "delta rule: heads of %d x %d have no kernel on tcgen05", v.dim, v.vdim);
-  LMB_CUDA(launch_k(delta_tc_kernel, dim3((unsigned)v.H, (unsigned)v.B), dim3(kThreads), kSmem, st, v, ctx->dev_err));
+  CUtensorMap kmap, qmap, vmap, gmap;
+  LMB_TRY(rows_map(&kmap, v.k, false, v.dim, v.G, v.total, v.k_pitch));
+  LMB_TRY(rows_map(&qmap, v.q, false, v.dim, v.G, v.total, v.q_pitch));
+  LMB_TRY(rows_map(&vmap, v.v, false, v.vdim, v.H, v.total, v.v_pitch));
+  LMB_TRY(rows_map(&gmap, v.decay, true, v.dim, v.H, v.total, v.decay_pitch));
+  LMB_CUDA(launch_k(delta_tc_kernel, dim3((unsigned)v.H, (unsigned)v.B), dim3(kThreads), kSmem, st, v, kmap, qmap, vmap, gmap, ctx->dev_err));
   ctx->launches++;
   return LMB200_OK;
 }
