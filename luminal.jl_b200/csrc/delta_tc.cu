@@ -26,7 +26,7 @@ constexpr float kLog2e = 1.4426950408889634f;
 constexpr float kDiagMax = 80.0f, kDecayMin = -150.0f;  // as in csrc/delta_chunk.cu
 constexpr int kThreads = 19 * 32;
 constexpr uint32_t cYO = 0, cS = 128, cSh = 256, cSl = 320, cXh = 256, cXl = 288, cUh = 384, cUl = 416, cBlk = 448;
-constexpr int kPv = kW, kPg = kW, kPt = 66;             // row pitches: raw rows, decay sums, float32 A and T
+constexpr int kPv = kW, kPg = kW, kPt = 72;             // row pitches: raw rows, decay sums, float32 A and T
 // shared memory; tiles in the 128-byte swizzle
 constexpr int kSub = 128 * 128, kSub64 = 64 * 128;      // sub-tiles [128 rows][64 columns], [64 rows][64 columns]
 constexpr int oKQh = 0, oKQl = oKQh + 2 * kSub;         // rows 0-63 kt, 64-127 qt
@@ -103,7 +103,7 @@ __global__ void __launch_bounds__(kThreads, 1) delta_tc_kernel(const DeltaView v
   const int h = blockIdx.x, b = blockIdx.y, D = v.dim, V = v.vdim, ld = (V + 3) & ~3, a = h / (v.H / v.G);
   if (tid == 0) {
     if (smem_u32(smem) & 1023) atomicExch(err, 1);       // the swizzle needs 1024-byte tiles
-    mbar_init(&tl.raw_full, 1); mbar_init(&tl.g_full, 1); mbar_init(&tl.v_full, 1); mbar_init(&tl.blk_done, 1); mbar_init(&tl.yo_done, 1); mbar_init(&tl.u_done, 1); mbar_init(&tl.o_done, 1); mbar_init(&tl.s_done, 1);
+    mbar_init(&tl.raw_full, 2); mbar_init(&tl.g_full, 1); mbar_init(&tl.v_full, 1); mbar_init(&tl.blk_done, 1); mbar_init(&tl.yo_done, 1); mbar_init(&tl.u_done, 1); mbar_init(&tl.o_done, 1); mbar_init(&tl.s_done, 1);
     mbar_init(&tl.raw_empty, 8); mbar_init(&tl.g_empty, 8); mbar_init(&tl.v_empty, 8); mbar_init(&tl.kb_ready, 8); mbar_init(&tl.kq_ready, 8); mbar_init(&tl.tb_ready, 8);
     mbar_init(&tl.s_ready, 8); mbar_init(&tl.x_ready, 8); mbar_init(&tl.u_ready, 8);
     mbar_init_fence();
@@ -124,19 +124,35 @@ __global__ void __launch_bounds__(kThreads, 1) delta_tc_kernel(const DeltaView v
 
   if (warp >= 17) {
     // ------------------------------ rows of log g, k and q; of v.  What a box takes in behind the portion counts as zero (beta, decay) ------------------------------
-    if (lane == 0) {
-      for (int c = 0; c < chunks; ++c) {
-        const int t0 = t_first + c * kC;
-        if (warp == 17) {
-          mbar_wait(&tl.g_empty, (c & 1) ^ 1, dead, err);
+    for (int c = 0; c < chunks; ++c) {
+      const int t0 = t_first + c * kC;
+      if (warp == 17) {
+        mbar_wait(&tl.g_empty, (c & 1) ^ 1, dead, err);
+        if (lane == 0) {
           mbar_expect_tx(&tl.g_full, kC * kW * 4);
           tma_3d(sG, &gmap, h, t0, &tl.g_full);
-          mbar_wait(&tl.raw_empty, (c & 1) ^ 1, dead, err);
+        }
+        mbar_wait(&tl.raw_empty, (c & 1) ^ 1, dead, err);
+        if (lane == 0) {
           mbar_expect_tx(&tl.raw_full, 2 * kC * kW * 2);
           tma_3d(sK, &kmap, a, t0, &tl.raw_full);
           tma_3d(sQ, &qmap, a, t0, &tl.raw_full);
-        } else {
-          mbar_wait(&tl.v_empty, (c & 1) ^ 1, dead, err);
+        }
+        float (*row)[kC] = tl.row[c & 1];                // the tokens' scalars go with them
+#pragma unroll
+        for (int r = lane; r < kC; r += 32) {
+          const bool ok = c * kC + r < n_all;
+          const int64_t t = (int64_t)t0 + (ok ? r : 0);
+          const float x = v.b[t * v.b_pitch + h], y = v.rk[t * v.G + a], z = v.rq[t * v.G + a];
+          row[0][r] = ok ? 1.0f / (1.0f + expf(-x)) : 0.f;
+          row[1][r] = ok ? y : 0.f;
+          row[2][r] = ok ? z : 0.f;
+        }
+        __syncwarp();
+        if (lane == 0) mbar_arrive(&tl.raw_full);
+      } else {
+        mbar_wait(&tl.v_empty, (c & 1) ^ 1, dead, err);
+        if (lane == 0) {
           mbar_expect_tx(&tl.v_full, kC * kW * 2);
           tma_3d(sV, &vmap, h, t0, &tl.v_full);
         }
@@ -197,25 +213,10 @@ __global__ void __launch_bounds__(kThreads, 1) delta_tc_kernel(const DeltaView v
     const int ch = pt >> 1, hf = pt & 1;                 // decay sums: channel, half of the chunk
     const int quad = warp & 3, side = pw >> 2;           // A and B: 32 rows of [A | B], half of their columns
     int n_mild = 0;                                      // phases of blk_done
-    float rb = 0.f, rk_ = 0.f, rq_ = 0.f;
-    auto fetch = [&](int c) {                            // scalars of token pt
-      const int64_t t = t_first + (int64_t)c * kC + pt;
-      if (pt >= kC) return;
-      const bool ok = c * kC + pt < n_all;
-      rb = ok ? v.b[t * v.b_pitch + h] : 0.f;
-      rk_ = ok ? v.rk[t * v.G + a] : 0.f;
-      rq_ = ok ? v.rq[t * v.G + a] : 0.f;
-    };
-    if (chunks > 0) fetch(0);
     for (int c = 0; c < chunks; ++c) {
       const int n = min(kC, n_all - c * kC);
-      float *beta = tl.row[c & 1][0], *rk = tl.row[c & 1][1], *rq = tl.row[c & 1][2], *E = tl.E[c & 1];
-      if (pt < kC) {
-        beta[pt] = pt < n ? 1.0f / (1.0f + expf(-rb)) : 0.f;
-        rk[pt] = rk_;
-        rq[pt] = rq_;
-      }
-      if (c + 1 < chunks) fetch(c + 1);
+      const float *beta = tl.row[c & 1][0], *rk = tl.row[c & 1][1], *rq = tl.row[c & 1][2];
+      float* E = tl.E[c & 1];
       // ---- decay sums (log2 units): in sG from the start of each block of 16 tokens, in R before the block
       mbar_wait(&tl.g_full, c & 1, dead, err);
       float tot[2];
@@ -417,6 +418,8 @@ __global__ void __launch_bounds__(kThreads, 1) delta_tc_kernel(const DeltaView v
       // ---- A in float32 over the decay sums, B as an operand
       float *sA = sG, *sT = sG + kC * kPt;
       if (mild) {
+        if (c) mbar_wait(&tl.s_done, (c - 1) & 1, dead, err);   // all products of the chunk before: kb, T and B are free
+        write_kb();                                      // while A and B are multiplied
         mbar_wait(&tl.blk_done, n_mild++ & 1, dead, err);
         fence_after();
         float x[32];
@@ -426,9 +429,11 @@ __global__ void __launch_bounds__(kThreads, 1) delta_tc_kernel(const DeltaView v
         if (quad < 2) {
           const float bt = beta[t];
 #pragma unroll
-          for (int i = 0; i < 32; i += 2) *reinterpret_cast<float2*>(sA + t * kPt + s0 + i) = make_float2(s0 + i < t ? x[i] * bt : 0.f, s0 + i + 1 < t ? x[i + 1] * bt : 0.f);
+          for (int i = 0; i < 32; i += 4) {
+            const auto z = [&](int j) { return s0 + i + j < t ? x[i + j] * bt : 0.f; };
+            *reinterpret_cast<float4*>(sA + t * kPt + s0 + i) = make_float4(z(0), z(1), z(2), z(3));
+          }
         } else {
-          if (c) mbar_wait(&tl.o_done, (c - 1) & 1, dead, err);
 #pragma unroll
           for (int i = 0; i < 32; i += 8) {
             uint4 hi, lo;
@@ -475,6 +480,9 @@ __global__ void __launch_bounds__(kThreads, 1) delta_tc_kernel(const DeltaView v
         put_a(rt1, st1, a1);
         if (pw < 4 && (pw & 1) == 0) put_a(rt2, st2, a2);
       }
+      fence_async_smem();
+      __syncwarp();
+      if (lane == 0) { mbar_arrive(&tl.kb_ready); mbar_arrive(&tl.raw_empty); }
       prep_sync();
       // ---- T = (I + A)^-1: 16 x 16 diagonal blocks, then twice [[P, 0], [R, Q]]^-1 = [[P', 0], [-Q' R P', Q']]
       if (pw < 4) {
@@ -520,7 +528,6 @@ __global__ void __launch_bounds__(kThreads, 1) delta_tc_kernel(const DeltaView v
         put_tile(sT + (32 + m0) * kPt + n0, x, -1.f);
       }
       prep_sync();
-      if (c) mbar_wait(&tl.u_done, (c - 1) & 1, dead, err);
       {                                                  // sixteen elements of a row, zero above the triangle
         const int r = pt >> 2, c0 = (pt & 3) * 16;
         const bool in = c0 <= r;
@@ -529,8 +536,8 @@ __global__ void __launch_bounds__(kThreads, 1) delta_tc_kernel(const DeltaView v
           const float* x = sT + r * kPt + c0 + i;
           uint4 hi = make_uint4(0, 0, 0, 0), lo = hi;
           if (in) {
-            const float2 x0 = *reinterpret_cast<const float2*>(x), x1 = *reinterpret_cast<const float2*>(x + 2), x2 = *reinterpret_cast<const float2*>(x + 4), x3 = *reinterpret_cast<const float2*>(x + 6);
-            split2(x0.x, x0.y, hi.x, lo.x); split2(x1.x, x1.y, hi.y, lo.y); split2(x2.x, x2.y, hi.z, lo.z); split2(x3.x, x3.y, hi.w, lo.w);
+            const float4 x0 = *reinterpret_cast<const float4*>(x), x1 = *reinterpret_cast<const float4*>(x + 4);
+            split2(x0.x, x0.y, hi.x, lo.x); split2(x0.z, x0.w, hi.y, lo.y); split2(x1.x, x1.y, hi.z, lo.z); split2(x1.z, x1.w, hi.w, lo.w);
           }
           const int to = swz(r, c0 + i, 0);
           *reinterpret_cast<uint4*>(smem + oTh + to) = hi;
@@ -540,14 +547,6 @@ __global__ void __launch_bounds__(kThreads, 1) delta_tc_kernel(const DeltaView v
       fence_async_smem();
       __syncwarp();
       if (lane == 0) { mbar_arrive(&tl.tb_ready); mbar_arrive(&tl.g_empty); }
-      // ---- kb
-      if (mild) {
-        if (c) mbar_wait(&tl.s_done, (c - 1) & 1, dead, err);
-        write_kb();
-        fence_async_smem();
-        __syncwarp();
-      }
-      if (lane == 0) { mbar_arrive(&tl.kb_ready); mbar_arrive(&tl.raw_empty); }
     }
   } else {
     // ------------------------------ value columns ------------------------------
