@@ -6,7 +6,9 @@
 //   X = beta (V - Y),  U^T = X^T T^T   T = (I + A)^-1, 64 x 64
 //   O^T += U^T B^T,   S^T = S^T diag(e^{G_end}) + U^T kb
 // every product as hi hi + lo hi + hi lo (x = hi + lo to about 2^-17), accumulated in float32.
-//   [A | B] = [kt | qt] (k e^{-G})^T   mild chunks (see there), from shared memory; other chunks with mma.sync, block by block
+//   [A | B] = [kt | qt] (k e^{-G})^T   mild chunks, from shared memory; other chunks with mma.sync, block by block
+// Mild: no channel decays by more than 2^-160 in the chunk.  There G counts from the middle, G - G_end / 2, so that e^G and e^-G stay within
+// 2^80, and the operand of the first product is S e^{G_end / 2}.  (A and B above their diagonals may overflow; those elements are dropped.)
 // Tensor memory columns: [Y then U | O] 128, S 128, [S hi | S lo, later X hi | X lo] 128, [U hi | U lo] 64, [A, B] 64 (lanes: tokens).
 // Warps: 0-7 own the value columns (two threads per column): they turn S, X and U into operands and write the outputs; 8-15 prepare the
 // next chunk (decay sums, kt, qt, kb, A and B, T in float32) while the others work on this one; 16 issues the other MMAs, 17
@@ -42,6 +44,7 @@ struct Tail {
   uint32_t tmem;
   alignas(16) float R[5][kW];                           // decay sums before blocks 1 .. 3 of 16 tokens, and of the whole chunk
   alignas(16) float E[2][kW];                           // e^{G_end}, by chunk parity
+  alignas(16) float M[2][kW];                           // e^{G_end / 2}, or 1 in other than mild chunks
   float row[2][3][kC];                                  // beta, 1 / |k|, 1 / |q| / sqrt(dim), by chunk parity
   float sum[4][kC];                                     // sums of squares of the outputs per 32 value columns
 };
@@ -242,14 +245,20 @@ __global__ void __launch_bounds__(kThreads, 1) delta_tc_kernel(const DeltaView v
       }
       int mild;
       {                                                  // over the preparing warps
-        int p = all >= -kDiagMax;
+        int p = all >= -2 * kDiagMax;
         asm volatile("{\n.reg .pred p, q;\nsetp.ne.s32 p, %1, 0;\nbarrier.red.and.pred q, 3, 256, p;\nselp.s32 %0, 1, 0, q;\n}\n" : "=r"(mild) : "r"(p) : "memory");
       }
+      if (!hf) tl.M[c & 1][ch] = mild ? ex2(0.5f * all) : 1.f;
       // ---- kt, qt, and k e^{-G} over the raw rows
       mbar_wait(&tl.raw_full, c & 1, dead, err);
       if (c) mbar_wait(&tl.yo_done, (c - 1) & 1, dead, err);
       {
         uint2 mh[8], ml[8];
+        float4 mid = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (mild) {
+          mid = *reinterpret_cast<const float4*>(&tl.R[4][(pt & 31) * 4]);
+          mid.x *= 0.5f; mid.y *= 0.5f; mid.z *= 0.5f; mid.w *= 0.5f;
+        }
 #pragma unroll
         for (int it = 0; it < 8; ++it) {
           const int r = (pt >> 5) + 8 * it, d = (pt & 31) * 4, at = r * kW + d;
@@ -262,7 +271,7 @@ __global__ void __launch_bounds__(kThreads, 1) delta_tc_kernel(const DeltaView v
           }
           const float2 k0 = unpack_bf16(ku.x), k1 = unpack_bf16(ku.y), q0 = unpack_bf16(qu.x), q1 = unpack_bf16(qu.y);
           const float kr = rk[r], qr = rq[r];
-          const float G[4] = {Rv.x + L.x, Rv.y + L.y, Rv.z + L.z, Rv.w + L.w};
+          const float G[4] = {Rv.x + L.x - mid.x, Rv.y + L.y - mid.y, Rv.z + L.z - mid.z, Rv.w + L.w - mid.w};
           const float k[4] = {k0.x * kr, k0.y * kr, k1.x * kr, k1.y * kr}, q[4] = {q0.x * qr, q0.y * qr, q1.x * qr, q1.y * qr};
           float e[4];
 #pragma unroll
@@ -394,7 +403,7 @@ __global__ void __launch_bounds__(kThreads, 1) delta_tc_kernel(const DeltaView v
           float2 k0, k1;
           float f[4];
           if (mild) {
-            const float4 X = *reinterpret_cast<const float4*>(E + d);
+            const float4 X = *reinterpret_cast<const float4*>(&tl.M[c & 1][d]);
             const uint2 ku = *reinterpret_cast<const uint2*>(smem + oK + to), lu = *reinterpret_cast<const uint2*>(smem + oQ + to);
             const float2 l0 = unpack_bf16(lu.x), l1 = unpack_bf16(lu.y);
             k0 = unpack_bf16(ku.x); k1 = unpack_bf16(ku.y);
@@ -557,7 +566,7 @@ __global__ void __launch_bounds__(kThreads, 1) delta_tc_kernel(const DeltaView v
     for (int c = 0; c < chunks; ++c) {
       const int n = min(kC, n_all - c * kC);
       const int64_t t0 = t_first + (int64_t)c * kC + half * 32;
-      const float *beta = tl.row[c & 1][0] + half * 32, *E = tl.E[c & 1];
+      const float *beta = tl.row[c & 1][0] + half * 32, *E = tl.E[c & 1], *M = tl.M[c & 1];
       // ---- S as an operand, and decayed
       mbar_wait(&tl.kq_ready, c & 1, dead, err);
       if (c) { mbar_wait(&tl.s_done, (c - 1) & 1, dead, err); fence_after(); }
@@ -573,7 +582,7 @@ __global__ void __launch_bounds__(kThreads, 1) delta_tc_kernel(const DeltaView v
         }
         uint32_t hi[8], lo[8], u[16];
 #pragma unroll
-        for (int i = 0; i < 16; i += 2) split2(x[i], x[i + 1], hi[i / 2], lo[i / 2]);
+        for (int i = 0; i < 16; i += 2) split2(x[i] * M[d0 + i], x[i + 1] * M[d0 + i + 1], hi[i / 2], lo[i / 2]);
 #pragma unroll
         for (int i = 0; i < 16; ++i) u[i] = __float_as_uint(x[i] * E[d0 + i]);
         tmem_st16_nowait(lanes + cS + d0, u);

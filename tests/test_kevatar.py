@@ -397,7 +397,7 @@ def test_delta_remembers_one_token(device, dtype, dims):
 @gpu
 @BOTH
 @pytest.mark.parametrize("dims", [(10, 14), (128, 128), (64, 64)])
-@pytest.mark.parametrize("rate", [(3.0, 4.0), (-6.0, -5.0), (0.5, -1.0), (1.0, 0.0), None])
+@pytest.mark.parametrize("rate", [(3.0, 4.0), (-6.0, -5.0), (0.5, -1.0), (0.5, 0.0), (1.0, -0.2), (1.0, 0.0), None])
 def test_delta_decays(device, dtype, dims, rate):
     """Decays from nearly none to a factor below any float within a few tokens, and both next to each other."""
     import luminal_jl_b200 as L
