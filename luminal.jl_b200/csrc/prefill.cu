@@ -114,11 +114,14 @@ __device__ __forceinline__ void segment_epilogue(const GemmParams& p, float (&v)
   if (sg.kind == SEG_GELU_TOKEN) {
     const __nv_bfloat16* table = reinterpret_cast<const __nv_bfloat16*>(sg.table);
     const int tok = t0 + lane < t_end ? sg.tokens[t0 + lane] : -1;
+    __nv_bfloat16 e[32];                                // all table reads first
 #pragma unroll
     for (int i = 0; i < 32; ++i) {
       const int tk = __shfl_sync(0xffffffffu, tok, i);
-      v[i] = tk >= 0 && tk < sg.table_rows && r < sg.rows ? gelu_ref(v[i]) * __bfloat162float(table[(int64_t)tk * sg.table_pitch + r]) : 0.f;
+      e[i] = tk >= 0 && tk < sg.table_rows && r < sg.rows ? __ldg(table + (int64_t)tk * sg.table_pitch + r) : __float2bfloat16_rn(0.f);
     }
+#pragma unroll
+    for (int i = 0; i < 32; ++i) v[i] = gelu_ref(v[i]) * __bfloat162float(e[i]);
   }
   if (sg.kind == SEG_ROT) {
     const int f = r % sg.rot_head - sg.rot_off;         // partner rows are neighbouring lanes
