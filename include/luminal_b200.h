@@ -419,7 +419,7 @@ int32_t lmb200_prefill_ragged(lmb200_session session, const int32_t* tokens, con
 /* The next lengths[b] >= 0 tokens of every sequence, appended at that sequence's position: `tokens` holds the ids of
  * sequence 0, then those of sequence 1, and so on.  want[n_want] (ascending places in that packed order) chooses the
  * positions whose logits come back, [n_want, vocab] in logits_out.  Prompts, portions of prompts and single tokens can be
- * mixed in one call; the result at a position does not depend on how its tokens were cut into calls, beyond rounding.
+ * mixed in one call.  Up to rounding, any division of a sequence into calls gives the same logits.
  * Replaces running the model over [batch, seq] tokens and slicing its logits (src/NN.jl:448-455). */
 int32_t lmb200_extend(lmb200_session session, const int32_t* tokens, const int32_t* lengths, int32_t n_want,
                       const int32_t* want, float* logits_out);
